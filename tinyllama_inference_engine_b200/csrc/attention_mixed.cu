@@ -7,6 +7,8 @@
 //   visible: 0 <= i - j, and i - j < window if window > 0; with keep_first > 0 the keys j < keep_first stay visible behind the window
 //   out_h = softmax_j(mixed_h) . v_j                                      (values of value_dim, keys of key_dim)
 //   out   = concat_h(out_h) * sigmoid(gate)                               (gate optional: H * value_dim columns of the same row, or H: one per head)
+// ``softcap`` > 0: the mixed score is bounded first, softcap * tanh(score / softcap).  ``sigmoid``: no softmax, the weight of a visible key is
+// sigmoid(score + shift_h) (``shifts`` optional, one per head), and a row's weights are not brought to a sum of one.
 // ``sinks`` (optional, one per head): the softmax's denominator also holds exp(sink_h), a weight that belongs to no key.
 // ``v_row_stride``: elements between two slots of the value plane (value_dim unless the values are a part of wider rows, as when
 // they are the leading columns of the keys themselves).
@@ -141,46 +143,144 @@ __global__ void __launch_bounds__(128) normed_store_kernel(T* __restrict__ rows,
   }
 }
 
-// Latent attention's cache write and rotation.  A row holds ``heads`` queries of [plain | rot] and, from ``latent_offset``, the
-// down projection [rank | rot].  The first ``rank`` columns are normalised (RMS, weight) into the latent; the last ``rot`` are a key
-// part that all heads share and that is rotated: pairs (2i, 2i + 1) of its first ``rot_dims`` columns turn by position * inv_freq[i]
-// (32-bit angles).  [latent | rotated part] goes into the token's cache row; the queries' rotated parts go into ``queries``
-// [T, heads, rank + rot] behind the ``rank`` columns that the product with the keys' expansion fills.
+// Biases, a norm and a rotation of every query and key, and the cache write.  A row of ``rows`` holds the products [q: heads x key_dim |
+// ... k at k_offset | ... v at v_offset].  Every vector gets its bias (null: none); q and k are divided by their root mean square and
+// multiplied by a weight (null: neither); their first ``rot_dims`` columns turn by position * inv_freq[i], cosines and sines times
+// ``amplitude``, columns (2i, 2i + 1) together if ``interleaved``, else column i with column i + rot_dims / 2; query head h is multiplied by
+// q_factors[h] (null: not).  q stays in place, k and v go into the token's page.  A warp per vector, which waits in shared memory as
+// 32-bit numbers between the passes.
 template <typename T>
-__global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__ rows, int row_stride, int latent_offset, const float* __restrict__ weight, float eps,
-                                                           const float* __restrict__ inv_freq, int rot_dims, const int* __restrict__ positions,
-                                                           const int* __restrict__ token_seq, const int* __restrict__ block_table, int table_stride,
-                                                           T* __restrict__ pages, long long page_stride, int heads, int plain, int rot, int rank, int page_size,
-                                                           int write_cache, T* __restrict__ queries) {
-  __shared__ float scratch[32];
+__global__ void __launch_bounds__(256) norm_rotary_store_kernel(T* __restrict__ rows, int row_stride, int k_offset, int v_offset, const float* __restrict__ q_bias,
+                                                                const float* __restrict__ k_bias, const float* __restrict__ v_bias, const float* __restrict__ q_weight,
+                                                                const float* __restrict__ k_weight, float eps, const float* __restrict__ q_factors,
+                                                                const float* __restrict__ inv_freq, int rot_dims, int interleaved, float amplitude,
+                                                                const int* __restrict__ positions, const int* __restrict__ token_seq,
+                                                                const int* __restrict__ block_table, int table_stride, T* __restrict__ k_pages, long long k_page_stride,
+                                                                T* __restrict__ v_pages, long long v_page_stride, int heads, int kv_heads, int key_dim, int value_dim,
+                                                                int page_size, int write_cache) {
+  extern __shared__ float turn_s[];   // the token's cosines [rot_dims / 2], its sines, then a vector per warp [key_dim]
   const int t = blockIdx.x;
   const int pos = positions[t];
   const int page = write_cache ? block_table[(size_t)token_seq[t] * table_stride + pos / page_size] : -1;
-  const T* row = rows + (size_t)t * row_stride;
-  T* cached = page >= 0 ? pages + (size_t)page * page_stride + (size_t)(pos % page_size) * (rank + rot) : nullptr;
-  float squares = 0.0f;
-  for (int d = threadIdx.x; d < rank; d += blockDim.x) {
-    const float v = to_float(row[latent_offset + d]);
-    squares += v * v;
+  const int slot = pos % page_size;
+  T* row = rows + (size_t)t * row_stride;
+  const int half = rot_dims / 2;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  float* vec = turn_s + rot_dims + (size_t)warp * key_dim;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sine, cosine;
+    sincosf((float)pos * inv_freq[i], &sine, &cosine);
+    turn_s[i] = cosine * amplitude;
+    turn_s[half + i] = sine * amplitude;
   }
-  const float inv = rsqrtf(block_sum(squares, scratch) / (float)rank + eps);
-  if (cached)
-    for (int d = threadIdx.x; d < rank; d += blockDim.x) cached[d] = from_float<T>(to_float(row[latent_offset + d]) * inv * weight[d]);
-  // the rot parts: the shared key part is vector ``heads`` and goes into the cache row, the queries' parts are vectors 0 .. heads - 1
-  // and go behind the ``rank`` columns of their head in ``queries``; a thread per pair of columns
+  if (page >= 0)
+    for (int i = threadIdx.x; i < kv_heads * value_dim; i += blockDim.x) {
+      const int head = i / value_dim, d = i - head * value_dim;
+      v_pages[(size_t)page * v_page_stride + ((size_t)head * page_size + slot) * value_dim + d] = from_float<T>(to_float(row[v_offset + i]) + (v_bias != nullptr ? v_bias[i] : 0.0f));
+    }
+  __syncthreads();
+  for (int h = warp; h < heads + kv_heads; h += warps) {
+    const bool is_key = h >= heads;
+    const int head = is_key ? h - heads : h;
+    T* src = row + (is_key ? k_offset : 0) + (size_t)head * key_dim;
+    T* dst = !is_key ? src : (page >= 0 ? k_pages + (size_t)page * k_page_stride + ((size_t)head * page_size + slot) * key_dim : nullptr);
+    const float* bias = is_key ? k_bias : q_bias;
+    const float* weight = is_key ? k_weight : q_weight;
+    float squares = 0.0f;
+    for (int d = lane; d < key_dim; d += 32) {
+      const float v = to_float(src[d]) + (bias != nullptr ? bias[head * key_dim + d] : 0.0f);
+      vec[d] = v;
+      squares += v * v;
+    }
+    const float inv = weight != nullptr ? 1.0f / sqrtf(warp_sum(squares) / (float)key_dim + eps) : 1.0f;
+    const float factor = (!is_key && q_factors != nullptr) ? q_factors[head] : 1.0f;
+    __syncwarp();
+    if (dst != nullptr)
+      for (int d = lane; d < key_dim; d += 32) {
+        float v = vec[d] * inv * (weight != nullptr ? weight[d] : 1.0f);
+        if (d < rot_dims) {
+          const int pair = interleaved ? d >> 1 : (d < half ? d : d - half);
+          const bool first = interleaved ? (d & 1) == 0 : d < half;
+          const int other = interleaved ? d ^ 1 : (first ? d + half : d - half);
+          const float u = vec[other] * inv * (weight != nullptr ? weight[other] : 1.0f);
+          v = first ? v * turn_s[pair] - u * turn_s[half + pair] : v * turn_s[pair] + u * turn_s[half + pair];
+        }
+        dst[d] = from_float<T>(v * factor);
+      }
+    __syncwarp();   // the next vector of this warp takes the same place
+  }
+}
+
+// Latent attention's norms, rotation and cache write, in up to three parts that a launch may hold or leave out:
+//   ``down_rows``    a row holds, from ``latent_offset``, the down projection [rank | rot].  The first ``rank`` columns are normalised (RMS,
+//                    weight) into the latent; the last ``rot`` are a key part that all heads share and that is rotated.  [latent |
+//                    rotated part] goes into the token's cache row.
+//   ``q_latent``     the q_rank columns from ``q_latent_offset`` of the same row, normalised the same way: what the queries are expanded from.
+//   ``query_rows``   ``heads`` queries of [plain | rot]; their rotated rot parts go into ``queries`` [T, heads, rank + rot] behind the ``rank``
+//                    columns that the product with the keys' expansion fills.
+// The first ``rot_dims`` columns of a rot part turn by position * inv_freq[i] (32-bit angles; cosines and sines times ``amplitude``), columns
+// (2i, 2i + 1) together if ``interleaved``, else column i with column i + rot_dims / 2.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__ down_rows, int down_stride, int latent_offset, const float* __restrict__ weight, float eps,
+                                                           const float* __restrict__ inv_freq, int rot_dims, int interleaved, float amplitude,
+                                                           const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ block_table,
+                                                           int table_stride, T* __restrict__ pages, long long page_stride, int heads, int plain, int rot, int rank,
+                                                           int page_size, int write_cache, const T* __restrict__ query_rows, int query_stride, T* __restrict__ queries,
+                                                           const float* __restrict__ q_latent_weight, int q_latent_offset, int q_rank, T* __restrict__ q_latent) {
+  __shared__ float scratch[32];
+  extern __shared__ float turn_s[];   // the token's cosines [rot_dims / 2], then its sines
+  const int t = blockIdx.x;
+  const int pos = positions[t];
+  const int half = rot_dims / 2;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sine, cosine;
+    sincosf((float)pos * inv_freq[i], &sine, &cosine);
+    turn_s[i] = cosine * amplitude;
+    turn_s[half + i] = sine * amplitude;
+  }
+  T* cached = nullptr;
+  const T* down = nullptr;
+  if (down_rows != nullptr) {
+    const int page = write_cache ? block_table[(size_t)token_seq[t] * table_stride + pos / page_size] : -1;
+    cached = page >= 0 ? pages + (size_t)page * page_stride + (size_t)(pos % page_size) * (rank + rot) : nullptr;
+    const T* row = down_rows + (size_t)t * down_stride;
+    down = row + latent_offset;
+    float squares = 0.0f;
+    for (int d = threadIdx.x; d < rank; d += blockDim.x) {
+      const float v = to_float(down[d]);
+      squares += v * v;
+    }
+    const float inv = rsqrtf(block_sum(squares, scratch) / (float)rank + eps);
+    if (cached)
+      for (int d = threadIdx.x; d < rank; d += blockDim.x) cached[d] = from_float<T>(to_float(down[d]) * inv * weight[d]);
+    if (q_latent != nullptr) {
+      const T* src = row + q_latent_offset;
+      T* dst = q_latent + (size_t)t * q_rank;
+      float q_squares = 0.0f;
+      for (int d = threadIdx.x; d < q_rank; d += blockDim.x) {
+        const float v = to_float(src[d]);
+        q_squares += v * v;
+      }
+      const float q_inv = rsqrtf(block_sum(q_squares, scratch) / (float)q_rank + eps);
+      for (int d = threadIdx.x; d < q_rank; d += blockDim.x) dst[d] = from_float<T>(to_float(src[d]) * q_inv * q_latent_weight[d]);
+    }
+  }
+  __syncthreads();   // the cosines and sines are in place
+  // the rot parts: a thread per pair of columns; vector ``heads`` is the shared key part
   const int pairs = rot / 2;
-  T* query_row = queries + (size_t)t * heads * (rank + rot);
-  for (int i = threadIdx.x; i < (heads + 1) * pairs; i += blockDim.x) {
-    const int vector = i / pairs, pair = i - vector * pairs;
-    const T* at = vector < heads ? row + vector * (plain + rot) + plain : row + latent_offset + rank;
-    T* to = vector < heads ? query_row + vector * (rank + rot) + rank : (cached ? cached + rank : nullptr);
-    if (!to) continue;
-    if (2 * pair + 1 < rot_dims) {
-      float sine, cosine;
-      sincosf((float)pos * inv_freq[pair], &sine, &cosine);
-      const float a = to_float(at[2 * pair]), b = to_float(at[2 * pair + 1]);
-      to[2 * pair] = from_float<T>(a * cosine - b * sine);
-      to[2 * pair + 1] = from_float<T>(b * cosine + a * sine);
+  const int first_vector = query_rows != nullptr ? 0 : heads, end_vector = cached != nullptr ? heads + 1 : heads;
+  const T* query_row = query_rows + (size_t)t * query_stride;
+  T* to_row = queries + (size_t)t * heads * (rank + rot);
+  for (int i = threadIdx.x; i < (end_vector - first_vector) * pairs; i += blockDim.x) {
+    const int vector = first_vector + i / pairs, pair = i % pairs;
+    const T* at = vector < heads ? query_row + vector * (plain + rot) + plain : down + rank;
+    T* to = vector < heads ? to_row + vector * (rank + rot) + rank : cached + rank;
+    if (pair < half) {
+      const int a_at = interleaved ? 2 * pair : pair, b_at = interleaved ? 2 * pair + 1 : pair + half;
+      const float cosine = turn_s[pair], sine = turn_s[half + pair];
+      const float a = to_float(at[a_at]), b = to_float(at[b_at]);
+      to[a_at] = from_float<T>(a * cosine - b * sine);
+      to[b_at] = from_float<T>(b * cosine + a * sine);
     } else {   // columns that do not rotate
       to[2 * pair] = at[2 * pair];
       to[2 * pair + 1] = at[2 * pair + 1];
@@ -305,7 +405,7 @@ __global__ void __launch_bounds__(kMixThreads) mixed_heads_attention_kernel(
     const T* __restrict__ v_pages, long long v_page_stride, const int* __restrict__ positions, const int* __restrict__ token_seq,
     const int* __restrict__ block_table, int table_stride, const float* __restrict__ slopes, const float* __restrict__ mix, T* __restrict__ out,
     int heads, int kv_heads, int key_dim, int value_dim, int page_size, int window, float scale, float* __restrict__ partial, int staged,
-    int keep_first, int gate_per_head, const float* __restrict__ sinks, int v_row_stride) {
+    int keep_first, int gate_per_head, const float* __restrict__ sinks, int v_row_stride, float softcap, int sigmoid, const float* __restrict__ shifts) {
   extern __shared__ __align__(16) unsigned char smem_bytes[];
   long long* k_at = reinterpret_cast<long long*>(smem_bytes);   // [32] where a key's row starts in its plane (head 0)
   long long* v_at = k_at + kMixKeys;
@@ -335,8 +435,9 @@ __global__ void __launch_bounds__(kMixThreads) mixed_heads_attention_kernel(
   if (mix)
     for (int i = tid; i < heads * heads; i += kMixThreads) mix_s[i] = mix[i];
   for (int i = tid; i < heads; i += kMixThreads) {
-    max_s[i] = -INFINITY;
-    sum_s[i] = 0.0f;
+    // sigmoid weights have no maximum and no denominator: every part's maximum is 0, and the parts' totals add up to 1
+    max_s[i] = sigmoid ? 0.0f : -INFINITY;
+    sum_s[i] = sigmoid && blockIdx.y == 0 ? 1.0f : 0.0f;
   }
 
   float acc[ACC];
@@ -408,6 +509,12 @@ __global__ void __launch_bounds__(kMixThreads) mixed_heads_attention_kernel(
         score = (part[0] + part[1]) + (part[2] + part[3]);
       } else {
         score = raw_s[h * kMixKeys + lane];
+      }
+      if (softcap > 0.0f) score = softcap * tanhf(score / softcap);
+      if (sigmoid) {
+        p_s[h * kMixKeys + lane] = lane < count ? 1.0f / (1.0f + expf(-(score + (shifts != nullptr ? shifts[h] : 0.0f)))) : 0.0f;
+        if (lane == 0) rescale_s[h] = 1.0f;
+        continue;
       }
       if (lane >= count) score = -INFINITY;
       const float before = max_s[h];
@@ -543,7 +650,7 @@ static int launch_mixed(const void* rows, int row_stride, int gate_offset, const
                         long long v_page_stride, const int* positions, const int* token_seq, const int* block_table, int table_stride,
                         const float* slopes, const float* mix, void* out, int tokens, int heads, int kv_heads, int key_dim, int value_dim,
                         int page_size, int window, float scale, size_t smem, int splits, float* partial, int keep_first, int gate_per_head,
-                        const float* sinks, int v_row_stride, cudaStream_t stream) {
+                        const float* sinks, int v_row_stride, float softcap, int sigmoid, const float* shifts, cudaStream_t stream) {
   auto kernel = mixed_heads_attention_kernel<T, ACC>;
   // room for a tile's keys and values of every key/value head behind the 32-bit part; without it rows are read from global memory
   const size_t tiles = (size_t)kv_heads * kMixKeys * ((size_t)staged_key_stride<T>(key_dim) + value_dim) * sizeof(T);
@@ -557,7 +664,7 @@ static int launch_mixed(const void* rows, int row_stride, int gate_offset, const
   kernel<<<dim3(tokens, splits), kMixThreads, smem, stream>>>((const T*)rows, row_stride, gate_offset, (const T*)k_pages, k_page_stride, (const T*)v_pages,
                                                               v_page_stride, positions, token_seq, block_table, table_stride, slopes, mix, (T*)out, heads,
                                                               kv_heads, key_dim, value_dim, page_size, window, scale, partial, staged, keep_first, gate_per_head,
-                                                              sinks, v_row_stride);
+                                                              sinks, v_row_stride, softcap, sigmoid, shifts);
   if (splits > 1)
     merge_mixed_kernel<T><<<dim3(tokens, heads), value_dim >= 128 ? 128 : (value_dim > 32 ? 64 : 32), 0, stream>>>(partial, (const T*)rows, row_stride, gate_offset,
                                                                                                                   (T*)out, heads, value_dim, splits, gate_per_head, sinks);
@@ -610,8 +717,9 @@ TLIE_EXPORT int tlie_mixed_heads_attention(int dtype, const void* rows, int row_
                                            const int* token_seq, const int* block_table, int table_stride, const float* slopes, const float* mix,
                                            void* out, int tokens, int heads, int kv_heads, int key_dim, int value_dim, int page_size, int window,
                                            float scale, int splits, float* partial, int keep_first, int gate_per_head, const float* sinks,
-                                           int v_row_stride, cudaStream_t stream) {
+                                           int v_row_stride, float softcap, int sigmoid, const float* shifts, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (sigmoid && sinks != nullptr) return (int)cudaErrorInvalidValue;
   if (keep_first < 0 || v_row_stride < value_dim) return (int)cudaErrorInvalidValue;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || key_dim <= 0 || value_dim <= 0 || splits < 1 || splits > 64 || (splits > 1 && partial == nullptr))
     return (int)cudaErrorInvalidValue;
@@ -623,7 +731,7 @@ TLIE_EXPORT int tlie_mixed_heads_attention(int dtype, const void* rows, int row_
 #define TLIE_MIXED(T, ACC)                                                                                                                    \
   return launch_mixed<T, ACC>(rows, row_stride, gate_offset, k_pages, k_page_stride, v_pages, v_page_stride, positions, token_seq, block_table, \
                               table_stride, slopes, mix, out, tokens, heads, kv_heads, key_dim, value_dim, page_size, window, scale, smem, splits, partial, \
-                              keep_first, gate_per_head, sinks, v_row_stride, stream)
+                              keep_first, gate_per_head, sinks, v_row_stride, softcap, sigmoid, shifts, stream)
   if (dtype == TLIE_F32) {
     if (outputs <= 4 * kMixThreads) TLIE_MIXED(float, 4);
     if (outputs <= 8 * kMixThreads) TLIE_MIXED(float, 8);
@@ -654,18 +762,48 @@ TLIE_EXPORT int tlie_normed_store(int dtype, void* rows, int row_stride, int k_o
   return (int)cudaGetLastError();
 }
 
-TLIE_EXPORT int tlie_latent_store(int dtype, const void* rows, int row_stride, int latent_offset, const float* weight, float eps, const float* inv_freq, int rot_dims,
-                                  const int* positions, const int* token_seq, const int* block_table, int table_stride, void* pages, long long page_stride,
-                                  int tokens, int heads, int plain, int rot, int rank, int page_size, int write_cache, void* queries, cudaStream_t stream) {
+// ``q_weight`` / ``k_weight`` null: no norm.  See norm_rotary_store_kernel.
+TLIE_EXPORT int tlie_norm_rotary_store(int dtype, void* rows, int row_stride, int k_offset, int v_offset, const float* q_bias, const float* k_bias, const float* v_bias,
+                                       const float* q_weight, const float* k_weight, float eps, const float* q_factors, const float* inv_freq, int rot_dims,
+                                       int interleaved, float amplitude, const int* positions, const int* token_seq, const int* block_table, int table_stride,
+                                       void* k_pages, long long k_page_stride, void* v_pages, long long v_page_stride, int tokens, int heads, int kv_heads, int key_dim,
+                                       int value_dim, int page_size, int write_cache, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (rot_dims < 0 || rot_dims > rot || (rot_dims & 1) || (rot & 1)) return (int)cudaErrorInvalidValue;
+  constexpr int kThreads = 256;
+  const size_t smem = ((size_t)rot_dims + (size_t)(kThreads / 32) * key_dim) * sizeof(float);
+  if (rot_dims < 0 || rot_dims % 2 || rot_dims > key_dim || key_dim <= 0 || smem > 48 * 1024 || (rot_dims > 0 && inv_freq == nullptr)) return (int)cudaErrorInvalidValue;
+#define TLIE_STORE(T)                                                                                                                                              \
+  norm_rotary_store_kernel<T><<<tokens, kThreads, smem, stream>>>((T*)rows, row_stride, k_offset, v_offset, q_bias, k_bias, v_bias, q_weight, k_weight, eps, q_factors, \
+                                                                  inv_freq, rot_dims, interleaved, amplitude, positions, token_seq, block_table, table_stride,     \
+                                                                  (T*)k_pages, k_page_stride, (T*)v_pages, v_page_stride, heads, kv_heads, key_dim, value_dim,       \
+                                                                  page_size, write_cache)
   if (dtype == TLIE_F32)
-    latent_store_kernel<float><<<tokens, 128, 0, stream>>>((const float*)rows, row_stride, latent_offset, weight, eps, inv_freq, rot_dims, positions, token_seq, block_table,
-                                                           table_stride, (float*)pages, page_stride, heads, plain, rot, rank, page_size, write_cache, (float*)queries);
+    TLIE_STORE(float);
   else
-    latent_store_kernel<__nv_bfloat16><<<tokens, 128, 0, stream>>>((const __nv_bfloat16*)rows, row_stride, latent_offset, weight, eps, inv_freq, rot_dims, positions, token_seq,
-                                                                   block_table, table_stride, (__nv_bfloat16*)pages, page_stride, heads, plain, rot, rank, page_size,
-                                                                   write_cache, (__nv_bfloat16*)queries);
+    TLIE_STORE(__nv_bfloat16);
+#undef TLIE_STORE
+  return (int)cudaGetLastError();
+}
+
+// ``down_rows``, ``query_rows`` and ``q_latent`` may each be null: that part is left out (``q_latent`` is read from the down rows, so it needs them).
+TLIE_EXPORT int tlie_latent_store(int dtype, const void* down_rows, int down_stride, int latent_offset, const float* weight, float eps, const float* inv_freq, int rot_dims,
+                                  int interleaved, float amplitude, const int* positions, const int* token_seq, const int* block_table, int table_stride, void* pages,
+                                  long long page_stride, int tokens, int heads, int plain, int rot, int rank, int page_size, int write_cache, const void* query_rows,
+                                  int query_stride, void* queries, const float* q_latent_weight, int q_latent_offset, int q_rank, void* q_latent, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (rot_dims < 0 || rot_dims > rot || (rot_dims & 1) || (rot & 1) || rot_dims > 8192) return (int)cudaErrorInvalidValue;
+  if ((q_latent != nullptr && (down_rows == nullptr || q_latent_weight == nullptr || q_rank <= 0)) || (query_rows != nullptr && queries == nullptr)) return (int)cudaErrorInvalidValue;
+  const size_t smem = (size_t)rot_dims * sizeof(float);
+#define TLIE_LATENT(T)                                                                                                                                             \
+  latent_store_kernel<T><<<tokens, 128, smem, stream>>>((const T*)down_rows, down_stride, latent_offset, weight, eps, inv_freq, rot_dims, interleaved, amplitude,     \
+                                                        positions, token_seq, block_table, table_stride, (T*)pages, page_stride, heads, plain, rot, rank, page_size, \
+                                                        write_cache, (const T*)query_rows, query_stride, (T*)queries, q_latent_weight, q_latent_offset, q_rank,     \
+                                                        (T*)q_latent)
+  if (dtype == TLIE_F32)
+    TLIE_LATENT(float);
+  else
+    TLIE_LATENT(__nv_bfloat16);
+#undef TLIE_LATENT
   return (int)cudaGetLastError();
 }
 

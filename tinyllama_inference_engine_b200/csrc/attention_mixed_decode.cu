@@ -10,6 +10,9 @@
 //   out  [16 heads x VALUE_DIM] += P_c [16 x 32] . V_c [32 x VALUE_DIM]
 // accumulates in registers across the tiles.  Nothing of the scores is rounded before the softmax.
 //
+// ``softcap`` and sigmoid weights (``sigmoid``, ``shifts``) as in the general kernel; a part's maximum is then 0 and the parts' totals add up to 1,
+// so that the merge is the same.
+//
 // Compile-time: KEY_DIM, VALUE_DIM (multiples of 16), KV_HEADS.  Heads per key/value head: at most 16.
 #include "common.cuh"
 #include "mma_utils.cuh"
@@ -54,7 +57,7 @@ __global__ void __launch_bounds__(kThreads)
                         long long k_page_stride, const __nv_bfloat16* __restrict__ v_pages, long long v_page_stride, const int* __restrict__ positions,
                         const int* __restrict__ token_seq, const int* __restrict__ block_table, int table_stride, const float* __restrict__ slopes,
                         const float* __restrict__ mix, __nv_bfloat16* __restrict__ out, int heads, int page_size, int window, float scale,
-                        float* __restrict__ partial, int keep_first, int gate_per_head) {
+                        float* __restrict__ partial, int keep_first, int gate_per_head, float softcap, int sigmoid, const float* __restrict__ shifts) {
   extern __shared__ __align__(16) unsigned char smem[];
   const DecodeSmem at(heads, mix != nullptr);
   long long* k_at = reinterpret_cast<long long*>(smem + at.rows);
@@ -90,8 +93,8 @@ __global__ void __launch_bounds__(kThreads)
   if (mix)
     for (int i = tid; i < heads * heads; i += kThreads) mix_s[i] = mix[i];
   for (int i = tid; i < heads; i += kThreads) {
-    max_s[i] = -INFINITY;
-    sum_s[i] = 0.0f;
+    max_s[i] = sigmoid ? 0.0f : -INFINITY;
+    sum_s[i] = sigmoid && blockIdx.y == 0 ? 1.0f : 0.0f;
   }
 
   float o[kGroupsPerWarp][kVD / 8][4];
@@ -191,6 +194,13 @@ __global__ void __launch_bounds__(kThreads)
         score = (part[0] + part[1]) + (part[2] + part[3]);
       } else {
         score = raw_s[h * kKeys + lane];
+      }
+      if (softcap > 0.0f) score = softcap * tanhf(score / softcap);
+      if (sigmoid) {
+        const float p = lane < count ? 1.0f / (1.0f + expf(-(score + (shifts != nullptr ? shifts[h] : 0.0f)))) : 0.0f;
+        p_s[(size_t)((h / group) * 16 + h % group) * kPRow + lane] = __float2bfloat16_rn(p);
+        if (lane == 0) shrink_s[h] = 1.0f;
+        continue;
       }
       if (lane >= count) score = -INFINITY;
       const float before = max_s[h];
@@ -334,7 +344,7 @@ TLIE_EXPORT long long tlie_mixed_decode_smem_bytes(int heads, int mixed) { retur
 TLIE_EXPORT int tlie_mixed_decode(const void* rows, int row_stride, int gate_offset, const void* k_pages, long long k_page_stride, const void* v_pages,
                                   long long v_page_stride, const int* positions, const int* token_seq, const int* block_table, int table_stride,
                                   const float* slopes, const float* mix, void* out, int tokens, int heads, int page_size, int window, float scale, int splits,
-                                  float* partial, int keep_first, int gate_per_head, cudaStream_t stream) {
+                                  float* partial, int keep_first, int gate_per_head, float softcap, int sigmoid, const float* shifts, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (keep_first < 0) return (int)cudaErrorInvalidValue;
   if (heads <= 0 || heads % kG != 0 || heads / kG > 16 || row_stride % 8 != 0 || (gate_offset >= 0 && !gate_per_head && gate_offset % 2 != 0) || splits < 1 || splits > 64 ||
@@ -349,7 +359,7 @@ TLIE_EXPORT int tlie_mixed_decode(const void* rows, int row_stride, int gate_off
   mixed_decode_kernel<<<dim3(tokens, splits), kThreads, smem, stream>>>((const __nv_bfloat16*)rows, row_stride, gate_offset, (const __nv_bfloat16*)k_pages,
                                                                        k_page_stride, (const __nv_bfloat16*)v_pages, v_page_stride, positions, token_seq,
                                                                        block_table, table_stride, slopes, mix, (__nv_bfloat16*)out, heads, page_size, window,
-                                                                       scale, partial, window > 0 ? keep_first : 0, gate_per_head);
+                                                                       scale, partial, window > 0 ? keep_first : 0, gate_per_head, softcap, sigmoid, shifts);
   if (splits > 1)
     merge_mixed_decode_kernel<<<dim3(tokens, heads), kVD >= 128 ? 128 : (kVD > 32 ? 64 : 32), 0, stream>>>(partial, (const __nv_bfloat16*)rows, row_stride,
                                                                                                         gate_offset, (__nv_bfloat16*)out, heads, splits, gate_per_head);

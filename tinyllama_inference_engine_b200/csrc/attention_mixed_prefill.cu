@@ -13,7 +13,10 @@
 // 64-key tiles (cp.async, a ring of chunks); Q'.K^T and P.V on mma.sync m16n8k16 with 32-bit accumulators, the
 // distance bias, the mask, the running maximum and sum in 32-bit; the output gate in the epilogue.
 //
-// Compile-time: KEY_DIM, VALUE_DIM (multiples of 16), PARTS (key heads per folded query).
+// SIGMOID_WEIGHTS 1: no softmax; the score is bounded, softcap * tanh(score / softcap), and a key's weight is sigmoid(score + shift_h), not brought
+// to a sum of one.  Nothing is rescaled then.  tanh and sigmoid are written with e^x and a reciprocal, in 32-bit.
+//
+// Compile-time: KEY_DIM, VALUE_DIM (multiples of 16), PARTS (key heads per folded query), SIGMOID_WEIGHTS.
 #include "common.cuh"
 #include "mma_utils.cuh"
 
@@ -25,6 +28,9 @@
 #endif
 #ifndef PARTS
 #define PARTS 1
+#endif
+#ifndef SIGMOID_WEIGHTS
+#define SIGMOID_WEIGHTS 0
 #endif
 
 namespace tlie {
@@ -132,11 +138,12 @@ __device__ __forceinline__ void load_plane(__nv_bfloat16* smem, const __nv_bfloa
 constexpr int kMinBlocks = (kRows > 0 && 2 * smem_for(kRows > 0 ? kRows : 16, kPartsPerChunk) <= kSmemLimit && kVD <= 64) ? 2 : 1;
 
 __global__ void __launch_bounds__(kThreads, kMinBlocks)
-    mixed_prefill_kernel(const __nv_bfloat16* __restrict__ folded, const __nv_bfloat16* __restrict__ rows, int row_stride, int gate_offset,
+    mixed_prefill_kernel(const __nv_bfloat16* __restrict__ folded, long long folded_stride, const __nv_bfloat16* __restrict__ rows, int row_stride, int gate_offset,
                          const __nv_bfloat16* __restrict__ k_pages, long long k_page_stride, const __nv_bfloat16* __restrict__ v_pages,
                          long long v_page_stride, const int* __restrict__ seq_starts, const int* __restrict__ first_positions,
                          const int* __restrict__ block_table, int table_stride, const float* __restrict__ slopes, __nv_bfloat16* __restrict__ out,
-                         int heads, int kv_heads, int page_size, int window, int mixed, int keep_first, int gate_per_head) {
+                         int heads, int kv_heads, int page_size, int window, int mixed, int keep_first, int gate_per_head, float softcap,
+                         const float* __restrict__ shifts) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __nv_bfloat16* q_smem = reinterpret_cast<__nv_bfloat16*>(smem_raw);            // [kRows][kQRow]
   __nv_bfloat16* k_ring = q_smem + (size_t)kRows * kQRow;                        // [kRing][kPartsPerChunk][64][kKRow]
@@ -162,7 +169,7 @@ __global__ void __launch_bounds__(kThreads, kMinBlocks)
   for (int idx = threadIdx.x; idx < kRows * kQChunks; idx += kThreads) {
     const int row = idx / kQChunks, chunk = idx - row * kQChunks;
     const bool valid = row < rows_here;
-    const __nv_bfloat16* src = folded + ((size_t)(row0 + (valid ? row : 0)) * heads + head) * (kParts * kD) + chunk * 8;
+    const __nv_bfloat16* src = folded + (size_t)(row0 + (valid ? row : 0)) * folded_stride + (size_t)head * (kParts * kD) + chunk * 8;
     cp_async_16(q_smem + (size_t)row * kQRow + chunk * 8, src, valid);
   }
 
@@ -201,8 +208,23 @@ __global__ void __launch_bounds__(kThreads, kMinBlocks)
   float o[kVD / 8][4];
 #pragma unroll
   for (int i = 0; i < kVD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+#if SIGMOID_WEIGHTS
+  // tanh(s / c) = 1 - 2 / (1 + e^(2 s / c)); sigmoid(z) = 1 / (1 + e^-z)
+  const float shift = (shifts != nullptr ? shifts[head] : 0.0f) * kLog2e;
+  const float to_exp = 2.0f * kLog2e / (softcap > 0.0f ? softcap : 1.0f), capped = softcap * kLog2e;
+  const int my_lo_max = my_lo[1];
+  auto bounded_sigmoid = [&](float s) {
+    float minus;   // -(score + shift) in units of log2
+    if (softcap > 0.0f)
+      minus = fmaf(2.0f * capped, __fdividef(1.0f, 1.0f + exp2_approx(s * to_exp)), -capped - shift);
+    else
+      minus = fmaf(s, -kLog2e, -shift);
+    return __fdividef(1.0f, 1.0f + exp2_approx(minus));
+  };
+#else
   float row_max[2] = {-INFINITY, -INFINITY};
   float row_sum[2] = {0.0f, 0.0f};
+#endif
 
   float s_frag[kKeys / 8][4];
   for (int c = 0; c < chunks; ++c) {
@@ -240,6 +262,25 @@ __global__ void __launch_bounds__(kThreads, kMinBlocks)
         }
       }
     }
+#if SIGMOID_WEIGHTS
+    if (first_part + kPartsPerChunk == kParts && tile_seen) {
+      unsigned pa[kKeys / 16][4];
+      const bool diagonal = key0 + kKeys > warp_first_pos + 1 || (window > 0 && key0 < my_lo_max);   // some key of the tile may be hidden from some row
+#pragma unroll
+      for (int j = 0; j < kKeys / 8; ++j) {
+        float w[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          w[e] = bounded_sigmoid(s_frag[j][e]);
+          if (diagonal) {
+            const int key = key0 + j * 8 + 2 * t + (e & 1);
+            if (!((key >= my_lo[e >> 1] || key < keep) && key <= my_pos[e >> 1])) w[e] = 0.0f;
+          }
+        }
+        pa[j >> 1][(j & 1) * 2 + 0] = pack_bf16(w[0], w[1]);
+        pa[j >> 1][(j & 1) * 2 + 1] = pack_bf16(w[2], w[3]);
+      }
+#else
     if (first_part + kPartsPerChunk == kParts && tile_seen) {
       // scores in units of log2: (dot - slope (i - j)) log2 e; keys outside a row's window or after it are masked
       float tile_max[2] = {-INFINITY, -INFINITY};
@@ -284,6 +325,7 @@ __global__ void __launch_bounds__(kThreads, kMinBlocks)
         o[i][2] *= rescale[1];
         o[i][3] *= rescale[1];
       }
+#endif
 #pragma unroll
       for (int kk = 0; kk < kKeys / 16; ++kk) {
 #pragma unroll
@@ -300,15 +342,21 @@ __global__ void __launch_bounds__(kThreads, kMinBlocks)
     __syncthreads();   // everyone is done with this chunk before the ring comes round to its buffer
   }
   cp_async_wait<0>();
+#if !SIGMOID_WEIGHTS
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     row_sum[r] += __shfl_xor_sync(0xffffffffu, row_sum[r], 1);
     row_sum[r] += __shfl_xor_sync(0xffffffffu, row_sum[r], 2);
   }
+#endif
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     if (my_row[r] >= rows_here) continue;
+#if SIGMOID_WEIGHTS
+    const float inv = 1.0f;
+#else
     const float inv = 1.0f / row_sum[r];
+#endif
     const size_t row = (size_t)(row0 + my_row[r]);
     __nv_bfloat16* dst = out + (row * heads + head) * kVD + 2 * t;
     const __nv_bfloat16* gate = (gate_offset >= 0 && !gate_per_head) ? rows + row * row_stride + gate_offset + (size_t)head * kVD + 2 * t : nullptr;
@@ -334,27 +382,34 @@ TLIE_EXPORT int tlie_mixed_prefill_tile_rows() { return kRows; }
 TLIE_EXPORT int tlie_mixed_prefill_folded_width() { return kParts * kD; }
 
 // ``folded``: scratch for the folded queries, bfloat16 [tokens, heads, PARTS * KEY_DIM].  ``slopes``: the folded slopes (or null).
+// ``folded`` null: the queries are taken from ``rows`` as they are (no mix, the scale already in them).
+// ``softcap`` and ``shifts`` (or null): SIGMOID_WEIGHTS only.
 // ``mix`` null: PARTS must be 1.  ``longest``: the most rows any entry of the step has.
 TLIE_EXPORT int tlie_mixed_prefill(const void* rows, int row_stride, int gate_offset, const float* mix, float scale, void* folded, const void* k_pages,
                                    long long k_page_stride, const void* v_pages, long long v_page_stride, const int* seq_starts,
                                    const int* first_positions, const int* block_table, int table_stride, const float* slopes, void* out, int tokens,
                                    int entries, int longest, int heads, int kv_heads, int page_size, int window, int keep_first, int gate_per_head,
-                                   cudaStream_t stream) {
+                                   float softcap, const float* shifts, cudaStream_t stream) {
   if (tokens <= 0 || entries <= 0) return 0;
   if (keep_first < 0) return (int)cudaErrorInvalidValue;
   if (kRows == 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || page_size % 16 != 0 || heads > 65535 || entries > 65535 ||
       (mix != nullptr ? kParts != kv_heads : kParts != 1) || row_stride % 8 != 0 || (gate_offset >= 0 && !gate_per_head && gate_offset % 2 != 0))
     return (int)cudaErrorInvalidValue;
+  if (!SIGMOID_WEIGHTS && (softcap > 0.0f || shifts != nullptr)) return (int)cudaErrorInvalidValue;
+  if (folded == nullptr && mix != nullptr) return (int)cudaErrorInvalidValue;
   const size_t fold_smem = ((size_t)heads * kD + (mix != nullptr ? (size_t)heads * heads : 0)) * sizeof(float);
   if (fold_smem > 200 * 1024) return (int)cudaErrorInvalidValue;
   cudaError_t e = cudaSuccess;
-  if (fold_smem > 48 * 1024) {
+  if (folded != nullptr && fold_smem > 48 * 1024) {
     e = cudaFuncSetAttribute(fold_queries_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)fold_smem);
     if (e != cudaSuccess) return (int)e;
   }
-  fold_queries_kernel<<<tokens, 256, fold_smem, stream>>>((const __nv_bfloat16*)rows, row_stride, mix, scale, (__nv_bfloat16*)folded, heads, heads / kv_heads);
-  e = cudaGetLastError();
-  if (e != cudaSuccess) return (int)e;
+  if (folded != nullptr) {
+    fold_queries_kernel<<<tokens, 256, fold_smem, stream>>>((const __nv_bfloat16*)rows, row_stride, mix, scale, (__nv_bfloat16*)folded, heads, heads / kv_heads);
+    e = cudaGetLastError();
+    if (e != cudaSuccess) return (int)e;
+  }
+  const long long folded_stride = folded != nullptr ? (long long)heads * kParts * kD : row_stride;
   constexpr size_t smem = smem_for(kRows > 0 ? kRows : 16, kPartsPerChunk);
   static bool configured = false;
   if (!configured) {
@@ -364,9 +419,9 @@ TLIE_EXPORT int tlie_mixed_prefill(const void* rows, int row_stride, int gate_of
   }
   const int tile_rows = kRows > 0 ? kRows : 16;
   const dim3 grid((longest + tile_rows - 1) / tile_rows, entries, heads);
-  mixed_prefill_kernel<<<grid, kThreads, smem, stream>>>((const __nv_bfloat16*)folded, (const __nv_bfloat16*)rows, row_stride, gate_offset,
+  mixed_prefill_kernel<<<grid, kThreads, smem, stream>>>((const __nv_bfloat16*)(folded != nullptr ? folded : rows), folded_stride, (const __nv_bfloat16*)rows, row_stride, gate_offset,
                                                          (const __nv_bfloat16*)k_pages, k_page_stride, (const __nv_bfloat16*)v_pages, v_page_stride,
                                                          seq_starts, first_positions, block_table, table_stride, slopes, (__nv_bfloat16*)out, heads,
-                                                         kv_heads, page_size, window, mix != nullptr ? 1 : 0, keep_first, gate_per_head);
+                                                         kv_heads, page_size, window, mix != nullptr ? 1 : 0, keep_first, gate_per_head, softcap, shifts);
   return (int)cudaGetLastError();
 }

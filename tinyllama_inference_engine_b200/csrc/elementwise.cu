@@ -265,27 +265,29 @@ __global__ void embedding_positions_kernel(const T* __restrict__ table, const T*
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = (dst[i] * inv) * norm_weight[i];   // every thread rereads what it wrote itself
 }
 
-// out[i] = act(in[i]), 32-bit inside: 0 the square of relu, 1 gelu in its tanh form, 2 silu.  In place is fine.
-__device__ __forceinline__ float activate(int kind, float z) {
+// out[i] = act(in[i]), 32-bit inside: 0 the square of relu, 1 gelu in its tanh form, 2 silu, 3 a z^2 + z / 2 above zero and
+// b (e^z - 1 - z) + z / 2 below (xIELU; the other kinds take no constants).  In place is fine.
+__device__ __forceinline__ float activate(int kind, float z, float a, float b) {
   if (kind == 0) {
     const float r = fmaxf(z, 0.0f);
     return r * r;
   }
   if (kind == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  if (kind == 3) return z > 0.0f ? a * z * z + 0.5f * z : b * (expm1f(z) - z) + 0.5f * z;
   return z / (1.0f + expf(-z));
 }
 
 template <typename T>
-__global__ void activation_kernel(const T* __restrict__ in, T* __restrict__ out, int kind, size_t count) {
+__global__ void activation_kernel(const T* __restrict__ in, T* __restrict__ out, int kind, float a, float b, size_t count) {
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < count; i += (size_t)gridDim.x * blockDim.x)
-    out[i] = from_float<T>(activate(kind, to_float(in[i])));
+    out[i] = from_float<T>(activate(kind, to_float(in[i]), a, b));
 }
 
 template <typename T>
-__global__ void activation_vec_kernel(const T* __restrict__ in, T* __restrict__ out, int kind, size_t count4) {
+__global__ void activation_vec_kernel(const T* __restrict__ in, T* __restrict__ out, int kind, float a, float b, size_t count4) {
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < count4; i += (size_t)gridDim.x * blockDim.x) {
     const float4 v = Vec4<T>::load(in + i * 4);
-    Vec4<T>::store(out + i * 4, make_float4(activate(kind, v.x), activate(kind, v.y), activate(kind, v.z), activate(kind, v.w)));
+    Vec4<T>::store(out + i * 4, make_float4(activate(kind, v.x, a, b), activate(kind, v.y, a, b), activate(kind, v.z, a, b), activate(kind, v.w, a, b)));
   }
 }
 
@@ -393,20 +395,20 @@ TLIE_EXPORT int tlie_embedding_positions(int dtype, const void* table, const voi
   return (int)cudaGetLastError();
 }
 
-TLIE_EXPORT int tlie_activation(int dtype, int kind, const void* in, void* out, long long count, cudaStream_t stream) {
+TLIE_EXPORT int tlie_activation(int dtype, int kind, const void* in, void* out, long long count, float a, float b, cudaStream_t stream) {
   if (count <= 0) return 0;
-  if (kind < 0 || kind > 2) return (int)cudaErrorInvalidValue;
+  if (kind < 0 || kind > 3) return (int)cudaErrorInvalidValue;
   if (count % 4 == 0) {
     const size_t count4 = (size_t)count / 4;
     if (dtype == TLIE_F32)
-      activation_vec_kernel<float><<<grid_for(count4, 256), 256, 0, stream>>>((const float*)in, (float*)out, kind, count4);
+      activation_vec_kernel<float><<<grid_for(count4, 256), 256, 0, stream>>>((const float*)in, (float*)out, kind, a, b, count4);
     else
-      activation_vec_kernel<__nv_bfloat16><<<grid_for(count4, 256), 256, 0, stream>>>((const __nv_bfloat16*)in, (__nv_bfloat16*)out, kind, count4);
+      activation_vec_kernel<__nv_bfloat16><<<grid_for(count4, 256), 256, 0, stream>>>((const __nv_bfloat16*)in, (__nv_bfloat16*)out, kind, a, b, count4);
     return (int)cudaGetLastError();
   }
   if (dtype == TLIE_F32)
-    activation_kernel<float><<<grid_for(count, 256), 256, 0, stream>>>((const float*)in, (float*)out, kind, (size_t)count);
+    activation_kernel<float><<<grid_for(count, 256), 256, 0, stream>>>((const float*)in, (float*)out, kind, a, b, (size_t)count);
   else
-    activation_kernel<__nv_bfloat16><<<grid_for(count, 256), 256, 0, stream>>>((const __nv_bfloat16*)in, (__nv_bfloat16*)out, kind, (size_t)count);
+    activation_kernel<__nv_bfloat16><<<grid_for(count, 256), 256, 0, stream>>>((const __nv_bfloat16*)in, (__nv_bfloat16*)out, kind, a, b, (size_t)count);
   return (int)cudaGetLastError();
 }

@@ -32,20 +32,24 @@ struct GemvArgs {
   const float* squares;
   int square_tiles;
   // STORE_BF16 may apply an activation to the (rounded) product before it is stored: 0 none, 1 the square of relu, 2 gelu in its
-  // tanh form, 3 silu.  The same roundings as a product stored and an elementwise kernel run over it.
+  // tanh form, 3 silu, 4 act_a z^2 + z / 2 above zero and act_b (e^z - 1 - z) + z / 2 below (xIELU).  The same roundings as a product
+  // stored and an elementwise kernel run over it.
   int activation;
+  float act_a, act_b;
+  const float* bias;        // STORE_BF16, no activation: [N] added to the 32-bit sum before it is rounded, or nullptr
   // GATED: how the two halves meet.  gate_kind 0: silu(gate) * up.  2: gelu (tanh form) of the gate times up.  1: with g = min(gate, gate_limit) and u = clamp(up, -gate_limit,
   // gate_limit): g * sigmoid(gate_alpha * g) * (u + gate_shift).
   int gate_kind;
   float gate_limit, gate_alpha, gate_shift;
 };
 
-__device__ __forceinline__ float gemv_activate(int kind, float z) {
+__device__ __forceinline__ float gemv_activate(int kind, float z, float a, float b) {
   if (kind == 1) {
     const float r = fmaxf(z, 0.0f);
     return r * r;
   }
   if (kind == 2) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  if (kind == 4) return z > 0.0f ? a * z * z + 0.5f * z : b * (expm1f(z) - z) + 0.5f * z;
   return z / (1.0f + expf(-z));
 }
 
@@ -160,8 +164,9 @@ __device__ __forceinline__ void gemv_reduce_store(const GemvArgs& a, const float
     const size_t o = (size_t)m * n_rows + n0 + r;
     if (EPI == EPI_STORE_BF16) {
       if (live) {
+        if (a.bias != nullptr) sum += __ldg(a.bias + n0 + r);
         __nv_bfloat16 stored = __float2bfloat16_rn(sum);
-        if (a.activation != 0) stored = __float2bfloat16_rn(gemv_activate(a.activation, __bfloat162float(stored)));
+        if (a.activation != 0) stored = __float2bfloat16_rn(gemv_activate(a.activation, __bfloat162float(stored), a.act_a, a.act_b));
         reinterpret_cast<__nv_bfloat16*>(a.out)[o] = stored;
       }
     } else if (EPI == EPI_STORE_F32) {

@@ -113,15 +113,16 @@ TLIE_EXPORT void tlie_gemv_set_wide_ctas(int on) { gemv_wide_ctas = on; }
 // squares per 16 columns in prepare_squares [M, ceil(N / 16)].  epilogue 0: bf16 out [M, N]; 1: 32-bit out; 2: out (32-bit [M, N]) += result;
 // 3: w holds [gate rows | up rows] (N even), out = silu(gate) * up as bf16 [M, N / 2] (gate_kind 2: gelu in its tanh form in the place of silu; gate_kind 1: the halves clamped at gate_limit,
 // min(gate) * sigmoid(gate_alpha * min(gate)) * (clamp(up) + gate_shift)).  activation (epilogue 0 only): 1 the square of
-// relu, 2 gelu in its tanh form, 3 silu, applied to the rounded product before it is stored.
+// relu, 2 gelu in its tanh form, 3 silu, 4 act_a z^2 + z / 2 above zero and act_b (e^z - 1 - z) + z / 2 below, applied to the rounded product before
+// it is stored.  bias (epilogue 0 only, or null): 32-bit [N], added to the sums before they are rounded.
 // Needs K % 8 == 0 (K % 4 == 0 suffices for x_mode 1 is NOT enough: weights are read 8 at a time), M <= 16.
 TLIE_EXPORT int tlie_gemv_fused(int x_mode, const void* x, int ldx, const int* rows, const float* norm_weight, float eps,
                                 const void* w, void* out, int M, int N, int K, int epilogue, const float* squares, int square_tiles,
                                 const float* prepare_weight, void* prepare_x, float* prepare_squares, int activation, int gate_kind, float gate_limit,
-                                float gate_alpha, float gate_shift, cudaStream_t stream) {
+                                float gate_alpha, float gate_shift, float act_a, float act_b, const float* bias, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (gate_kind < 0 || gate_kind > 2 || (gate_kind != 0 && epilogue != EPI_GATED)) return (int)cudaErrorInvalidValue;
-  if (activation < 0 || activation > 3 || (activation != 0 && epilogue != EPI_STORE_BF16)) return (int)cudaErrorInvalidValue;
+  if (activation < 0 || activation > 4 || ((activation != 0 || bias != nullptr) && epilogue != EPI_STORE_BF16)) return (int)cudaErrorInvalidValue;
   if (K <= 0 || K % 8 != 0 || M > 16 || ((x_mode == X_PLAIN || x_mode == X_PREPARED) && ldx % 8 != 0) || (epilogue == EPI_GATED && (N & 1)) ||
       (x_mode == X_PREPARED && (squares == nullptr || square_tiles <= 0)) ||
       (prepare_weight != nullptr && (epilogue != EPI_ACCUM || prepare_x == nullptr || prepare_squares == nullptr)))
@@ -144,6 +145,9 @@ TLIE_EXPORT int tlie_gemv_fused(int x_mode, const void* x, int ldx, const int* r
   a.prepare_x = (__nv_bfloat16*)prepare_x;
   a.prepare_squares = prepare_squares;
   a.activation = activation;
+  a.act_a = act_a;
+  a.act_b = act_b;
+  a.bias = bias;
   a.gate_kind = gate_kind;
   a.gate_limit = gate_limit;
   a.gate_alpha = gate_alpha;

@@ -1,22 +1,30 @@
 // A feed-forward of routed experts: every token goes through ``top`` of ``experts`` small gated feed-forwards, chosen by a router.
 //
-//   moe_route     per token: z = W_router x (32-bit), s = sigmoid(z), choice = s + correction.  Experts form ``groups`` equal groups
-//                 of neighbours; a group's score is the sum of its two largest choice scores; only experts of the ``keep`` best
-//                 groups can be chosen.  The ``top`` largest choice scores among them are chosen (ties: the lower index); their
+//   moe_route     per token: z = W_router x (32-bit), s = sigmoid(z) or (``softmax``) softmax(z) over all experts, choice = s + correction.
+//                 Experts form ``groups`` equal groups of neighbours; a group's score is the sum of its two largest choice scores, or
+//                 (``group_best``) its largest; only experts of the ``keep`` best groups can be chosen.  The ``top`` largest choice scores among them are chosen (ties: the lower index); their
 //                 weights are s / (sum of the chosen s + 1e-20) * route_scale (``normalize`` 0: s * route_scale, the scores as they are).
+//                 ``shared_gate``: the router has one row more, and sigmoid of its product with the token is what the shared branch is
+//                 multiplied by.
 //   moe_gate_up   per (token, chosen expert): act(W_gate x) * (W_up x), straight from the expert's rows (steps of few rows, and the
 //                 32-bit path): a warp per output, the sums in a fixed order.
 //   moe_down      per token: sum over its chosen experts of weight * W_down act, plus the shared branch if there is one.
 //                 ``weight_input``: the weight multiplies what the expert reads instead (moe_gate_up scales the token as it loads it,
 //                 moe_down adds the experts' outputs as they are).
 //
+//
 // Expert weights are stacked: gate_up [experts][2 ff][width] (gate rows, then up rows), down [experts][width][ff].
-// Activation codes: 0 silu, 1 gelu in its tanh form.
+// Activation codes: 0 silu, 1 gelu in its tanh form, both times the up half; 2 the square of relu, for experts without a gate
+// (gate_up is then [experts][ff][width], the up rows alone).
 #include "common.cuh"
 
 namespace tlie {
 
 __device__ __forceinline__ float moe_act(float z, int kind) {
+  if (kind == 2) {
+    const float r = fmaxf(z, 0.0f);
+    return r * r;
+  }
   if (kind == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   return z / (1.0f + expf(-z));
 }
@@ -220,9 +228,29 @@ __device__ __forceinline__ int warp_argmax(const float* values, int n, int lane,
 
 constexpr int kRouteWarps = 4;
 
+// One warp turns s [experts] from router logits into their softmax and fills choice [experts].
+__device__ __forceinline__ void route_softmax(float* s, float* choice, const float* __restrict__ correction, int lane, int experts) {
+  float highest = -INFINITY;
+  for (int e = lane; e < experts; e += 32) highest = fmaxf(highest, s[e]);
+  highest = warp_max(highest);
+  float total = 0.0f;
+  for (int e = lane; e < experts; e += 32) {
+    const float p = expf(s[e] - highest);
+    s[e] = p;
+    total += p;
+  }
+  total = warp_sum(total);
+  for (int e = lane; e < experts; e += 32) {
+    const float p = s[e] / total;
+    s[e] = p;
+    choice[e] = p + (correction != nullptr ? correction[e] : 0.0f);
+  }
+  __syncwarp();
+}
+
 // One warp chooses a token's experts from s [experts] and choice [experts] (shared memory, written before); group_score [groups] is scratch.
 __device__ __forceinline__ void route_select(float* s, float* choice, float* group_score, int* __restrict__ ids, float* __restrict__ weights, int t, int lane,
-                                             int experts, int groups, int keep, int top, float route_scale, int normalize) {
+                                             int experts, int groups, int keep, int top, float route_scale, int normalize, int group_best) {
   const int per = experts / groups;
   if (groups > 1 && keep < groups) {
     for (int g = lane; g < groups; g += 32) {
@@ -236,7 +264,7 @@ __device__ __forceinline__ void route_select(float* s, float* choice, float* gro
           second = c;
         }
       }
-      group_score[g] = per > 1 ? first + second : first;
+      group_score[g] = (per > 1 && !group_best) ? first + second : first;
     }
     __syncwarp();
     // the ``keep`` best groups are marked by a score of +inf; the others' experts leave the choice
@@ -287,7 +315,8 @@ __device__ __forceinline__ void route_select(float* s, float* choice, float* gro
 template <typename T>
 __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router, const float* __restrict__ correction,
                                                                      int* __restrict__ ids, float* __restrict__ weights, int tokens, int width, int experts,
-                                                                     int groups, int keep, int top, float route_scale, int normalize) {
+                                                                     int groups, int keep, int top, float route_scale, int normalize, int softmax, int group_best,
+                                                                     float* __restrict__ shared_gate) {
   extern __shared__ float route_smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kRouteWarps + warp;
@@ -296,19 +325,25 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const T* __
   float* choice = s + experts;
   float* group_score = choice + experts;
   const T* row = x + (size_t)t * width;
-  for (int e = 0; e < experts; ++e) {
+  const int router_rows = experts + (shared_gate != nullptr ? 1 : 0);   // the last row, if there is one more, is the shared branch's gate
+  for (int e = 0; e < router_rows; ++e) {
     const float* w = router + (size_t)e * width;
     float sum = 0.0f;
     for (int d = lane; d < width; d += 32) sum = fmaf(w[d], to_float(row[d]), sum);
     sum = warp_sum(sum);
     if (lane == 0) {
       const float score = 1.0f / (1.0f + expf(-sum));
-      s[e] = score;
-      choice[e] = score + (correction != nullptr ? correction[e] : 0.0f);
+      if (e == experts) {
+        shared_gate[t] = score;
+      } else {
+        s[e] = softmax ? sum : score;
+        choice[e] = score + (correction != nullptr ? correction[e] : 0.0f);
+      }
     }
   }
   __syncwarp();
-  route_select(s, choice, group_score, ids, weights, t, lane, experts, groups, keep, top, route_scale, normalize);
+  if (softmax) route_softmax(s, choice, correction, lane, experts);
+  route_select(s, choice, group_score, ids, weights, t, lane, experts, groups, keep, top, route_scale, normalize, group_best);
 }
 
 constexpr int kRouteTiledWarps = 8;    // steps of many tokens (four share a CTA); a CTA of one token has 16 warps
@@ -322,7 +357,8 @@ template <typename T, int TOK, int WARPS>
 __global__ void __launch_bounds__(WARPS * 32) moe_route_tiled_kernel(const T* __restrict__ x, const float* __restrict__ router,
                                                                                 const float* __restrict__ correction, int* __restrict__ ids,
                                                                                 float* __restrict__ weights, int tokens, int width, int experts, int groups, int keep,
-                                                                                int top, float route_scale, int normalize) {
+                                                                                int top, float route_scale, int normalize, int softmax, int group_best,
+                                                                                float* __restrict__ shared_gate) {
   extern __shared__ __align__(16) float route_smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t0 = blockIdx.x * TOK;
@@ -338,10 +374,11 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_tiled_kernel(const T* __
   __syncthreads();
   // two experts of a warp side by side and four pieces of each ahead: a row at a time with one piece in flight made a step of few
   // tokens wait for memory once per 512 bytes of a row.  An expert past the end reads the last one again and writes nothing.
-  for (int e0 = warp; e0 < experts; e0 += 2 * WARPS) {
+  const int router_rows = experts + (shared_gate != nullptr ? 1 : 0);   // the last row, if there is one more, is the shared branch's gate
+  for (int e0 = warp; e0 < router_rows; e0 += 2 * WARPS) {
     const int e1 = e0 + WARPS;
     const float* w0 = router + (size_t)e0 * width;
-    const float* w1 = router + (size_t)min(e1, experts - 1) * width;
+    const float* w1 = router + (size_t)min(e1, router_rows - 1) * width;
     float sum[2][TOK];
 #pragma unroll
     for (int i = 0; i < TOK; ++i) sum[0][i] = sum[1][i] = 0.0f;
@@ -365,15 +402,19 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_tiled_kernel(const T* __
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int e = j == 0 ? e0 : e1;
-      if (e >= experts) break;
-      const float shift = correction != nullptr ? correction[e] : 0.0f;
+      if (e >= router_rows) break;
+      const float shift = (correction != nullptr && e < experts) ? correction[e] : 0.0f;
 #pragma unroll
       for (int i = 0; i < TOK; ++i) {
         const float z = warp_sum(sum[j][i]);
         if (lane == 0) {
           const float score = 1.0f / (1.0f + expf(-z));
-          tables[(size_t)i * per_token + e] = score;
-          tables[(size_t)i * per_token + experts + e] = score + shift;
+          if (e == experts) {
+            if (t0 + i < tokens) shared_gate[t0 + i] = score;
+          } else {
+            tables[(size_t)i * per_token + e] = softmax ? z : score;
+            tables[(size_t)i * per_token + experts + e] = score + shift;
+          }
         }
       }
     }
@@ -382,7 +423,8 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_tiled_kernel(const T* __
   for (int i = warp; i < TOK; i += WARPS) {
     if (t0 + i >= tokens) break;
     float* s = tables + (size_t)i * per_token;
-    route_select(s, s + experts, s + 2 * experts, ids, weights, t0 + i, lane, experts, groups, keep, top, route_scale, normalize);
+    if (softmax) route_softmax(s, s + experts, correction, lane, experts);
+    route_select(s, s + experts, s + 2 * experts, ids, weights, t0 + i, lane, experts, groups, keep, top, route_scale, normalize, group_best);
   }
 }
 
@@ -390,8 +432,8 @@ constexpr int kMoeWarps = 8;
 constexpr int kGateUpOutputs = 32;   // outputs of one CTA of the direct first half
 constexpr int kDownOutputs = 32;
 
-// grid (tokens * top, ceil(ff / 32)); act [tokens * top][ff]
-template <typename T>
+// grid (tokens * top, ceil(ff / (GATED ? 32 : 64))); act [tokens * top][ff].  GATED false: experts of one up matrix, act(W_up x).
+template <typename T, bool GATED>
 __global__ void __launch_bounds__(kMoeWarps * 32) moe_gate_up_kernel(const T* __restrict__ x, const T* __restrict__ gate_up, const int* __restrict__ ids,
                                                                      const float* __restrict__ input_weights, T* __restrict__ act, int width, int ff, int top, int kind) {
   extern __shared__ float moe_x[];
@@ -400,36 +442,41 @@ __global__ void __launch_bounds__(kMoeWarps * 32) moe_gate_up_kernel(const T* __
   const float scale = input_weights != nullptr ? input_weights[slot] : 1.0f;   // an expert that reads its token times the token's weight
   for (int d = threadIdx.x; d < width; d += blockDim.x) moe_x[d] = to_float(x[(size_t)t * width + d]) * scale;
   __syncthreads();
-  const T* expert = gate_up + (size_t)ids[slot] * 2 * ff * width;
+  const T* expert = gate_up + (size_t)ids[slot] * (GATED ? 2 : 1) * ff * width;
   const bool vector = rows_are_vectors(expert, width);
-  // a warp's outputs (warp, warp + kMoeWarps, ...) four at a time: four gate rows and four up rows side by side.  Outputs past the end
+  // eight of the expert's rows side by side per warp: four outputs' gate and up rows, or eight outputs' up rows.  Outputs past the end
   // read the last row again and store nothing.
-  constexpr int kPerWarp = kGateUpOutputs / kMoeWarps;
-  static_assert(kPerWarp == 4, "four outputs per warp");
-  const T* rows[2 * kPerWarp];
+  constexpr int kRows = 8, kPerWarp = GATED ? kRows / 2 : kRows;
+  constexpr int kOutputs = GATED ? kGateUpOutputs : 2 * kGateUpOutputs;
+  static_assert(kPerWarp * kMoeWarps == kOutputs, "a CTA's outputs are dealt to its warps");
+  const T* rows[kRows];
   int f[kPerWarp];
 #pragma unroll
   for (int j = 0; j < kPerWarp; ++j) {
-    f[j] = blockIdx.y * kGateUpOutputs + warp + j * kMoeWarps;
+    f[j] = blockIdx.y * kOutputs + warp + j * kMoeWarps;
     const int row = min(f[j], ff - 1);
-    rows[2 * j] = expert + (size_t)row * width;
-    rows[2 * j + 1] = expert + (size_t)(ff + row) * width;
+    if (GATED) {
+      rows[2 * j] = expert + (size_t)row * width;
+      rows[2 * j + 1] = expert + (size_t)(ff + row) * width;
+    } else {
+      rows[j] = expert + (size_t)row * width;
+    }
   }
-  float sums[2 * kPerWarp];
-  lane_dot_n<2 * kPerWarp>(rows, moe_x, width, lane, vector, sums);
+  float sums[kRows];
+  lane_dot_n<kRows>(rows, moe_x, width, lane, vector, sums);
 #pragma unroll
   for (int j = 0; j < kPerWarp; ++j) {
-    const float g = warp_sum(sums[2 * j]);
-    const float u = warp_sum(sums[2 * j + 1]);
+    const float g = warp_sum(sums[GATED ? 2 * j : j]);
+    const float u = GATED ? warp_sum(sums[2 * j + 1]) : 1.0f;
     if (lane == 0 && f[j] < ff) act[(size_t)slot * ff + f[j]] = from_float<T>(moe_act(g, kind) * u);
   }
 }
 
-// grid (tokens, ceil(width / 32)); out[t] = sum_k weight_k * W_down[e_k] act[t, k]  (+ shared[t])
+// grid (tokens, ceil(width / 32)); out[t] = sum_k weight_k * W_down[e_k] act[t, k]  (+ shared[t], times shared_gate[t] if given)
 template <typename T>
 __global__ void __launch_bounds__(kMoeWarps * 32, 4) moe_down_kernel(const T* __restrict__ act, const T* __restrict__ down, const int* __restrict__ ids,
-                                                                  const float* __restrict__ weights, const T* __restrict__ shared, T* __restrict__ out, int width,
-                                                                  int ff, int top) {
+                                                                  const float* __restrict__ weights, const T* __restrict__ shared,
+                                                                  const float* __restrict__ shared_gate, T* __restrict__ out, int width, int ff, int top) {
   extern __shared__ float moe_act_rows[];   // [top][ff]
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -471,7 +518,7 @@ __global__ void __launch_bounds__(kMoeWarps * 32, 4) moe_down_kernel(const T* __
     for (int o = 0; o < 2; ++o) {
       if (n[o] >= width) continue;
       float value = total[o];
-      if (shared != nullptr) value += to_float(shared[(size_t)t * width + n[o]]);
+      if (shared != nullptr) value += to_float(shared[(size_t)t * width + n[o]]) * (shared_gate != nullptr ? shared_gate[t] : 1.0f);
       if (lane == 0) out[(size_t)t * width + n[o]] = from_float<T>(value);
     }
   }
@@ -482,7 +529,8 @@ __global__ void __launch_bounds__(kMoeWarps * 32, 4) moe_down_kernel(const T* __
 using namespace tlie;
 
 TLIE_EXPORT int tlie_moe_route(int dtype, const void* x, const float* router, const float* correction, int* ids, float* weights, int tokens, int width, int experts,
-                               int groups, int keep, int top, float route_scale, int normalize, cudaStream_t stream) {
+                               int groups, int keep, int top, float route_scale, int normalize, int softmax, int group_best, float* shared_gate,
+                               cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (experts <= 0 || groups <= 0 || experts % groups != 0 || keep <= 0 || keep > groups || top <= 0 || top > keep * (experts / groups))
     return (int)cudaErrorInvalidValue;
@@ -499,7 +547,7 @@ TLIE_EXPORT int tlie_moe_route(int dtype, const void* x, const float* router, co
     if (tiled > 48 * 1024) e = cudaFuncSetAttribute(moe_route_tiled_kernel<T, TOK, (TOK == 1 ? 16 : kRouteTiledWarps)>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tiled);             \
     if (e == cudaSuccess)                                                                                                                                 \
       moe_route_tiled_kernel<T, TOK, (TOK == 1 ? 16 : kRouteTiledWarps)><<<blocks, (TOK == 1 ? 16 : kRouteTiledWarps) * 32, tiled, stream>>>((const T*)x, router, correction, ids, weights, tokens, width, experts, groups, keep, \
-                                                                                     top, route_scale, normalize);                                                  \
+                                                                                     top, route_scale, normalize, softmax, group_best, shared_gate);                \
   } while (0)
       if (dtype == TLIE_F32) {
         if (tok == 4) TLIE_ROUTE_TILED(float, 4); else TLIE_ROUTE_TILED(float, 1);
@@ -514,42 +562,54 @@ TLIE_EXPORT int tlie_moe_route(int dtype, const void* x, const float* router, co
   if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
   const int blocks = (tokens + kRouteWarps - 1) / kRouteWarps;
   if (dtype == TLIE_F32)
-    moe_route_kernel<float><<<blocks, kRouteWarps * 32, smem, stream>>>((const float*)x, router, correction, ids, weights, tokens, width, experts, groups, keep, top, route_scale, normalize);
+    moe_route_kernel<float><<<blocks, kRouteWarps * 32, smem, stream>>>((const float*)x, router, correction, ids, weights, tokens, width, experts, groups, keep, top, route_scale, normalize, softmax, group_best, shared_gate);
   else
     moe_route_kernel<__nv_bfloat16><<<blocks, kRouteWarps * 32, smem, stream>>>((const __nv_bfloat16*)x, router, correction, ids, weights, tokens, width, experts, groups,
-                                                                              keep, top, route_scale, normalize);
+                                                                              keep, top, route_scale, normalize, softmax, group_best, shared_gate);
+  return (int)cudaGetLastError();
+}
+
+template <typename T, bool GATED>
+static int launch_moe_first(const void* x, const void* gate_up, const int* ids, const float* input_weights, void* act, int tokens, int width, int ff, int top, int kind,
+                            cudaStream_t stream) {
+  const size_t x_smem = (size_t)width * sizeof(float);
+  if (x_smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+  if (x_smem > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(moe_gate_up_kernel<T, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)x_smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  constexpr int kOutputs = GATED ? kGateUpOutputs : 2 * kGateUpOutputs;
+  moe_gate_up_kernel<T, GATED><<<dim3(tokens * top, (ff + kOutputs - 1) / kOutputs), kMoeWarps * 32, x_smem, stream>>>((const T*)x, (const T*)gate_up, ids, input_weights,
+                                                                                                                    (T*)act, width, ff, top, kind);
   return (int)cudaGetLastError();
 }
 
 template <typename T>
-static int launch_moe_experts(const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, void* act, void* out,
-                              int tokens, int width, int ff, int top, int kind, int weight_input, cudaStream_t stream) {
-  const size_t x_smem = (size_t)width * sizeof(float), act_smem = (size_t)top * ff * sizeof(float);
-  if (x_smem > 200 * 1024 || act_smem > 200 * 1024) return (int)cudaErrorInvalidValue;
-  cudaError_t e;
-  if (x_smem > 48 * 1024) {
-    e = cudaFuncSetAttribute(moe_gate_up_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)x_smem);
-    if (e != cudaSuccess) return (int)e;
-  }
+static int launch_moe_experts(const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, const float* shared_gate, void* act,
+                              void* out, int tokens, int width, int ff, int top, int kind, int weight_input, cudaStream_t stream) {
+  const size_t act_smem = (size_t)top * ff * sizeof(float);
+  if (act_smem > 200 * 1024) return (int)cudaErrorInvalidValue;
   if (act_smem > 48 * 1024) {
-    e = cudaFuncSetAttribute(moe_down_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)act_smem);
+    const cudaError_t e = cudaFuncSetAttribute(moe_down_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)act_smem);
     if (e != cudaSuccess) return (int)e;
   }
-  moe_gate_up_kernel<T><<<dim3(tokens * top, (ff + kGateUpOutputs - 1) / kGateUpOutputs), kMoeWarps * 32, x_smem, stream>>>(
-      (const T*)x, (const T*)gate_up, ids, weight_input ? weights : nullptr, (T*)act, width, ff, top, kind);
-  e = cudaGetLastError();
-  if (e != cudaSuccess) return (int)e;
+  const float* input_weights = weight_input ? weights : nullptr;
+  const int rc = kind == 2 ? launch_moe_first<T, false>(x, gate_up, ids, input_weights, act, tokens, width, ff, top, kind, stream)
+                           : launch_moe_first<T, true>(x, gate_up, ids, input_weights, act, tokens, width, ff, top, kind, stream);
+  if (rc != 0) return rc;
   moe_down_kernel<T><<<dim3(tokens, (width + kDownOutputs - 1) / kDownOutputs), kMoeWarps * 32, act_smem, stream>>>(
-      (const T*)act, (const T*)down, ids, weight_input ? nullptr : weights, (const T*)shared, (T*)out, width, ff, top);
+      (const T*)act, (const T*)down, ids, weight_input ? nullptr : weights, (const T*)shared, shared_gate, (T*)out, width, ff, top);
   return (int)cudaGetLastError();
 }
 
-// ``act``: scratch [tokens * top, ff] of ``dtype``; ``shared`` [tokens, width] or null; ``out`` [tokens, width].  ``weight_input`` 1: a chosen expert reads
-// the token times its weight and its output is added as it is (out[t] = sum_k expert_k(weight_k x[t])); 0: the weight multiplies the expert's output.
-TLIE_EXPORT int tlie_moe_experts(int dtype, const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, void* act,
-                                 void* out, int tokens, int width, int ff, int top, int kind, int weight_input, cudaStream_t stream) {
+// ``act``: scratch [tokens * top, ff] of ``dtype``; ``shared`` [tokens, width] or null, times ``shared_gate`` [tokens] (32-bit) unless that is null; ``out`` [tokens, width].
+// ``weight_input`` 1: a chosen expert reads the token times its weight and its output is added as it is (out[t] = sum_k expert_k(weight_k x[t])); 0: the weight
+// multiplies the expert's output.  ``kind`` 2: experts without a gate.
+TLIE_EXPORT int tlie_moe_experts(int dtype, const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared,
+                                 const float* shared_gate, void* act, void* out, int tokens, int width, int ff, int top, int kind, int weight_input, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if ((long long)tokens * top > 2147483647LL / 2 || kind < 0 || kind > 1) return (int)cudaErrorInvalidValue;
-  if (dtype == TLIE_F32) return launch_moe_experts<float>(x, gate_up, down, ids, weights, shared, act, out, tokens, width, ff, top, kind, weight_input, stream);
-  return launch_moe_experts<__nv_bfloat16>(x, gate_up, down, ids, weights, shared, act, out, tokens, width, ff, top, kind, weight_input, stream);
+  if ((long long)tokens * top > 2147483647LL / 2 || kind < 0 || kind > 2) return (int)cudaErrorInvalidValue;
+  if (dtype == TLIE_F32)
+    return launch_moe_experts<float>(x, gate_up, down, ids, weights, shared, shared_gate, act, out, tokens, width, ff, top, kind, weight_input, stream);
+  return launch_moe_experts<__nv_bfloat16>(x, gate_up, down, ids, weights, shared, shared_gate, act, out, tokens, width, ff, top, kind, weight_input, stream);
 }

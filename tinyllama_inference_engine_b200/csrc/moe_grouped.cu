@@ -11,7 +11,8 @@
 //                act(w g) * (w u) in the gated epilogue, 32-bit, and no weight behind W_down)
 //                64 x 64 tiles (the gated one: 64 gate and the 64 up columns beside them), k in blocks of 32 through two cp.async
 //                stages, mma.sync m16n8k16 with 32-bit accumulators, a warp per 16 rows.
-//   moe_combine  out[t] = sum_k y[t * top + k] + shared[t]: the chosen experts in the order they were chosen, so that a row's
+//                <PLAIN>  act[p] = act(W_up[e] x[token(p)]), for experts without a gate.
+//   moe_combine  out[t] = sum_k y[t * top + k] + shared[t] (times shared_gate[t] if given): the chosen experts in the order they were chosen, so that a row's
 //                sum does not depend on what else is in the step.
 #include "common.cuh"
 #include "mma_utils.cuh"
@@ -23,6 +24,10 @@ constexpr int kGRow = kGK + 8;   // padded shared-memory rows (elements)
 constexpr int kGThreads = 128;
 
 __device__ __forceinline__ float grouped_act(float z, int kind) {
+  if (kind == 2) {
+    const float r = fmaxf(z, 0.0f);
+    return r * r;
+  }
   if (kind == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   return z / (1.0f + expf(-z));
 }
@@ -55,12 +60,15 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
 }
 
 // GATED: a [tokens][K] gathered by slot / top, w [experts][2 N][K], out bfloat16 [slots][N] by sorted row.
+// PLAIN: as GATED with w [experts][N][K].
 // DOWN:  a [slots][K] by sorted row, w [experts][N][K], out 32-bit [slots][N] by slot, times the slot's weight.
-template <bool GATED>
+enum { GROUPED_DOWN = 0, GROUPED_GATED = 1, GROUPED_PLAIN = 2 };
+template <int MODE>
 __global__ void __launch_bounds__(kGThreads) moe_grouped_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __restrict__ w, const int* __restrict__ sorted_slots,
                                                                 const int* __restrict__ meta, const float* __restrict__ weights, void* __restrict__ out, int N, int K,
                                                                 int top, int kind, int weight_input) {
-  constexpr int kB = GATED ? 2 : 1;
+  constexpr bool FIRST = MODE != GROUPED_DOWN;   // the rows are the tokens' own, gathered
+  constexpr int kB = MODE == GROUPED_GATED ? 2 : 1;
   __shared__ __align__(16) __nv_bfloat16 a_s[2][kGM][kGRow];
   __shared__ __align__(16) __nv_bfloat16 b_s[2][kB][kGN][kGRow];
   __shared__ int row_slot[kGM];
@@ -71,7 +79,7 @@ __global__ void __launch_bounds__(kGThreads) moe_grouped_kernel(const __nv_bfloa
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x < kGM) row_slot[threadIdx.x] = threadIdx.x < rows ? sorted_slots[row0 + threadIdx.x] : 0;
   __syncthreads();
-  const __nv_bfloat16* w_e = w + (size_t)expert * (GATED ? 2 : 1) * N * K;
+  const __nv_bfloat16* w_e = w + (size_t)expert * kB * N * K;
   auto issue = [&](int kb) {
     const int k0 = kb * kGK;
     if (k0 < K) {
@@ -79,7 +87,7 @@ __global__ void __launch_bounds__(kGThreads) moe_grouped_kernel(const __nv_bfloa
       for (int idx = threadIdx.x; idx < kGM * (kGK / 8); idx += kGThreads) {
         const int row = idx / (kGK / 8), chunk = idx % (kGK / 8);
         const bool valid = row < rows && k0 + chunk * 8 < K;
-        const size_t source = GATED ? (size_t)(row_slot[row] / top) : (size_t)(row0 + row);
+        const size_t source = FIRST ? (size_t)(row_slot[row] / top) : (size_t)(row0 + row);
         cp_async_16(&a_s[stage][row][chunk * 8], valid ? a + source * K + k0 + chunk * 8 : a, valid);
       }
       for (int idx = threadIdx.x; idx < kB * kGN * (kGK / 8); idx += kGThreads) {
@@ -124,7 +132,7 @@ __global__ void __launch_bounds__(kGThreads) moe_grouped_kernel(const __nv_bfloa
   for (int r = 0; r < 2; ++r) {
     const int row = warp * 16 + g + 8 * r;
     if (row >= rows) continue;
-    if (GATED) {
+    if (FIRST) {
       __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)(row0 + row) * N;
       const float scale = weight_input ? weights[row_slot[row]] : 1.0f;
 #pragma unroll
@@ -132,7 +140,8 @@ __global__ void __launch_bounds__(kGThreads) moe_grouped_kernel(const __nv_bfloa
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
           const int n = n0 + j * 8 + 2 * t + c;
-          if (n < N) dst[n] = __float2bfloat16_rn(grouped_act(scale * acc[0][j][r * 2 + c], kind) * (scale * acc[kB - 1][j][r * 2 + c]));
+          const float up = MODE == GROUPED_GATED ? scale * acc[kB - 1][j][r * 2 + c] : 1.0f;
+          if (n < N) dst[n] = __float2bfloat16_rn(grouped_act(scale * acc[0][j][r * 2 + c], kind) * up);
         }
     } else {
       const int slot = row_slot[row];
@@ -149,13 +158,14 @@ __global__ void __launch_bounds__(kGThreads) moe_grouped_kernel(const __nv_bfloa
   }
 }
 
-__global__ void moe_combine_kernel(const float* __restrict__ y, const __nv_bfloat16* __restrict__ shared, __nv_bfloat16* __restrict__ out, int width, int top, size_t total) {
+__global__ void moe_combine_kernel(const float* __restrict__ y, const __nv_bfloat16* __restrict__ shared, const float* __restrict__ shared_gate,
+                                   __nv_bfloat16* __restrict__ out, int width, int top, size_t total) {
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const size_t t = i / width;
     const int n = (int)(i - t * width);
     float sum = 0.0f;
     for (int k = 0; k < top; ++k) sum += y[(t * top + k) * width + n];
-    if (shared != nullptr) sum += __bfloat162float(shared[i]);
+    if (shared != nullptr) sum += __bfloat162float(shared[i]) * (shared_gate != nullptr ? shared_gate[t] : 1.0f);
     out[i] = __float2bfloat16_rn(sum);
   }
 }
@@ -165,28 +175,30 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const __nv_bfloa
 using namespace tlie;
 
 // Scratch: sorted_slots int32 [tokens * top], meta int32 [1 + 3 * (tokens * top / 64 + experts)], act bfloat16 [tokens * top, ff],
-// y 32-bit [tokens * top, width].  ``shared`` bfloat16 [tokens, width] or null.
-TLIE_EXPORT int tlie_moe_grouped(const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, int* sorted_slots,
+// y 32-bit [tokens * top, width].  ``shared`` bfloat16 [tokens, width] or null, times ``shared_gate`` [tokens] unless that is null.
+TLIE_EXPORT int tlie_moe_grouped(const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, const float* shared_gate, int* sorted_slots,
                                  int* meta, void* act, float* y, void* out, int tokens, int width, int ff, int experts, int top, int kind, int weight_input,
                                  cudaStream_t stream) {
   if (tokens <= 0) return 0;
   const long long slots = (long long)tokens * top;
-  if (width % 8 != 0 || ff % 8 != 0 || experts <= 0 || experts > 4096 || slots > (1LL << 30) || kind < 0 || kind > 1) return (int)cudaErrorInvalidValue;
+  if (width % 8 != 0 || ff % 8 != 0 || experts <= 0 || experts > 4096 || slots > (1LL << 30) || kind < 0 || kind > 2) return (int)cudaErrorInvalidValue;
   const int max_tiles = (int)(slots / kGM) + experts;
   moe_sort_kernel<<<1, 1024, 2 * experts * sizeof(int), stream>>>(ids, (int)slots, experts, sorted_slots, meta);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
-  moe_grouped_kernel<true><<<dim3(max_tiles, (ff + kGN - 1) / kGN), kGThreads, 0, stream>>>((const __nv_bfloat16*)x, (const __nv_bfloat16*)gate_up, sorted_slots, meta,
-                                                                                            weights, act, ff, width, top, kind, weight_input);
+  auto first = kind == 2 ? moe_grouped_kernel<GROUPED_PLAIN> : moe_grouped_kernel<GROUPED_GATED>;
+  first<<<dim3(max_tiles, (ff + kGN - 1) / kGN), kGThreads, 0, stream>>>((const __nv_bfloat16*)x, (const __nv_bfloat16*)gate_up, sorted_slots, meta, weights, act, ff, width,
+                                                                         top, kind, weight_input);
   e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
-  moe_grouped_kernel<false><<<dim3(max_tiles, (width + kGN - 1) / kGN), kGThreads, 0, stream>>>((const __nv_bfloat16*)act, (const __nv_bfloat16*)down, sorted_slots, meta,
+  moe_grouped_kernel<GROUPED_DOWN><<<dim3(max_tiles, (width + kGN - 1) / kGN), kGThreads, 0, stream>>>((const __nv_bfloat16*)act, (const __nv_bfloat16*)down, sorted_slots, meta,
                                                                                                 weights, y, width, ff, top, kind, weight_input);
   e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   const size_t total = (size_t)tokens * width;
   const size_t blocks = (total + 255) / 256;
   const size_t most = (size_t)device_sm_count() * 16;
-  moe_combine_kernel<<<(int)(blocks < most ? blocks : most), 256, 0, stream>>>(y, (const __nv_bfloat16*)shared, (__nv_bfloat16*)out, width, top, total);
+  moe_combine_kernel<<<(int)(blocks < most ? blocks : most), 256, 0, stream>>>(y, (const __nv_bfloat16*)shared, shared_gate, (__nv_bfloat16*)out, width, top,
+                                                                                             total);
   return (int)cudaGetLastError();
 }

@@ -10,8 +10,9 @@
 //   moe_gather     xs[row] = x[token(row)] (zeros for padding rows), so that TMA fetches an expert's rows as one box.  Where the weight
 //                  multiplies what an expert reads (``weight_input``), the row is gathered times its weight and the sum below takes no weights.
 //   moe_tc <GATED> act[row] = act(W_gate[e] xs[row]) * (W_up[e] xs[row])      tile 128 x (128 gate + 128 up columns)
+//          <PLAIN> act[row] = act(W_up[e] xs[row]), experts without a gate     tile 128 x 256
 //          <DOWN>  y[row]   = W_down[e] act[row]                               32-bit, tile 128 x 256
-//   moe_tc_combine out[t] = sum_k weight[t, k] y[row(t, k)] + shared[t]: the chosen experts in the order they were chosen, so
+//   moe_tc_combine out[t] = sum_k weight[t, k] y[row(t, k)] + shared[t] (times shared_gate[t] if given): the chosen experts in the order they were chosen, so
 //                  that a token's sum does not depend on what else is in the step.
 // Roles (warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 epilogue), the ring of stages, the two alternating accumulators in
 // tensor memory and the bounded waits are those of gemm_tcgen05.cu.  Tiles are walked with the row tile fastest: the CTAs that
@@ -33,6 +34,10 @@ static_assert(kTcSmemBytes <= 227 * 1024, "shared memory of one CTA");
 
 template <int ACT>
 __device__ __forceinline__ float tc_act(float z) {
+  if (ACT == 2) {
+    const float r = fmaxf(z, 0.0f);
+    return r * r;
+  }
   if (ACT == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   return z / (1.0f + expf(-z));
 }
@@ -91,20 +96,21 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const __nv_bfloat16* __
   }
 }
 
-// One warp's 32 rows of a gated tile: act(gate) * up of 32 columns at a time as bfloat16 into a staging box, written by a bulk
-// tensor store (columns past N are clipped by the tensor map).
-template <int ACT>
-__device__ __forceinline__ void tc_store_gated(uint32_t tmem_acc, int row0, int n0, int N, const CUtensorMap* map_out, uint8_t* staging, int lane, int& boxes) {
+// One warp's 32 rows of a gated tile: act(gate) * up of 32 columns at a time (GATED false: act of a plain tile's columns) as bfloat16 into
+// a staging box, written by a bulk tensor store (columns past N are clipped by the tensor map).
+template <int ACT, bool GATED>
+__device__ __forceinline__ void tc_store_activated(uint32_t tmem_acc, int row0, int n0, int N, const CUtensorMap* map_out, uint8_t* staging, int lane, int& boxes) {
   const int swizzle = (lane >> 1) & 3;   // 64-byte swizzle: 16-byte chunk j of row r lies at chunk j ^ ((r / 2) % 4)
 #pragma unroll 1
-  for (int c = 0; c < (kTcBN / 2) / kStoreCols && n0 + c * kStoreCols < N; ++c) {
+  for (int c = 0; c < (GATED ? kTcBN / 2 : kTcBN) / kStoreCols && n0 + c * kStoreCols < N; ++c) {
     uint32_t gate[32], up[32], packed[kStoreCols / 2];
     tmem_load_32(tmem_acc + c * kStoreCols, gate);
-    tmem_load_32(tmem_acc + kTcBN / 2 + c * kStoreCols, up);
+    if (GATED) tmem_load_32(tmem_acc + kTcBN / 2 + c * kStoreCols, up);
     asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
 #pragma unroll
     for (int i = 0; i < kStoreCols / 2; ++i)
-      packed[i] = pack_bf16(tc_act<ACT>(__uint_as_float(gate[2 * i])) * __uint_as_float(up[2 * i]), tc_act<ACT>(__uint_as_float(gate[2 * i + 1])) * __uint_as_float(up[2 * i + 1]));
+      packed[i] = GATED ? pack_bf16(tc_act<ACT>(__uint_as_float(gate[2 * i])) * __uint_as_float(up[2 * i]), tc_act<ACT>(__uint_as_float(gate[2 * i + 1])) * __uint_as_float(up[2 * i + 1]))
+                        : pack_bf16(tc_act<ACT>(__uint_as_float(gate[2 * i])), tc_act<ACT>(__uint_as_float(gate[2 * i + 1])));
     uint8_t* box = staging + (boxes % kTcStoreBuffers) * kTcBoxBytes;
     ++boxes;
     if (lane == 0) bulk_wait_read<kTcStoreBuffers - 1>();   // the store that last read this box is done with it
@@ -147,10 +153,12 @@ __device__ __forceinline__ void tc_store_f32(uint32_t tmem_acc, int row0, int n0
 }
 
 // GATED: a = gathered rows [rows, K = width], b = gate_up [experts * 2 N, K] with N = ff, out = act bfloat16 [rows, N].
+// PLAIN: as GATED with b = up [experts * N, K].
 // DOWN:  a = act [rows, K = ff], b = down [experts * N, K] with N = width, out = y 32-bit [rows, N].
 // Rows of B past an expert's own (the last column block of an N that is no multiple of the tile) belong to the next expert or are
 // filled with zeros; their columns are never stored.
-template <bool GATED, int ACT>
+enum { TC_DOWN = 0, TC_GATED = 1, TC_PLAIN = 2 };
+template <int MODE, int ACT>
 __global__ void __launch_bounds__(kGemmThreads)
     moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const __grid_constant__ CUtensorMap map_out,
                   const int* __restrict__ meta, int N, int K, int* __restrict__ error_flag) {
@@ -165,6 +173,7 @@ __global__ void __launch_bounds__(kGemmThreads)
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  constexpr bool GATED = MODE == TC_GATED;
   constexpr int kTileN = GATED ? kTcBN / 2 : kTcBN;   // output columns of a tile
   const int n_blocks = (N + kTileN - 1) / kTileN;
   const int k_blocks = (K + kBK - 1) / kBK;
@@ -256,8 +265,8 @@ __global__ void __launch_bounds__(kGemmThreads)
       if (!mbar_wait(&accum_full[acc], (local >> 1) & 1, abort_flag)) break;
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
       const uint32_t tmem_acc = tmem_base + acc * kTcBN + ((uint32_t)(sub * 32) << 16);
-      if (GATED)
-        tc_store_gated<ACT>(tmem_acc, m0 + sub * 32, n0, N, &map_out, my_staging, lane, boxes);
+      if (MODE != TC_DOWN)
+        tc_store_activated<ACT, GATED>(tmem_acc, m0 + sub * 32, n0, N, &map_out, my_staging, lane, boxes);
       else
         tc_store_f32(tmem_acc, m0 + sub * 32, n0, N, &map_out, my_staging, lane, boxes);
       asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -279,7 +288,8 @@ __global__ void __launch_bounds__(kGemmThreads)
 
 // four columns a thread
 __global__ void __launch_bounds__(256) moe_tc_combine_kernel(const float* __restrict__ y, const int* __restrict__ row_of_slot, const float* __restrict__ weights,
-                                                             const __nv_bfloat16* __restrict__ shared, __nv_bfloat16* __restrict__ out, int width, int top, size_t quads) {
+                                                             const __nv_bfloat16* __restrict__ shared, const float* __restrict__ shared_gate,
+                                                             __nv_bfloat16* __restrict__ out, int width, int top, size_t quads) {
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < quads; i += (size_t)gridDim.x * blockDim.x) {
     const size_t t = i / (width / 4);
     const int n = (int)(i - t * (width / 4)) * 4;
@@ -295,10 +305,11 @@ __global__ void __launch_bounds__(256) moe_tc_combine_kernel(const float* __rest
     if (shared != nullptr) {
       const uint2 s = *reinterpret_cast<const uint2*>(shared + t * width + n);
       const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&s.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&s.y);
-      sum.x += __low2float(lo);
-      sum.y += __high2float(lo);
-      sum.z += __low2float(hi);
-      sum.w += __high2float(hi);
+      const float share = shared_gate != nullptr ? shared_gate[t] : 1.0f;
+      sum.x = fmaf(share, __low2float(lo), sum.x);
+      sum.y = fmaf(share, __high2float(lo), sum.y);
+      sum.z = fmaf(share, __low2float(hi), sum.z);
+      sum.w = fmaf(share, __high2float(hi), sum.w);
     }
     uint2 packed;
     packed.x = pack_bf16(sum.x, sum.y);
@@ -307,21 +318,22 @@ __global__ void __launch_bounds__(256) moe_tc_combine_kernel(const float* __rest
   }
 }
 
-template <bool GATED, int ACT>
+template <int MODE, int ACT>
 static int launch_moe_tc(const void* a, const void* b, void* out, const int* meta, int max_rows, int b_rows, int N, int K, int* error_flag, cudaStream_t stream) {
+  constexpr bool GATED = MODE == TC_GATED;
   CUtensorMap map_a, map_b, map_out;
   if (!make_map(&map_a, a, max_rows, K, kBM) || !make_map(&map_b, b, b_rows, K, GATED ? kTcBN / 2 : kTcBN)) return (int)cudaErrorInvalidValue;
-  if (!(GATED ? make_store_map(&map_out, out, max_rows, N) : make_add_map(&map_out, out, max_rows, N))) return (int)cudaErrorInvalidValue;
+  if (!(MODE != TC_DOWN ? make_store_map(&map_out, out, max_rows, N) : make_add_map(&map_out, out, max_rows, N))) return (int)cudaErrorInvalidValue;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(moe_tc_kernel<GATED, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmemBytes);
+    cudaError_t e = cudaFuncSetAttribute(moe_tc_kernel<MODE, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmemBytes);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   constexpr int kTileN = GATED ? kTcBN / 2 : kTcBN;
   const long long most = (long long)(max_rows / kBM) * ((N + kTileN - 1) / kTileN);
   const int sm_count = device_sm_count();
-  return (int)launch_pdl(moe_tc_kernel<GATED, ACT>, dim3((unsigned)(most < sm_count ? most : sm_count)), dim3(kGemmThreads), kTcSmemBytes, stream, map_a, map_b, map_out,
+  return (int)launch_pdl(moe_tc_kernel<MODE, ACT>, dim3((unsigned)(most < sm_count ? most : sm_count)), dim3(kGemmThreads), kTcSmemBytes, stream, map_a, map_b, map_out,
                          meta, N, K, error_flag);
 }
 
@@ -331,13 +343,13 @@ using namespace tlie;
 
 // Scratch, with max_rows = (tokens * top / 128 + experts) * 128: row_of_slot int32 [tokens * top], token_of_row int32 [max_rows],
 // meta int32 [1 + max_rows / 128], xs bfloat16 [max_rows, width], act bfloat16 [max_rows, ff], y 32-bit [max_rows, width].
-// ``shared`` bfloat16 [tokens, width] or null.  All of 16-byte aligned bases; width and ff multiples of 8.
-TLIE_EXPORT int tlie_moe_grouped_tc(const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, int* row_of_slot,
+// ``shared`` bfloat16 [tokens, width] or null, times ``shared_gate`` [tokens] unless that is null.  All of 16-byte aligned bases; width and ff multiples of 8.
+TLIE_EXPORT int tlie_moe_grouped_tc(const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, const float* shared_gate, int* row_of_slot,
                                     int* token_of_row, int* meta, void* xs, void* act, float* y, void* out, int tokens, int width, int ff, int experts, int top,
                                     int kind, int weight_input, int* error_flag, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   const long long slots = (long long)tokens * top;
-  if (width % 8 != 0 || ff % 8 != 0 || experts <= 0 || experts > 4096 || slots > (1LL << 30) || kind < 0 || kind > 1 || error_flag == nullptr) return (int)cudaErrorInvalidValue;
+  if (width % 8 != 0 || ff % 8 != 0 || experts <= 0 || experts > 4096 || slots > (1LL << 30) || kind < 0 || kind > 2 || error_flag == nullptr) return (int)cudaErrorInvalidValue;
   if ((long long)experts * 2 * ff > 2147483647LL || (long long)experts * width > 2147483647LL) return (int)cudaErrorInvalidValue;
   const int max_rows = ((int)(slots / kBM) + experts) * kBM;
   moe_layout_kernel<<<1, 1024, 2 * experts * sizeof(int), stream>>>(ids, (int)slots, experts, top, max_rows, row_of_slot, token_of_row, meta);
@@ -346,14 +358,15 @@ TLIE_EXPORT int tlie_moe_grouped_tc(const void* x, const void* gate_up, const vo
   moe_gather_kernel<<<max_rows / 8, 256, 0, stream>>>((const __nv_bfloat16*)x, token_of_row, meta, weight_input ? weights : nullptr, (__nv_bfloat16*)xs, width, top);
   e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
-  int rc = kind == 1 ? launch_moe_tc<true, 1>(xs, gate_up, act, meta, max_rows, experts * 2 * ff, ff, width, error_flag, stream)
-                     : launch_moe_tc<true, 0>(xs, gate_up, act, meta, max_rows, experts * 2 * ff, ff, width, error_flag, stream);
+  int rc = kind == 2   ? launch_moe_tc<TC_PLAIN, 2>(xs, gate_up, act, meta, max_rows, experts * ff, ff, width, error_flag, stream)
+           : kind == 1 ? launch_moe_tc<TC_GATED, 1>(xs, gate_up, act, meta, max_rows, experts * 2 * ff, ff, width, error_flag, stream)
+                       : launch_moe_tc<TC_GATED, 0>(xs, gate_up, act, meta, max_rows, experts * 2 * ff, ff, width, error_flag, stream);
   if (rc != 0) return rc;
-  rc = launch_moe_tc<false, 0>(act, down, y, meta, max_rows, experts * width, width, ff, error_flag, stream);
+  rc = launch_moe_tc<TC_DOWN, 0>(act, down, y, meta, max_rows, experts * width, width, ff, error_flag, stream);
   if (rc != 0) return rc;
   const size_t quads = (size_t)tokens * (width / 4);
   const size_t blocks = (quads + 255) / 256;
   const size_t most = (size_t)device_sm_count() * 16;
-  moe_tc_combine_kernel<<<(int)(blocks < most ? blocks : most), 256, 0, stream>>>(y, row_of_slot, weight_input ? nullptr : weights, (const __nv_bfloat16*)shared, (__nv_bfloat16*)out, width, top, quads);
+  moe_tc_combine_kernel<<<(int)(blocks < most ? blocks : most), 256, 0, stream>>>(y, row_of_slot, weight_input ? nullptr : weights, (const __nv_bfloat16*)shared, shared_gate, (__nv_bfloat16*)out, width, top, quads);
   return (int)cudaGetLastError();
 }

@@ -1,9 +1,10 @@
 // Norms around a residual branch, for layers that normalise a sublayer's output before it joins the stream:
 //
-//   residual[t] += norm(y[t]) * post_weight          (if y is given)
-//   out[r]       = norm(residual[rows[r]]) * next_weight   (if out is given; rows null: every row in order)
+//   residual[t] += norm(y[t]) * post_weight + post_bias          (if y is given; the bias may be null)
+//   out[r]       = norm(residual[rows[r]]) * next_weight + next_bias   (if out is given; rows null: every row in order; bias null: none)
+//   out[r]       = residual[rows[r]]                              (next_weight null: the finished stream, rounded to out's type)
 //
-// in one kernel, a CTA per row.  ``centred`` 1: (x - mean) / sqrt(mean((x - mean)^2) + eps), the layer norm without a bias;
+// in one kernel, a CTA per row.  ``centred`` 1: (x - mean) / sqrt(mean((x - mean)^2) + eps), the layer norm;
 // 0: x / sqrt(mean(x^2) + eps).  ``groups`` > 1: the statistics are taken over each of that many equal consecutive parts of the row.  The row waits in shared memory as 32-bit numbers between the passes; mean, variance (of
 // the deviations, after the mean is known), the sum into the stream and the second norm are 32-bit whatever y and out are
 // stored as.  The order of a row's sums depends on the block size alone.
@@ -76,7 +77,8 @@ __device__ __forceinline__ void store8(__nv_bfloat16* dst, const float (&v)[8]) 
 // eight numbers t, t + block, ...  Which of the two kernels runs depends on the width alone, so a row's bits do not depend on the step.
 template <typename TY, typename TO>
 __global__ void __launch_bounds__(kNormThreads) branch_norm_wide_kernel(float* __restrict__ residual, const TY* __restrict__ y, const float* __restrict__ post_weight,
-                                                                        const float* __restrict__ next_weight, TO* __restrict__ out, const int* __restrict__ rows,
+                                                                        const float* __restrict__ post_bias, const float* __restrict__ next_weight,
+                                                                        const float* __restrict__ next_bias, TO* __restrict__ out, const int* __restrict__ rows,
                                                                         float eps, int centred, int width, int groups) {
   extern __shared__ __align__(16) float norm_row[];
   __shared__ float scratch[32];
@@ -84,7 +86,11 @@ __global__ void __launch_bounds__(kNormThreads) branch_norm_wide_kernel(float* _
   const int source = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
   float* stream = residual + (size_t)source * width;
   const int part = width / groups;   // a multiple of 8 here: a run of eight lies in one group
-  float a[8], b[8], w[8];
+  TO* dst = out + (size_t)blockIdx.x * width;
+  const bool copies = out != nullptr && next_weight == nullptr;   // the finished stream itself is what is read next
+  float a[8], b[8], w[8], c[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) c[j] = 0.0f;
   if (y != nullptr) {
     const TY* branch = y + (size_t)source * width;
     for (int i = threadIdx.x * 8; i < width; i += blockDim.x * 8) {
@@ -96,36 +102,46 @@ __global__ void __launch_bounds__(kNormThreads) branch_norm_wide_kernel(float* _
     for (int i = threadIdx.x * 8; i < width; i += blockDim.x * 8) {   // a thread's own runs again
       load8(stream + i, b);
       load8(post_weight + i, w);
+      if (post_bias != nullptr) load8(post_bias + i, c);
       load8(norm_row + i, a);
       const float mean = means[i / part], inv = invs[i / part];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) b[j] = b[j] + ((a[j] - mean) * inv) * w[j];
+      for (int j = 0; j < 8; ++j) b[j] = b[j] + (((a[j] - mean) * inv) * w[j] + c[j]);
       store8(stream + i, b);
-      store8(norm_row + i, b);
+      if (copies)
+        store8(dst + i, b);
+      else
+        store8(norm_row + i, b);
     }
   } else {
     for (int i = threadIdx.x * 8; i < width; i += blockDim.x * 8) {
       load8(stream + i, b);
-      store8(norm_row + i, b);
+      if (copies)
+        store8(dst + i, b);
+      else
+        store8(norm_row + i, b);
     }
   }
-  if (out == nullptr) return;
+  if (out == nullptr || copies) return;
   __syncthreads();
   group_statistics(norm_row, width, groups, centred, eps, scratch, means, invs);
-  TO* dst = out + (size_t)blockIdx.x * width;
+#pragma unroll
+  for (int j = 0; j < 8; ++j) c[j] = 0.0f;
   for (int i = threadIdx.x * 8; i < width; i += blockDim.x * 8) {
     load8(next_weight + i, w);
+    if (next_bias != nullptr) load8(next_bias + i, c);
     load8(norm_row + i, a);
     const float mean = means[i / part], inv = invs[i / part];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) a[j] = ((a[j] - mean) * inv) * w[j];
+    for (int j = 0; j < 8; ++j) a[j] = ((a[j] - mean) * inv) * w[j] + c[j];
     store8(dst + i, a);
   }
 }
 
 template <typename TY, typename TO>
 __global__ void __launch_bounds__(kNormThreads) branch_norm_kernel(float* __restrict__ residual, const TY* __restrict__ y, const float* __restrict__ post_weight,
-                                                                   const float* __restrict__ next_weight, TO* __restrict__ out, const int* __restrict__ rows,
+                                                                   const float* __restrict__ post_bias, const float* __restrict__ next_weight,
+                                                                   const float* __restrict__ next_bias, TO* __restrict__ out, const int* __restrict__ rows,
                                                                    float eps, int centred, int width, int groups) {
   extern __shared__ float norm_row[];
   __shared__ float scratch[32];
@@ -139,7 +155,7 @@ __global__ void __launch_bounds__(kNormThreads) branch_norm_kernel(float* __rest
     __syncthreads();
     group_statistics(norm_row, width, groups, centred, eps, scratch, means, invs);
     for (int i = threadIdx.x; i < width; i += blockDim.x) {   // every thread rereads what it wrote itself
-      const float v = stream[i] + ((norm_row[i] - means[i / part]) * invs[i / part]) * post_weight[i];
+      const float v = stream[i] + (((norm_row[i] - means[i / part]) * invs[i / part]) * post_weight[i] + (post_bias != nullptr ? post_bias[i] : 0.0f));
       stream[i] = v;
       norm_row[i] = v;
     }
@@ -147,10 +163,15 @@ __global__ void __launch_bounds__(kNormThreads) branch_norm_kernel(float* __rest
     for (int i = threadIdx.x; i < width; i += blockDim.x) norm_row[i] = stream[i];
   }
   if (out == nullptr) return;
+  TO* dst = out + (size_t)blockIdx.x * width;
+  if (next_weight == nullptr) {   // the finished stream itself is what is read next (a thread's own numbers again)
+    for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = from_float<TO>(norm_row[i]);
+    return;
+  }
   __syncthreads();
   group_statistics(norm_row, width, groups, centred, eps, scratch, means, invs);
-  TO* dst = out + (size_t)blockIdx.x * width;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = from_float<TO>(((norm_row[i] - means[i / part]) * invs[i / part]) * next_weight[i]);
+  for (int i = threadIdx.x; i < width; i += blockDim.x)
+    dst[i] = from_float<TO>(((norm_row[i] - means[i / part]) * invs[i / part]) * next_weight[i] + (next_bias != nullptr ? next_bias[i] : 0.0f));
 }
 
 template <typename T>
@@ -172,8 +193,8 @@ __global__ void stream_with_embedding_kernel(const float* __restrict__ residual,
 }
 
 template <typename TY, typename TO>
-static int launch_branch_norm(float* residual, const void* y, const float* post_weight, const float* next_weight, void* out, const int* rows, float eps,
-                              int centred, int count, int width, int groups, cudaStream_t stream) {
+static int launch_branch_norm(float* residual, const void* y, const float* post_weight, const float* post_bias, const float* next_weight, const float* next_bias,
+                              void* out, const int* rows, float eps, int centred, int count, int width, int groups, cudaStream_t stream) {
   const size_t smem = (size_t)width * sizeof(float);
   if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
   if (smem > 48 * 1024) {
@@ -181,15 +202,16 @@ static int launch_branch_norm(float* residual, const void* y, const float* post_
     if (e != cudaSuccess) return (int)e;
   }
   const auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-  if (width % 8 == 0 && (width / groups) % 8 == 0 && aligned(residual) && aligned(y) && aligned(post_weight) && aligned(next_weight) && aligned(out)) {
+  if (width % 8 == 0 && (width / groups) % 8 == 0 && aligned(residual) && aligned(y) && aligned(post_weight) && aligned(post_bias) && aligned(next_weight) &&
+      aligned(next_bias) && aligned(out)) {
     if (smem > 48 * 1024) {
       cudaError_t e = cudaFuncSetAttribute(branch_norm_wide_kernel<TY, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return (int)e;
     }
-    branch_norm_wide_kernel<TY, TO><<<count, kNormThreads, smem, stream>>>(residual, (const TY*)y, post_weight, next_weight, (TO*)out, rows, eps, centred, width, groups);
+    branch_norm_wide_kernel<TY, TO><<<count, kNormThreads, smem, stream>>>(residual, (const TY*)y, post_weight, post_bias, next_weight, next_bias, (TO*)out, rows, eps, centred, width, groups);
     return (int)cudaGetLastError();
   }
-  branch_norm_kernel<TY, TO><<<count, kNormThreads, smem, stream>>>(residual, (const TY*)y, post_weight, next_weight, (TO*)out, rows, eps, centred, width, groups);
+  branch_norm_kernel<TY, TO><<<count, kNormThreads, smem, stream>>>(residual, (const TY*)y, post_weight, post_bias, next_weight, next_bias, (TO*)out, rows, eps, centred, width, groups);
   return (int)cudaGetLastError();
 }
 
@@ -199,14 +221,15 @@ using namespace tlie;
 
 // ``count`` rows are worked on: all of the stream's, or with ``rows`` the listed ones (then y must be null: a gathered norm adds nothing).
 // ``y`` and ``out`` are of ``dtype``; either may be null.
+// ``post_bias`` / ``next_bias`` null: a norm without a bias; ``next_weight`` null: ``out`` is the finished stream, rounded.
 // ``groups``: the norms' statistics are taken over each of that many equal consecutive parts of a row (1: over the whole row).
-TLIE_EXPORT int tlie_branch_norm(int dtype, float* residual, const void* y, const float* post_weight, const float* next_weight, void* out, const int* rows,
-                                 float eps, int centred, int count, int width, int groups, cudaStream_t stream) {
+TLIE_EXPORT int tlie_branch_norm(int dtype, float* residual, const void* y, const float* post_weight, const float* post_bias, const float* next_weight,
+                                 const float* next_bias, void* out, const int* rows, float eps, int centred, int count, int width, int groups, cudaStream_t stream) {
   if (count <= 0) return 0;
-  if (groups < 1 || groups > kNormMaxGroups || width % groups != 0 || width <= 0 || (rows != nullptr && y != nullptr) || (y != nullptr && post_weight == nullptr) || (out != nullptr && next_weight == nullptr))
+  if (groups < 1 || groups > kNormMaxGroups || width % groups != 0 || width <= 0 || (rows != nullptr && y != nullptr) || (y != nullptr && post_weight == nullptr))
     return (int)cudaErrorInvalidValue;
-  if (dtype == TLIE_F32) return launch_branch_norm<float, float>(residual, y, post_weight, next_weight, out, rows, eps, centred, count, width, groups, stream);
-  return launch_branch_norm<__nv_bfloat16, __nv_bfloat16>(residual, y, post_weight, next_weight, out, rows, eps, centred, count, width, groups, stream);
+  if (dtype == TLIE_F32) return launch_branch_norm<float, float>(residual, y, post_weight, post_bias, next_weight, next_bias, out, rows, eps, centred, count, width, groups, stream);
+  return launch_branch_norm<__nv_bfloat16, __nv_bfloat16>(residual, y, post_weight, post_bias, next_weight, next_bias, out, rows, eps, centred, count, width, groups, stream);
 }
 
 TLIE_EXPORT int tlie_stream_with_embedding(int dtype, const float* residual, const void* table, const int* ids, float scale, void* out, int rows, int width,

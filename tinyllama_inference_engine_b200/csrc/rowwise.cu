@@ -6,7 +6,9 @@
 //   scale_rows          x *= factor (32-bit, in place)
 //   gather_gated        out[t, d] = act(z[t, d]) * table[ids[t], offset + d]           a slice of a second token table, gated
 //   unit_norm_add       residual[t] += y[t] / sqrt(mean(y[t]^2) + eps) * weight        a normalised branch joins the stream
-//   head_linear         out[t, h, :] = W[h] . x[t, h, :]  per head, operands with strides of their own, 32-bit sums in a fixed order
+//   head_linear         out[t, h, :] = W[h] . x[t, h, :]  per head, operands with strides of their own, 32-bit sums in a fixed order; optionally gated
+//   sigmoid_gate        x[t, i] *= sigmoid(gate[t, i])
+//   add_bias            x[t, i] += bias[i]
 // Storage float or bfloat16, arithmetic 32-bit.
 #include "common.cuh"
 
@@ -111,11 +113,40 @@ __global__ void unit_norm_add_kernel(float* __restrict__ residual, const T* __re
   for (int i = threadIdx.x + kKept * blockDim.x; i < hidden; i += blockDim.x) residual[row * hidden + i] += to_float(y[row * hidden + i]) * inv * weight[i];
 }
 
-// out[t, h, n] = sum_k x[t, h, k] * w[h, n, k]: a warp per output, the lanes taking k in turns (neighbouring lanes read neighbouring
+// x[t, i] *= sigmoid(gate[t, i]), rows of both with strides of their own.
+template <typename T>
+__global__ void sigmoid_gate_kernel(T* __restrict__ x, long long x_row, const T* __restrict__ gate, long long gate_row, int width, size_t total) {
+  for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / width;
+    const int c = (int)(i - t * width);
+    T* at = x + t * x_row + c;
+    *at = from_float<T>(to_float(*at) * (1.0f / (1.0f + expf(-to_float(gate[t * gate_row + c])))));
+  }
+}
+
+// the same, eight bfloat16 numbers a thread (width and strides multiples of 8, 16-byte aligned bases)
+__global__ void sigmoid_gate_vec_kernel(__nv_bfloat16* __restrict__ x, long long x_row, const __nv_bfloat16* __restrict__ gate, long long gate_row, int width8, size_t total8) {
+  for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total8; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / width8;
+    const int c = (int)(i - t * width8) * 8;
+    uint4 raw = *reinterpret_cast<const uint4*>(x + t * x_row + c);
+    const uint4 graw = *reinterpret_cast<const uint4*>(gate + t * gate_row + c);
+    __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&raw);
+    const __nv_bfloat162* gates = reinterpret_cast<const __nv_bfloat162*>(&graw);
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      const float2 v = __bfloat1622float2(pairs[n]), g = __bfloat1622float2(gates[n]);
+      pairs[n] = __floats2bfloat162_rn(v.x * (1.0f / (1.0f + expf(-g.x))), v.y * (1.0f / (1.0f + expf(-g.y))));
+    }
+    *reinterpret_cast<uint4*>(x + t * x_row + c) = raw;
+  }
+}
+
+// out[t, h, n] = sum_k x[t, h, k] * w[h, n, k], times sigmoid(gate[t, h N + n]) if there is a gate: a warp per output, the lanes taking k in turns (neighbouring lanes read neighbouring
 // elements) and adding up in a fixed order, so a row's bits depend on the row alone.
 template <typename T>
 __global__ void head_linear_kernel(const T* __restrict__ x, long long x_row, long long x_head, const T* __restrict__ w, T* __restrict__ out, long long out_row,
-                                   long long out_head, int heads, int n_out, int k_in, size_t total) {
+                                   long long out_head, int heads, int n_out, int k_in, const T* __restrict__ gate, long long gate_row, size_t total) {
   const int lane = threadIdx.x & 31;
   const size_t warps = ((size_t)gridDim.x * blockDim.x) >> 5;
   for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) >> 5; i < total; i += warps) {
@@ -127,8 +158,18 @@ __global__ void head_linear_kernel(const T* __restrict__ x, long long x_row, lon
     float sum = 0.0f;
     for (int k = lane; k < k_in; k += 32) sum += to_float(xr[k]) * to_float(wr[k]);
     sum = warp_sum(sum);
-    if (lane == 0) out[t * out_row + h * out_head + n] = from_float<T>(sum);
+    if (lane == 0) {
+      if (gate != nullptr) sum *= 1.0f / (1.0f + expf(-to_float(gate[t * gate_row + (long long)h * n_out + n])));
+      out[t * out_row + h * out_head + n] = from_float<T>(sum);
+    }
   }
+}
+
+// x[t, c] += bias[c], 32-bit inside.
+template <typename T>
+__global__ void add_bias_kernel(T* __restrict__ x, const float* __restrict__ bias, int width, size_t count) {
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < count) x[i] = from_float<T>(to_float(x[i]) + bias[i % width]);
 }
 
 static inline int blocks_for(size_t total, int threads) {
@@ -198,10 +239,33 @@ TLIE_EXPORT int tlie_unit_norm_add(int dtype, float* residual, const void* y, co
 }
 
 TLIE_EXPORT int tlie_head_linear(int dtype, const void* x, long long x_row, long long x_head, const void* w, void* out, long long out_row, long long out_head,
-                                 int rows, int heads, int n_out, int k_in, cudaStream_t stream) {
+                                 int rows, int heads, int n_out, int k_in, const void* gate, long long gate_row, cudaStream_t stream) {
   const size_t total = (size_t)rows * heads * n_out;
   if (total == 0) return 0;
   TLIE_BY_TYPE(dtype, (head_linear_kernel<T><<<blocks_for(total * 32, 256), 256, 0, stream>>>((const T*)x, x_row, x_head, (const T*)w, (T*)out, out_row, out_head, heads,
-                                                                                       n_out, k_in, total)));
+                                                                                       n_out, k_in, (const T*)gate, gate_row, total)));
+  return (int)cudaGetLastError();
+}
+
+TLIE_EXPORT int tlie_add_bias(int dtype, void* x, const float* bias, int rows, int width, cudaStream_t stream) {
+  const size_t count = (size_t)rows * width;
+  if (count == 0) return 0;
+  const int blocks = (int)((count + 255) / 256);
+  if (dtype == TLIE_F32)
+    add_bias_kernel<float><<<blocks, 256, 0, stream>>>((float*)x, bias, width, count);
+  else
+    add_bias_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((__nv_bfloat16*)x, bias, width, count);
+  return (int)cudaGetLastError();
+}
+
+TLIE_EXPORT int tlie_sigmoid_gate(int dtype, void* x, long long x_row, const void* gate, long long gate_row, int rows, int width, cudaStream_t stream) {
+  const size_t total = (size_t)rows * width;
+  if (total == 0) return 0;
+  const auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (dtype == TLIE_BF16 && width % 8 == 0 && x_row % 8 == 0 && gate_row % 8 == 0 && aligned(x) && aligned(gate)) {
+    sigmoid_gate_vec_kernel<<<blocks_for(total / 8, 256), 256, 0, stream>>>((__nv_bfloat16*)x, x_row, (const __nv_bfloat16*)gate, gate_row, width / 8, total / 8);
+    return (int)cudaGetLastError();
+  }
+  TLIE_BY_TYPE(dtype, (sigmoid_gate_kernel<T><<<blocks_for(total, 256), 256, 0, stream>>>((T*)x, x_row, (const T*)gate, gate_row, width, total)));
   return (int)cudaGetLastError();
 }

@@ -8,7 +8,6 @@
 //   conv_residual        out[t, c] = x[t, c] + sum_j taps[c, j] x[t - n + 1 + j, c]  (zeros before a request's start; the last n - 1
 //                        inputs of a request are its state, moved on by ``conv_inputs_keep``).  32-bit inside.
 //   scaled_sum           out = a * x + b * y, 32-bit inside: two branches that read the same input join.
-//   add_bias             x[t, c] += bias[c], 32-bit inside.
 #include <cstdint>
 #include "common.cuh"
 
@@ -187,12 +186,6 @@ __global__ void scaled_sum_kernel(const T* __restrict__ x, const T* __restrict__
   if (i < count) out[i] = from_float<T>(a * to_float(x[i]) + b * to_float(y[i]));
 }
 
-template <typename T>
-__global__ void add_bias_kernel(T* __restrict__ x, const float* __restrict__ bias, int width, size_t count) {
-  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < count) x[i] = from_float<T>(to_float(x[i]) + bias[i % width]);
-}
-
 }  // namespace tlie
 
 using namespace tlie;
@@ -265,13 +258,3 @@ TLIE_EXPORT int tlie_scaled_sum(int dtype, const void* x, const void* y, float a
   return (int)cudaGetLastError();
 }
 
-TLIE_EXPORT int tlie_add_bias(int dtype, void* x, const float* bias, int rows, int width, cudaStream_t stream) {
-  const size_t count = (size_t)rows * width;
-  if (count == 0) return 0;
-  const int blocks = (int)((count + 255) / 256);
-  if (dtype == TLIE_F32)
-    add_bias_kernel<float><<<blocks, 256, 0, stream>>>((float*)x, bias, width, count);
-  else
-    add_bias_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((__nv_bfloat16*)x, bias, width, count);
-  return (int)cudaGetLastError();
-}

@@ -150,17 +150,19 @@ def embedding_positions(table, place_table, ids, positions, norm_weight, eps: fl
            "embedding_positions")
 
 
-ACTIVATIONS = {"relu_squared": 0, "gelu_tanh": 1, "silu": 2}
+ACTIVATIONS = {"relu_squared": 0, "gelu_tanh": 1, "silu": 2, "xielu": 3}
 
 
-def activation(kind: str, x, out) -> None:
+def activation(kind: str, x, out, constants=(0.0, 0.0)) -> None:
     """out = act(x) element by element, 32-bit inside (``out`` may be ``x``): the square of relu, gelu in its tanh form
-    0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), or silu."""
+    0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), silu, or xielu with ``constants`` = (a, b): a z^2 + z / 2 for z > 0 and
+    b (e^z - 1 - z) + z / 2 below."""
     if kind not in ACTIVATIONS:
         raise KernelError(f"no activation {kind!r}; known: {sorted(ACTIVATIONS)}", code="invalid_argument")
     if out.shape != x.shape or out.dtype != x.dtype:
         raise KernelError("activation: the output must have the input's shape and dtype", code="invalid_shape")
-    _check(core().tlie_activation(_code(x), c_int(ACTIVATIONS[kind]), _ptr(x), _ptr(out), c_longlong(x.numel()), _stream()), "activation")
+    _check(core().tlie_activation(_code(x), c_int(ACTIVATIONS[kind]), _ptr(x), _ptr(out), c_longlong(x.numel()), c_float(constants[0]),
+                                   c_float(constants[1]), _stream()), "activation")
 
 
 def add_rmsnorm(residual, delta, weight, eps: float, out, rows=None) -> None:
@@ -205,10 +207,11 @@ def gate_mul(gate_up, out, kind: str = "silu") -> None:
     _check(core().tlie_gate_mul(_code(out), _ptr(gate_up), _ptr(out), c_int(rows), c_int(inter), c_int(GATE_KINDS[kind]), _stream()), "gate_mul")
 
 
-def branch_norm(residual, y, post_weight, next_weight, out, eps: float, centred: bool = True, rows=None, groups: int = 1) -> None:
-    """One kernel around a residual branch: ``residual += norm(y) * post_weight`` (if ``y`` is given), then
-    ``out = norm(residual[rows]) * next_weight`` (if ``out`` is given; ``rows`` None: every row in order, and only then may ``y`` be given).
-    ``centred``: the layer norm without a bias, (x - mean) / sqrt(mean((x - mean)^2) + eps); else x / sqrt(mean(x^2) + eps).
+def branch_norm(residual, y, post_weight, next_weight, out, eps: float, centred: bool = True, rows=None, groups: int = 1, post_bias=None, next_bias=None) -> None:
+    """One kernel around a residual branch: ``residual += norm(y) * post_weight + post_bias`` (if ``y`` is given), then
+    ``out = norm(residual[rows]) * next_weight + next_bias`` (if ``out`` is given; ``rows`` None: every row in order, and only then may ``y``
+    be given).  A bias may be None; ``next_weight`` None with an ``out``: ``out`` is the finished stream itself, rounded to its dtype.
+    ``centred``: the layer norm, (x - mean) / sqrt(mean((x - mean)^2) + eps); else x / sqrt(mean(x^2) + eps).
     ``groups``: the statistics are taken over each of that many equal consecutive parts of a row.
     The stream, the statistics and the weights are 32-bit; ``y`` and ``out`` share a dtype."""
     width = residual.shape[1]
@@ -217,15 +220,16 @@ def branch_norm(residual, y, post_weight, next_weight, out, eps: float, centred:
     count = residual.shape[0] if rows is None else rows.shape[0]
     if residual.dtype != torch.float32 or (y is not None and (y.shape != residual.shape or rows is not None)) or (out is not None and out.shape != (count, width)):
         raise KernelError("branch_norm: a 32-bit stream [T, width], y of its shape, out [rows, width]", code="invalid_shape")
-    for weight in (post_weight, next_weight):
+    for weight in (post_weight, next_weight, post_bias, next_bias):
         if weight is not None and (weight.dtype != torch.float32 or weight.numel() != width):
-            raise KernelError("branch_norm: norm weights are 32-bit [width]", code="invalid_shape")
+            raise KernelError("branch_norm: norm weights and biases are 32-bit [width]", code="invalid_shape")
     if y is not None and out is not None and y.dtype != out.dtype:
         raise KernelError("branch_norm: y and out share a dtype", code="invalid_dtype")
     if y is None and out is None:
         return
     _check(core().tlie_branch_norm(_code(y if y is not None else out), _ptr(residual), _ptr(y), _ptr(post_weight if y is not None else None),
-                                   _ptr(next_weight if out is not None else None), _ptr(out), _i32(rows, "rows"), c_float(eps), c_int(1 if centred else 0),
+                                   _ptr(post_bias if y is not None else None), _ptr(next_weight if out is not None else None), _ptr(next_bias if out is not None else None),
+                                   _ptr(out), _i32(rows, "rows"), c_float(eps), c_int(1 if centred else 0),
                                    c_int(count), c_int(width), c_int(groups), _stream()), "branch_norm")
 
 
@@ -291,8 +295,9 @@ def unit_norm_add(residual, y, weight, eps: float) -> None:
 HEAD_LINEAR_LIBRARY_ROWS = 64    # from this many bfloat16 rows on the per-head product is one batched library product
 
 
-def head_linear(x, weight, out) -> None:
-    """out[t, h, :] = weight[h] . x[t, h, :] for every head: x [T, H, K] and out [T, H, N] may be views with strides of their own
+def head_linear(x, weight, out, gate=None) -> None:
+    """out[t, h, :] = weight[h] . x[t, h, :] for every head, times sigmoid(gate[t, h, :]) if a ``gate`` [T, H N] is given (its rows may be a run of columns of
+    wider ones): x [T, H, K] and out [T, H, N] may be views with strides of their own
     (last axis contiguous), weight [H, N, K] contiguous.  32-bit sums, ascending k (a row's bits depend on the row alone) in the
     engine's own kernel; bfloat16 steps of many rows go to the library's batched product, as the other products of their size do."""
     rows, heads, k_in = x.shape
@@ -301,13 +306,20 @@ def head_linear(x, weight, out) -> None:
         raise KernelError("head_linear: x [T, H, K], weight [H, N, K], out [T, H, N] with contiguous last axes", code="invalid_shape")
     if x.dtype != weight.dtype or out.dtype != x.dtype:
         raise KernelError("head_linear: one dtype for x, weight and out", code="invalid_dtype")
+    if gate is not None and (gate.shape != (rows, heads * n_out) or gate.dtype != out.dtype or gate.stride(1) != 1 or out.stride(1) != n_out):
+        raise KernelError("head_linear: the gate is [T, H N] of the output's dtype, the output's heads side by side", code="invalid_shape")
     if not x.is_cuda:
         raise KernelError("this engine has no CPU path: a kernel was given a tensor that is not on a CUDA device")
+    gate_ptr, gate_stride = (c_void_p(0), 0) if gate is None else (c_void_p(gate.data_ptr()), gate.stride(0))
     if x.dtype == torch.bfloat16 and rows >= HEAD_LINEAR_LIBRARY_ROWS:
         torch.bmm(x.transpose(0, 1), weight.transpose(1, 2), out=out.transpose(0, 1))
+        if gate is not None:
+            _check(core().tlie_sigmoid_gate(_code(out), c_void_p(out.data_ptr()), c_longlong(out.stride(0)), gate_ptr, c_longlong(gate_stride), c_int(rows),
+                                            c_int(heads * n_out), _stream()), "sigmoid_gate")
         return
     _check(core().tlie_head_linear(_code(x), c_void_p(x.data_ptr()), c_longlong(x.stride(0)), c_longlong(x.stride(1)), _ptr(weight), c_void_p(out.data_ptr()),
-                                   c_longlong(out.stride(0)), c_longlong(out.stride(1)), c_int(rows), c_int(heads), c_int(n_out), c_int(k_in), _stream()), "head_linear")
+                                   c_longlong(out.stride(0)), c_longlong(out.stride(1)), c_int(rows), c_int(heads), c_int(n_out), c_int(k_in), gate_ptr,
+                                   c_longlong(gate_stride), _stream()), "head_linear")
 
 
 def linear(x, weight, out) -> None:
@@ -359,6 +371,16 @@ class LazyNorm:
         return self._materialize()
 
 
+class StreamCopy(LazyNorm):
+    """The finished residual stream beside a copy of it in the activations' dtype (the stream itself in the 32-bit path): what a block
+    leaves pending when the next one reads the stream without a norm.  No norm is prepared here: nobody's weight is this one's."""
+
+    def __init__(self, residual, copy):
+        super().__init__(residual, None, 0.0, None, lambda: copy)
+        self.prepared = None
+        self.copy = copy
+
+
 def norm_linear(x: "LazyNorm", weight, out, gated: bool = False, clamp=None) -> None:
     """out = rmsnorm(residual) * norm_weight . weight^T in one kernel (``gated``: silu(gate) * up of the two halves; with ``clamp`` =
     (limit, alpha, shift) the clamped gate of ``clamped_gate_mul`` instead)."""
@@ -381,26 +403,36 @@ def norm_linear(x: "LazyNorm", weight, out, gated: bool = False, clamp=None) -> 
         linear(x.tensor(), weight, out)
 
 
-def linear_activated(x, weight, out, kind: str) -> None:
+def linear_activated(x, weight, out, kind: str, constants=(0.0, 0.0)) -> None:
     """out = act(x . weight^T), the activation applied to the product as it is stored (rounded to the output's dtype first, as when
     the product is stored and ``activation`` run over it).  ``x``: a tensor or a ``LazyNorm``.  One kernel for up to 16 bfloat16 rows
-    (norm in front, activation behind); a product and an elementwise kernel otherwise."""
+    (norm in front, activation behind); a product and an elementwise kernel otherwise.  ``constants``: what ``activation`` takes."""
     lazy = isinstance(x, LazyNorm)
     if out.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and fast.gemv_fits(out.shape[0], weight.shape[1], norm=lazy, N=None if lazy else weight.shape[0]):
         if lazy and x.prepared is not None:
-            fast.gemv_fused(x.prepared[0], weight, out, prepared=(x.prepared[1], x.eps), activation=kind)
+            fast.gemv_fused(x.prepared[0], weight, out, prepared=(x.prepared[1], x.eps), activation=kind, constants=constants)
             return
         if lazy:
-            fast.gemv_fused(x.residual, weight, out, norm=(x.weight, x.eps, x.rows), activation=kind)
+            fast.gemv_fused(x.residual, weight, out, norm=(x.weight, x.eps, x.rows), activation=kind, constants=constants)
             return
         if x.dtype == torch.bfloat16 and x.stride(1) == 1 and x.stride(0) % 8 == 0:
-            fast.gemv_fused(x, weight, out, activation=kind)
+            fast.gemv_fused(x, weight, out, activation=kind, constants=constants)
             return
     if lazy:
         norm_linear(x, weight, out)
     else:
         linear(x, weight, out)
-    activation(kind, out, out)
+    activation(kind, out, out, constants)
+
+
+def linear_bias(x, weight, bias, out) -> None:
+    """out = x . weight^T + bias (32-bit [N]).  Up to 16 bfloat16 rows: one kernel, the bias added to the 32-bit sums; otherwise the product
+    and a kernel that adds the bias."""
+    if out.dtype == torch.bfloat16 and fast.gemv_fits(x.shape[0], weight.shape[1], norm=False, N=weight.shape[0]) and x.stride(1) == 1 and x.stride(0) % 8 == 0:
+        fast.gemv_fused(x, weight, out, bias=bias)
+        return
+    linear(x, weight, out)
+    add_bias(out, bias)
 
 
 def can_accumulate(rows: int, weight) -> bool:
@@ -735,7 +767,7 @@ def add_bias(x, bias) -> None:
     """x[t, c] += bias[c] in place (``bias`` 32-bit [width]), 32-bit inside."""
     if bias.dtype != torch.float32 or x.dim() != 2 or bias.numel() != x.shape[1]:
         raise KernelError("add_bias: x [rows, width], bias 32-bit [width]", code="invalid_shape")
-    _check(sequence_library().tlie_add_bias(_code(x), _ptr(x), _ptr(bias), c_int(x.shape[0]), c_int(x.shape[1]), _stream()), "add_bias")
+    _check(core().tlie_add_bias(_code(x), _ptr(x), _ptr(bias), c_int(x.shape[0]), c_int(x.shape[1]), _stream()), "add_bias")
 
 
 def scaled_sum(x, y, a: float, b: float, out) -> None:
@@ -786,21 +818,37 @@ def _latent_plane(cache, width: int):
     return pages
 
 
-def latent_store(rows, latent_offset: int, weight, eps: float, inv_freq, rot_dims: int, positions, token_seq, cache, queries, heads: int, plain: int, rot: int, rank: int) -> None:
-    """Latent attention's cache write and rotation: ``rows[:, latent_offset:]`` = [rank | rot] becomes [rms-normed latent (32-bit ``weight``) |
-    rotated shared key part] in the token's cache row; the ``rot`` columns behind the ``plain`` ones of every query head are rotated into
-    ``queries`` [T, heads * (rank + rot)], behind each head's first ``rank`` columns (which are left alone).
-    Pairs (2i, 2i + 1) of the first ``rot_dims`` columns turn by position * inv_freq[i]."""
+def latent_store(rows, latent_offset: int, weight, eps: float, inv_freq, rot_dims: int, positions, token_seq, cache, queries, heads: int, plain: int, rot: int, rank: int,
+                 interleaved: bool = True, amplitude: float = 1.0, query_rows=None, q_latent=None) -> None:
+    """Latent attention's norms, rotation and cache write: ``rows[:, latent_offset:]`` = [rank | rot] becomes [rms-normed latent (32-bit ``weight``) |
+    rotated shared key part] in the token's cache row (``rows`` None: this part is left out); the ``rot`` columns behind the ``plain`` ones of
+    every query head of ``query_rows`` [T, heads * (plain + rot)] (None: of the first columns of ``rows``) are rotated into ``queries``
+    [T, heads * (rank + rot)], behind each head's first ``rank`` columns, which are left alone (``queries`` None: this part is left out).
+    The first ``rot_dims`` columns turn by position * inv_freq[i], cosines and sines times ``amplitude``: columns (2i, 2i + 1) together if
+    ``interleaved``, else column i with column i + rot_dims / 2.  ``q_latent`` = (offset, 32-bit weight, out): the queries' own latent, the columns of
+    ``rows`` from ``offset`` on, rms-normed into ``out`` [T, its width]."""
     pages = _latent_plane(cache, rank + rot)
-    if queries.shape != (rows.shape[0], heads * (rank + rot)) or queries.dtype != rows.dtype:
+    some = rows if rows is not None else query_rows
+    tokens = some.shape[0]
+    if queries is not None and (queries.shape != (tokens, heads * (rank + rot)) or queries.dtype != some.dtype):
         raise KernelError("latent_store: queries must be [rows, heads * (rank + rot)] of the rows' dtype", code="invalid_shape")
-    if pages.dtype != rows.dtype or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dims // 2 or weight.dtype != torch.float32 or weight.numel() != rank:
+    if pages.dtype != some.dtype or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dims // 2 or weight.dtype != torch.float32 or weight.numel() != rank:
         raise KernelError("latent_store: pages of the rows' dtype; inv_freq [rot_dims / 2] and weight [rank] 32-bit", code="invalid_shape")
+    from_rows = queries is not None and query_rows is None
+    source = rows if from_rows else query_rows
+    if queries is not None and (source.shape[1] < heads * (plain + rot) or source.shape[0] != tokens or source.dtype != some.dtype):
+        raise KernelError("latent_store: the queries' rows are [T, heads * (plain + rot)] of one dtype with the others", code="invalid_shape")
+    q_offset, q_weight, q_out = q_latent if q_latent is not None else (0, None, None)
+    if q_out is not None and (rows is None or q_out.shape[0] != tokens or q_out.dtype != rows.dtype or q_weight.dtype != torch.float32 or q_weight.numel() != q_out.shape[1]):
+        raise KernelError("latent_store: the queries' latent is [T, its width] of the rows' dtype under a 32-bit weight", code="invalid_shape")
     table = cache.block_table
-    _check(mixed_attention().tlie_latent_store(_code(rows), _ptr(rows), c_int(rows.shape[1]), c_int(latent_offset), _ptr(weight), c_float(eps), _ptr(inv_freq), c_int(rot_dims),
-                                               _i32(positions, "positions"), _i32(token_seq, "token_seq"), _i32(table, "block_table"), c_int(table.shape[1]), _ptr(pages),
-                                               c_longlong(cache.page_size * (rank + rot)), c_int(rows.shape[0]), c_int(heads), c_int(plain), c_int(rot), c_int(rank),
-                                               c_int(cache.page_size), c_int(1 if cache.writes else 0), _ptr(queries), _stream()), "latent_store")
+    _check(mixed_attention().tlie_latent_store(_code(some), _ptr(rows), c_int(0 if rows is None else rows.shape[1]), c_int(latent_offset), _ptr(weight), c_float(eps),
+                                               _ptr(inv_freq), c_int(rot_dims), c_int(1 if interleaved else 0), c_float(amplitude), _i32(positions, "positions"),
+                                               _i32(token_seq, "token_seq"), _i32(table, "block_table"), c_int(table.shape[1]), _ptr(pages),
+                                               c_longlong(cache.page_size * (rank + rot)), c_int(tokens), c_int(heads), c_int(plain), c_int(rot), c_int(rank),
+                                               c_int(cache.page_size), c_int(1 if cache.writes else 0), _ptr(source if queries is not None else None),
+                                               c_int(0 if queries is None else source.shape[1]), _ptr(queries), _ptr(q_weight), c_int(q_offset),
+                                               c_int(0 if q_out is None else q_out.shape[1]), _ptr(q_out), _stream()), "latent_store")
 
 
 def store_kv_planes(rows, k_offset: int, v_offset: int, positions, token_seq, cache, kv_heads: int, key_dim: int, value_dim: int) -> None:
@@ -836,9 +884,33 @@ def rotary_store_planes(rows, k_offset: int, v_offset: int, biases, inv_freq, ro
                                                       c_int(1 if cache.writes else 0), _stream()), "rotary_store_planes")
 
 
+def norm_rotary_store(rows, k_offset: int, v_offset: int, biases, q_weight, k_weight, eps: float, q_factors, inv_freq, rot_dims: int, interleaved: bool, amplitude: float,
+                      positions, token_seq, cache, heads: int, kv_heads: int, key_dim: int, value_dim: int) -> None:
+    """Biases, a norm, a partial rotation and the cache write in one kernel.  Every q, k and v vector of ``rows`` gets its bias (``biases`` =
+    (q, k, v), 32-bit or None each, or None); q and k are divided by their root mean square (``eps`` inside the root) and multiplied by
+    ``q_weight`` / ``k_weight`` (32-bit [key_dim]; None: no norm); their first ``rot_dims`` columns turn by position * inv_freq[i], cosines and
+    sines times ``amplitude``, columns (2i, 2i + 1) together if ``interleaved``, else column i with column i + rot_dims / 2; query head h is
+    multiplied by ``q_factors[h]`` (32-bit [heads] or None).  q is left in place, k goes into the key plane and v into the value plane of the
+    token's page."""
+    pages, k_ptr, k_stride, v_ptr, v_stride = _plane_pointers(cache, kv_heads, key_dim, value_dim)
+    if pages.dtype != rows.dtype or rot_dims % 2 or rot_dims > key_dim or (rot_dims > 0 and (inv_freq is None or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dims // 2)):
+        raise KernelError("norm_rotary_store: pages of the rows' dtype; inv_freq 32-bit [rot_dims / 2], rot_dims even and at most key_dim", code="invalid_shape")
+    q_bias, k_bias, v_bias = biases if biases is not None else (None, None, None)
+    for tensor, count in ((q_bias, heads * key_dim), (k_bias, kv_heads * key_dim), (v_bias, kv_heads * value_dim), (q_weight, key_dim), (k_weight, key_dim), (q_factors, heads)):
+        if tensor is not None and (tensor.dtype != torch.float32 or tensor.numel() != count):
+            raise KernelError("norm_rotary_store: biases (one number per column), norm weights [key_dim] and factors [heads] are 32-bit", code="invalid_shape")
+    table = cache.block_table
+    _check(mixed_attention().tlie_norm_rotary_store(_code(rows), _ptr(rows), c_int(rows.shape[1]), c_int(k_offset), c_int(v_offset), _ptr(q_bias), _ptr(k_bias), _ptr(v_bias),
+                                                    _ptr(q_weight), _ptr(k_weight), c_float(eps), _ptr(q_factors), _ptr(inv_freq if rot_dims > 0 else None), c_int(rot_dims),
+                                                    c_int(1 if interleaved else 0), c_float(amplitude), _i32(positions, "positions"), _i32(token_seq, "token_seq"),
+                                                    _i32(table, "block_table"), c_int(table.shape[1]), k_ptr, c_longlong(k_stride), v_ptr, c_longlong(v_stride),
+                                                    c_int(rows.shape[0]), c_int(heads), c_int(kv_heads), c_int(key_dim), c_int(value_dim), c_int(cache.page_size),
+                                                    c_int(1 if cache.writes else 0), _stream()), "norm_rotary_store")
+
+
 def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, slopes, mix, out, heads: int, kv_heads: int, key_dim: int, value_dim: int,
                           window: int, scale: float, batch=None, folded_slopes=None, keep_first: int = 0, gate_per_head: bool = False, sinks=None,
-                          values_in_keys: bool = False) -> None:
+                          values_in_keys: bool = False, softcap: float = 0.0, sigmoid: bool = False, shifts=None) -> None:
     """Attention over the paged keys with a distance bias, the heads' scores mixed before the softmax, and an output gate.
 
     ``rows`` [T, >= heads * key_dim]: each row starts with its query heads; ``gate_offset`` (>= 0) names the column where
@@ -848,7 +920,9 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
     ``batch``: the step's context, from which a faster kernel is chosen where one fits; ``folded_slopes``: ``fast.folded_slopes(slopes, mix)``
     if the caller keeps it (it is worked out here otherwise).  ``keep_first``: with a window, the keys at positions below it stay visible.
     ``gate_per_head``: the gate is ``heads`` columns, one per head.  ``sinks`` (32-bit [heads]): exp(sink_h) joins the softmax's denominator.
-    ``values_in_keys``: the cache has one plane of one key/value head whose rows are the keys and whose first ``value_dim`` columns are the values."""
+    ``values_in_keys``: the cache has one plane of one key/value head whose rows are the keys and whose first ``value_dim`` columns are the values.
+    ``softcap`` > 0: a score is bounded, softcap * tanh(score / softcap), before it is turned into a weight.  ``sigmoid``: no softmax, the weight of
+    a visible key is sigmoid(score + shifts[h]) (``shifts`` 32-bit [heads] or None) and the weights of a row are not brought to a sum of one."""
     tokens = rows.shape[0]
     if heads % kv_heads != 0 or out.shape != (tokens, heads * value_dim) or out.dtype != rows.dtype:
         raise KernelError("mixed_heads_attention: out must be [rows, heads * value_dim] of the rows' dtype, heads a multiple of kv heads", code="invalid_shape")
@@ -857,6 +931,8 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
             raise KernelError(f"mixed_heads_attention: {name} must be 32-bit with {count} elements", code="invalid_shape")
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != heads):
         raise KernelError("mixed_heads_attention: sinks must be 32-bit with one element per head", code="invalid_shape")
+    if (shifts is not None and (not sigmoid or shifts.dtype != torch.float32 or shifts.numel() != heads)) or (sigmoid and sinks is not None):
+        raise KernelError("mixed_heads_attention: shifts are 32-bit, one per head, and belong to sigmoid weights, which take no sinks", code="invalid_shape")
     v_row_stride = value_dim
     if values_in_keys:
         if kv_heads != 1 or value_dim > key_dim:
@@ -870,16 +946,16 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
     if pages.dtype != rows.dtype:
         raise KernelError("mixed_heads_attention: pages and rows differ in dtype", code="invalid_dtype")
     table = cache.block_table
-    if (values_in_keys and window == 0 and gate_offset < 0 and slopes is None and mix is None and rows.shape[1] == heads * key_dim
+    if (values_in_keys and window == 0 and not sigmoid and softcap == 0.0 and gate_offset < 0 and slopes is None and mix is None and rows.shape[1] == heads * key_dim
             and fast.latent_prefill_takes(batch, rows, key_dim, value_dim)):
         fast.latent_prefill(rows, batch, table, k_ptr, k_stride, sinks, out, heads, key_dim, value_dim, cache.page_size, scale)
         return
     plain_options = sinks is None and not values_in_keys   # what the tensor-core kernels with two planes know
-    if plain_options and rows.dtype == torch.bfloat16 and fast.mixed_prefill_takes(batch, rows, cache.page_size, kv_heads if mix is not None else 1, key_dim, value_dim, gate_offset,
-                                                                                   gate_per_head):
+    if plain_options and (sigmoid or softcap == 0.0) and rows.dtype == torch.bfloat16 and fast.mixed_prefill_takes(batch, rows, cache.page_size, kv_heads if mix is not None else 1, key_dim, value_dim, gate_offset,
+                                                                                   gate_per_head, sigmoid):
         folded = folded_slopes if folded_slopes is not None else fast.folded_slopes(slopes, mix)
         fast.mixed_prefill(rows, gate_offset, batch, table, (k_ptr, k_stride, v_ptr, v_stride), folded, mix, out, heads, kv_heads, key_dim, value_dim,
-                           cache.page_size, window, scale, keep_first if window > 0 else 0, gate_per_head)
+                           cache.page_size, window, scale, keep_first if window > 0 else 0, gate_per_head, softcap, sigmoid, shifts)
         return
     # few rows over long contexts (decode steps): every row's keys are dealt to several CTAs
     splits, partial = 1, None
@@ -888,7 +964,7 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
         splits = max(1, min(2 * fast.sm_count() // tokens, -(-reach // 32), 64))   # down to one tile of 32 keys per CTA
         if plain_options and fast.mixed_decode_takes(rows, heads, kv_heads, key_dim, value_dim, gate_offset, mix is not None, gate_per_head):
             fast.mixed_decode(rows, gate_offset, positions, token_seq, table, (k_ptr, k_stride, v_ptr, v_stride), slopes, mix, out, heads, kv_heads, key_dim,
-                              value_dim, cache.page_size, window, scale, splits, keep_first if window > 0 else 0, gate_per_head)
+                              value_dim, cache.page_size, window, scale, splits, keep_first if window > 0 else 0, gate_per_head, softcap, sigmoid, shifts)
             return
         if splits > 1:
             partial = fast.mixed_scratch(rows.device, tokens * splits * (heads * value_dim + 2 * heads), torch.float32)
@@ -896,7 +972,8 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
                                                         c_longlong(v_stride), _i32(positions, "positions"), _i32(token_seq, "token_seq"), _i32(table, "block_table"),
                                                         c_int(table.shape[1]), _ptr(slopes), _ptr(mix), _ptr(out), c_int(tokens), c_int(heads), c_int(kv_heads),
                                                         c_int(key_dim), c_int(value_dim), c_int(cache.page_size), c_int(window), c_float(scale), c_int(splits), _ptr(partial),
-                                                        c_int(keep_first if window > 0 else 0), c_int(1 if gate_per_head else 0), _ptr(sinks), c_int(v_row_stride), _stream()),
+                                                        c_int(keep_first if window > 0 else 0), c_int(1 if gate_per_head else 0), _ptr(sinks), c_int(v_row_stride), c_float(softcap),
+                                                        c_int(1 if sigmoid else 0), _ptr(shifts), _stream()),
            "mixed_heads_attention")
 
 
@@ -971,43 +1048,63 @@ def moe_library():
     return load_library("tlie_moe", MOE_SOURCES)
 
 
-def moe_route(x, router, correction, ids, weights, groups: int, keep: int, route_scale: float, normalize: bool = True) -> None:
-    """Per token of ``x`` [T, width]: s = sigmoid(router x) (``router`` 32-bit [experts, width], sums in 32-bit), choice = s + ``correction``
-    (32-bit [experts] or None).  Experts form ``groups`` equal groups of neighbours; a group's score is the sum of its two largest choice
-    scores and only experts of the ``keep`` best groups can be chosen.  ``ids`` int32 [T, top] receives the experts of the ``top`` largest
+ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}
+GROUP_SCORES = {"two_best": 0, "best": 1}
+
+
+def moe_route(x, router, correction, ids, weights, groups: int, keep: int, route_scale: float, normalize: bool = True, scores: str = "sigmoid",
+              group_score: str = "two_best", shared_gate=None) -> None:
+    """Per token of ``x`` [T, width]: s = sigmoid(router x), or with ``scores`` "softmax" softmax(router x) over all experts (``router`` 32-bit
+    [experts, width], sums in 32-bit), choice = s + ``correction`` (32-bit [experts] or None).  Experts form ``groups`` equal groups of
+    neighbours; a group's score is the sum of its two largest choice scores (``group_score`` "best": its largest) and only experts of the
+    ``keep`` best groups can be chosen.  ``ids`` int32 [T, top] receives the experts of the ``top`` largest
     choice scores (the lower index on ties), ``weights`` 32-bit [T, top] their s / (sum of the chosen s + 1e-20) * ``route_scale``
-    (``normalize`` False: s * ``route_scale``, the scores as they are)."""
+    (``normalize`` False: s * ``route_scale``, the scores as they are).  ``shared_gate`` (32-bit [T]): the router then has one row more, and
+    ``shared_gate`` receives the sigmoid of that row's product with the token."""
     tokens, width = x.shape
-    experts, top = router.shape[0], ids.shape[1]
+    experts, top = router.shape[0] - (0 if shared_gate is None else 1), ids.shape[1]
+    if scores not in ROUTER_SCORES or group_score not in GROUP_SCORES:
+        raise KernelError(f"moe_route: no scores {scores!r} or no group score {group_score!r}", code="invalid_argument")
+    if shared_gate is not None and (shared_gate.dtype != torch.float32 or shared_gate.numel() != tokens):
+        raise KernelError("moe_route: the shared branch's gate is 32-bit, one number per token", code="invalid_shape")
     if router.dtype != torch.float32 or router.shape[1] != width or ids.dtype != torch.int32 or ids.shape != (tokens, top) or weights.dtype != torch.float32 or weights.shape != (tokens, top):
         raise KernelError("moe_route: a 32-bit router [experts, width], int32 ids and 32-bit weights [T, top]", code="invalid_shape")
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != experts):
         raise KernelError("moe_route: the correction is 32-bit [experts]", code="invalid_shape")
     _check(moe_library().tlie_moe_route(_code(x), _ptr(x), _ptr(router), _ptr(correction), _ptr(ids), _ptr(weights), c_int(tokens), c_int(width), c_int(experts),
-                                        c_int(groups), c_int(keep), c_int(top), c_float(route_scale), c_int(1 if normalize else 0), _stream()), "moe_route")
+                                        c_int(groups), c_int(keep), c_int(top), c_float(route_scale), c_int(1 if normalize else 0), c_int(ROUTER_SCORES[scores]),
+                                        c_int(GROUP_SCORES[group_score]), _ptr(shared_gate), _stream()), "moe_route")
 
 
-def moe_experts(x, gate_up, down, ids, weights, shared, out, activation: str = "silu", batch=None, weight_input: bool = False) -> None:
+EXPERT_KINDS = {**GATE_KINDS, "relu_squared": 2}   # the last: experts without a gate
+
+
+def moe_experts(x, gate_up, down, ids, weights, shared, out, activation: str = "silu", batch=None, weight_input: bool = False, shared_gate=None) -> None:
     """out[t] = sum_k weights[t, k] * W_down[e] (act(W_gate[e] x[t]) * (W_up[e] x[t])) for e = ids[t, k], plus ``shared[t]`` if given.
     ``gate_up`` [experts, 2 ff, width] (an expert's gate rows, then its up rows), ``down`` [experts, width, ff].  Steps of few rows and the
     32-bit path read each chosen expert's rows directly; bfloat16 prompt portions sort the (token, expert) pairs by expert and run
     the experts' products on the tensor cores.  ``weight_input``: the weight multiplies what the expert reads instead of what it returns,
-    out[t] = sum_k expert_e(weights[t, k] x[t]) (the two differ: the experts are not linear)."""
+    out[t] = sum_k expert_e(weights[t, k] x[t]) (the two differ: the experts are not linear).  ``activation`` "relu_squared": experts without a
+    gate, W_down[e] act(W_up[e] x[t]), ``gate_up`` [experts, ff, width] holding the up rows alone.  ``shared_gate`` (32-bit [T]): ``shared[t]`` is
+    multiplied by it."""
+    if activation not in EXPERT_KINDS:
+        raise KernelError(f"moe_experts: no activation {activation!r}", code="invalid_argument")
+    kind = EXPERT_KINDS[activation]
     tokens, width = x.shape
-    experts, two_ff, _ = gate_up.shape
-    ff, top = two_ff // 2, ids.shape[1]
-    if gate_up.shape != (experts, 2 * ff, width) or down.shape != (experts, width, ff) or out.shape != (tokens, width) or gate_up.dtype != x.dtype or down.dtype != x.dtype or out.dtype != x.dtype:
+    experts, first_rows, _ = gate_up.shape
+    ff, top = first_rows if kind == 2 else first_rows // 2, ids.shape[1]
+    if gate_up.shape != (experts, ff if kind == 2 else 2 * ff, width) or down.shape != (experts, width, ff) or out.shape != (tokens, width) or gate_up.dtype != x.dtype or down.dtype != x.dtype or out.dtype != x.dtype:
         raise KernelError("moe_experts: gate_up [experts, 2 ff, width], down [experts, width, ff], out [T, width], one dtype", code="invalid_shape")
     if shared is not None and (shared.shape != out.shape or shared.dtype != out.dtype):
         raise KernelError("moe_experts: the shared branch has the output's shape and dtype", code="invalid_shape")
-    if activation not in GATE_KINDS:
-        raise KernelError(f"moe_experts: no activation {activation!r}", code="invalid_argument")
+    if shared_gate is not None and (shared is None or shared_gate.dtype != torch.float32 or shared_gate.numel() != tokens):
+        raise KernelError("moe_experts: the shared branch's gate is 32-bit, one number per token, beside a shared branch", code="invalid_shape")
     if x.dtype == torch.bfloat16 and fast.moe_grouped_takes(tokens, top, width, ff, experts):
-        fast.moe_grouped(x, gate_up, down, ids, weights, shared, out, GATE_KINDS[activation], weight_input)
+        fast.moe_grouped(x, gate_up, down, ids, weights, shared, out, kind, weight_input, shared_gate)
         return
     act = fast.mixed_scratch(x.device, tokens * top * ff, x.dtype)
-    _check(moe_library().tlie_moe_experts(_code(x), _ptr(x), _ptr(gate_up), _ptr(down), _ptr(ids), _ptr(weights), _ptr(shared), _ptr(act), _ptr(out), c_int(tokens),
-                                          c_int(width), c_int(ff), c_int(top), c_int(GATE_KINDS[activation]), c_int(1 if weight_input else 0), _stream()), "moe_experts")
+    _check(moe_library().tlie_moe_experts(_code(x), _ptr(x), _ptr(gate_up), _ptr(down), _ptr(ids), _ptr(weights), _ptr(shared), _ptr(shared_gate), _ptr(act), _ptr(out),
+                                          c_int(tokens), c_int(width), c_int(ff), c_int(top), c_int(kind), c_int(1 if weight_input else 0), _stream()), "moe_experts")
 
 
 # --- sampling ------------------------------------------------------------------------------

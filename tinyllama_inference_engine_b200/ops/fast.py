@@ -98,13 +98,14 @@ def prepared_norm_buffers(rows: int, width: int, device) -> tuple:
     return (torch.empty((rows, width), dtype=torch.bfloat16, device=device), torch.empty((rows, -(-width // 16)), dtype=torch.float32, device=device))
 
 
-GEMV_ACTIVATIONS = {None: 0, "relu_squared": 1, "gelu_tanh": 2, "silu": 3}
+GEMV_ACTIVATIONS = {None: 0, "relu_squared": 1, "gelu_tanh": 2, "silu": 3, "xielu": 4}
 
 
 GEMV_GATES = {"silu": 0, "gelu_tanh": 2}   # the gated epilogue's activation (1 is the clamped gate, chosen by ``clamp``)
 
 
-def gemv_fused(x, weight, out, *, norm=None, epilogue: str = "store", prepared=None, prepare=None, activation: str | None = None, clamp=None, gate: str = "silu") -> None:
+def gemv_fused(x, weight, out, *, norm=None, epilogue: str = "store", prepared=None, prepare=None, activation: str | None = None, constants=(0.0, 0.0),
+               clamp=None, gate: str = "silu", bias=None) -> None:
     """out (+)= f(x) . weight^T for up to 16 rows, one kernel.
 
     norm      None: ``x`` is bfloat16 [M, K].  (norm_weight, eps, rows): ``x`` is the 32-bit residual stream and
@@ -115,7 +116,9 @@ def gemv_fused(x, weight, out, *, norm=None, epilogue: str = "store", prepared=N
               "gated": weight is [gate rows | up rows], out [M, N / 2] = silu(gate) * up; with ``clamp`` = (limit, alpha, shift) instead
               g * sigmoid(alpha * g) * (u + shift) for g = min(gate, limit), u = clamp(up, -limit, limit); with ``gate`` = "gelu_tanh" the gate's
               activation is gelu in its tanh form.
-    activation ("store" into bfloat16 only) "relu_squared", "gelu_tanh" or "silu": applied to the rounded product before it is stored.
+    activation ("store" into bfloat16 only) "relu_squared", "gelu_tanh", "silu" or "xielu" (which takes two ``constants``, see ``ops.activation``): applied to
+              the rounded product before it is stored.
+    bias      ("store" into bfloat16 only) 32-bit [N], added to the sums before they are rounded.
     prepare   ("accumulate" only) (norm_weight [N], x_out bfloat16 [M, N], squares_out [M, ceil(N / 16)]): also store
               bfloat16(out * norm_weight) and the rows' sums of squares per 16 columns, for a later call with ``prepared``.
     """
@@ -131,6 +134,8 @@ def gemv_fused(x, weight, out, *, norm=None, epilogue: str = "store", prepared=N
         raise KernelError("gemv_fused accumulates into the 32-bit residual only", code="invalid_dtype")
     if activation is not None and (epilogue != "store" or out.dtype != torch.bfloat16 or activation not in GEMV_ACTIVATIONS):
         raise KernelError("gemv_fused applies an activation only when it stores bfloat16", code="invalid_argument")
+    if bias is not None and (epilogue != "store" or out.dtype != torch.bfloat16 or bias.dtype != torch.float32 or bias.numel() != N):
+        raise KernelError("gemv_fused adds a 32-bit bias [N] only when it stores bfloat16", code="invalid_argument")
     if out.shape[1] != (N // 2 if epilogue == "gated" else N):
         raise KernelError("gemv_fused: the output's width does not fit the weight", code="invalid_shape")
     consume = (c_void_p(0), c_int(0))
@@ -159,8 +164,8 @@ def gemv_fused(x, weight, out, *, norm=None, epilogue: str = "store", prepared=N
             raise KernelError("gemv_fused: prepare takes a 32-bit norm weight [N], bfloat16 [M, N] and 32-bit [M, ceil(N / 16)], with accumulate", code="invalid_shape")
         emit = (ops._ptr(norm_weight), ops._ptr(x_out), ops._ptr(squares_out))
     ops._check(gemv_library().tlie_gemv_fused(*args, ops._ptr(weight), ops._ptr(out), c_int(M), c_int(N), c_int(K), c_int(code), *consume, *emit, c_int(GEMV_ACTIVATIONS[activation]),
-                                             c_int(GEMV_GATES[gate] if clamp is None else 1), *(c_float(float(v)) for v in (clamp or (0.0, 0.0, 0.0))), ops._stream()),
-               "gemv_fused")
+                                             c_int(GEMV_GATES[gate] if clamp is None else 1), *(c_float(float(v)) for v in (clamp or (0.0, 0.0, 0.0))), *(c_float(float(v)) for v in constants), ops._ptr(bias),
+                                             ops._stream()), "gemv_fused")
 
 
 # --- tensor-core product for 17 to 127 rows (tcgen05 with the operands swapped, K cut over a cluster) -----------------
@@ -696,13 +701,16 @@ use_mixed_prefill = True
 MIXED_PREFILL_MIN_ROWS = 8    # a step whose longest entry has fewer rows stays on the general kernel (a tile is at least 16 rows)
 
 
-def mixed_prefill_library(key_dim: int, value_dim: int, parts: int):
-    """The kernel set of one (key width, value width, key heads per folded query): compiled when a model of these sizes first runs a prompt."""
-    lib = load_library(f"tlie_attn_mixed_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "PARTS": parts})
-    return lib
+def mixed_prefill_library(key_dim: int, value_dim: int, parts: int, sigmoid: bool = False):
+    """The kernel set of one (key width, value width, key heads per folded query, kind of weights): compiled when a model of these sizes first runs a prompt."""
+    defines = {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "PARTS": parts}
+    if sigmoid:
+        return load_library(f"tlie_attn_sigmoid_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], {**defines, "SIGMOID_WEIGHTS": 1})
+    return load_library(f"tlie_attn_mixed_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], defines)
 
 
-def mixed_prefill_takes(batch, rows, page_size: int, parts: int, key_dim: int, value_dim: int, gate_offset: int, gate_per_head: bool = False) -> bool:
+def mixed_prefill_takes(batch, rows, page_size: int, parts: int, key_dim: int, value_dim: int, gate_offset: int, gate_per_head: bool = False,
+                        sigmoid: bool = False) -> bool:
     """Whether a step's attention with mixed heads runs on the tensor-core kernel: bfloat16, a prompt portion among the entries,
     widths that are multiples of 16, and tiles that fit shared memory (the kernel set says how many rows its tile has: 0 = none)."""
     if not use_mixed_prefill or batch is None or batch.max_q_len < MIXED_PREFILL_MIN_ROWS or rows.dtype != torch.bfloat16:
@@ -711,7 +719,7 @@ def mixed_prefill_takes(batch, rows, page_size: int, parts: int, key_dim: int, v
         return False
     if ((parts * key_dim + 8) * 16 + 3 * 64 * (key_dim + 8) + (3 if parts == 1 else 2) * 64 * (value_dim + 8)) * 2 > 227 * 1024:
         return False   # not even 16 rows of folded queries fit beside the rings of keys and values
-    return mixed_prefill_library(key_dim, value_dim, parts).tlie_mixed_prefill_tile_rows() > 0
+    return mixed_prefill_library(key_dim, value_dim, parts, sigmoid).tlie_mixed_prefill_tile_rows() > 0
 
 
 def folded_slopes(slopes, mix):
@@ -736,25 +744,29 @@ def mixed_scratch(device: torch.device, elements: int, dtype: torch.dtype) -> to
 
 
 def mixed_prefill(rows, gate_offset: int, batch, block_table, planes, folded, mix, out, heads: int, kv_heads: int, key_dim: int, value_dim: int,
-                  page_size: int, window: int, scale: float, keep_first: int = 0, gate_per_head: bool = False) -> None:
+                  page_size: int, window: int, scale: float, keep_first: int = 0, gate_per_head: bool = False, softcap: float = 0.0, sigmoid: bool = False,
+                  shifts=None) -> None:
     """Attention with mixed heads for a step that carries prompt portions (csrc/attention_mixed_prefill.cu): the mix is folded into
     the queries by a first kernel, the second is flash attention over the concatenated key heads.  ``planes``: (key plane pointer,
     its page stride in elements, value plane pointer, its page stride); ``folded``: the folded slopes (``folded_slopes``) or None.
-    ``keep_first``: with a window, the keys below this position stay visible; ``gate_per_head``: the gate is one column per head."""
+    ``keep_first``: with a window, the keys below this position stay visible; ``gate_per_head``: the gate is one column per head.
+    With nothing to fold (no mix, ``scale`` 1) the first kernel is left out and the queries are read where they are.  ``sigmoid``, ``softcap``,
+    ``shifts``: see ``ops.mixed_heads_attention``."""
     ops = _ops()
     parts = kv_heads if mix is not None else 1
     tokens = rows.shape[0]
     need = tokens * heads * parts * key_dim
-    held = mixed_scratch(rows.device, need, torch.bfloat16)
+    held = None if mix is None and scale == 1.0 else mixed_scratch(rows.device, need, torch.bfloat16)
     k_ptr, k_stride, v_ptr, v_stride = planes
     ops._check(
-        mixed_prefill_library(key_dim, value_dim, parts).tlie_mixed_prefill(
+        mixed_prefill_library(key_dim, value_dim, parts, sigmoid).tlie_mixed_prefill(
             ops._ptr(rows), c_int(rows.shape[1]), c_int(gate_offset), ops._ptr(mix), c_float(scale), ops._ptr(held), k_ptr, c_longlong(k_stride), v_ptr,
             c_longlong(v_stride), ops._i32(batch.seq_starts, "seq_starts"), ops._i32(batch.first_positions, "first_positions"), ops._i32(block_table, "block_table"),
             c_int(block_table.shape[1]), ops._ptr(folded), ops._ptr(out), c_int(tokens), c_int(batch.num_seqs), c_int(batch.max_q_len),
-            c_int(heads), c_int(kv_heads), c_int(page_size), c_int(window), c_int(keep_first), c_int(1 if gate_per_head else 0), ops._stream()),
+            c_int(heads), c_int(kv_heads), c_int(page_size), c_int(window), c_int(keep_first), c_int(1 if gate_per_head else 0), c_float(softcap),
+            ops._ptr(shifts), ops._stream()),
         "mixed_prefill")
-    ops.launch_count += 1   # two kernels: the fold and the attention
+    ops.launch_count += 0 if held is None else 1   # two kernels: the fold and the attention
 
 
 # --- latent attention, prompt portions on the tensor cores -----------------------------------------------------------------------------
@@ -828,7 +840,8 @@ def mixed_decode_takes(rows, heads: int, kv_heads: int, key_dim: int, value_dim:
 
 
 def mixed_decode(rows, gate_offset: int, positions, token_seq, block_table, planes, slopes, mix, out, heads: int, kv_heads: int, key_dim: int, value_dim: int,
-                 page_size: int, window: int, scale: float, splits: int, keep_first: int = 0, gate_per_head: bool = False) -> None:
+                 page_size: int, window: int, scale: float, splits: int, keep_first: int = 0, gate_per_head: bool = False, softcap: float = 0.0,
+                 sigmoid: bool = False, shifts=None) -> None:
     """Attention with mixed heads for a step of few rows (csrc/attention_mixed_decode.cu).  ``planes`` as in ``mixed_prefill``;
     ``splits``: CTAs that share a row's key tiles (their parts are merged by a second kernel)."""
     ops = _ops()
@@ -840,7 +853,7 @@ def mixed_decode(rows, gate_offset: int, positions, token_seq, block_table, plan
             ops._ptr(rows), c_int(rows.shape[1]), c_int(gate_offset), k_ptr, c_longlong(k_stride), v_ptr, c_longlong(v_stride), ops._i32(positions, "positions"),
             ops._i32(token_seq, "token_seq"), ops._i32(block_table, "block_table"), c_int(block_table.shape[1]), ops._ptr(slopes), ops._ptr(mix), ops._ptr(out),
             c_int(tokens), c_int(heads), c_int(page_size), c_int(window), c_float(scale), c_int(splits), ops._ptr(partial), c_int(keep_first),
-            c_int(1 if gate_per_head else 0), ops._stream()),
+            c_int(1 if gate_per_head else 0), c_float(softcap), c_int(1 if sigmoid else 0), ops._ptr(shifts), ops._stream()),
         "mixed_decode")
 
 
@@ -953,11 +966,11 @@ def moe_grouped_takes(tokens: int, top: int, width: int, ff: int, experts: int) 
     return use_moe_grouped and tokens >= MOE_GROUPED_MIN_ROWS and tokens * top >= MOE_GROUPED_MIN_SLOTS and width % 8 == 0 and ff % 8 == 0 and experts <= 4096
 
 
-def moe_grouped(x, gate_up, down, ids, weights, shared, out, kind: int, weight_input: bool = False) -> None:
+def moe_grouped(x, gate_up, down, ids, weights, shared, out, kind: int, weight_input: bool = False, shared_gate=None) -> None:
     ops = _ops()
     tokens, width = x.shape
-    experts, two_ff, _ = gate_up.shape
-    ff, top = two_ff // 2, ids.shape[1]
+    experts, _, ff = down.shape
+    top = ids.shape[1]
     slots = tokens * top
     device = x.device
     if use_moe_tc and slots >= MOE_TC_MIN_ROWS_PER_EXPERT * experts and width >= 64 and ff >= 64:   # a TMA box is 64 numbers of a row
@@ -969,7 +982,8 @@ def moe_grouped(x, gate_up, down, ids, weights, shared, out, kind: int, weight_i
         xs = named_scratch(device, "moe_rows", max_rows * width, torch.bfloat16)
         act = named_scratch(device, "moe_act", max_rows * ff, torch.bfloat16)
         y = named_scratch(device, "moe_by_row", max_rows * width, torch.float32)
-        ops._check(ops.moe_library().tlie_moe_grouped_tc(ops._ptr(x), ops._ptr(gate_up), ops._ptr(down), ops._ptr(ids), ops._ptr(weights), ops._ptr(shared), ops._ptr(row_of_slot),
+        ops._check(ops.moe_library().tlie_moe_grouped_tc(ops._ptr(x), ops._ptr(gate_up), ops._ptr(down), ops._ptr(ids), ops._ptr(weights), ops._ptr(shared), ops._ptr(shared_gate),
+                                                         ops._ptr(row_of_slot),
                                                          ops._ptr(token_of_row), ops._ptr(meta), ops._ptr(xs), ops._ptr(act), ops._ptr(y), ops._ptr(out), c_int(tokens), c_int(width),
                                                          c_int(ff), c_int(experts), c_int(top), c_int(kind), c_int(1 if weight_input else 0), ops._ptr(tcgen05_error_flag(device)), ops._stream()), "moe_grouped_tc")
         ops.launch_count += 4   # five kernels: the layout, the gathered rows, two products over all experts, the sum
@@ -978,7 +992,7 @@ def moe_grouped(x, gate_up, down, ids, weights, shared, out, kind: int, weight_i
     meta = named_scratch(device, "moe_tiles", 1 + 3 * (slots // 64 + experts), torch.int32)
     act = named_scratch(device, "moe_act", slots * ff, torch.bfloat16)
     y = named_scratch(device, "moe_by_slot", slots * width, torch.float32)
-    ops._check(ops.moe_library().tlie_moe_grouped(ops._ptr(x), ops._ptr(gate_up), ops._ptr(down), ops._ptr(ids), ops._ptr(weights), ops._ptr(shared), ops._ptr(sorted_slots),
+    ops._check(ops.moe_library().tlie_moe_grouped(ops._ptr(x), ops._ptr(gate_up), ops._ptr(down), ops._ptr(ids), ops._ptr(weights), ops._ptr(shared), ops._ptr(shared_gate), ops._ptr(sorted_slots),
                                                   ops._ptr(meta), ops._ptr(act), ops._ptr(y), ops._ptr(out), c_int(tokens), c_int(width), c_int(ff), c_int(experts), c_int(top),
                                                   c_int(kind), c_int(1 if weight_input else 0), ops._stream()), "moe_grouped")
     ops.launch_count += 3   # four kernels: the sort, two products per expert, the sum

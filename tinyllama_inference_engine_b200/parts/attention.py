@@ -1,13 +1,15 @@
 """Attention over the paged cache: grouped-query attention with a position encoding; attention whose heads are biased by
 distance, mixed before the softmax and gated after it; attention with normalised queries and keys under a window that keeps
-the first tokens; and latent attention, which caches one small vector per token for all heads."""
+the first tokens; attention whose keys are each weighed by a sigmoid of their own; and latent attention, which caches one small vector
+per token for all heads."""
 from __future__ import annotations
 
-import numpy as np
 import torch
 
 from .. import ops
+from ..errors import ConfigError
 from .base import CacheNeed, LayerCache, Mixer, build_part, register_part
+from .position import rotation_frequencies
 from .spec import PartSpec, TensorSpec
 
 
@@ -164,9 +166,7 @@ class MixedHeadsAttention(Mixer):
         self.rot_dims = int(spec.get("rot_dims", 0) or 0)
         self.inv_freq = None
         if self.rot_dims:
-            # frequencies in 64-bit, rounded once: the angle is float(position) * frequency in 32-bit inside the kernel
-            exponent = -2.0 * np.arange(self.rot_dims // 2, dtype=np.float64) / float(self.rot_dims)
-            self.inv_freq = torch.from_numpy(np.power(float(spec["rot_base"]), exponent).astype(np.float32)).to(runtime.device)
+            self.inv_freq = torch.from_numpy(rotation_frequencies(self.rot_dims, spec["rot_base"])[0]).to(runtime.device)
         if self.biases is not None or self.rot_dims:
             # the kernels of few rows take neither: such a layer is handed finished tensors and returns its output
             self.accepts_lazy_norm = self.fuses_residual_add = self.prepares_next_norm = False
@@ -248,8 +248,6 @@ class NormedKeyAttention(Mixer):
         self.scale, self.eps = float(spec["scale"]), float(spec["eps"])
         self.values_are_keys = spec.get("values", "projection") == "keys"
         if self.values_are_keys and self.value_dim != self.key_dim:
-            from ..errors import ConfigError
-
             raise ConfigError(f"{prefix}: values that are the keys have the keys' width ({self.key_dim}), not {self.value_dim}")
         dtype = runtime.dtype
         stacked = [weights.get(f"{prefix}.q", dtype), weights.get(f"{prefix}.k", dtype)]
@@ -292,14 +290,90 @@ class NormedKeyAttention(Mixer):
         return out
 
 
+class SigmoidAttention(Mixer):
+    """Grouped heads whose visible keys are each weighed by a sigmoid of their own: no softmax, nothing is brought to a sum of one.
+
+    q, k and v have biases.  q and k are divided by their root mean square per head and multiplied by a weight; their first ``rot_dims``
+    columns then turn by position.  Score of head h: (q . k) * scale * temp_h, bounded by ``softcap`` * tanh(score / ``softcap``) if that is positive; the
+    weight of key j <= i is sigmoid(score + shift_h); head h's sum of weighted values is multiplied by sigmoid((W_g x)_h), one number per
+    head; out = W_o concat(heads) + b_o.
+
+    params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``key_dim``, ``value_dim``, ``scale``, ``eps``, ``softcap`` (0: unbounded), ``rot_dims``, ``rot_base``, optional
+    ``rot_scaling`` (``position.rotation_frequencies``), ``rot_layout`` ("interleaved": columns (2i, 2i + 1) turn together; "halves": column i with column
+    i + rot_dims / 2).
+    tensors: ``<prefix>.q`` [heads * key_dim, hidden], ``<prefix>.k`` [kv * key_dim, hidden], ``<prefix>.v`` [kv * value_dim, hidden], ``<prefix>.o`` [hidden, heads *
+    value_dim], each with its ``.b``; ``<prefix>.{q,k}.norm`` [key_dim], ``<prefix>.temp`` and ``<prefix>.pb`` [heads] (temperatures and shifts), ``<prefix>.g``
+    [heads, hidden].  q, k, v and the gate are one stacked product; scale and temperature are multiplied into the queries in 32-bit
+    before these are rounded.  The cache holds two planes per token: the normed, turned keys and the values.  Norms, angles, scores,
+    weights and the gate are 32-bit.
+    """
+
+    capturable = True
+
+    @classmethod
+    def _sizes(cls, spec: PartSpec) -> tuple[int, int, int, int, int]:
+        return int(spec["hidden_size"]), int(spec["num_heads"]), int(spec["num_kv_heads"]), int(spec["key_dim"]), int(spec["value_dim"])
+
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
+        hidden, heads, kv, dim, vdim = cls._sizes(spec)
+        specs = []
+        for name, rows, columns in (("q", heads * dim, hidden), ("k", kv * dim, hidden), ("v", kv * vdim, hidden), ("o", hidden, heads * vdim)):
+            specs += [TensorSpec(f"{prefix}.{name}", (rows, columns), std=columns ** -0.5), TensorSpec(f"{prefix}.{name}.b", (rows,), std=0.2)]
+        return specs + [TensorSpec(f"{prefix}.q.norm", (dim,), init="norm", std=0.1), TensorSpec(f"{prefix}.k.norm", (dim,), init="norm", std=0.1),
+                        TensorSpec(f"{prefix}.temp", (heads,), init="norm", std=0.2), TensorSpec(f"{prefix}.pb", (heads,), std=1.0), TensorSpec(f"{prefix}.g", (heads, hidden), std=hidden ** -0.5)]
+
+    @classmethod
+    def cache_need(cls, spec: PartSpec) -> CacheNeed:
+        _, _, kv, dim, vdim = cls._sizes(spec)
+        return CacheNeed("pages", planes=((kv, dim), (kv, vdim)))
+
+    def __init__(self, spec, prefix, weights, runtime):
+        super().__init__(spec, prefix, weights, runtime)
+        self.hidden, self.heads, self.kv_heads, self.dim, self.vdim = self._sizes(spec)
+        self.eps, self.softcap = float(spec["eps"]), float(spec.get("softcap", 0.0) or 0.0)
+        dtype = runtime.dtype
+        stacked = [weights.get(f"{prefix}.{n}", dtype) for n in ("q", "k", "v", "g")]
+        self.k_offset = self.heads * self.dim
+        self.v_offset = self.k_offset + self.kv_heads * self.dim
+        self.gate_offset = self.v_offset + self.kv_heads * self.vdim
+        width = self.gate_offset + self.heads
+        if width % 8:   # rows of the stacked product start on 16-byte boundaries (what the tensor-core attention kernels read them by)
+            stacked.append(torch.zeros((8 - width % 8, self.hidden), dtype=dtype, device=stacked[0].device))
+        self.w_in = torch.cat(stacked, dim=0).contiguous()
+        self.w_o = weights.get(f"{prefix}.o", dtype).contiguous()
+        vector = lambda name: weights.get(f"{prefix}.{name}", torch.float32).contiguous()
+        self.biases, self.out_bias = tuple(vector(f"{n}.b") for n in ("q", "k", "v")), vector("o.b")
+        self.q_weight, self.k_weight, self.shifts = vector("q.norm"), vector("k.norm"), vector("pb")
+        self.factors = (vector("temp") * float(spec["scale"])).contiguous()
+        self.rot_dims, self.interleaved = int(spec.get("rot_dims", 0) or 0), spec.get("rot_layout", "interleaved") == "interleaved"
+        frequencies, self.amplitude = rotation_frequencies(self.rot_dims, spec.get("rot_base", 10000.0), spec.get("rot_scaling"))
+        self.inv_freq = torch.from_numpy(frequencies).to(runtime.device)
+
+    def forward(self, x, ctx, cache: LayerCache):
+        ws, dtype, tokens = self.runtime.workspace, self.runtime.dtype, x.shape[0]
+        rows = ws.get("qkv_gate", tokens, self.w_in.shape[0], dtype)
+        ops.linear(x, self.w_in, rows)
+        ops.norm_rotary_store(rows, self.k_offset, self.v_offset, self.biases, self.q_weight, self.k_weight, self.eps, self.factors, self.inv_freq, self.rot_dims,
+                              self.interleaved, self.amplitude, ctx.positions, ctx.token_seq, cache, self.heads, self.kv_heads, self.dim, self.vdim)
+        mixed = ws.get("attention", tokens, self.heads * self.vdim, dtype)
+        ops.mixed_heads_attention(rows, self.gate_offset, ctx.positions, ctx.token_seq, cache, None, None, mixed, self.heads, self.kv_heads, self.dim, self.vdim, 0, 1.0,
+                                  batch=ctx, gate_per_head=True, softcap=self.softcap, sigmoid=True, shifts=self.shifts)
+        out = ws.get("mixer_out", tokens, self.hidden, dtype)
+        ops.linear_bias(mixed, self.w_o, self.out_bias, out)
+        return out
+
+
 class LatentAttention(Mixer):
     """Attention whose keys and values are expanded from one latent vector per token, with a rotated key part shared by all heads
     and, optionally, a sink in the softmax.
 
     Per token: q = W_q x, head by head [plain | rot]; W_dkv x = [rank | rot]; the latent c is the first ``rank`` columns under an RMS norm
-    with a weight, the last ``rot`` columns are one key part for every head, rotated by position like the queries' rot parts (pairs
-    (2i, 2i + 1) of the first ``rot_dims`` columns by angle position * base^(-2i / rot_dims)).  Head h has keys [W_uk,h c | shared part]
+    with a weight, the last ``rot`` columns are one key part for every head, rotated by position like the queries' rot parts (the first
+    ``rot_dims`` columns by angle position * frequency).  Head h has keys [W_uk,h c | shared part]
     and values W_uv,h c; causal; softmax whose denominator also holds exp(sink_h) if ``sink``; out = W_o concat(heads).
+    ``query_rank`` > 0: the queries pass a latent of their own, q = W_uq norm(W_dq x) with an RMS norm and a weight.
+    ``output_gate``: the concatenated heads are multiplied element by element by sigmoid(W_g x).
 
     Only [c | rotated part] is cached (one plane, one head, rank + rot wide).  The products with W_uk and W_uv are moved across the
     attention: q~_h = W_uk,h^T q_plain,h, so that the score is [q~_h | q_rot,h] . [c_j | rot_j] and head h's weighted sum of latents,
@@ -307,8 +381,12 @@ class LatentAttention(Mixer):
     head whose values are the first ``rank`` columns of its keys.
 
     params: ``hidden_size``, ``num_heads``, ``plain_dim``, ``rot_dim``, ``value_dim``, ``rank``, ``scale``, ``eps``, ``rot_dims``, ``rot_base``,
-    ``sink``.  tensors: ``<prefix>.q`` [heads * (plain + rot), hidden], ``<prefix>.dkv`` [rank + rot, hidden], ``<prefix>.dkv.norm`` [rank],
-    ``<prefix>.uk`` [heads * plain, rank], ``<prefix>.uv`` [heads * value_dim, rank], ``<prefix>.sink`` [heads], ``<prefix>.o`` [hidden, heads * value_dim].
+    ``sink``, optional ``query_rank`` (0), ``output_gate`` (False), ``rot_layout`` ("interleaved": columns (2i, 2i + 1) turn together; "halves": column i with
+    column i + rot_dims / 2), ``rot_scaling`` (``position.rotation_frequencies``; cosines and sines are multiplied by its amplitude).
+    tensors: ``<prefix>.q`` [heads * (plain + rot), hidden] (with a query latent instead ``<prefix>.dq`` [query_rank, hidden], ``<prefix>.dq.norm`` [query_rank],
+    ``<prefix>.uq`` [heads * (plain + rot), query_rank]), ``<prefix>.dkv`` [rank + rot, hidden], ``<prefix>.dkv.norm`` [rank],
+    ``<prefix>.uk`` [heads * plain, rank], ``<prefix>.uv`` [heads * value_dim, rank], ``<prefix>.sink`` [heads], ``<prefix>.g`` [heads * value_dim, hidden],
+    ``<prefix>.o`` [hidden, heads * value_dim].
     """
 
     capturable = True
@@ -319,12 +397,20 @@ class LatentAttention(Mixer):
     @classmethod
     def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
         hidden, heads, plain, rot, vdim, rank = (int(spec[k]) for k in ("hidden_size", "num_heads", "plain_dim", "rot_dim", "value_dim", "rank"))
+        query_rank = int(spec.get("query_rank", 0) or 0)
         std = hidden ** -0.5
-        specs = [TensorSpec(f"{prefix}.q", (heads * (plain + rot), hidden), std=std), TensorSpec(f"{prefix}.dkv", (rank + rot, hidden), std=std),
-                 TensorSpec(f"{prefix}.dkv.norm", (rank,), init="norm", std=0.1), TensorSpec(f"{prefix}.uk", (heads * plain, rank), std=rank ** -0.5),
-                 TensorSpec(f"{prefix}.uv", (heads * vdim, rank), std=rank ** -0.5)]
+        if query_rank:
+            specs = [TensorSpec(f"{prefix}.dq", (query_rank, hidden), std=std), TensorSpec(f"{prefix}.dq.norm", (query_rank,), init="norm", std=0.1),
+                     TensorSpec(f"{prefix}.uq", (heads * (plain + rot), query_rank), std=query_rank ** -0.5)]
+        else:
+            specs = [TensorSpec(f"{prefix}.q", (heads * (plain + rot), hidden), std=std)]
+        specs += [TensorSpec(f"{prefix}.dkv", (rank + rot, hidden), std=std),
+                  TensorSpec(f"{prefix}.dkv.norm", (rank,), init="norm", std=0.1), TensorSpec(f"{prefix}.uk", (heads * plain, rank), std=rank ** -0.5),
+                  TensorSpec(f"{prefix}.uv", (heads * vdim, rank), std=rank ** -0.5)]
         if spec.get("sink"):
             specs.append(TensorSpec(f"{prefix}.sink", (heads,), std=1.0))
+        if spec.get("output_gate"):
+            specs.append(TensorSpec(f"{prefix}.g", (heads * vdim, hidden), std=std))
         return specs + [TensorSpec(f"{prefix}.o", (hidden, heads * vdim), std=(heads * vdim) ** -0.5)]
 
     @classmethod
@@ -334,20 +420,37 @@ class LatentAttention(Mixer):
     def __init__(self, spec, prefix, weights, runtime):
         super().__init__(spec, prefix, weights, runtime)
         self.hidden, self.heads, self.plain, self.rot, self.vdim, self.rank = (int(spec[k]) for k in ("hidden_size", "num_heads", "plain_dim", "rot_dim", "value_dim", "rank"))
+        self.query_rank = int(spec.get("query_rank", 0) or 0)
         self.scale, self.eps = float(spec["scale"]), float(spec["eps"])
-        self.rot_dims = int(spec["rot_dims"])
+        self.rot_dims, self.interleaved = int(spec["rot_dims"]), spec.get("rot_layout", "interleaved") == "interleaved"
         dtype = runtime.dtype
-        self.w_in = torch.cat([weights.get(f"{prefix}.q", dtype), weights.get(f"{prefix}.dkv", dtype)], dim=0).contiguous()
-        self.latent_offset = self.heads * (self.plain + self.rot)
+        # one stacked product: [queries (or their latent) | latent and shared key part | gate], every piece starting on a 16-byte boundary of its row
+        pieces = [weights.get(f"{prefix}.{'dq' if self.query_rank else 'q'}", dtype), weights.get(f"{prefix}.dkv", dtype)]
+        if spec.get("output_gate"):
+            pieces.append(weights.get(f"{prefix}.g", dtype))
+        stacked, offsets, width = [], [], 0
+        for piece in pieces:
+            if width % 8 and (self.query_rank or spec.get("output_gate")):
+                stacked.append(torch.zeros((8 - width % 8, self.hidden), dtype=dtype, device=piece.device))
+                width += stacked[-1].shape[0]
+            offsets.append(width)
+            stacked.append(piece)
+            width += piece.shape[0]
+        self.w_in = torch.cat(stacked, dim=0).contiguous()
+        self.latent_offset = offsets[1]
+        self.gate_offset = offsets[2] if spec.get("output_gate") else -1
+        self.query_width = self.heads * (self.plain + self.rot)
+        if self.query_rank:
+            self.query_weight = weights.get(f"{prefix}.dq.norm", torch.float32).contiguous()
+            self.w_uq = weights.get(f"{prefix}.uq", dtype).contiguous()
         self.latent_weight = weights.get(f"{prefix}.dkv.norm", torch.float32).contiguous()
         # W_uk per head, transposed: [heads, rank, plain], the operand of q~ = W_uk^T q; W_uv per head [heads, vdim, rank]
         self.w_uk_t = weights.get(f"{prefix}.uk", dtype).view(self.heads, self.plain, self.rank).transpose(1, 2).contiguous()
         self.w_uv = weights.get(f"{prefix}.uv", dtype).view(self.heads, self.vdim, self.rank).contiguous()
         self.sinks = weights.get(f"{prefix}.sink", torch.float32).contiguous() if spec.get("sink") else None
         self.w_o = weights.get(f"{prefix}.o", dtype).contiguous()
-        # frequencies in 64-bit, rounded once: the angle is float(position) * frequency in 32-bit inside the kernel
-        exponent = -2.0 * np.arange(self.rot_dims // 2, dtype=np.float64) / float(self.rot_dims)
-        self.inv_freq = torch.from_numpy(np.power(float(spec["rot_base"]), exponent).astype(np.float32)).to(runtime.device)
+        frequencies, self.amplitude = rotation_frequencies(self.rot_dims, spec["rot_base"], spec.get("rot_scaling"))
+        self.inv_freq = torch.from_numpy(frequencies).to(runtime.device)
 
     def adds_to_residual(self, rows: int) -> bool:
         return ops.can_accumulate(rows, self.w_o)
@@ -361,16 +464,26 @@ class LatentAttention(Mixer):
             ops.linear(x, self.w_in, rows)
         width = self.rank + self.rot
         flat_queries = ws.get("latent_queries", tokens, self.heads * width, dtype)
-        ops.latent_store(rows, self.latent_offset, self.latent_weight, self.eps, self.inv_freq, self.rot_dims, ctx.positions, ctx.token_seq, cache, flat_queries,
-                         self.heads, self.plain, self.rot, self.rank)
+        rotation = (self.inv_freq, self.rot_dims, ctx.positions, ctx.token_seq, cache)
+        sizes = (self.heads, self.plain, self.rot, self.rank, self.interleaved, self.amplitude)
+        if self.query_rank:
+            query_latent = ws.get("query_latent", tokens, self.query_rank, dtype)
+            ops.latent_store(rows, self.latent_offset, self.latent_weight, self.eps, *rotation, None, *sizes, q_latent=(0, self.query_weight, query_latent))
+            query_rows = ws.get("latent_query_rows", tokens, self.query_width, dtype)
+            ops.linear(query_latent, self.w_uq, query_rows)
+            ops.latent_store(None, 0, self.latent_weight, self.eps, *rotation, flat_queries, *sizes, query_rows=query_rows)
+        else:
+            query_rows = rows[:, : self.query_width]
+            ops.latent_store(rows, self.latent_offset, self.latent_weight, self.eps, *rotation, flat_queries, *sizes)
         queries = flat_queries.view(tokens, self.heads, width)
-        per_head = rows[:, : self.latent_offset].view(tokens, self.heads, self.plain + self.rot)
+        per_head = query_rows.view(tokens, self.heads, self.plain + self.rot)
         ops.head_linear(per_head[:, :, : self.plain], self.w_uk_t, queries[:, :, : self.rank])
         summed = ws.get("latent_sums", tokens, self.heads * self.rank, dtype)
         ops.mixed_heads_attention(flat_queries, -1, ctx.positions, ctx.token_seq, cache, None, None, summed, self.heads, 1, width,
                                   self.rank, 0, self.scale, batch=ctx, sinks=self.sinks, values_in_keys=True)
         mixed = ws.get("attention", tokens, self.heads * self.vdim, dtype)
-        ops.head_linear(summed.view(tokens, self.heads, self.rank), self.w_uv, mixed.view(tokens, self.heads, self.vdim))
+        gate = rows[:, self.gate_offset : self.gate_offset + self.heads * self.vdim] if self.gate_offset >= 0 else None
+        ops.head_linear(summed.view(tokens, self.heads, self.rank), self.w_uv, mixed.view(tokens, self.heads, self.vdim), gate)
         if accumulate_into is not None:
             ops.linear_accumulate(mixed, self.w_o, accumulate_into, prepare)
             return None
@@ -436,9 +549,7 @@ class DifferentialAttention(Mixer):
         # lambda: one number for the layer, worked out once in 32-bit
         l = {name: weights.get(f"{prefix}.{name}", torch.float32) for name in ("lq1", "lk1", "lq2", "lk2")}
         self.lam = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum())) + self.diff
-        # frequencies in 64-bit, rounded once: the angle is float(position) * frequency in 32-bit inside the kernel
-        exponent = -2.0 * np.arange(self.rot_dims // 2, dtype=np.float64) / float(max(self.rot_dims, 1))
-        self.inv_freq = torch.from_numpy(np.power(float(spec.get("rot_base", 10000.0)), exponent).astype(np.float32)).to(runtime.device)
+        self.inv_freq = torch.from_numpy(rotation_frequencies(self.rot_dims, spec.get("rot_base", 10000.0))[0]).to(runtime.device)
 
     def forward(self, x, ctx, cache: LayerCache):
         ws, dtype, tokens = self.runtime.workspace, self.runtime.dtype, x.shape[0]
@@ -459,3 +570,4 @@ register_part("mixer", "differential_attention", DifferentialAttention)
 register_part("mixer", "mixed_heads_attention", MixedHeadsAttention)
 register_part("mixer", "normed_key_attention", NormedKeyAttention)
 register_part("mixer", "latent_attention", LatentAttention)
+register_part("mixer", "sigmoid_attention", SigmoidAttention)

@@ -194,6 +194,70 @@ class SandwichNormBlock(Block):
         return residual, None
 
 
+class OutputNormBlock(Block):
+    """x -> x + norm(mixer(x)) -> x + norm'(feed_forward(x)): the sublayers read the stream itself, and a norm stands on each one's output
+    before that joins the stream.
+
+    params: ``mixer``, ``feed_forward`` (or None), ``mixer_norm``, ``feed_forward_norm`` (PartSpecs of a norm kind that offers ``join_stream``), each with its
+    tensor-name suffix (``*_name``).  A branch's norm, its sum into the 32-bit stream and the rounded copy that the next sublayer reads
+    are one kernel; the copy behind the last sublayer goes to the next block as an ``ops.StreamCopy``.
+    """
+
+    _SLOTS = (("mixer", "mixer"), ("mixer_norm", "norm"), ("feed_forward", "feed_forward"), ("feed_forward_norm", "norm"))
+
+    capturable = True
+    accepts_next_norm = True
+
+    @classmethod
+    def _slots(cls, spec: PartSpec):
+        return [pair for pair in cls._SLOTS if spec.get("feed_forward") is not None or not pair[0].startswith("feed_forward")]
+
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
+        specs: list[TensorSpec] = []
+        for slot, category in cls._slots(spec):
+            child = spec[slot]
+            specs += part_class(category, child).tensor_specs(child, f"{prefix}.{spec[slot + '_name']}")
+        return specs
+
+    @classmethod
+    def cache_need(cls, spec: PartSpec) -> CacheNeed:
+        return part_class("mixer", spec["mixer"]).cache_need(spec["mixer"])
+
+    def __init__(self, spec, prefix, weights, runtime):
+        super().__init__(spec, prefix, weights, runtime)
+        self.feed_forward = self.feed_forward_norm = None
+        for slot, category in self._slots(spec):
+            setattr(self, slot, build_part(category, spec[slot], f"{prefix}.{spec[slot + '_name']}", weights, runtime))
+
+    def _stream(self, residual, pending):
+        """The finished stream as a product's operand, whoever ran before."""
+        from .. import ops
+
+        if isinstance(pending, ops.StreamCopy):
+            return pending.copy
+        if isinstance(pending, ops.LazyNorm):
+            pending = None   # the residual is complete
+        if self.runtime.dtype == torch.float32:
+            if pending is not None:
+                ops.add_(residual, pending)
+            return residual
+        x = self.runtime.workspace.get("stream_rounded", residual.shape[0], residual.shape[1], self.runtime.dtype)
+        ops.complete_and_round(residual, pending, x)
+        return x
+
+    def forward(self, residual, pending, ctx, cache: LayerCache, next_norm=None):
+        from .. import ops
+
+        branch, norm = self.mixer.forward(self._stream(residual, pending), ctx, cache), self.mixer_norm
+        if self.feed_forward is not None:
+            branch, norm = self.feed_forward.forward(norm.join_stream(residual, branch), ctx), self.feed_forward_norm
+        if next_norm is None:
+            return residual, ops.StreamCopy(residual, norm.join_stream(residual, branch))
+        norm.join(residual, branch)   # what reads the stream next norms it first: no copy
+        return residual, None
+
+
 class StreamInputMixBlock(Block):
     """x -> W [x ; x0]: the stream and the embedding's output x0 (the token's table row times a constant), side by side, through one
     product that gives the new stream (what a model does before each pass of a run of layers that it repeats).  It keeps nothing
@@ -230,6 +294,7 @@ class StreamInputMixBlock(Block):
         return mixed, None
 
 
+register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "pre_norm_residual", PreNormResidualBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)
 register_part("block", "stream_input_mix", StreamInputMixBlock)

@@ -5,7 +5,7 @@ import torch
 
 from .. import ops
 from ..errors import ConfigError
-from .base import FeedForward, register_part
+from .base import FeedForward, build_part, part_class, register_part
 from .spec import PartSpec, TensorSpec
 
 
@@ -102,8 +102,10 @@ class GatedMLP(FeedForward):
 class DenseMLP(FeedForward):
     """down( act(up(x)) ), no gate and no biases.
 
-    params: ``hidden_size``, ``intermediate_size``, ``activation`` ("relu_squared", "gelu_tanh" or "silu"; ops.ACTIVATIONS),
+    params: ``hidden_size``, ``intermediate_size``, ``activation`` ("relu_squared", "gelu_tanh", "silu" or "xielu"; ops.ACTIVATIONS),
     optional ``up_name`` / ``down_name`` (the tensors are ``<prefix>.<name>``: "up" and "down" unless given).
+    "xielu" has two learned numbers (p, q), the tensor ``<prefix>.act`` [2]: softplus(p) z^2 + z / 2 for z > 0 and
+    (1/2 + softplus(q)) (e^z - 1 - z) + z / 2 below; both softplus are worked out once, at load time.
     The activation is computed in 32-bit on the first product's (rounded) output.  With few rows the norm in front and the
     activation behind are applied inside the first product and the residual add inside the second, as the gated feed-forward does.
     """
@@ -121,7 +123,8 @@ class DenseMLP(FeedForward):
     def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
         hidden, inter = spec["hidden_size"], spec["intermediate_size"]
         up, down = cls._names(spec, prefix)
-        return [TensorSpec(up, (inter, hidden), std=hidden ** -0.5), TensorSpec(down, (hidden, inter), std=inter ** -0.5)]
+        specs = [TensorSpec(up, (inter, hidden), std=hidden ** -0.5), TensorSpec(down, (hidden, inter), std=inter ** -0.5)]
+        return specs + ([TensorSpec(f"{prefix}.act", (2,), std=0.5)] if spec.get("activation") == "xielu" else [])
 
     def __init__(self, spec, prefix, weights, runtime):
         super().__init__(spec, prefix, weights, runtime)
@@ -133,6 +136,10 @@ class DenseMLP(FeedForward):
         up, down = self._names(spec, prefix)
         self.w_up = weights.get(up, runtime.dtype).contiguous()
         self.w_down = weights.get(down, runtime.dtype).contiguous()
+        self.constants = (0.0, 0.0)
+        if self.activation == "xielu":
+            p, q = torch.nn.functional.softplus(weights.get(f"{prefix}.act", torch.float32).double()).tolist()
+            self.constants = (p, 0.5 + q)
 
     def adds_to_residual(self, rows: int) -> bool:
         return ops.can_accumulate(rows, self.w_down)
@@ -140,7 +147,7 @@ class DenseMLP(FeedForward):
     def forward(self, x, ctx, accumulate_into=None, prepare=None):
         ws, dtype, tokens = self.runtime.workspace, self.runtime.dtype, x.shape[0]
         act = ws.get("activated", tokens, self.inter, dtype)
-        ops.linear_activated(x, self.w_up, act, self.activation)   # few rows: norm, product and activation are one kernel
+        ops.linear_activated(x, self.w_up, act, self.activation, self.constants)   # few rows: norm, product and activation are one kernel
         if accumulate_into is not None:
             ops.linear_accumulate(act, self.w_down, accumulate_into, prepare)
             return None
@@ -159,12 +166,15 @@ class RoutedExperts(FeedForward):
     s / (sum of the chosen s + 1e-20) * ``route_scale``.  out = sum_k weight_k expert_k(x) + shared(x).
     ``normalize`` False: the weights are the chosen experts' scores as they are (times ``route_scale``).  ``weight_input`` True: the weight
     multiplies what the expert reads and not what it returns, out = sum_k expert_k(weight_k x) + shared(x).
+    ``scores`` "softmax": s = softmax(z) over all experts.  ``group_score`` "best": a group's score is its largest choice score.
+    ``activation`` "relu_squared": experts (and the shared one) without a gate, W_down act(W_up x).  ``shared_gate`` True: the shared expert's output is
+    multiplied by sigmoid(w x), one number per token, w the tensor ``<prefix>.shared.sg`` [1, hidden]: a row more in the router's product.
 
     params: ``hidden_size``, ``experts``, ``top``, ``expert_size`` (an expert's inner width), ``groups``, ``keep_groups``, ``route_scale``,
     ``activation`` ("silu" or "gelu_tanh"), ``shared_size`` (0 or None: no shared expert), ``correction`` (whether the tensor exists),
-    ``normalize`` (True), ``weight_input`` (False).
+    ``normalize`` (True), ``weight_input`` (False), ``scores`` ("sigmoid"), ``group_score`` ("two_best"), ``shared_gate`` (False).
     tensors: ``<prefix>.router`` [experts, hidden], ``<prefix>.correction`` [experts], ``<prefix>.e<i>.{gate,up,down}``,
-    ``<prefix>.shared.{gate,up,down}``.  The experts' gate and up rows are stacked per expert at load time, [experts, 2 ff, hidden].
+    ``<prefix>.shared.{gate,up,down}`` (without a gate: up and down).  The experts' gate and up rows are stacked per expert at load time, [experts, 2 ff, hidden].
     """
 
     capturable = True
@@ -174,21 +184,29 @@ class RoutedExperts(FeedForward):
         size = int(spec.get("shared_size") or 0)
         if size <= 0:
             return None
-        return PartSpec("gated_mlp", {"hidden_size": spec["hidden_size"], "intermediate_size": size, "activation": spec.get("activation", "silu"), "names": ("gate", "up", "down")})
+        sizes = {"hidden_size": spec["hidden_size"], "intermediate_size": size, "activation": spec.get("activation", "silu")}
+        return PartSpec("gated_mlp", {**sizes, "names": ("gate", "up", "down")}) if cls._gated(spec) else PartSpec("dense_mlp", sizes)
+
+    @classmethod
+    def _gated(cls, spec: PartSpec) -> bool:
+        return spec.get("activation", "silu") in ops.GATE_KINDS
 
     @classmethod
     def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
         hidden, ff = int(spec["hidden_size"]), int(spec["expert_size"])
         specs = []
         for e in range(int(spec["experts"])):
-            specs += [TensorSpec(f"{prefix}.e{e}.gate", (ff, hidden), std=hidden ** -0.5), TensorSpec(f"{prefix}.e{e}.up", (ff, hidden), std=hidden ** -0.5),
-                      TensorSpec(f"{prefix}.e{e}.down", (hidden, ff), std=ff ** -0.5)]
+            if cls._gated(spec):
+                specs.append(TensorSpec(f"{prefix}.e{e}.gate", (ff, hidden), std=hidden ** -0.5))
+            specs += [TensorSpec(f"{prefix}.e{e}.up", (ff, hidden), std=hidden ** -0.5), TensorSpec(f"{prefix}.e{e}.down", (hidden, ff), std=ff ** -0.5)]
         specs.append(TensorSpec(f"{prefix}.router", (int(spec["experts"]), hidden), std=hidden ** -0.5))
         if spec.get("correction", True):
             specs.append(TensorSpec(f"{prefix}.correction", (int(spec["experts"]),), std=0.1))
         shared = cls._shared_spec(spec)
         if shared is not None:
-            specs += GatedMLP.tensor_specs(shared, f"{prefix}.shared")
+            specs += part_class("feed_forward", shared).tensor_specs(shared, f"{prefix}.shared")
+            if spec.get("shared_gate"):
+                specs.append(TensorSpec(f"{prefix}.shared.sg", (1, hidden), std=hidden ** -0.5))
         return specs
 
     def __init__(self, spec, prefix, weights, runtime):
@@ -200,24 +218,34 @@ class RoutedExperts(FeedForward):
         self.normalize, self.weight_input = bool(spec.get("normalize", True)), bool(spec.get("weight_input", False))
         if self.experts % self.groups or not 0 < self.keep <= self.groups or not 0 < self.top <= self.keep * (self.experts // self.groups):
             raise ConfigError(f"{prefix}: {self.experts} experts in {self.groups} groups of which {self.keep} are kept cannot give {self.top} per token")
-        if self.activation not in ops.GATE_KINDS:
+        if self.activation not in ops.EXPERT_KINDS:
             raise ConfigError(f"{prefix}: experts have no activation {self.activation!r}")
         dtype = runtime.dtype
-        self.w_gate_up = torch.stack([torch.cat([weights.get(f"{prefix}.e{e}.gate", dtype), weights.get(f"{prefix}.e{e}.up", dtype)], dim=0) for e in range(self.experts)]).contiguous()
+        first = ("gate", "up") if self._gated(spec) else ("up",)
+        self.w_gate_up = torch.stack([torch.cat([weights.get(f"{prefix}.e{e}.{name}", dtype) for name in first], dim=0) for e in range(self.experts)]).contiguous()
         self.w_down = torch.stack([weights.get(f"{prefix}.e{e}.down", dtype) for e in range(self.experts)]).contiguous()
         self.router = weights.get(f"{prefix}.router", torch.float32).contiguous()
         self.correction = weights.get(f"{prefix}.correction", torch.float32).contiguous() if spec.get("correction", True) else None
+        self.scores, self.group_score = spec.get("scores", "sigmoid"), spec.get("group_score", "two_best")
+        if self.scores not in ops.ROUTER_SCORES or self.group_score not in ops.GROUP_SCORES:
+            raise ConfigError(f"{prefix}: a router has no scores {self.scores!r} or no group score {self.group_score!r}")
         shared = self._shared_spec(spec)
-        self.shared = None if shared is None else GatedMLP(shared, f"{prefix}.shared", weights, runtime)
+        self.shared = None if shared is None else build_part("feed_forward", shared, f"{prefix}.shared", weights, runtime)
+        self.gates_shared = self.shared is not None and bool(spec.get("shared_gate", False))
+        if self.gates_shared:
+            self.router = torch.cat([self.router, weights.get(f"{prefix}.shared.sg", torch.float32)], dim=0).contiguous()
 
     def forward(self, x, ctx):
         ws, dtype, tokens = self.runtime.workspace, self.runtime.dtype, x.shape[0]
         ids = ws.get("expert_ids", tokens, self.top, torch.int32)
         weights = ws.get("expert_weights", tokens, self.top, torch.float32)
-        ops.moe_route(x, self.router, self.correction, ids, weights, self.groups, self.keep, self.route_scale, normalize=self.normalize)
+        shared_gate = ws.get("shared_gate", tokens, 1, torch.float32) if self.gates_shared else None
+        ops.moe_route(x, self.router, self.correction, ids, weights, self.groups, self.keep, self.route_scale, normalize=self.normalize, scores=self.scores,
+                      group_score=self.group_score, shared_gate=shared_gate)
         shared = None if self.shared is None else self.shared.forward(x, ctx)
         out = ws.get("routed_out", tokens, self.hidden, dtype)
-        ops.moe_experts(x, self.w_gate_up, self.w_down, ids, weights, shared, out, self.activation, batch=ctx, weight_input=self.weight_input)
+        ops.moe_experts(x, self.w_gate_up, self.w_down, ids, weights, shared, out, self.activation, batch=ctx, weight_input=self.weight_input,
+                        shared_gate=shared_gate)
         return out
 
 

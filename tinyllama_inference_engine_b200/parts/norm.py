@@ -1,4 +1,4 @@
-"""RMSNorm, with the residual add fused in front of it; and the layer norm without a bias."""
+"""RMSNorm, with the residual add fused in front of it; and the layer norm, with and without a bias."""
 from __future__ import annotations
 
 import torch
@@ -53,12 +53,14 @@ class RMSNorm(Norm):
 
 
 class LayerNorm(Norm):
-    """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight: a layer norm with a weight and no bias.
+    """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight (+ bias): a layer norm.
 
-    params: ``size``, ``eps``, optional ``suffix`` (what follows the prefix in the tensor's name, ".weight" unless given).
-    tensors: ``<prefix><suffix> [size]``.  Mean, variance, scale and the residual sum are 32-bit in both precisions; the weight is held
-    in 32-bit.  ``forward`` adds ``delta`` into the stream first, as the RMS norm does; ``join`` is what a block calls that normalises a
+    params: ``size``, ``eps``, optional ``suffix`` (what follows the prefix in the tensor's name, ".weight" unless given), optional ``bias`` (whether there
+    is a tensor of the same name with ".b" added).
+    tensors: ``<prefix><suffix> [size]``, ``<prefix><suffix>.b [size]``.  Mean, variance, scale and the residual sum are 32-bit in both precisions; weight and
+    bias are held in 32-bit.  ``forward`` adds ``delta`` into the stream first, as the RMS norm does; ``join`` is what a block calls that normalises a
     branch before it joins the stream: ``residual += self(y)``, and in the same kernel the next norm of the stream if one is named.
+    ``join_stream`` is the same for a block whose next sublayer reads the stream itself.
     """
 
     capturable = True
@@ -68,29 +70,42 @@ class LayerNorm(Norm):
 
     @classmethod
     def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
-        return [TensorSpec(f"{prefix}{spec.get('suffix', '.weight')}", (spec["size"],), init="norm", std=0.1)]
+        name = f"{prefix}{spec.get('suffix', '.weight')}"
+        return [TensorSpec(name, (spec["size"],), init="norm", std=0.1)] + ([TensorSpec(f"{name}.b", (spec["size"],), std=0.2)] if spec.get("bias") else [])
 
     def __init__(self, spec, prefix, weights, runtime):
         super().__init__(spec, prefix, weights, runtime)
         self.size = int(spec["size"])
         self.eps = float(spec["eps"])
-        self.weight = weights.get(f"{prefix}{spec.get('suffix', '.weight')}", torch.float32).contiguous()
+        name = f"{prefix}{spec.get('suffix', '.weight')}"
+        self.weight = weights.get(name, torch.float32).contiguous()
+        self.bias = weights.get(f"{name}.b", torch.float32).contiguous() if spec.get("bias") else None
 
     def forward(self, residual, delta=None, rows=None, lazy: bool = False):
         if delta is not None:
             ops.add_(residual, delta)
         count = residual.shape[0] if rows is None else rows.shape[0]
         out = self.runtime.workspace.get("normed" if rows is None else "normed_rows", count, self.size, self.runtime.dtype)
-        ops.branch_norm(residual, None, None, self.weight, out, self.eps, self.centred, rows, groups=self.groups)
+        ops.branch_norm(residual, None, None, self.weight, out, self.eps, self.centred, rows, groups=self.groups, next_bias=self.bias)
         return out
 
     def join(self, residual, branch, following: "LayerNorm | None" = None):
         """``residual += self(branch)``; with ``following`` (a norm of this kind and eps) also returns ``following(residual)``, one kernel."""
         if following is None:
-            ops.branch_norm(residual, branch, self.weight, None, None, self.eps, self.centred, groups=self.groups)
+            ops.branch_norm(residual, branch, self.weight, None, None, self.eps, self.centred, groups=self.groups, post_bias=self.bias)
             return None
         out = self.runtime.workspace.get("normed", residual.shape[0], self.size, self.runtime.dtype)
-        ops.branch_norm(residual, branch, self.weight, following.weight, out, self.eps, self.centred, groups=self.groups)
+        ops.branch_norm(residual, branch, self.weight, following.weight, out, self.eps, self.centred, groups=self.groups, post_bias=self.bias, next_bias=following.bias)
+        return out
+
+    def join_stream(self, residual, branch):
+        """``residual += self(branch)``; returns the finished stream as the next product's operand: rounded by the same kernel, or in the 32-bit
+        path the stream itself."""
+        if self.runtime.dtype == torch.float32:
+            self.join(residual, branch)
+            return residual
+        out = self.runtime.workspace.get("stream_rounded", residual.shape[0], self.size, self.runtime.dtype)
+        ops.branch_norm(residual, branch, self.weight, None, out, self.eps, self.centred, groups=self.groups, post_bias=self.bias)
         return out
 
 
