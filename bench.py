@@ -455,6 +455,40 @@ def kilurax_config(size: dict, extra: dict) -> dict:
             "embedding": {"scale": size["width"] ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}}, "canon": {"taps": extra["taps"]}, "layers": layers}
 
 
+# `--designs nopuzen`: Nopuzen (latent attention whose queries pass a latent of their own, with a stretched rotation and a gate per element;
+# attention with biased projections, normed and rotated queries and keys and sigmoid weights; layer norms with a bias on the sublayers'
+# outputs; every second layer a mixture of experts without a gate behind a softmax router beside a gated shared expert, the others two
+# products with xIELU between them) beside Redasun, the closest of the engine's designs (layer norms around every sublayer, attention with
+# normed and rotated queries and keys over pages, every second layer a mixture of experts beside a shared one), at equal width, layer count,
+# vocabulary, feed-forward and expert widths.
+NOPUZEN_SIZES = {
+    "w2048": dict(latent=dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=768), attention=dict(heads=16, kv_heads=4, dim=128, vdim=128, softcap=30.0),
+                  experts=32, top=4, groups=(8, 4), expert_ff=1408, shared_ff=1408, pattern=("latent_attention", "attention", "latent_attention", "latent_attention")),
+    "w4096": dict(latent=dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536), attention=dict(heads=32, kv_heads=8, dim=128, vdim=128, softcap=30.0),
+                  experts=32, top=4, groups=(8, 4), expert_ff=3584, shared_ff=3584, pattern=("latent_attention", "attention")),
+}
+
+
+def nopuzen_config(size: dict, extra: dict) -> dict:
+    layers = []
+    for index in range(size["layers"]):
+        kind = extra["pattern"][index % len(extra["pattern"])]
+        if kind == "attention":
+            a = extra["attention"]
+            mixer = {**a, "scale": a["dim"] ** -0.5, "rot": {"base": 500000.0, "dims": a["dim"]}}
+        else:
+            l = extra["latent"]
+            mixer = {**l, "scale": (l["dim"] + l["rot_dim"]) ** -0.5,
+                     "rot": {"base": 10000.0, "dims": l["rot_dim"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        if index % 2 == 0:
+            mlp = {"kind": "dense", "ff": size["ff"]}
+        else:
+            mlp = {"kind": "moe", "expert": {"ff": extra["expert_ff"]}, "shared": {"ff": extra["shared_ff"]},
+                   "router": {"experts": extra["experts"], "top": extra["top"], "scale": 2.0, "groups": {"count": extra["groups"][0], "keep": extra["groups"][1]}}}
+        layers.append({"type": kind, "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Nopuzen", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-5}, "layers": layers}
+
+
 def run_designs(args) -> dict:
     import numpy as np
     import torch
@@ -871,13 +905,136 @@ def run_designs(args) -> dict:
                 out["attention_decode"] = {"ms": ms, "gbs": moved / ms / 1e6, "frac": moved / (ms / 1e3) / 1e9 / peak["hbm_gbs"], "store_ms": store_ms, "like_store_ms": like_store_ms}
         return out
 
+    def nopuzen_kernel_numbers(size: dict, extra: dict) -> dict:
+        """Nopuzen's own kernels alone against their rooflines, beside like kernels of the other designs at the same sizes: sigmoid attention beside the
+        Llama path's and beside softmax over the same planes (Zirutar's attention), its norm + rotation + cache write beside Redasun's; latent
+        attention (the kernel is Zirutar's) and what stands around it; experts without a gate beside gated ones; the softmax router beside the sigmoid
+        one; the norm of a branch and the stream's copy beside the branch norm and the next norm; xIELU beside the gelu gate."""
+        a, l, W, page, bf16 = extra["attention"], extra["latent"], size["width"], 64, torch.bfloat16
+        H, G, D = a["heads"], a["kv_heads"], a["dim"]
+        LH, rank, rot, plain, vdim, q_rank = l["heads"], l["kv_rank"], l["rot_dim"], l["dim"], l["vdim"], l["q_rank"]
+        E, top, F = extra["experts"], extra["top"], extra["expert_ff"]
+        out = {}
+        pages_needed = -(-(context + 1) // page) * batch + -(-prompt_tokens // page)
+        pages = torch.randn(pages_needed, 2, G, page, D, device=device).to(bf16)
+        diff_planes = (torch.randn(pages_needed, G, page, D, device=device).to(bf16), torch.randn(pages_needed, G // 2, page, D, device=device).to(bf16))
+        latent_pages = torch.randn(pages_needed, 1, 1, page, rank + rot, device=device).to(bf16)
+        inv_freq = torch.tensor([10000.0 ** (-2.0 * i / D) for i in range(D // 2)], dtype=torch.float32, device=device)
+        latent_freq = torch.tensor([10000.0 ** (-2.0 * i / rot) for i in range(rot // 2)], dtype=torch.float32, device=device)
+        ones, factors, shifts = torch.ones(W, device=device), torch.full((H,), D ** -0.5, device=device), torch.linspace(-6.0, 0.0, H, device=device)
+        biases = (torch.zeros(H * D, device=device), torch.zeros(G * D, device=device), torch.zeros(G * D, device=device))
+        up, down = (torch.randn(E, F, W, device=device) * W ** -0.5).to(bf16), (torch.randn(E, W, F, device=device) * F ** -0.5).to(bf16)
+        gate_up = (torch.randn(E, 2 * F, W, device=device) * W ** -0.5).to(bf16)
+        router = torch.randn(E + 1, W, device=device) * W ** -0.5
+        w_up, w_down = (torch.randn(size["ff"], W, device=device) * W ** -0.5).to(bf16), (torch.randn(W, size["ff"], device=device) * size["ff"] ** -0.5).to(bf16)
+        w_gate_up = (torch.randn(2 * size["ff"], W, device=device) * W ** -0.5).to(bf16)
+        w_uk, w_uv = (torch.randn(LH, rank, plain, device=device) * plain ** -0.5).to(bf16), (torch.randn(LH, vdim, rank, device=device) * rank ** -0.5).to(bf16)
+
+        def context_for(lens, firsts):
+            table_width = size["positions"] // page
+            rows, at = [], 0
+            for n, f in zip(lens, firsts):
+                count = -(-(f + n) // page)
+                rows.append(list(range(at, at + count)) + [-1] * (table_width - count))
+                at += count
+            entries = [StepEntry(i, [0] * n, []) for i, n in enumerate(lens)]
+            return pack_step(entries, list(firsts), list(range(len(lens))), [rows], device)
+
+        def against_bytes(ms, moved, like_ms=None, like_moved=None, **more):
+            line = {"ms": ms, "gbs": moved / ms / 1e6, "frac": moved / (ms / 1e3) / 1e9 / peak["hbm_gbs"], **more}
+            return line if like_ms is None else {**line, "like_ms": like_ms, "like_frac": (like_moved or moved) / (like_ms / 1e3) / 1e9 / peak["hbm_gbs"]}
+
+        def against_flops(ms, flops, like_ms=None, like_flops=None, **more):
+            line = {"ms": ms, "tflops": flops / ms / 1e9, "frac": flops / (ms / 1e3) / (peak["bf16_tflops"] * 1e12), **more}
+            return line if like_ms is None else {**line, "like_ms": like_ms, "like_frac": (like_flops or flops) / (like_ms / 1e3) / (peak["bf16_tflops"] * 1e12)}
+
+        for name, lens, firsts in (("prefill", [prompt_tokens], [0]), ("decode", [1] * batch, [context] * batch)):
+            ctx, tokens, prompt = context_for(lens, firsts), sum(lens), name == "prefill"
+            causal = sum(f + i + 1 for n, f in zip(lens, firsts) for i in range(n))
+            cache = LayerCache(CacheNeed("pages"), True, pages, ctx.block_tables[0], page)
+            # sigmoid attention
+            gate_at = (H + 2 * G) * D
+            rows = torch.randn(tokens, gate_at + -(-H // 8) * 8, device=device).to(bf16)
+            store_ms = timed(lambda: ops.norm_rotary_store(rows, H * D, (H + G) * D, biases, ones[:D], ones[:D], 1e-5, factors, inv_freq, D, True, 1.0, ctx.positions, ctx.token_seq, cache,
+                                                           H, G, D, D))
+            mixed = torch.empty(tokens, H * D, dtype=bf16, device=device)
+            ms = timed(lambda: ops.mixed_heads_attention(rows, gate_at, ctx.positions, ctx.token_seq, cache, None, None, mixed, H, G, D, D, 0, 1.0, batch=ctx, gate_per_head=True,
+                                                         softcap=a["softcap"], sigmoid=True, shifts=shifts))
+            softmax_ms = timed(lambda: ops.mixed_heads_attention(rows, gate_at, ctx.positions, ctx.token_seq, cache, None, None, mixed, H, G, D, D, 0, D ** -0.5, batch=ctx,
+                                                                 gate_per_head=True))
+            qkv = torch.randn(tokens, (H + 2 * G) * D, device=device).to(bf16)
+            like_ms = timed(lambda: ops.paged_attention(qkv, pages, ctx.positions, ctx.token_seq, ctx.block_tables[0], mixed, H, G, D, page, 0, D ** -0.5, batch=ctx))
+            out[f"sigmoid_attention_{name}"] = (against_flops(ms, causal * H * 4.0 * D, like_ms, softmax_over_planes_ms=softmax_ms) if prompt
+                                                else against_bytes(ms, causal * G * 4.0 * D, like_ms, softmax_over_planes_ms=softmax_ms))
+            diff_cache = LayerCache(CacheNeed("pages"), True, None, ctx.block_tables[0], page, None, diff_planes)   # as many vectors per token: two maps of half the heads
+            diff_rows = torch.randn(tokens, (H + G + G // 2) * D, device=device).to(bf16)
+            like_ms = timed(lambda: ops.diff_store(diff_rows, H * D, (H + G) * D, ones[:D], ones[:D], 1e-5, inv_freq, D, ctx.positions, ctx.token_seq, diff_cache, H // 2, G // 2, D, D))
+            out[f"norm_rotary_store_{name}"] = against_bytes(store_ms, tokens * D * 2.0 * (2 * H + 4 * G), like_ms, tokens * D * 2.0 * (2 * H + 3 * G))
+            # latent attention and what stands around it
+            latent_cache = LayerCache(CacheNeed("pages"), True, latent_pages, ctx.block_tables[0], page)
+            queries, summed = torch.randn(tokens, LH * (rank + rot), device=device).to(bf16), torch.empty(tokens, LH * rank, dtype=bf16, device=device)
+            ms = timed(lambda: ops.mixed_heads_attention(queries, -1, ctx.positions, ctx.token_seq, latent_cache, None, None, summed, LH, 1, rank + rot, rank, 0, (plain + rot) ** -0.5,
+                                                         batch=ctx, values_in_keys=True))
+            out[f"latent_attention_{name}"] = against_flops(ms, causal * LH * 2.0 * (2 * rank + rot)) if prompt else against_bytes(ms, causal * (rank + rot) * 2.0)
+            down_rows, q_latent = torch.randn(tokens, q_rank + rank + rot + LH * vdim, device=device).to(bf16), torch.empty(tokens, q_rank, dtype=bf16, device=device)
+            q_rows = torch.randn(tokens, LH * (plain + rot), device=device).to(bf16)
+            sizes = (LH, plain, rot, rank, False, 1.1)
+            first_ms = timed(lambda: ops.latent_store(down_rows, q_rank, ones[:rank], 1e-5, latent_freq, rot, ctx.positions, ctx.token_seq, latent_cache, None, *sizes,
+                                                      q_latent=(0, ones[:q_rank], q_latent)))
+            second_ms = timed(lambda: ops.latent_store(None, 0, ones[:rank], 1e-5, latent_freq, rot, ctx.positions, ctx.token_seq, latent_cache, queries, *sizes, query_rows=q_rows))
+            like_rows = torch.randn(tokens, LH * (plain + rot) + rank + rot, device=device).to(bf16)
+            like_ms = timed(lambda: ops.latent_store(like_rows, LH * (plain + rot), ones[:rank], 1e-5, latent_freq, rot, ctx.positions, ctx.token_seq, latent_cache, queries, *sizes))
+            out[f"latent_store_{name}"] = against_bytes(first_ms + second_ms, tokens * 4.0 * (q_rank + rank + rot + LH * rot), like_ms, tokens * 4.0 * (rank + rot + LH * rot), down_ms=first_ms,
+                                                        queries_ms=second_ms)
+            gated, gate = torch.empty(tokens, LH * vdim, dtype=bf16, device=device), down_rows[:, q_rank + rank + rot :]
+            ms = timed(lambda: ops.head_linear(summed.view(tokens, LH, rank), w_uv, gated.view(tokens, LH, vdim), gate))
+            like_ms = timed(lambda: ops.head_linear(summed.view(tokens, LH, rank), w_uv, gated.view(tokens, LH, vdim)))
+            expand_ms = timed(lambda: ops.head_linear(q_rows.view(tokens, LH, plain + rot)[:, :, :plain], w_uk, queries.view(tokens, LH, rank + rot)[:, :, :rank]))
+            out[f"values_expanded_and_gated_{name}"] = (against_flops(ms, tokens * LH * 2.0 * rank * vdim, like_ms, keys_folded_ms=expand_ms) if prompt
+                                                        else against_bytes(ms, LH * rank * vdim * 2.0, like_ms, keys_folded_ms=expand_ms))
+            # router and experts
+            x = torch.randn(tokens, W, device=device).to(bf16)
+            ids, weights, shared_gate = torch.empty(tokens, top, dtype=torch.int32, device=device), torch.empty(tokens, top, device=device), torch.empty(tokens, 1, device=device)
+            like_route_ms = timed(lambda: ops.moe_route(x, router[:E], None, ids, weights, extra["groups"][0], extra["groups"][1], 2.0))
+            route_ms = timed(lambda: ops.moe_route(x, router, None, ids, weights, extra["groups"][0], extra["groups"][1], 2.0, normalize=False, scores="softmax", group_score="best",
+                                                   shared_gate=shared_gate))
+            out[f"router_{name}"] = against_bytes(route_ms, tokens * W * 2.0 + E * W * 4.0, like_route_ms)
+            shared, routed = torch.randn(tokens, W, device=device).to(bf16), torch.empty(tokens, W, dtype=bf16, device=device)
+            ms = timed(lambda: ops.moe_experts(x, up, down, ids, weights, shared, routed, "relu_squared", batch=ctx, shared_gate=shared_gate))
+            like_ms = timed(lambda: ops.moe_experts(x, gate_up, down, ids, weights, shared, routed, "silu", batch=ctx))
+            chosen = len(torch.unique(ids))
+            out[f"experts_{name}"] = (against_flops(ms, tokens * top * 4.0 * F * W, like_ms, tokens * top * 6.0 * F * W) if prompt
+                                      else against_bytes(ms, chosen * 4.0 * F * W, like_ms, chosen * 6.0 * F * W, experts_read=chosen))
+            # the dense feed-forward
+            act, ff_out = torch.empty(tokens, size["ff"], dtype=bf16, device=device), torch.empty(tokens, W, dtype=bf16, device=device)
+
+            def dense():
+                ops.linear_activated(x, w_up, act, "xielu", (0.7, 1.2))
+                ops.linear(act, w_down, ff_out)
+
+            def like_dense():
+                ops.linear_gated(x, w_gate_up, act, activation="gelu_tanh")
+                ops.linear(act, w_down, ff_out)
+
+            ms, like_ms = timed(dense), timed(like_dense)
+            out[f"dense_{name}"] = (against_flops(ms, tokens * 4.0 * size["ff"] * W, like_ms, tokens * 6.0 * size["ff"] * W) if prompt
+                                    else against_bytes(ms, 4.0 * size["ff"] * W, like_ms, 6.0 * size["ff"] * W))
+            # the norm on a branch and the stream's copy
+            stream, y, copy = torch.zeros(tokens, W, device=device), torch.randn(tokens, W, device=device).to(bf16), torch.empty(tokens, W, dtype=bf16, device=device)
+            ms = timed(lambda: ops.branch_norm(stream, y, ones, None, copy, 1e-5, post_bias=ones))
+            like_ms = timed(lambda: ops.branch_norm(stream, y, ones, ones, copy, 1e-5))
+            out[f"norms_{name}"] = against_bytes(ms, tokens * W * 12.0, like_ms)
+        return out
+
     results = {}
     which = args.designs
     with ClockSampler() as clocks:
         for key, size in DESIGN_SIZES.items():
             marutar, llama = design_configs(size)
             base = Path(tempfile.gettempdir()) / f"tlie_b200_designs_{os.getuid()}_{key}"
-            if which == "kilurax":
+            if which == "nopuzen":
+                pair = (("nopuzen", nopuzen_config(size, NOPUZEN_SIZES[key])), ("redasun", redasun_config(size, REDASUN_SIZES[key])))
+            elif which == "kilurax":
                 pair = (("kilurax", kilurax_config(size, KILURAX_SIZES[key])), ("redasun", redasun_config(size, REDASUN_SIZES[key])))
             elif which == "redasun":
                 pair = (("redasun", redasun_config(size, REDASUN_SIZES[key])), ("llama", llama))
@@ -889,7 +1046,9 @@ def run_designs(args) -> dict:
                 if not (folders[name] / "model.safetensors").exists():
                     write_random_model(folders[name], config, seed=0)
             results[key] = {name: model_numbers(folders[name]) for name, _ in pair}
-            if which == "kilurax":
+            if which == "nopuzen":
+                results[key]["kernels"] = nopuzen_kernel_numbers(size, NOPUZEN_SIZES[key])
+            elif which == "kilurax":
                 results[key]["kernels"] = kilurax_kernel_numbers(size, KILURAX_SIZES[key], ZIRUTAR_SIZES[key])
             elif which == "redasun":
                 results[key]["kernels"] = redasun_kernel_numbers(size, REDASUN_SIZES[key])
@@ -898,12 +1057,14 @@ def run_designs(args) -> dict:
             results[key]["sizes"] = {k: v for k, v in size.items() if k != "pattern"} | {"pattern": "/".join(size["pattern"])}
             if which == "redasun":
                 results[key]["sizes"] = {k: v for k, v in size.items() if k in ("width", "ff", "vocab", "layers")} | {k: (list(v) if isinstance(v, tuple) else v) for k, v in REDASUN_SIZES[key].items()}
+            if which == "nopuzen":
+                results[key]["sizes"] = {k: v for k, v in size.items() if k in ("width", "ff", "vocab", "layers")} | {k: (list(v) if isinstance(v, tuple) else v) for k, v in NOPUZEN_SIZES[key].items()}
             if which == "kilurax":
                 results[key]["sizes"] = {k: v for k, v in size.items() if k in ("width", "vocab", "layers")} | {k: (list(v) if isinstance(v, tuple) else v) for k, v in KILURAX_SIZES[key].items()}
             if which == "zirutar":
                 results[key]["sizes"] |= {k: v for k, v in ZIRUTAR_SIZES[key].items() if k != "pattern"} | {"zirutar_pattern": "/".join(ZIRUTAR_SIZES[key]["pattern"])}
     names = {"marutar": "Marutar beside the Llama decoder", "zirutar": "Zirutar beside Marutar", "redasun": "Redasun beside the Llama decoder",
-             "kilurax": "Kilurax beside Redasun"}[which]
+             "kilurax": "Kilurax beside Redasun", "nopuzen": "Nopuzen beside Redasun"}[which]
     return {"metric": f"prompt and decode throughput of {names} at equal sizes", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16",
             "data": "synthetic (random weights, uniform random token ids)", "impl": "engine", "higher_is_better": True,
             "config": {"prompt_tokens": prompt_tokens, "decode_context": context, "decode_batch": batch, "decode_steps": steps, "page_size": 64, "peaks": peak_kind,
@@ -964,9 +1125,9 @@ def main() -> int:
     parser.add_argument("--impl", default="engine", choices=["engine", "reference"])
     parser.add_argument("--reference-points", action="store_true", help="with --impl reference: also time batch 1 and 64 (minutes)")
     parser.add_argument("--sections", default="decode,e2e,prefill,points,mixed", help="which measurements to take (fewer for profiling runs; `mixed` adds requests of mixed length through the scheduler)")
-    parser.add_argument("--designs", nargs="?", const="marutar", default=None, choices=["marutar", "zirutar", "redasun", "kilurax"],
+    parser.add_argument("--designs", nargs="?", const="marutar", default=None, choices=["marutar", "zirutar", "redasun", "kilurax", "nopuzen"],
                         help="instead of the headline workload: another design beside the closest existing one at equal sizes (prompt and decode throughput through "
-                             "the engine, and the design's own kernels against their rooflines): Marutar beside the Llama decoder (the default), Zirutar beside Marutar, Redasun beside the Llama decoder, or Kilurax beside Redasun")
+                             "the engine, and the design's own kernels against their rooflines): Marutar beside the Llama decoder (the default), Zirutar beside Marutar, Redasun beside the Llama decoder, Kilurax beside Redasun, or Nopuzen beside Redasun")
     args = parser.parse_args()
     if args.gpus != 1:
         print(f"bench.py measures one GPU only: this engine is single-GPU by design (asked for {args.gpus})")

@@ -130,20 +130,23 @@ def embedding_positions(table, place_table, ids, positions, norm_weight, eps, re
     _store(residual, x)
 
 
-def activation(kind, x, out) -> None:
+def activation(kind, x, out, constants=(0.0, 0.0)) -> None:
     z = x.float()
     if kind == "relu_squared":
         y = torch.relu(z) ** 2
     elif kind == "gelu_tanh":
         y = 0.5 * z * (1.0 + torch.tanh(0.7978845608028654 * (z + 0.044715 * z ** 3)))
+    elif kind == "xielu":
+        a, b = constants
+        y = torch.where(z > 0, a * z * z, b * (torch.expm1(z.clamp(max=0.0)) - z)) + 0.5 * z
     else:
         y = z * torch.sigmoid(z)
     _store(out, y)
 
 
-def linear_activated(x, weight, out, kind) -> None:
+def linear_activated(x, weight, out, kind, constants=(0.0, 0.0)) -> None:
     linear(x, weight, out)
-    activation(kind, out, out)
+    activation(kind, out, out, constants)
 
 
 def mingru_scan(zxg, bias_z, bias_x, state, seq_starts, state_slots, out, max_rows) -> None:
