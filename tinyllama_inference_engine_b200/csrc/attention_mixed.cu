@@ -148,7 +148,7 @@ __global__ void __launch_bounds__(128) normed_store_kernel(T* __restrict__ rows,
 // multiplied by a weight (null: neither); their first ``rot_dims`` columns turn by position * inv_freq[i], cosines and sines times
 // ``amplitude``, columns (2i, 2i + 1) together if ``interleaved``, else column i with column i + rot_dims / 2; query head h is multiplied by
 // q_factors[h] (null: not).  q stays in place, k and v go into the token's page.  A warp per vector, which waits in shared memory as
-// 32-bit numbers between the passes.
+// 32-bit numbers between the passes; gridDim.y CTAs share a token's vectors (steps of few rows).
 template <typename T>
 __global__ void __launch_bounds__(256) norm_rotary_store_kernel(T* __restrict__ rows, int row_stride, int k_offset, int v_offset, const float* __restrict__ q_bias,
                                                                 const float* __restrict__ k_bias, const float* __restrict__ v_bias, const float* __restrict__ q_weight,
@@ -174,12 +174,12 @@ __global__ void __launch_bounds__(256) norm_rotary_store_kernel(T* __restrict__ 
     turn_s[half + i] = sine * amplitude;
   }
   if (page >= 0)
-    for (int i = threadIdx.x; i < kv_heads * value_dim; i += blockDim.x) {
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < kv_heads * value_dim; i += gridDim.y * blockDim.x) {
       const int head = i / value_dim, d = i - head * value_dim;
       v_pages[(size_t)page * v_page_stride + ((size_t)head * page_size + slot) * value_dim + d] = from_float<T>(to_float(row[v_offset + i]) + (v_bias != nullptr ? v_bias[i] : 0.0f));
     }
   __syncthreads();
-  for (int h = warp; h < heads + kv_heads; h += warps) {
+  for (int h = blockIdx.y * warps + warp; h < heads + kv_heads; h += gridDim.y * warps) {
     const bool is_key = h >= heads;
     const int head = is_key ? h - heads : h;
     T* src = row + (is_key ? k_offset : 0) + (size_t)head * key_dim;
@@ -221,7 +221,7 @@ __global__ void __launch_bounds__(256) norm_rotary_store_kernel(T* __restrict__ 
 // The first ``rot_dims`` columns of a rot part turn by position * inv_freq[i] (32-bit angles; cosines and sines times ``amplitude``), columns
 // (2i, 2i + 1) together if ``interleaved``, else column i with column i + rot_dims / 2.
 template <typename T>
-__global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__ down_rows, int down_stride, int latent_offset, const float* __restrict__ weight, float eps,
+__global__ void __launch_bounds__(256) latent_store_kernel(const T* __restrict__ down_rows, int down_stride, int latent_offset, const float* __restrict__ weight, float eps,
                                                            const float* __restrict__ inv_freq, int rot_dims, int interleaved, float amplitude,
                                                            const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ block_table,
                                                            int table_stride, T* __restrict__ pages, long long page_stride, int heads, int plain, int rot, int rank,
@@ -245,24 +245,41 @@ __global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__
     cached = page >= 0 ? pages + (size_t)page * page_stride + (size_t)(pos % page_size) * (rank + rot) : nullptr;
     const T* row = down_rows + (size_t)t * down_stride;
     down = row + latent_offset;
-    float squares = 0.0f;
-    for (int d = threadIdx.x; d < rank; d += blockDim.x) {
-      const float v = to_float(down[d]);
-      squares += v * v;
+    // both latents' numbers are asked for before either sum is formed, and stay in registers between the passes (eight a thread; longer
+    // latents read the rest again)
+    constexpr int kHeld = 8;
+    const T* q_src = q_latent != nullptr ? row + q_latent_offset : nullptr;
+    float held[kHeld], q_held[kHeld];
+#pragma unroll
+    for (int n = 0; n < kHeld; ++n) {
+      const int d = threadIdx.x + n * blockDim.x;
+      held[n] = d < rank ? to_float(down[d]) : 0.0f;
+      q_held[n] = (q_src != nullptr && d < q_rank) ? to_float(q_src[d]) : 0.0f;
     }
+    float squares = 0.0f, q_squares = 0.0f;
+#pragma unroll
+    for (int n = 0; n < kHeld; ++n) squares += held[n] * held[n], q_squares += q_held[n] * q_held[n];
+    for (int d = threadIdx.x + kHeld * blockDim.x; d < rank; d += blockDim.x) squares += to_float(down[d]) * to_float(down[d]);
+    if (q_src != nullptr)
+      for (int d = threadIdx.x + kHeld * blockDim.x; d < q_rank; d += blockDim.x) q_squares += to_float(q_src[d]) * to_float(q_src[d]);
     const float inv = rsqrtf(block_sum(squares, scratch) / (float)rank + eps);
-    if (cached)
-      for (int d = threadIdx.x; d < rank; d += blockDim.x) cached[d] = from_float<T>(to_float(down[d]) * inv * weight[d]);
-    if (q_latent != nullptr) {
-      const T* src = row + q_latent_offset;
-      T* dst = q_latent + (size_t)t * q_rank;
-      float q_squares = 0.0f;
-      for (int d = threadIdx.x; d < q_rank; d += blockDim.x) {
-        const float v = to_float(src[d]);
-        q_squares += v * v;
+    if (cached) {
+#pragma unroll
+      for (int n = 0; n < kHeld; ++n) {
+        const int d = threadIdx.x + n * blockDim.x;
+        if (d < rank) cached[d] = from_float<T>(held[n] * inv * weight[d]);
       }
+      for (int d = threadIdx.x + kHeld * blockDim.x; d < rank; d += blockDim.x) cached[d] = from_float<T>(to_float(down[d]) * inv * weight[d]);
+    }
+    if (q_src != nullptr) {
+      T* dst = q_latent + (size_t)t * q_rank;
       const float q_inv = rsqrtf(block_sum(q_squares, scratch) / (float)q_rank + eps);
-      for (int d = threadIdx.x; d < q_rank; d += blockDim.x) dst[d] = from_float<T>(to_float(src[d]) * q_inv * q_latent_weight[d]);
+#pragma unroll
+      for (int n = 0; n < kHeld; ++n) {
+        const int d = threadIdx.x + n * blockDim.x;
+        if (d < q_rank) dst[d] = from_float<T>(q_held[n] * q_inv * q_latent_weight[d]);
+      }
+      for (int d = threadIdx.x + kHeld * blockDim.x; d < q_rank; d += blockDim.x) dst[d] = from_float<T>(to_float(q_src[d]) * q_inv * q_latent_weight[d]);
     }
   }
   __syncthreads();   // the cosines and sines are in place
@@ -627,6 +644,28 @@ __global__ void merge_mixed_kernel(const float* __restrict__ partial, const T* _
   }
   __syncthreads();
   const float inv = scratch[0];
+  if (value_dim % 4 == 0 && part_size % 4 == 0 && (reinterpret_cast<uintptr_t>(partial) & 15) == 0 && gate_offset < 0) {
+    // four neighbours at a time, eight parts' loads in flight
+    for (int d = threadIdx.x * 4; d < value_dim; d += blockDim.x * 4) {
+      const float* at = mine + h * value_dim + d;
+      float4 total = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
+      for (int s = 0; s < splits; ++s) {
+        const float4 v = *reinterpret_cast<const float4*>(at + (size_t)s * part_size);
+        const float w = weight_s[s];
+        total.x = fmaf(v.x, w, total.x);
+        total.y = fmaf(v.y, w, total.y);
+        total.z = fmaf(v.z, w, total.z);
+        total.w = fmaf(v.w, w, total.w);
+      }
+      T* dst = out + (size_t)t * outputs + h * value_dim + d;
+      dst[0] = from_float<T>(total.x * inv);
+      dst[1] = from_float<T>(total.y * inv);
+      dst[2] = from_float<T>(total.z * inv);
+      dst[3] = from_float<T>(total.w * inv);
+    }
+    return;
+  }
   for (int d = threadIdx.x; d < value_dim; d += blockDim.x) {
     const int o = h * value_dim + d;
     float value[4] = {0.0f, 0.0f, 0.0f, 0.0f};
@@ -772,8 +811,9 @@ TLIE_EXPORT int tlie_norm_rotary_store(int dtype, void* rows, int row_stride, in
   constexpr int kThreads = 256;
   const size_t smem = ((size_t)rot_dims + (size_t)(kThreads / 32) * key_dim) * sizeof(float);
   if (rot_dims < 0 || rot_dims % 2 || rot_dims > key_dim || key_dim <= 0 || smem > 48 * 1024 || (rot_dims > 0 && inv_freq == nullptr)) return (int)cudaErrorInvalidValue;
+  const int shares = tokens < 64 ? (heads + kv_heads + kThreads / 32 - 1) / (kThreads / 32) : 1;
 #define TLIE_STORE(T)                                                                                                                                              \
-  norm_rotary_store_kernel<T><<<tokens, kThreads, smem, stream>>>((T*)rows, row_stride, k_offset, v_offset, q_bias, k_bias, v_bias, q_weight, k_weight, eps, q_factors, \
+  norm_rotary_store_kernel<T><<<dim3(tokens, shares), kThreads, smem, stream>>>((T*)rows, row_stride, k_offset, v_offset, q_bias, k_bias, v_bias, q_weight, k_weight, eps, q_factors, \
                                                                   inv_freq, rot_dims, interleaved, amplitude, positions, token_seq, block_table, table_stride,     \
                                                                   (T*)k_pages, k_page_stride, (T*)v_pages, v_page_stride, heads, kv_heads, key_dim, value_dim,       \
                                                                   page_size, write_cache)
@@ -795,7 +835,7 @@ TLIE_EXPORT int tlie_latent_store(int dtype, const void* down_rows, int down_str
   if ((q_latent != nullptr && (down_rows == nullptr || q_latent_weight == nullptr || q_rank <= 0)) || (query_rows != nullptr && queries == nullptr)) return (int)cudaErrorInvalidValue;
   const size_t smem = (size_t)rot_dims * sizeof(float);
 #define TLIE_LATENT(T)                                                                                                                                             \
-  latent_store_kernel<T><<<tokens, 128, smem, stream>>>((const T*)down_rows, down_stride, latent_offset, weight, eps, inv_freq, rot_dims, interleaved, amplitude,     \
+  latent_store_kernel<T><<<tokens, 256, smem, stream>>>((const T*)down_rows, down_stride, latent_offset, weight, eps, inv_freq, rot_dims, interleaved, amplitude,     \
                                                         positions, token_seq, block_table, table_stride, (T*)pages, page_stride, heads, plain, rot, rank, page_size, \
                                                         write_cache, (const T*)query_rows, query_stride, (T*)queries, q_latent_weight, q_latent_offset, q_rank,     \
                                                         (T*)q_latent)

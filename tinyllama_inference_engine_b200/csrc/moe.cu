@@ -181,14 +181,16 @@ __device__ __forceinline__ void lane_dot_sides(const __nv_bfloat16* const (&w)[2
       for (int k = 0; k < K; ++k) {
         const __nv_bfloat162* p0 = reinterpret_cast<const __nv_bfloat162*>(&raw[0][k]);
         const __nv_bfloat162* p1 = reinterpret_cast<const __nv_bfloat162*>(&raw[1][k]);
+        // 16 bytes a read: eight numbers read one at a time, 32 bytes apart from lane to lane, meet in the same banks eight at a time
+        const float4 lo = *reinterpret_cast<const float4*>(x[k] + d), hi = *reinterpret_cast<const float4*>(x[k] + d + 4);
+        const float v[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const float2 a0 = __bfloat1622float2(p0[i]), a1 = __bfloat1622float2(p1[i]);
-          const float v0 = x[k][d + 2 * i], v1 = x[k][d + 2 * i + 1];
-          sums[0][k] = fmaf(a0.x, v0, sums[0][k]);
-          sums[1][k] = fmaf(a1.x, v0, sums[1][k]);
-          sums[0][k] = fmaf(a0.y, v1, sums[0][k]);
-          sums[1][k] = fmaf(a1.y, v1, sums[1][k]);
+          sums[0][k] = fmaf(a0.x, v[2 * i], sums[0][k]);
+          sums[1][k] = fmaf(a1.x, v[2 * i], sums[1][k]);
+          sums[0][k] = fmaf(a0.y, v[2 * i + 1], sums[0][k]);
+          sums[1][k] = fmaf(a1.y, v[2 * i + 1], sums[1][k]);
         }
       }
     }
@@ -346,7 +348,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const T* __
   route_select(s, choice, group_score, ids, weights, t, lane, experts, groups, keep, top, route_scale, normalize, group_best);
 }
 
-constexpr int kRouteTiledWarps = 8;    // steps of many tokens (four share a CTA); a CTA of one token has 16 warps
+constexpr int kRouteTiledWarps = 8;    // steps of many tokens (four share a CTA); a CTA of one token has 32 warps
 
 // Rows of a multiple of 4 numbers: a CTA of eight warps per TOK tokens.  The tokens' rows wait in shared memory as 32-bit numbers; a warp
 // takes every eighth expert and reads its row of the router once for all TOK tokens, 16 bytes a lane at a time, so that the router
@@ -373,15 +375,29 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_tiled_kernel(const T* __
   }
   __syncthreads();
   // two experts of a warp side by side and four pieces of each ahead: a row at a time with one piece in flight made a step of few
-  // tokens wait for memory once per 512 bytes of a row.  An expert past the end reads the last one again and writes nothing.
+  // tokens wait for memory once per 512 bytes of a row.
   const int router_rows = experts + (shared_gate != nullptr ? 1 : 0);   // the last row, if there is one more, is the shared branch's gate
   for (int e0 = warp; e0 < router_rows; e0 += 2 * WARPS) {
     const int e1 = e0 + WARPS;
     const float* w0 = router + (size_t)e0 * width;
-    const float* w1 = router + (size_t)min(e1, router_rows - 1) * width;
+    const float* w1 = router + (size_t)(e1 < router_rows ? e1 : e0) * width;
     float sum[2][TOK];
 #pragma unroll
     for (int i = 0; i < TOK; ++i) sum[0][i] = sum[1][i] = 0.0f;
+    if (e1 >= router_rows) {   // a warp with one row left: eight of its pieces ahead (a token's sum runs over the columns in the same order)
+#pragma unroll 8
+      for (int d = lane * 4; d < width; d += 128) {
+        const float4 a0 = *reinterpret_cast<const float4*>(w0 + d);
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) {
+          const float4 b = *reinterpret_cast<const float4*>(xs + (size_t)i * width + d);
+          sum[0][i] = fmaf(a0.x, b.x, sum[0][i]);
+          sum[0][i] = fmaf(a0.y, b.y, sum[0][i]);
+          sum[0][i] = fmaf(a0.z, b.z, sum[0][i]);
+          sum[0][i] = fmaf(a0.w, b.w, sum[0][i]);
+        }
+      }
+    } else
 #pragma unroll 4
     for (int d = lane * 4; d < width; d += 128) {
       const float4 a0 = *reinterpret_cast<const float4*>(w0 + d);
@@ -436,7 +452,7 @@ constexpr int kDownOutputs = 32;
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(kMoeWarps * 32) moe_gate_up_kernel(const T* __restrict__ x, const T* __restrict__ gate_up, const int* __restrict__ ids,
                                                                      const float* __restrict__ input_weights, T* __restrict__ act, int width, int ff, int top, int kind) {
-  extern __shared__ float moe_x[];
+  extern __shared__ __align__(16) float moe_x[];
   const int slot = blockIdx.x, t = slot / top;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float scale = input_weights != nullptr ? input_weights[slot] : 1.0f;   // an expert that reads its token times the token's weight
@@ -477,7 +493,7 @@ template <typename T>
 __global__ void __launch_bounds__(kMoeWarps * 32, 4) moe_down_kernel(const T* __restrict__ act, const T* __restrict__ down, const int* __restrict__ ids,
                                                                   const float* __restrict__ weights, const T* __restrict__ shared,
                                                                   const float* __restrict__ shared_gate, T* __restrict__ out, int width, int ff, int top) {
-  extern __shared__ float moe_act_rows[];   // [top][ff]
+  extern __shared__ __align__(16) float moe_act_rows[];   // [top][ff]
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int i = threadIdx.x; i < top * ff; i += blockDim.x) moe_act_rows[i] = to_float(act[(size_t)t * top * ff + i]);
@@ -544,9 +560,9 @@ TLIE_EXPORT int tlie_moe_route(int dtype, const void* x, const float* router, co
       cudaError_t e = cudaSuccess;
 #define TLIE_ROUTE_TILED(T, TOK)                                                                                                                          \
   do {                                                                                                                                                    \
-    if (tiled > 48 * 1024) e = cudaFuncSetAttribute(moe_route_tiled_kernel<T, TOK, (TOK == 1 ? 16 : kRouteTiledWarps)>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tiled);             \
+    if (tiled > 48 * 1024) e = cudaFuncSetAttribute(moe_route_tiled_kernel<T, TOK, (TOK == 1 ? 32 : kRouteTiledWarps)>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tiled);             \
     if (e == cudaSuccess)                                                                                                                                 \
-      moe_route_tiled_kernel<T, TOK, (TOK == 1 ? 16 : kRouteTiledWarps)><<<blocks, (TOK == 1 ? 16 : kRouteTiledWarps) * 32, tiled, stream>>>((const T*)x, router, correction, ids, weights, tokens, width, experts, groups, keep, \
+      moe_route_tiled_kernel<T, TOK, (TOK == 1 ? 32 : kRouteTiledWarps)><<<blocks, (TOK == 1 ? 32 : kRouteTiledWarps) * 32, tiled, stream>>>((const T*)x, router, correction, ids, weights, tokens, width, experts, groups, keep, \
                                                                                      top, route_scale, normalize, softmax, group_best, shared_gate);                \
   } while (0)
       if (dtype == TLIE_F32) {

@@ -11,6 +11,7 @@
 //   add_bias            x[t, i] += bias[i]
 // Storage float or bfloat16, arithmetic 32-bit.
 #include "common.cuh"
+#include "mma_utils.cuh"
 
 namespace tlie {
 
@@ -172,6 +173,58 @@ __global__ void add_bias_kernel(T* __restrict__ x, const float* __restrict__ bia
   if (i < count) x[i] = from_float<T>(to_float(x[i]) + bias[i % width]);
 }
 
+// The same for bfloat16 steps of up to 16 rows on the tensor cores: a CTA takes 16 outputs of one head for every row of the step, so a weight is read
+// once however many rows there are (a warp per output and row read it once per row).  16 weight rows are the A operand of an m16n8k16
+// MMA, eight rows of x the B operand; the contraction index is permuted so that a thread's 16-byte loads feed two MMAs; the four warps
+// split K and meet in shared memory.  K a multiple of 8, rows on 16-byte boundaries.
+constexpr int kHeadWarps = 4;
+template <int MT>
+__global__ void __launch_bounds__(kHeadWarps * 32) head_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, long long x_row, long long x_head,
+                                                                          const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out, long long out_row,
+                                                                          long long out_head, int rows, int n_out, int k_in, const __nv_bfloat16* __restrict__ gate,
+                                                                          long long gate_row) {
+  __shared__ float red[kHeadWarps][16][MT * 8 + 1];
+  const int h = blockIdx.y, n0 = blockIdx.x * 16;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const __nv_bfloat16* w0 = w + ((size_t)h * n_out + min(n0 + g, n_out - 1)) * k_in + t * 8;
+  const __nv_bfloat16* w1 = w + ((size_t)h * n_out + min(n0 + g + 8, n_out - 1)) * k_in + t * 8;
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  float acc[MT][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m) acc[m][0] = acc[m][1] = acc[m][2] = acc[m][3] = 0.0f;
+  const int blocks = (k_in + 31) / 32;
+#pragma unroll 4
+  for (int kb = warp; kb < blocks; kb += kHeadWarps) {
+    const bool valid = kb * 32 + t * 8 < k_in;
+    const uint4 a0 = valid ? *reinterpret_cast<const uint4*>(w0 + kb * 32) : zero, a1 = valid ? *reinterpret_cast<const uint4*>(w1 + kb * 32) : zero;
+    const unsigned lo[4] = {a0.x, a1.x, a0.y, a1.y}, hi[4] = {a0.z, a1.z, a0.w, a1.w};
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const int row = m * 8 + g;
+      const uint4 v = valid && row < rows ? *reinterpret_cast<const uint4*>(x + row * x_row + h * x_head + kb * 32 + t * 8) : zero;
+      mma_bf16(acc[m], lo, v.x, v.y);
+      mma_bf16(acc[m], hi, v.z, v.w);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m) {
+    red[warp][g][m * 8 + 2 * t] = acc[m][0];
+    red[warp][g][m * 8 + 2 * t + 1] = acc[m][1];
+    red[warp][g + 8][m * 8 + 2 * t] = acc[m][2];
+    red[warp][g + 8][m * 8 + 2 * t + 1] = acc[m][3];
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < 16 * MT * 8; i += kHeadWarps * 32) {
+    const int n = i & 15, row = i >> 4;
+    if (row >= rows || n0 + n >= n_out) continue;
+    float sum = 0.0f;
+#pragma unroll
+    for (int k = 0; k < kHeadWarps; ++k) sum += red[k][n][row];
+    if (gate != nullptr) sum *= 1.0f / (1.0f + expf(-__bfloat162float(gate[row * gate_row + (long long)h * n_out + n0 + n])));
+    out[row * out_row + h * out_head + n0 + n] = __float2bfloat16_rn(sum);
+  }
+}
+
 static inline int blocks_for(size_t total, int threads) {
   const size_t wanted = (total + threads - 1) / threads;
   const size_t most = (size_t)device_sm_count() * 16;
@@ -242,6 +295,19 @@ TLIE_EXPORT int tlie_head_linear(int dtype, const void* x, long long x_row, long
                                  int rows, int heads, int n_out, int k_in, const void* gate, long long gate_row, cudaStream_t stream) {
   const size_t total = (size_t)rows * heads * n_out;
   if (total == 0) return 0;
+  const auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (dtype == TLIE_BF16 && rows <= 16 && k_in % 8 == 0 && x_row % 8 == 0 && x_head % 8 == 0 && aligned(x) && aligned(w) && heads <= 65535) {
+    const dim3 grid((n_out + 15) / 16, heads);
+#define TLIE_HEAD_MMA(MT)                                                                                                                                          \
+  head_linear_mma_kernel<MT><<<grid, kHeadWarps * 32, 0, stream>>>((const __nv_bfloat16*)x, x_row, x_head, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, out_row, out_head, \
+                                                                   rows, n_out, k_in, (const __nv_bfloat16*)gate, gate_row)
+    if (rows <= 8)
+      TLIE_HEAD_MMA(1);
+    else
+      TLIE_HEAD_MMA(2);
+#undef TLIE_HEAD_MMA
+    return (int)cudaGetLastError();
+  }
   TLIE_BY_TYPE(dtype, (head_linear_kernel<T><<<blocks_for(total * 32, 256), 256, 0, stream>>>((const T*)x, x_row, x_head, (const T*)w, (T*)out, out_row, out_head, heads,
                                                                                        n_out, k_in, (const T*)gate, gate_row, total)));
   return (int)cudaGetLastError();

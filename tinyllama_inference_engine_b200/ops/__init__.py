@@ -298,8 +298,9 @@ HEAD_LINEAR_LIBRARY_ROWS = 64    # from this many bfloat16 rows on the per-head 
 def head_linear(x, weight, out, gate=None) -> None:
     """out[t, h, :] = weight[h] . x[t, h, :] for every head, times sigmoid(gate[t, h, :]) if a ``gate`` [T, H N] is given (its rows may be a run of columns of
     wider ones): x [T, H, K] and out [T, H, N] may be views with strides of their own
-    (last axis contiguous), weight [H, N, K] contiguous.  32-bit sums, ascending k (a row's bits depend on the row alone) in the
-    engine's own kernel; bfloat16 steps of many rows go to the library's batched product, as the other products of their size do."""
+    (last axis contiguous), weight [H, N, K] contiguous.  32-bit sums in an order that the row's own width gives; bfloat16 steps of up to 16 rows
+    run on the tensor cores (a weight read once for all rows), bfloat16 steps of many rows go to the library's batched product, as the
+    other products of their size do."""
     rows, heads, k_in = x.shape
     n_out = weight.shape[1]
     if weight.shape != (heads, n_out, k_in) or out.shape != (rows, heads, n_out) or x.stride(2) != 1 or out.stride(2) != 1 or not weight.is_contiguous():
