@@ -427,6 +427,56 @@ def test_sigmoid_attention_kernels(dtype, atol, heads, kv, dim, vdim, rot, inter
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("dim,heads,kv,page_size,softcap", [(64, 4, 2, 64, 4.0), (128, 8, 2, 64, 4.0), (128, 3, 3, 128, 30.0), (64, 16, 1, 64, 0.0)])
+def test_sigmoid_attention_in_tensor_memory(dim, heads, kv, page_size, softcap, monkeypatch):
+    """Prompt portions whose heads are 64 or 128 wide run on the tcgen05 kernel, decoding requests at the step's head on the kernel of few rows:
+    portions from position 0 and behind cached keys (a request's keys in an earlier step), page borders, a portion of 129 rows, loud scores."""
+    from tinyllama_inference_engine_b200 import ops
+    from tinyllama_inference_engine_b200.engine.batch import pack_step
+    from tinyllama_inference_engine_b200.ops import fast
+    from tinyllama_inference_engine_b200.parts.base import CacheNeed, LayerCache
+
+    g = torch.Generator().manual_seed(dim + heads)
+    lens, firsts = [1, 1, 300, 129, 200], [70, 200, 0, 130, 1]
+    totals = [f + n for n, f in zip(lens, firsts)]
+    table, count = _scrambled_table(totals, page_size, g)
+    columns = (heads + 2 * kv) * dim + heads
+    columns += -columns % 8
+    rows = [torch.randn(t, columns, generator=g).bfloat16() for t in totals]
+    for r in rows:      # some keys stand out for some queries of their head
+        r[-1, :dim] = r[5, heads * dim : (heads + 1) * dim] * 2.0
+    pages = torch.full((count, 2, kv, page_size, dim), float("nan")).bfloat16().cuda()
+    temps, shifts = (1 + 0.5 * torch.rand(heads, generator=g)) * 2.0 * dim ** -0.5, torch.linspace(-5.0, 1.0, heads)
+    gate_at, k_at, v_at = (heads + 2 * kv) * dim, heads * dim, (heads + kv) * dim
+    device = [temps.cuda(), shifts.cuda(), torch.zeros(0, device="cuda")]
+    want = []
+    for r in rows:
+        x, total = r.double(), r.shape[0]
+        q = (x[:, :k_at].view(total, heads, dim) * temps.double()[:, None]).bfloat16().double()
+        sizes = {"heads": heads, "kv_heads": kv, "scale": 1.0, "softcap": softcap if softcap > 0 else 1e6}
+        o = plain_nopuzen.sigmoid_heads(q, x[:, k_at:v_at].view(total, kv, dim), x[:, v_at:gate_at].view(total, kv, dim), torch.ones(heads).double(), shifts.double(), sizes, torch.arange(total))
+        want.append((o * torch.sigmoid(x[:, gate_at : gate_at + heads])[:, :, None]).reshape(total, heads * dim))
+    calls = []
+    kernel = fast.prefill_attention_tc
+    monkeypatch.setattr(fast, "prefill_attention_tc", lambda *a, **k: (calls.append(1), kernel(*a, **k)))
+    for pieces in ([(r, 0, f) for r, f in enumerate(firsts) if f > 0], [(r, f, n) for r, (n, f) in enumerate(zip(lens, firsts))]):
+        entries = [StepEntry(r, [0] * n, []) for r, _, n in pieces]
+        ctx = pack_step(entries, [a for _, a, _ in pieces], list(range(len(pieces))), [[table[r].tolist() for r, _, _ in pieces]], torch.device("cuda:0"))
+        cache = LayerCache(CacheNeed("pages"), True, pages, ctx.block_tables[0], page_size)
+        index = [(r, a + i) for r, a, n in pieces for i in range(n)]
+        step_rows = torch.stack([rows[r][p] for r, p in index]).cuda().contiguous()
+        ops.norm_rotary_store(step_rows, k_at, v_at, None, None, None, 1e-5, device[0], device[2], 0, True, 1.0, ctx.positions, ctx.token_seq, cache, heads, kv, dim, dim)
+        out = torch.full((len(index), heads * dim), float("nan"), dtype=torch.bfloat16, device="cuda")
+        ops.mixed_heads_attention(step_rows, gate_at, ctx.positions, ctx.token_seq, cache, None, None, out, heads, kv, dim, dim, 0, 1.0, batch=ctx, gate_per_head=True, softcap=softcap,
+                                  sigmoid=True, shifts=device[1])
+        assert int(fast.tcgen05_error_flag(out.device)) == 0, "a bounded wait inside the kernel gave up"
+        for (r, p), row in zip(index, out.cpu().double()):
+            rms_of = lambda v: float((v * v).mean().sqrt())
+            assert rms_of(row - want[r][p]) <= 1e-2 * max(0.5, rms_of(want[r][p])), (r, p)
+    assert len(calls) == 2
+
+
+@pytest.mark.gpu
 @pytest.mark.parametrize("dtype,atol", [(torch.float32, 2e-5), (torch.bfloat16, 3e-2)])
 @pytest.mark.parametrize("heads,dim,rot,vdim,rank,q_rank,interleaved", [(4, 16, 16, 32, 32, 24, False), (1, 20, 6, 10, 96, 40, False), (3, 10, 2, 7, 20, 13, True), (16, 32, 64, 32, 128, 48, False)])
 @pytest.mark.parametrize("long_tail", [False, True])
@@ -644,6 +694,21 @@ def test_long_decoding_and_other_page_sizes(cases, dtype):
     for page_size in (64, 32):
         trace_tools.run_and_compare(_runner(folder, dtype, max_tokens=2048, page_size=page_size), trace_tools.tail_decode(more, tail=150), full,
                                     atol=TOLERANCE[dtype] * scale, over_vocabulary=RMS[dtype], allowed_over=LOOSE_ROWS[dtype])
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dim,kv", [(64, 2), (128, 1)])
+def test_long_portions_beside_decoded_tokens(tmp_path, dim, kv):
+    """Portions of up to 200 rows beside single tokens with pages of 64: the tensor-memory kernel, the kernel of few rows at the step's head and the
+    ones between them, in one model."""
+    folder = write_random_model(tmp_path / "m", _config(64, 47, [_attention(4, kv, dim, dim, _dense(64)), _latent(4, 64, 64, 64, 64, 48, _dense(96), scaling=(4.0, 100, 8.0, 1.0))]), 3)
+    config, tensors = load_plain(folder)
+    requests = trace_tools.make_requests(47, [500, 230, 64, 300], seed=9)
+    full = {rid: _logits(config, tensors, tokens) for rid, tokens in requests.items()}
+    scale = max(float(v.abs().max()) for v in full.values())
+    for steps in (trace_tools.whole(requests), trace_tools.tail_decode(requests, tail=20), trace_tools.portions(requests, sizes=(200, 65, 2, 128)),
+                  trace_tools.mixed(requests, seed=2, max_portion=200)[0]):
+        trace_tools.run_and_compare(_runner(folder, "bfloat16", max_tokens=2048, page_size=64), steps, full, atol=TOLERANCE["bfloat16"] * scale, over_vocabulary=True)
 
 
 @pytest.mark.gpu

@@ -27,6 +27,11 @@
 //     before P of that tile is handed over, and the output is read once, after the last tile, and divided by the sum;
 //   * the kernel is launched as a programmatic dependent: barriers and tensor memory are set up while the kernel before
 //     it drains, global memory is touched only after the dependency wait.
+// SIGMOID_WEIGHTS 1 (a build of its own): no softmax.  The score is bounded, softcap * tanh(score / softcap), and a key's weight is
+// sigmoid(score + shift_h); nothing is brought to a sum of one, so there is no maximum, no sum and no rescaling, and the output is read
+// as it is.  tanh and sigmoid are e^x and a reciprocal each, in 32-bit; one reciprocal serves two scores (1 / a = b / (a b)), so that a
+// score costs three operations of the exponential unit.  In both kinds the output may be multiplied by sigmoid(gate), one number per
+// (row, head), as it is read out.
 // Roles: warp 0 TMA producer, warp 1 issuer of the score products and tensor-memory owner, warp 2 issuer of the P . V products,
 // warp 3 idle, warps 4..7 softmax (128 threads).  The launch gives every thread 128 registers (two CTAs of 256 threads fill the
 // register file); the first four warps hand most of theirs back at once (setmaxnreg) and the softmax warps, whose threads hold a
@@ -46,8 +51,13 @@
 // 4,096 tokens: by 3 to 24 %) than pairs of a heavy and a light tile (paired_attention_tiles), which the kernel also takes.
 #include "tcgen05_utils.cuh"
 
+#ifndef SIGMOID_WEIGHTS
+#define SIGMOID_WEIGHTS 0
+#endif
+
 namespace tlie {
 
+constexpr bool kSigmoidTC = SIGMOID_WEIGHTS != 0;
 constexpr int kRowsTC = 128;      // query rows per CTA
 constexpr int kKeysTC = 64;       // keys per tile (one box)
 constexpr int kBoxDims = 64;      // dims of one box: 128 bytes, the swizzle span
@@ -149,6 +159,25 @@ __device__ __forceinline__ Float2Bits add2(Float2Bits a, Float2Bits b) {
   return r;
 }
 
+__device__ __forceinline__ Float2Bits mul2(Float2Bits a, Float2Bits b) {
+  Float2Bits r;
+  asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(r.bits) : "l"(a.bits), "l"(b.bits));
+  return r;
+}
+__device__ __forceinline__ float reciprocal_approx(float x) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(x));
+  return r;
+}
+// 1 / (1 + 2^x) for two numbers with one reciprocal.  Exponents above 60 are taken as 60: the result, 2^-60, is as good as zero, and the
+// product of two denominators stays in range.
+__device__ __forceinline__ void inverse_one_plus_exp2(float x0, float x1, float& r0, float& r1) {
+  float a, b;
+  unpair(add2(pair_of(exp2_approx(fminf(x0, 60.0f)), exp2_approx(fminf(x1, 60.0f))), pair_of(1.0f, 1.0f)), a, b);
+  const float r = reciprocal_approx(a * b);
+  unpair(mul2(pair_of(b, a), pair_of(r, r)), r0, r1);
+}
+
 // Where a CTA's time goes, when compiled with TLIE_ATTN_TIMELINE: one thread of each role of CTA (0, 0) reports the cycles of its
 // whole loop (slot 6 of its group: softmax 0-7, issuer 8-15, producer 16-23), its tiles (slot 7) and, with TLIE_ATTN_TIMELINE_SLOT = k,
 // the cycles spent between stamp k - 1 and stamp k (slot k).  One slot per build: more would cost registers the kernel does not have.
@@ -192,7 +221,8 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
     prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                                 const int* __restrict__ tiles, const int* __restrict__ seq_starts, const int* __restrict__ first_positions,
                                 const int* __restrict__ block_table, int table_stride, __nv_bfloat16* __restrict__ out, int q_heads,
-                                int kv_heads, int page_size, int window, float scale, int* __restrict__ error_flag) {
+                                int kv_heads, int page_size, int window, float scale, float softcap, const float* __restrict__ shifts,
+                                const __nv_bfloat16* __restrict__ gate, int gate_stride, int* __restrict__ error_flag) {
   extern __shared__ uint8_t smem_raw[];
   using Smem = SmemTC<kD>;
   constexpr int kKvStages = Smem::kStages;
@@ -412,6 +442,10 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
     const int row = sub * 32 + lane;
     const uint32_t lane_base = (uint32_t)(sub * 32) << 16;
     const float sl2 = scale * kLog2eTC;
+    // sigmoid weights, in units of log2: without a bound the exponent is -(score + shift); with one see the loop
+    const float sig_to_exp = softcap > 0.0f ? 2.0f * sl2 / softcap : sl2;
+    const float sig_twice_cap = softcap > 0.0f ? 2.0f * softcap * kLog2eTC : -1.0f;
+    const float sig_base = -(softcap + (shifts != nullptr ? shifts[head] : 0.0f)) * kLog2eTC;
     int g = 0;
     bool ok = true;
     // Where tile g, g - 1 and g - 2 lie in the K / V rings (stage and phase bit of their barriers).
@@ -437,7 +471,31 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
         float sc[kKeysTC];
         tmem_ld64(tmem + lane_base + b * kKeysTC, sc);
         TL(2)
+        uint32_t packed[kKeysTC / 2];
         const bool need_mask = key0 + kKeysTC - 1 > t.pos0 || (window > 0 && key0 < t.pos0 + t.rows_here - window);
+        if constexpr (kSigmoidTC) {
+          // with u = 1 / (1 + e^(2 s / c)): c tanh(s / c) = c - 2 c u, and the weight is 1 / (1 + e^-(c - 2 c u + shift))
+          const Float2Bits to_exp2 = pair_of(sig_to_exp, sig_to_exp), twice_cap2 = pair_of(sig_twice_cap, sig_twice_cap), base2 = pair_of(sig_base, sig_base);
+#pragma unroll
+          for (int i = 0; i < kKeysTC / 2; ++i) {
+            float x0, x1, w0, w1;
+            Float2Bits score = mul2(pair_of(sc[2 * i], sc[2 * i + 1]), to_exp2);
+            if (softcap > 0.0f) {
+              float u0, u1;
+              unpair(score, x0, x1);
+              inverse_one_plus_exp2(x0, x1, u0, u1);
+              score = pair_of(u0, u1);
+            }
+            unpair(fma2(score, twice_cap2, base2), x0, x1);
+            inverse_one_plus_exp2(x0, x1, w0, w1);
+            if (need_mask) {
+              const int key = key0 + 2 * i;
+              w0 = (key >= my_lo && key <= my_pos) ? w0 : 0.0f;
+              w1 = (key + 1 >= my_lo && key + 1 <= my_pos) ? w1 : 0.0f;
+            }
+            packed[i] = pack_bf16(w0, w1);
+          }
+        } else {
         float tile_max = -INFINITY;
         if (need_mask) {
 #pragma unroll
@@ -484,7 +542,6 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
         }
         const float base = (reference == -INFINITY) ? 0.0f : reference;   // a row that has seen no key yet: every p is 0
         TL(3)
-        uint32_t packed[kKeysTC / 2];
         const Float2Bits scale2 = pair_of(sl2, sl2), minus_base2 = pair_of(-base, -base);
         Float2Bits sums = pair_of(0.0f, 0.0f);   // the even keys' sum and the odd keys'
         // (Taking a share of the exponentials on the FMA pipe, by a polynomial, was measured: a quarter of them gains 2 %, half
@@ -500,6 +557,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
         float sum0, sum1;
         unpair(sums, sum0, sum1);
         row_sum += sum0 + sum1;
+        }
         TL(4)
         // P over the first 32 columns of this tile's scores: key 2 i in the lower half of column i, key 2 i + 1 in the upper.  The
         // buffer is free for it: its scores were issued after the product that read P of two tiles back had completed.
@@ -528,7 +586,8 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
       if (ok) ok = mbar_wait(&sm.o_full[u], 0, abort_flag);
       if (ok) {
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        const float inv = 1.0f / row_sum;
+        float inv = kSigmoidTC ? 1.0f : 1.0f / row_sum;
+        if (gate != nullptr && row < t.rows_here) inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(t.row0 + row) * gate_stride + head])));
 #pragma unroll
         for (int half = 0; half < kSubTiles; ++half) {   // 64 columns of the output at a time (the load is warp-wide: every row takes part)
           float o[64];
@@ -587,7 +646,8 @@ TLIE_EXPORT int tlie_prefill_attention_tc_timeline(long long* host) { return (in
 template <int kD>
 static int launch_attention_tc(const void* q, int q_row_stride, int tokens, const void* pages, int num_pages, const int* tiles, int n_tiles,
                                const int* seq_starts, const int* first_positions, const int* block_table, int table_stride, void* out, int q_heads,
-                               int kv_heads, int page_size, int window, float scale, int* error_flag, cudaStream_t stream) {
+                               int kv_heads, int page_size, int window, float scale, float softcap, const float* shifts, const void* gate, int gate_stride,
+                               int* error_flag, cudaStream_t stream) {
   CUtensorMap map_q, map_kv;
   if (!make_map_2d(&map_q, q, tokens, (long long)q_heads * kD, q_row_stride, kRowsTC)) return (int)cudaErrorInvalidValue;
   if (!make_map_2d(&map_kv, pages, (long long)num_pages * 2 * kv_heads * page_size, kD, kD, kKeysTC)) return (int)cudaErrorInvalidValue;
@@ -605,23 +665,25 @@ static int launch_attention_tc(const void* q, int q_row_stride, int tokens, cons
   }
   dim3 grid(q_heads, n_tiles);
   return (int)launch_pdl(prefill_attention_tc_kernel<kD>, grid, dim3(kThreadsTC), (size_t)smem, stream, map_q, map_kv, tiles, seq_starts, first_positions,
-                         block_table, table_stride, (__nv_bfloat16*)out, q_heads, kv_heads, page_size, window, scale, error_flag);
+                         block_table, table_stride, (__nv_bfloat16*)out, q_heads, kv_heads, page_size, window, scale, softcap, shifts, (const __nv_bfloat16*)gate, gate_stride, error_flag);
 }
 
 // q: the step's rows [tokens, q_row_stride] starting with the rotated q heads (head size 64 or 128); pages: one layer's pool
 // [num_pages, 2, kv_heads, page_size, head size]; tiles: int32 [n_tiles, 4] work items of one or two 128-row tiles (request, first
-// row, request or -1, first row); error_flag: device int, zero.
+// row, request or -1, first row); error_flag: device int, zero.  softcap (0: none) and shifts (32-bit [q_heads] or null): SIGMOID_WEIGHTS only.
+// gate (or null): bfloat16, one number per (token, head), rows gate_stride elements apart; the output is multiplied by its sigmoid.
 TLIE_EXPORT int tlie_prefill_attention_tc(const void* q, int q_row_stride, int tokens, const void* pages, int num_pages, const int* tiles,
                                           int n_tiles, const int* seq_starts, const int* first_positions, const int* block_table,
                                           int table_stride, void* out, int q_heads, int kv_heads, int head_dim, int page_size, int window, float scale,
-                                          int* error_flag, cudaStream_t stream) {
+                                          float softcap, const float* shifts, const void* gate, int gate_stride, int* error_flag, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
+  if (!kSigmoidTC && (softcap > 0.0f || shifts != nullptr)) return (int)cudaErrorInvalidValue;
   if (kv_heads <= 0 || q_heads % kv_heads != 0 || n_tiles > 65535 || page_size % kKeysTC != 0 || q_row_stride % 8 != 0 || error_flag == nullptr ||
       (head_dim != 64 && head_dim != 128))
     return (int)cudaErrorInvalidValue;
   if (head_dim == 64)
     return launch_attention_tc<64>(q, q_row_stride, tokens, pages, num_pages, tiles, n_tiles, seq_starts, first_positions, block_table, table_stride, out,
-                                   q_heads, kv_heads, page_size, window, scale, error_flag, stream);
+                                   q_heads, kv_heads, page_size, window, scale, softcap, shifts, gate, gate_stride, error_flag, stream);
   return launch_attention_tc<128>(q, q_row_stride, tokens, pages, num_pages, tiles, n_tiles, seq_starts, first_positions, block_table, table_stride, out,
-                                  q_heads, kv_heads, page_size, window, scale, error_flag, stream);
+                                  q_heads, kv_heads, page_size, window, scale, softcap, shifts, gate, gate_stride, error_flag, stream);
 }

@@ -952,6 +952,10 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
         fast.latent_prefill(rows, batch, table, k_ptr, k_stride, sinks, out, heads, key_dim, value_dim, cache.page_size, scale)
         return
     plain_options = sinks is None and not values_in_keys   # what the tensor-core kernels with two planes know
+    if (plain_options and sigmoid and slopes is None and mix is None and window == 0 and rows.dtype == torch.bfloat16 and cache.pages is not None and key_dim == value_dim
+            and rows.shape[1] % 8 == 0 and (gate_offset < 0 or gate_per_head) and _tensor_memory_attention(rows, gate_offset, positions, token_seq, cache, out, heads, kv_heads, key_dim,
+                                                                                                           scale, batch, softcap, shifts)):
+        return
     if plain_options and (sigmoid or softcap == 0.0) and rows.dtype == torch.bfloat16 and fast.mixed_prefill_takes(batch, rows, cache.page_size, kv_heads if mix is not None else 1, key_dim, value_dim, gate_offset,
                                                                                    gate_per_head, sigmoid):
         folded = folded_slopes if folded_slopes is not None else fast.folded_slopes(slopes, mix)
@@ -976,6 +980,26 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
                                                         c_int(keep_first if window > 0 else 0), c_int(1 if gate_per_head else 0), _ptr(sinks), c_int(v_row_stride), c_float(softcap),
                                                         c_int(1 if sigmoid else 0), _ptr(shifts), _stream()),
            "mixed_heads_attention")
+
+
+def _tensor_memory_attention(rows, gate_offset: int, positions, token_seq, cache, out, heads: int, kv_heads: int, dim: int, scale: float, batch, softcap: float, shifts) -> bool:
+    """Attention with sigmoid weights for a step that carries prompt portions, on the tensor-memory kernel; decoding requests at the step's head
+    run on the kernel of few rows.  False: the step or the sizes are not for it."""
+    host_q_lens = getattr(batch, "host_q_lens", None)
+    if host_q_lens is None:
+        return False
+    lead = fast.leading_single_rows(host_q_lens)
+    tiles = fast.tc_attention_tiles(batch, dim, cache.page_size, lead)
+    if tiles is None or (lead and not fast.mixed_decode_takes(rows, heads, kv_heads, dim, dim, gate_offset, False, True)):
+        return False
+    if lead:
+        planes = _plane_pointers(cache, kv_heads, dim, dim)[1:]
+        splits = max(1, min(2 * fast.sm_count() // lead, -(-batch.max_seq_len // 32), 64))
+        fast.mixed_decode(rows[:lead], gate_offset, positions[:lead], token_seq[:lead], cache.block_table, planes, None, None, out[:lead], heads, kv_heads, dim, dim, cache.page_size, 0,
+                          scale, splits, 0, True, softcap, True, shifts)
+    fast.prefill_attention_tc(rows, cache.pages, tiles, batch.seq_starts, batch.first_positions, cache.block_table, out, heads, kv_heads, dim, cache.page_size, 0, scale, softcap, True,
+                              shifts, gate_offset)
+    return True
 
 
 # --- differential attention --------------------------------------------------------------------

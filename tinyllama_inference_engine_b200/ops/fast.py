@@ -27,6 +27,7 @@ def sm_count() -> int:
 
 DEFAULT_HEAD_DIMS = (64, 128)
 DEFAULT_MIXED_PREFILL_SETS = ((64, 64, 4), (128, 128, 8))   # (key width, value width, key heads per folded query) built ahead; others on first use
+DEFAULT_SIGMOID_SETS = ((64, 64, 4), (128, 128, 4))   # (key width, value width, key/value heads) of attention with sigmoid weights built ahead; others on first use
 DEFAULT_DIFF_SETS = ((64, 128), (128, 128))   # (key width per map, value width) of differential attention built ahead; others on first use
 _scratch: dict[torch.device, list[torch.Tensor]] = {}
 
@@ -39,12 +40,17 @@ def build_all() -> list:
     built.append(build_library("tlie_gemm_skinny", ["gemm_skinny.cu"]))
     built.append(build_library("tlie_gemm_tcgen05", TCGEN05_SOURCES))
     built.append(build_library("tlie_attn_prefill_tc", ["attention_prefill_tc.cu"]))
+    built.append(build_library("tlie_attn_prefill_tc_sigmoid", ["attention_prefill_tc.cu"], {"SIGMOID_WEIGHTS": 1}))
     built.append(build_library("tlie_probes", ["probes.cu"]))
     for key_dim, value_dim, parts in DEFAULT_MIXED_PREFILL_SETS:
         built.append(build_library(f"tlie_attn_mixed_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "PARTS": parts}))
         built.append(build_library(f"tlie_attn_mixed_decode_k{key_dim}_v{value_dim}_g{parts}", ["attention_mixed_decode.cu"],
                                    {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "KV_HEADS": parts}))
     built.append(build_library("tlie_attn_latent_k576_v512", ["attention_latent_prefill.cu"], {"KEY_DIM": 576, "VALUE_DIM": 512}))   # other widths on first use
+    for key_dim, value_dim, kv_heads in DEFAULT_SIGMOID_SETS:
+        built.append(build_library(f"tlie_attn_sigmoid_k{key_dim}_v{value_dim}_p1", ["attention_mixed_prefill.cu"], {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "PARTS": 1, "SIGMOID_WEIGHTS": 1}))
+        built.append(build_library(f"tlie_attn_mixed_decode_k{key_dim}_v{value_dim}_g{kv_heads}", ["attention_mixed_decode.cu"],
+                                   {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "KV_HEADS": kv_heads}))
     for key_dim, value_dim in DEFAULT_DIFF_SETS:
         built.append(build_library(f"tlie_attn_diff_k{key_dim}_v{value_dim}", ["attention_diff_prefill.cu"], {"KEY_DIM": key_dim, "VALUE_DIM": value_dim}))
     return built
@@ -647,19 +653,37 @@ TC_ATTENTION_HEAD_DIMS = (64, 128)
 TC_ATTENTION_MIN_ROWS_PER_TILE = 32
 
 
+def tc_attention_library(sigmoid: bool = False):
+    if sigmoid:
+        return load_library("tlie_attn_prefill_tc_sigmoid", ["attention_prefill_tc.cu"], {"SIGMOID_WEIGHTS": 1})
+    return load_library("tlie_attn_prefill_tc", ["attention_prefill_tc.cu"])
+
+
+def tc_attention_tiles(batch, head_dim: int, page_size: int, lead: int):
+    """The step's row tiles for the tensor-memory kernel, or None if the step or the sizes are not for it (``lead``: the single rows at the
+    step's head, which the tiles leave out)."""
+    tiles = batch.plan("attention_tiles_tc")
+    if not use_tc_attention or tiles is None or head_dim not in TC_ATTENTION_HEAD_DIMS or page_size % 64 != 0:
+        return None
+    return tiles if batch.num_tokens - lead >= TC_ATTENTION_MIN_ROWS_PER_TILE * tiles.shape[0] else None
+
+
 def prefill_attention_tc(qkv, pages, tiles, seq_starts, first_positions, block_table, out, q_heads: int, kv_heads: int, head_dim: int, page_size: int,
-                         window: int, scale: float) -> None:
-    """Flash attention of the work items in ``tiles`` (int32 [n, 4], see ``paired_attention_tiles``) on the 5th-generation tensor cores; head size 64 or 128, bfloat16."""
+                         window: int, scale: float, softcap: float = 0.0, sigmoid: bool = False, shifts=None, gate_offset: int = -1) -> None:
+    """Flash attention of the work items in ``tiles`` (int32 [n, 4], see ``paired_attention_tiles``) on the 5th-generation tensor cores; head size 64 or 128, bfloat16.
+    ``sigmoid``, ``softcap``, ``shifts``: weights without a softmax (see ``ops.mixed_heads_attention``), a build of its own.  ``gate_offset`` >= 0: the column
+    of ``qkv`` where one gate per head starts, whose sigmoid multiplies the head's output."""
     ops = _ops()
     if head_dim not in TC_ATTENTION_HEAD_DIMS or page_size % 64 != 0:
         raise KernelError("the tensor-memory attention takes head sizes 64 and 128 and pages of a multiple of 64 keys", code="invalid_shape")
-    lib = load_library("tlie_attn_prefill_tc", ["attention_prefill_tc.cu"])
+    lib = tc_attention_library(sigmoid)
+    gate = c_void_p(0) if gate_offset < 0 else c_void_p(qkv.data_ptr() + gate_offset * qkv.element_size())
     ops._check(
         lib.tlie_prefill_attention_tc(
             ops._ptr(qkv), c_int(qkv.shape[1]), c_int(qkv.shape[0]), ops._ptr(pages), c_int(pages.shape[0]), ops._i32(tiles, "tiles"), c_int(tiles.shape[0]),
             ops._i32(seq_starts, "seq_starts"), ops._i32(first_positions, "first_positions"), ops._i32(block_table, "block_table"),
             c_int(block_table.shape[1]), ops._ptr(out), c_int(q_heads), c_int(kv_heads), c_int(head_dim), c_int(page_size), c_int(window), c_float(scale),
-            ops._ptr(tcgen05_error_flag(qkv.device)), ops._stream(),
+            c_float(softcap), ops._ptr(shifts), gate, c_int(qkv.shape[1]), ops._ptr(tcgen05_error_flag(qkv.device)), ops._stream(),
         ),
         "prefill_attention_tc",
     )
@@ -683,9 +707,8 @@ def paged_attention_bf16(qkv, pages, positions, token_seq, block_table, out, q_h
         else:
             prefill_attention(qkv, pages, batch.plan("attention_tiles_lead"), batch.seq_starts, batch.first_positions, block_table, out, q_heads, kv_heads,
                               head_dim, page_size, window, scale)
-    tc_tiles = batch.plan("attention_tiles_tc")
-    if (use_tc_attention and tc_tiles is not None and head_dim in TC_ATTENTION_HEAD_DIMS and page_size % 64 == 0 and pages.is_contiguous()
-            and batch.num_tokens - lead >= TC_ATTENTION_MIN_ROWS_PER_TILE * tc_tiles.shape[0]):
+    tc_tiles = tc_attention_tiles(batch, head_dim, page_size, lead)
+    if tc_tiles is not None and pages.is_contiguous():
         prefill_attention_tc(qkv, pages, tc_tiles, batch.seq_starts, batch.first_positions, block_table, out, q_heads, kv_heads, head_dim, page_size, window, scale)
         return True
     tiles = batch.plan("attention_tiles")
