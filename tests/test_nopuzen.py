@@ -533,6 +533,42 @@ def test_latent_attention_kernels(dtype, atol, heads, dim, rot, vdim, rank, q_ra
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("heads,dim,rot,vdim", [(3, 128, 64, 128), (4, 64, 64, 64), (2, 64, 128, 64), (1, 128, 64, 64), (2, 64, 64, 128)])
+def test_latent_attention_over_the_steps_own_rows(heads, dim, rot, vdim):
+    """A step that begins all its requests: expanded keys with a part that the heads share, through the tensor-memory kernel; row tiles that
+    end inside a key tile, requests next to one another in the same matrices, a key that stands out."""
+    from tinyllama_inference_engine_b200.engine.batch import pack_step
+    from tinyllama_inference_engine_b200.ops import fast
+
+    g = torch.Generator().manual_seed(dim + rot + vdim)
+    lens = [300, 129, 64, 2, 200, 127]
+    starts = np.concatenate([[0], np.cumsum(lens)])
+    tokens = int(starts[-1])
+    queries = torch.randn(tokens, heads, dim + rot, generator=g).bfloat16()
+    keys, values, shared = torch.randn(tokens, heads, dim, generator=g), torch.randn(tokens, heads, vdim, generator=g), torch.randn(tokens, rot, generator=g)
+    keys[3] = queries[250, :, :dim].float() * 3.0                          # far back in the first request, and late in another one
+    keys[starts[4] + 150] = queries[starts[4] + 190, :, :dim].float() * 5.0
+    keys, values, shared = keys.bfloat16(), values.bfloat16(), shared.bfloat16()
+    scale = 1.5 * (dim + rot) ** -0.5
+    want = torch.empty(tokens, heads, vdim, dtype=torch.float64)
+    for a, b in zip(starts[:-1], starts[1:]):
+        score = torch.einsum("ihd,jhd->hij", queries[a:b, :, :dim].double(), keys[a:b].double()) + torch.einsum("ihd,jd->hij", queries[a:b, :, dim:].double(), shared[a:b].double())
+        score = (score * scale).masked_fill(torch.arange(b - a)[:, None] < torch.arange(b - a)[None, :], float("-inf"))
+        want[a:b] = torch.einsum("hij,jhd->ihd", torch.softmax(score, dim=-1), values[a:b].double())
+    ctx = pack_step([StepEntry(i, [0] * n, []) for i, n in enumerate(lens)], [0] * len(lens), list(range(len(lens))), [[[0]] * len(lens)], torch.device("cuda:0"))
+    tiles = fast.latent_rows_tiles(ctx)
+    assert tiles is not None and fast.latent_rows_fit(dim, rot, vdim, torch.bfloat16)
+    later = pack_step([StepEntry(0, [0] * 300, [])], [1], [0], [[[0]]], torch.device("cuda:0"))
+    assert fast.latent_rows_tiles(later) is None          # a step behind cached tokens is not for this kernel
+    expanded = torch.cat([keys.reshape(tokens, -1), values.reshape(tokens, -1)], dim=1).cuda()
+    out = torch.full((tokens, heads * vdim), float("nan"), dtype=torch.bfloat16, device="cuda")
+    fast.latent_rows(queries.view(tokens, -1).cuda(), expanded, shared.cuda(), tiles, ctx, out, heads, dim, rot, vdim, scale)
+    assert int(fast.tcgen05_error_flag(out.device)) == 0, "a bounded wait inside the kernel gave up"
+    error = (out.cpu().double() - want.reshape(tokens, -1)).abs().max(dim=1).values
+    assert float(error.max()) <= 3e-2, int(error.argmax())
+
+
+@pytest.mark.gpu
 @pytest.mark.parametrize("tokens", [50, 1300])    # a CTA per token; four tokens per CTA (a step of many rows), the last CTA short of rows
 @pytest.mark.parametrize("experts,groups,keep,top,width", [(8, 4, 2, 3, 64), (6, 1, 1, 2, 44), (9, 3, 2, 4, 40), (4, 4, 3, 2, 32), (64, 8, 4, 8, 128), (5, 5, 1, 1, 24), (12, 2, 1, 6, 48),
                                                            (10, 5, 2, 3, 42), (7, 1, 1, 7, 17)])    # rows that are no multiple of four numbers: the general form
@@ -698,9 +734,14 @@ def test_long_decoding_and_other_page_sizes(cases, dtype):
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dim,kv", [(64, 2), (128, 1)])
-def test_long_portions_beside_decoded_tokens(tmp_path, dim, kv):
-    """Portions of up to 200 rows beside single tokens with pages of 64: the tensor-memory kernel, the kernel of few rows at the step's head and the
-    ones between them, in one model."""
+def test_long_portions_beside_decoded_tokens(tmp_path, dim, kv, monkeypatch):
+    """Portions of up to 200 rows beside single tokens with pages of 64: the tensor-memory kernels (steps that begin their requests attend to their
+    own expanded rows in the latent layer, later portions to the cache), the kernel of few rows at the step's head and the ones between
+    them, in one model."""
+    from tinyllama_inference_engine_b200.ops import fast
+
+    calls, kernel = [], fast.latent_rows
+    monkeypatch.setattr(fast, "latent_rows", lambda *a: (calls.append(a[0].shape[0]), kernel(*a)))
     folder = write_random_model(tmp_path / "m", _config(64, 47, [_attention(4, kv, dim, dim, _dense(64)), _latent(4, 64, 64, 64, 64, 48, _dense(96), scaling=(4.0, 100, 8.0, 1.0))]), 3)
     config, tensors = load_plain(folder)
     requests = trace_tools.make_requests(47, [500, 230, 64, 300], seed=9)
@@ -709,6 +750,7 @@ def test_long_portions_beside_decoded_tokens(tmp_path, dim, kv):
     for steps in (trace_tools.whole(requests), trace_tools.tail_decode(requests, tail=20), trace_tools.portions(requests, sizes=(200, 65, 2, 128)),
                   trace_tools.mixed(requests, seed=2, max_portion=200)[0]):
         trace_tools.run_and_compare(_runner(folder, "bfloat16", max_tokens=2048, page_size=64), steps, full, atol=TOLERANCE["bfloat16"] * scale, over_vocabulary=True)
+    assert 500 in calls and 200 in calls      # whole prompts and first portions
 
 
 @pytest.mark.gpu

@@ -214,7 +214,8 @@ __global__ void __launch_bounds__(256) norm_rotary_store_kernel(T* __restrict__ 
 // Latent attention's norms, rotation and cache write, in up to three parts that a launch may hold or leave out:
 //   ``down_rows``    a row holds, from ``latent_offset``, the down projection [rank | rot].  The first ``rank`` columns are normalised (RMS,
 //                    weight) into the latent; the last ``rot`` are a key part that all heads share and that is rotated.  [latent |
-//                    rotated part] goes into the token's cache row.
+//                    rotated part] goes into the token's cache row, and into ``latent_out`` [T, rank] and ``shared_out`` [T, rot] if these
+//                    are given (the step's own rows as a product's operand).
 //   ``q_latent``     the q_rank columns from ``q_latent_offset`` of the same row, normalised the same way: what the queries are expanded from.
 //   ``query_rows``   ``heads`` queries of [plain | rot]; their rotated rot parts go into ``queries`` [T, heads, rank + rot] behind the ``rank``
 //                    columns that the product with the keys' expansion fills.
@@ -225,8 +226,9 @@ __global__ void __launch_bounds__(256) latent_store_kernel(const T* __restrict__
                                                            const float* __restrict__ inv_freq, int rot_dims, int interleaved, float amplitude,
                                                            const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ block_table,
                                                            int table_stride, T* __restrict__ pages, long long page_stride, int heads, int plain, int rot, int rank,
-                                                           int page_size, int write_cache, const T* __restrict__ query_rows, int query_stride, T* __restrict__ queries,
-                                                           const float* __restrict__ q_latent_weight, int q_latent_offset, int q_rank, T* __restrict__ q_latent) {
+                                                           int page_size, int write_cache, const T* query_rows, int query_stride, T* queries,
+                                                           const float* __restrict__ q_latent_weight, int q_latent_offset, int q_rank, T* __restrict__ q_latent,
+                                                           T* __restrict__ latent_out, T* __restrict__ shared_out) {
   __shared__ float scratch[32];
   extern __shared__ float turn_s[];   // the token's cosines [rot_dims / 2], then its sines
   const int t = blockIdx.x;
@@ -263,13 +265,19 @@ __global__ void __launch_bounds__(256) latent_store_kernel(const T* __restrict__
     if (q_src != nullptr)
       for (int d = threadIdx.x + kHeld * blockDim.x; d < q_rank; d += blockDim.x) q_squares += to_float(q_src[d]) * to_float(q_src[d]);
     const float inv = rsqrtf(block_sum(squares, scratch) / (float)rank + eps);
-    if (cached) {
+    T* mine = latent_out != nullptr ? latent_out + (size_t)t * rank : nullptr;
 #pragma unroll
-      for (int n = 0; n < kHeld; ++n) {
-        const int d = threadIdx.x + n * blockDim.x;
-        if (d < rank) cached[d] = from_float<T>(held[n] * inv * weight[d]);
-      }
-      for (int d = threadIdx.x + kHeld * blockDim.x; d < rank; d += blockDim.x) cached[d] = from_float<T>(to_float(down[d]) * inv * weight[d]);
+    for (int n = 0; n < kHeld; ++n) {
+      const int d = threadIdx.x + n * blockDim.x;
+      if (d >= rank) continue;
+      const T v = from_float<T>(held[n] * inv * weight[d]);
+      if (cached != nullptr) cached[d] = v;
+      if (mine != nullptr) mine[d] = v;
+    }
+    for (int d = threadIdx.x + kHeld * blockDim.x; d < rank; d += blockDim.x) {
+      const T v = from_float<T>(to_float(down[d]) * inv * weight[d]);
+      if (cached != nullptr) cached[d] = v;
+      if (mine != nullptr) mine[d] = v;
     }
     if (q_src != nullptr) {
       T* dst = q_latent + (size_t)t * q_rank;
@@ -285,22 +293,25 @@ __global__ void __launch_bounds__(256) latent_store_kernel(const T* __restrict__
   __syncthreads();   // the cosines and sines are in place
   // the rot parts: a thread per pair of columns; vector ``heads`` is the shared key part
   const int pairs = rot / 2;
-  const int first_vector = query_rows != nullptr ? 0 : heads, end_vector = cached != nullptr ? heads + 1 : heads;
+  const int first_vector = query_rows != nullptr ? 0 : heads, end_vector = (cached != nullptr || shared_out != nullptr) ? heads + 1 : heads;
   const T* query_row = query_rows + (size_t)t * query_stride;
   T* to_row = queries + (size_t)t * heads * (rank + rot);
   for (int i = threadIdx.x; i < (end_vector - first_vector) * pairs; i += blockDim.x) {
     const int vector = first_vector + i / pairs, pair = i % pairs;
     const T* at = vector < heads ? query_row + vector * (plain + rot) + plain : down + rank;
-    T* to = vector < heads ? to_row + vector * (rank + rot) + rank : cached + rank;
+    T* to = vector < heads ? to_row + vector * (rank + rot) + rank : (cached != nullptr ? cached + rank : shared_out + (size_t)t * rot);
+    T* also = (vector == heads && cached != nullptr && shared_out != nullptr) ? shared_out + (size_t)t * rot : nullptr;
     if (pair < half) {
       const int a_at = interleaved ? 2 * pair : pair, b_at = interleaved ? 2 * pair + 1 : pair + half;
       const float cosine = turn_s[pair], sine = turn_s[half + pair];
       const float a = to_float(at[a_at]), b = to_float(at[b_at]);
-      to[a_at] = from_float<T>(a * cosine - b * sine);
-      to[b_at] = from_float<T>(b * cosine + a * sine);
+      const T first = from_float<T>(a * cosine - b * sine), second = from_float<T>(b * cosine + a * sine);
+      to[a_at] = first, to[b_at] = second;
+      if (also != nullptr) also[a_at] = first, also[b_at] = second;
     } else {   // columns that do not rotate
-      to[2 * pair] = at[2 * pair];
-      to[2 * pair + 1] = at[2 * pair + 1];
+      const T first = at[2 * pair], second = at[2 * pair + 1];
+      to[2 * pair] = first, to[2 * pair + 1] = second;
+      if (also != nullptr) also[2 * pair] = first, also[2 * pair + 1] = second;
     }
   }
 }
@@ -829,16 +840,18 @@ TLIE_EXPORT int tlie_norm_rotary_store(int dtype, void* rows, int row_stride, in
 TLIE_EXPORT int tlie_latent_store(int dtype, const void* down_rows, int down_stride, int latent_offset, const float* weight, float eps, const float* inv_freq, int rot_dims,
                                   int interleaved, float amplitude, const int* positions, const int* token_seq, const int* block_table, int table_stride, void* pages,
                                   long long page_stride, int tokens, int heads, int plain, int rot, int rank, int page_size, int write_cache, const void* query_rows,
-                                  int query_stride, void* queries, const float* q_latent_weight, int q_latent_offset, int q_rank, void* q_latent, cudaStream_t stream) {
+                                  int query_stride, void* queries, const float* q_latent_weight, int q_latent_offset, int q_rank, void* q_latent, void* latent_out, void* shared_out,
+                                  cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (rot_dims < 0 || rot_dims > rot || (rot_dims & 1) || (rot & 1) || rot_dims > 8192) return (int)cudaErrorInvalidValue;
   if ((q_latent != nullptr && (down_rows == nullptr || q_latent_weight == nullptr || q_rank <= 0)) || (query_rows != nullptr && queries == nullptr)) return (int)cudaErrorInvalidValue;
+  if ((latent_out != nullptr || shared_out != nullptr) && down_rows == nullptr) return (int)cudaErrorInvalidValue;
   const size_t smem = (size_t)rot_dims * sizeof(float);
 #define TLIE_LATENT(T)                                                                                                                                             \
   latent_store_kernel<T><<<tokens, 256, smem, stream>>>((const T*)down_rows, down_stride, latent_offset, weight, eps, inv_freq, rot_dims, interleaved, amplitude,     \
                                                         positions, token_seq, block_table, table_stride, (T*)pages, page_stride, heads, plain, rot, rank, page_size, \
                                                         write_cache, (const T*)query_rows, query_stride, (T*)queries, q_latent_weight, q_latent_offset, q_rank,     \
-                                                        (T*)q_latent)
+                                                        (T*)q_latent, (T*)latent_out, (T*)shared_out)
   if (dtype == TLIE_F32)
     TLIE_LATENT(float);
   else

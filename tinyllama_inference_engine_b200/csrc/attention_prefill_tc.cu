@@ -32,6 +32,9 @@
 // as it is.  tanh and sigmoid are e^x and a reciprocal each, in 32-bit; one reciprocal serves two scores (1 / a = b / (a b)), so that a
 // score costs three operations of the exponential unit.  In both kinds the output may be multiplied by sigmoid(gate), one number per
 // (row, head), as it is read out.
+// LATENT_ROWS 1 (a build of its own, KEY_DIM / ROT_DIM / VALUE_DIM): the keys and values are rows of the step itself and not of pages, which is all a
+// step sees whose requests all start in it.  A key is a head's own columns beside ROT_DIM columns that every head shares (latent
+// attention with its keys and values expanded): the two come from matrices of their own, a box each.
 // Roles: warp 0 TMA producer, warp 1 issuer of the score products and tensor-memory owner, warp 2 issuer of the P . V products,
 // warp 3 idle, warps 4..7 softmax (128 threads).  The launch gives every thread 128 registers (two CTAs of 256 threads fill the
 // register file); the first four warps hand most of theirs back at once (setmaxnreg) and the softmax warps, whose threads hold a
@@ -54,6 +57,10 @@
 #ifndef SIGMOID_WEIGHTS
 #define SIGMOID_WEIGHTS 0
 #endif
+#ifndef LATENT_ROWS
+#define LATENT_ROWS 0
+#endif
+#include <type_traits>
 
 namespace tlie {
 
@@ -199,34 +206,36 @@ __device__ long long tlie_attn_stamps[24];
 #endif
 
 // A tile of D dims is D / 64 sub-tiles of 64 dims side by side in memory, each [rows][64] in the 128-byte swizzle.
-template <int D>
+template <int KD, int VD>
 struct SmemTC {
-  static constexpr int kStages = D <= 64 ? 3 : 2;
+  static constexpr int kKStages = KD <= 64 ? 3 : 2;
+  static constexpr int kVStages = KD <= 64 ? 3 : (KD <= 128 ? 2 : 1);   // keys of 192: one V buffer, so that two CTAs still share an SM (its load runs under the next softmax)
   // all tiles are 1024-byte aligned (the struct is placed on a 1024-byte boundary)
-  __nv_bfloat16 q[kRowsTC * D];                      // 16 KB per 64 dims
-  __nv_bfloat16 k[kStages][kKeysTC * D];             // 8 KB per 64 dims each
-  __nv_bfloat16 v[kStages][kKeysTC * D];
+  __nv_bfloat16 q[kRowsTC * KD];                      // 16 KB per 64 dims
+  __nv_bfloat16 k[kKStages][kKeysTC * KD];             // 8 KB per 64 dims each
+  __nv_bfloat16 v[kVStages][kKeysTC * VD];
   // k_full / v_full: a tile has landed.  s_done: the scores of the tile in this K stage are computed (the softmax threads wait for it,
   // and the producer before it loads K again).  v_done: the P . V of the tile in this V stage is done (the producer waits for it, and the
-  // softmax threads before they touch O, and the score issuer before it writes the S buffer that holds this tile's P).  p_full: the
-  // softmax threads have written P.
-  uint64_t q_full, q_empty, k_full[kStages], s_done[kStages], v_full[kStages], v_done[kStages], p_full[2], o_full[2], o_read;
+  // softmax threads before they touch O).  p_read: the P . V that read this S buffer's P is done (the score issuer waits for it before it
+  // writes the buffer again).  p_full: the softmax threads have written P.
+  uint64_t q_full, q_empty, k_full[kKStages], s_done[kKStages], v_full[kVStages], v_done[kVStages], p_read[2], p_full[2], o_full[2], o_read;
   uint32_t tmem_base;
   int abort_flag;
 };
 
 // tiles: [n_items][4] = (request, first row, request, first row): one or two 128-row tiles per CTA (second request -1: none)
-template <int kD>
+template <int kD, int kVD>
 __global__ void __launch_bounds__(kThreadsTC, 2)
-    prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
+    prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_v,
+                                const __grid_constant__ CUtensorMap map_rot,
                                 const int* __restrict__ tiles, const int* __restrict__ seq_starts, const int* __restrict__ first_positions,
                                 const int* __restrict__ block_table, int table_stride, __nv_bfloat16* __restrict__ out, int q_heads,
                                 int kv_heads, int page_size, int window, float scale, float softcap, const float* __restrict__ shifts,
                                 const __nv_bfloat16* __restrict__ gate, int gate_stride, int* __restrict__ error_flag) {
   extern __shared__ uint8_t smem_raw[];
-  using Smem = SmemTC<kD>;
-  constexpr int kKvStages = Smem::kStages;
-  constexpr int kSubTiles = kD / kBoxDims;
+  using Smem = SmemTC<kD, kVD>;
+  constexpr int kKStages = Smem::kKStages, kVStages = Smem::kVStages;
+  constexpr int kKSubTiles = kD / kBoxDims, kSubTiles = kVD / kBoxDims;
   Smem& sm = *reinterpret_cast<Smem*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   volatile int* abort_flag = &sm.abort_flag;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -238,19 +247,19 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
   const int* item = tiles + (size_t)blockIdx.y * 4;
   const int head = blockIdx.x;
   const int kvh = head / (q_heads / kv_heads);
-  // S0 [0,64), S1 [64,128), O of the first row tile [128, 128 + D), of the second [128 + D, 128 + 2 D)
-  // (head size 128: both row tiles use [128, 256), one after the other)
+  // S0 [0,64), S1 [64,128), O of the first row tile [128, 128 + D), of the second [128 + D, 128 + 2 D), D the values' width
+  // (values of 128: both row tiles use [128, 256), one after the other)
   constexpr int kTmemCols = 256;
   constexpr int kOutCol0 = 2 * kKeysTC;
-  constexpr bool kCompact = kD > 64;
-  constexpr int kOutStride = kCompact ? 0 : kD;
-  if (kCompact && (smem_u32(smem_raw) & 1023u) != 0) {   // no room was asked for to align by hand: the tiles must lie on 1 KB boundaries as they are
+  constexpr bool kCompact = kVD > 64;
+  constexpr int kOutStride = kCompact ? 0 : kVD;
+  if (kD > 64 && (smem_u32(smem_raw) & 1023u) != 0) {   // no room was asked for to align by hand: the tiles must lie on 1 KB boundaries as they are
     if (threadIdx.x == 0) atomicOr(error_flag, 1);
     return;
   }
 
   struct RowTile {
-    int row0, rows_here, pos0, n_keys, first_kt, num_kt;
+    int row0, rows_here, pos0, n_keys, first_kt, num_kt, key_row0;
     const int* table;
   };
   auto row_tile = [&](int u) {
@@ -259,10 +268,11 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
     t.row0 = item[2 * u + 1];
     if (seq < 0) {
       t.num_kt = 0;
-      t.rows_here = t.pos0 = t.n_keys = t.first_kt = 0;
+      t.rows_here = t.pos0 = t.n_keys = t.first_kt = t.key_row0 = 0;
       t.table = block_table;
       return t;
     }
+    t.key_row0 = seq_starts[seq];
     t.rows_here = min(kRowsTC, seq_starts[seq + 1] - t.row0);
     t.pos0 = first_positions[seq] + (t.row0 - seq_starts[seq]);
     t.n_keys = t.pos0 + t.rows_here;                 // keys the last row of the tile sees
@@ -276,13 +286,16 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
   if (threadIdx.x == 0) {
     mbar_init(&sm.q_full, 1);
     mbar_init(&sm.q_empty, 1);
-    for (int s = 0; s < kKvStages; ++s) {
+    for (int s = 0; s < kKStages; ++s) {
       mbar_init(&sm.k_full[s], 1);
       mbar_init(&sm.s_done[s], 1);
+    }
+    for (int s = 0; s < kVStages; ++s) {
       mbar_init(&sm.v_full[s], 1);
       mbar_init(&sm.v_done[s], 1);
     }
     for (int b = 0; b < 2; ++b) {
+      mbar_init(&sm.p_read[b], 1);
       mbar_init(&sm.p_full[b], 4);   // one arrival per softmax warp
     }
     mbar_init(&sm.o_full[0], 1);   // used once each: all products of a row tile are done
@@ -313,15 +326,23 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
       const RowTile t0 = row_tile(0), t1 = row_tile(1);
       const int n0 = t0.num_kt, G = n0 + t1.num_kt;
       const int tiles_per_page = page_size / kKeysTC;
-      RingPosition<kKvStages> k_ring, v_ring;
+      RingPosition<kKStages> k_ring;
+      RingPosition<kVStages> v_ring;
       TL_BEGIN(blockIdx.x == 0 && blockIdx.y == 0)
       const uint32_t k_addr = smem_u32(sm.k), v_addr = smem_u32(sm.v);
       const uint32_t k_full = smem_u32(sm.k_full), k_empty = smem_u32(sm.s_done), v_full = smem_u32(sm.v_full), v_empty = smem_u32(sm.v_done);
       // One tile of K (plane 0 of the page) or of V (plane 1).  The page's number is asked for before the wait for a free buffer,
       // so that its trip to memory runs under the wait.
-      auto load = [&](int g, int plane, RingPosition<kKvStages>& ring, uint32_t tiles_addr, uint32_t full, uint32_t empty) {
+      auto load = [&](int g, auto is_v, auto& ring, uint32_t tiles_addr, uint32_t full, uint32_t empty) {
+        constexpr bool kIsV = decltype(is_v)::value;
+        constexpr int kWidth = kIsV ? kVD : kD, kBoxes = kIsV ? kSubTiles : kKSubTiles;
         const RowTile& t = g >= n0 ? t1 : t0;
         const int kt = t.first_kt + (g >= n0 ? g - n0 : g);
+        int row;
+#if LATENT_ROWS
+        row = t.key_row0 + kt * kKeysTC;   // the keys are rows of the step
+        TL(0)
+#else
         int page_index = kt, in_page = 0;
         if (tiles_per_page != 1) {
           page_index = kt / tiles_per_page;
@@ -329,26 +350,41 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
         }
         const int page = t.table[page_index];
         TL(0)
+        row = ((page * 2 + (kIsV ? 1 : 0)) * kv_heads + kvh) * page_size + in_page;   // row of the [rows, head size] view of the pool
+#endif
         if (!mbar_wait(empty + 8 * ring.stage, ring.phase ^ 1, abort_flag)) return false;
         TL(1)
-        const int row = ((page * 2 + plane) * kv_heads + kvh) * page_size + in_page;   // row of the [rows, head size] view of the pool
         const uint32_t bar = full + 8 * ring.stage;
-        mbar_expect_tx(bar, kKeysTC * kD * 2);
+        mbar_expect_tx(bar, kKeysTC * kWidth * 2);
 #pragma unroll
-        for (int c = 0; c < kSubTiles; ++c)
-          tma_load_2d(tiles_addr + ring.stage * (kKeysTC * kD * 2) + c * (kKeysTC * kBoxDims * 2), &map_kv, c * kBoxDims, row, bar);
+        for (int c = 0; c < kBoxes; ++c) {
+          const uint32_t dst = tiles_addr + ring.stage * (kKeysTC * kWidth * 2) + c * (kKeysTC * kBoxDims * 2);
+#if LATENT_ROWS
+          constexpr int kPlain = kD - ROT_DIM;   // a head's own key columns; the rotated ones behind them are the same for every head
+          if (kIsV)
+            tma_load_2d(dst, &map_v, head * kVD + c * kBoxDims, row, bar);
+          else if (c * kBoxDims < kPlain)
+            tma_load_2d(dst, &map_kv, head * kPlain + c * kBoxDims, row, bar);
+          else
+            tma_load_2d(dst, &map_rot, c * kBoxDims - kPlain, row, bar);
+#else
+          tma_load_2d(dst, &map_kv, c * kBoxDims, row, bar);
+#endif
+        }
         ring.advance();
         return true;
       };
+      constexpr std::false_type keys{};
+      constexpr std::true_type values{};
       auto load_q = [&](const RowTile& t) {
         mbar_expect_tx(&sm.q_full, kRowsTC * kD * 2);
 #pragma unroll
-        for (int c = 0; c < kSubTiles; ++c) tma_load_2d(sm.q + c * kRowsTC * kBoxDims, &map_q, head * kD + c * kBoxDims, t.row0, &sm.q_full);
+        for (int c = 0; c < kKSubTiles; ++c) tma_load_2d(sm.q + c * kRowsTC * kBoxDims, &map_q, head * kD + c * kBoxDims, t.row0, &sm.q_full);
       };
       bool ok = G > 0;
       if (ok) {
         load_q(n0 > 0 ? t0 : t1);
-        ok = load(0, 0, k_ring, k_addr, k_full, k_empty);
+        ok = load(0, keys, k_ring, k_addr, k_full, k_empty);
       }
       for (int g = 0; g < G && ok; ++g) {   // K of the next tile, then V of this one
         if (g + 1 < G) {
@@ -356,9 +392,9 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
             ok = mbar_wait(&sm.q_empty, 0, abort_flag);
             if (ok) load_q(t1);
           }
-          if (ok) ok = load(g + 1, 0, k_ring, k_addr, k_full, k_empty);
+          if (ok) ok = load(g + 1, keys, k_ring, k_addr, k_full, k_empty);
         }
-        if (ok) ok = load(g, 1, v_ring, v_addr, v_full, v_empty);
+        if (ok) ok = load(g, values, v_ring, v_addr, v_full, v_empty);
         TL_COUNT()
       }
       TL_END(16)
@@ -369,12 +405,12 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
       constexpr uint32_t kTileLow = (kKeysTC * kD * 2) >> 4;               // one K tile further, in descriptor units
       const int n0 = row_tile(0).num_kt, G = n0 + row_tile(1).num_kt;
       const uint32_t q_low = umma_desc_low(smem_u32(sm.q)), k_low = umma_desc_low(smem_u32(sm.k));
-      const uint32_t k_full = smem_u32(sm.k_full), s_done = smem_u32(sm.s_done), v_done = smem_u32(sm.v_done);
-      RingPosition<kKvStages> ring, before, two_before;   // where tile g, g - 1, g - 2 lie in the rings
+      const uint32_t k_full = smem_u32(sm.k_full), s_done = smem_u32(sm.s_done), p_read = smem_u32(sm.p_read);
+      RingPosition<kKStages> ring;
       int q_phase = 0;
       bool ok = true;
       TL_BEGIN(blockIdx.x == 0 && blockIdx.y == 0)
-      for (int g = 0; g < G && ok; ++g, two_before = before, before = ring, ring.advance()) {
+      for (int g = 0; g < G && ok; ++g, ring.advance()) {
         const uint32_t b = g & 1;
         TL(0)
         if (g == 0 || g == n0) {    // a row tile begins: its Q
@@ -385,7 +421,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
         TL(1)
         // This S buffer still holds P of tile g - 2: the product that reads it must be done.  (Its barrier cannot be further on than that:
         // the product that completes it next needs the scores issued here.)
-        if (ok && g > 1) ok = mbar_wait(v_done + 8 * two_before.stage, two_before.phase, abort_flag);
+        if (ok && g > 1) ok = mbar_wait(p_read + 8 * b, ((g >> 1) & 1) ^ 1, abort_flag);
         if (!ok) break;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         TL(2)
@@ -404,15 +440,15 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
     }
   } else if (warp == 2) {
     if (lane == 0) {   // issuer of the P . V products: O += P(g) . V(g) as soon as P(g) is written
-      constexpr uint32_t idesc_pv = instr_desc_b_mn(kRowsTC, kD);          // B = V tile, MN-major
-      constexpr uint32_t kTileLow = (kKeysTC * kD * 2) >> 4;
+      constexpr uint32_t idesc_pv = instr_desc_b_mn(kRowsTC, kVD);         // B = V tile, MN-major
+      constexpr uint32_t kTileLow = (kKeysTC * kVD * 2) >> 4;
       // V is the MN-major operand: its dims run along N.  Beyond 64 dims the next sub-tile of 64 lies kKeysTC * 128 bytes on,
       // which the descriptor's leading-dimension offset says (bits 16-29, in 16-byte units); one sub-tile needs none.
       constexpr uint32_t kVLeading = kSubTiles > 1 ? ((uint32_t)(kKeysTC * kBoxDims * 2) >> 4) : 1u;
       const int n0 = row_tile(0).num_kt, G = n0 + row_tile(1).num_kt;
       const uint32_t v_low = ((smem_u32(sm.v) >> 4) & 0x3FFF) | (kVLeading << 16);
-      const uint32_t v_full = smem_u32(sm.v_full), v_done = smem_u32(sm.v_done), p_full = smem_u32(sm.p_full);
-      RingPosition<kKvStages> ring;
+      const uint32_t v_full = smem_u32(sm.v_full), v_done = smem_u32(sm.v_done), p_full = smem_u32(sm.p_full), p_read = smem_u32(sm.p_read);
+      RingPosition<kVStages> ring;
       bool ok = true;
       TL_BEGIN(false)
       for (int g = 0; g < G && ok; ++g, ring.advance()) {
@@ -431,6 +467,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
         for (int kk = 0; kk < kKeysTC / 16; ++kk)   // 16 keys further: 8 columns of P, 16 rows (2048 bytes) down in a V sub-tile
           umma_bf16_a_tmem(tmem_o, p_tile + kk * 8, v_tile + kk * ((16 * kBoxDims * 2) >> 4), idesc_pv, (!first_of_row_tile || kk > 0) ? 1u : 0u);
         umma_commit(v_done + 8 * ring.stage);
+        umma_commit(p_read + 8 * b);
         if (g + 1 == n0) umma_commit(&sm.o_full[0]);   // a row tile's output is complete when this fires
         if (g + 1 == G && G > n0) umma_commit(&sm.o_full[1]);
       }
@@ -448,8 +485,9 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
     const float sig_base = -(softcap + (shifts != nullptr ? shifts[head] : 0.0f)) * kLog2eTC;
     int g = 0;
     bool ok = true;
-    // Where tile g, g - 1 and g - 2 lie in the K / V rings (stage and phase bit of their barriers).
-    RingPosition<kKvStages> at, before, two_before;
+    // Where tile g lies in the K and V rings and tile g - 1 in the V ring (stage and phase bit of their barriers).
+    RingPosition<kKStages> at;
+    RingPosition<kVStages> v_at, v_before;
     TL_BEGIN(blockIdx.x == 0 && blockIdx.y == 0 && warp == kFirstSoftmaxWarpTC && lane == 0)
     for (int u = 0; u < 2 && ok; ++u) {
       const RowTile t = row_tile(u);
@@ -459,7 +497,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
       const uint32_t tmem_o = tmem + lane_base + kOutCol0 + u * kOutStride;
       // The row's reference maximum (times scale * log2 e) that the exponents are taken against, and the sum against it.
       float reference = -INFINITY, row_sum = 0.0f;
-      for (int j = 0; j < t.num_kt && ok; ++j, ++g, two_before = before, before = at, at.advance()) {
+      for (int j = 0; j < t.num_kt && ok; ++j, ++g, v_before = v_at, v_at.advance(), at.advance()) {
         const int b = g & 1;
         const int key0 = (t.first_kt + j) * kKeysTC;
         TL(0)
@@ -524,7 +562,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
           const bool grown = scaled_max > reference + kLazyRescale;
           if (__any_sync(0xffffffffu, grown)) {
             // The product that last added to O must be done (the one of this tile waits for this P, so its barrier cannot be further on).
-            ok = mbar_wait(&sm.v_done[before.stage], before.phase, abort_flag);
+            ok = mbar_wait(&sm.v_done[v_before.stage], v_before.phase, abort_flag);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
             const float alpha = grown ? exp2f(reference - scaled_max) : 1.0f;
@@ -567,9 +605,9 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
         if (key0 + kKeysTC > t.n_keys) {
           const int first_bad = t.n_keys - key0;
           // V of this tile must have landed first (its scores being there says nothing about it: K and V arrive on their own)
-          ok = mbar_wait(&sm.v_full[at.stage], at.phase, abort_flag);
+          ok = mbar_wait(&sm.v_full[v_at.stage], v_at.phase, abort_flag);
           if (!ok) break;
-          uint8_t* v_tile = reinterpret_cast<uint8_t*>(sm.v[at.stage]);
+          uint8_t* v_tile = reinterpret_cast<uint8_t*>(sm.v[v_at.stage]);
           for (int r = first_bad + (row >> 3); r < kKeysTC; r += kRowsTC / 8)
 #pragma unroll
             for (int c = 0; c < kSubTiles; ++c)
@@ -593,7 +631,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
           float o[64];
           tmem_ld64(tmem_o + half * 64, o);
           if (row < t.rows_here) {
-            __nv_bfloat16* dst = out + ((size_t)(t.row0 + row) * q_heads + head) * kD + half * 64;
+            __nv_bfloat16* dst = out + ((size_t)(t.row0 + row) * q_heads + head) * kVD + half * 64;
 #pragma unroll
             for (int c = 0; c < 8; ++c)
               *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(pack_bf16(o[c * 8] * inv, o[c * 8 + 1] * inv), pack_bf16(o[c * 8 + 2] * inv, o[c * 8 + 3] * inv),
@@ -643,31 +681,50 @@ TLIE_EXPORT int tlie_prefill_attention_tc_tile_rows() { return kRowsTC; }
 TLIE_EXPORT int tlie_prefill_attention_tc_timeline(long long* host) { return (int)cudaMemcpyFromSymbol(host, tlie_attn_stamps, sizeof(long long) * 24); }
 #endif
 
-template <int kD>
-static int launch_attention_tc(const void* q, int q_row_stride, int tokens, const void* pages, int num_pages, const int* tiles, int n_tiles,
+template <int kD, int kVD>
+static int launch_attention_tc(const CUtensorMap& map_q, const CUtensorMap& map_kv, const CUtensorMap& map_v, const CUtensorMap& map_rot, const int* tiles, int n_tiles,
                                const int* seq_starts, const int* first_positions, const int* block_table, int table_stride, void* out, int q_heads,
                                int kv_heads, int page_size, int window, float scale, float softcap, const float* shifts, const void* gate, int gate_stride,
                                int* error_flag, cudaStream_t stream) {
-  CUtensorMap map_q, map_kv;
-  if (!make_map_2d(&map_q, q, tokens, (long long)q_heads * kD, q_row_stride, kRowsTC)) return (int)cudaErrorInvalidValue;
-  if (!make_map_2d(&map_kv, pages, (long long)num_pages * 2 * kv_heads * page_size, kD, kD, kKeysTC)) return (int)cudaErrorInvalidValue;
-  // head size 128: exactly the structure, no room to align it by hand (the kernel checks that it need not): 1 KB more and two CTAs no longer share an SM
+  // keys of 128 and more: exactly the structure, no room to align it by hand (the kernel checks that it need not): 1 KB more and two CTAs no longer share an SM
 #ifdef TLIE_ATTN_ONE_PER_SM   // for measurements: so much shared memory that a CTA has its SM to itself
   const int smem = 200 * 1024;
 #else
-  const int smem = (int)sizeof(SmemTC<kD>) + (kD <= 64 ? 1024 : 0);
+  const int smem = (int)sizeof(SmemTC<kD, kVD>) + (kD <= 64 ? 1024 : 0);
 #endif
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<kD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<kD, kVD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   dim3 grid(q_heads, n_tiles);
-  return (int)launch_pdl(prefill_attention_tc_kernel<kD>, grid, dim3(kThreadsTC), (size_t)smem, stream, map_q, map_kv, tiles, seq_starts, first_positions,
-                         block_table, table_stride, (__nv_bfloat16*)out, q_heads, kv_heads, page_size, window, scale, softcap, shifts, (const __nv_bfloat16*)gate, gate_stride, error_flag);
+  return (int)launch_pdl(prefill_attention_tc_kernel<kD, kVD>, grid, dim3(kThreadsTC), (size_t)smem, stream, map_q, map_kv, map_v, map_rot, tiles, seq_starts, first_positions,
+                         block_table, table_stride, (__nv_bfloat16*)out, q_heads, kv_heads, page_size, window, scale, softcap, shifts, (const __nv_bfloat16*)gate, gate_stride,
+                         error_flag);
 }
 
+#if LATENT_ROWS
+// Attention of a step's rows among themselves with keys of [a head's own columns | ROT_DIM columns that all heads share] and values of VALUE_DIM.  q: rows of
+// heads x KEY_DIM.  expanded: rows of [heads x (KEY_DIM - ROT_DIM) keys | heads x VALUE_DIM values]; shared: rows of ROT_DIM.  Row r of all three is token r of the
+// step; a request's tokens attend to its own earlier tokens in the step.
+TLIE_EXPORT int tlie_prefill_attention_rows(const void* q, const void* expanded, const void* shared, int tokens, const int* tiles, int n_tiles, const int* seq_starts,
+                                            const int* first_positions, void* out, int heads, float scale, int* error_flag, cudaStream_t stream) {
+  if (n_tiles <= 0) return 0;
+  constexpr int kPlain = KEY_DIM - ROT_DIM;
+  static_assert(KEY_DIM % kBoxDims == 0 && ROT_DIM % kBoxDims == 0 && VALUE_DIM % kBoxDims == 0 && kPlain > 0 && VALUE_DIM <= 128, "widths are multiples of a box");
+  if (heads <= 0 || n_tiles > 65535 || error_flag == nullptr) return (int)cudaErrorInvalidValue;
+  CUtensorMap map_q, map_k, map_v, map_rot;
+  const long long stride = (long long)heads * (kPlain + VALUE_DIM);
+  const __nv_bfloat16* values = (const __nv_bfloat16*)expanded + (long long)heads * kPlain;
+  if (!make_map_2d(&map_q, q, tokens, (long long)heads * KEY_DIM, (long long)heads * KEY_DIM, kRowsTC) ||
+      !make_map_2d(&map_k, expanded, tokens, (long long)heads * kPlain, stride, kKeysTC) || !make_map_2d(&map_v, values, tokens, (long long)heads * VALUE_DIM, stride, kKeysTC) ||
+      !make_map_2d(&map_rot, shared, tokens, ROT_DIM, ROT_DIM, kKeysTC))
+    return (int)cudaErrorInvalidValue;
+  return launch_attention_tc<KEY_DIM, VALUE_DIM>(map_q, map_k, map_v, map_rot, tiles, n_tiles, seq_starts, first_positions, nullptr, 0, out, heads, heads, kKeysTC, 0, scale, 0.0f,
+                                                 nullptr, nullptr, 0, error_flag, stream);
+}
+#else
 // q: the step's rows [tokens, q_row_stride] starting with the rotated q heads (head size 64 or 128); pages: one layer's pool
 // [num_pages, 2, kv_heads, page_size, head size]; tiles: int32 [n_tiles, 4] work items of one or two 128-row tiles (request, first
 // row, request or -1, first row); error_flag: device int, zero.  softcap (0: none) and shifts (32-bit [q_heads] or null): SIGMOID_WEIGHTS only.
@@ -681,9 +738,11 @@ TLIE_EXPORT int tlie_prefill_attention_tc(const void* q, int q_row_stride, int t
   if (kv_heads <= 0 || q_heads % kv_heads != 0 || n_tiles > 65535 || page_size % kKeysTC != 0 || q_row_stride % 8 != 0 || error_flag == nullptr ||
       (head_dim != 64 && head_dim != 128))
     return (int)cudaErrorInvalidValue;
-  if (head_dim == 64)
-    return launch_attention_tc<64>(q, q_row_stride, tokens, pages, num_pages, tiles, n_tiles, seq_starts, first_positions, block_table, table_stride, out,
-                                   q_heads, kv_heads, page_size, window, scale, softcap, shifts, gate, gate_stride, error_flag, stream);
-  return launch_attention_tc<128>(q, q_row_stride, tokens, pages, num_pages, tiles, n_tiles, seq_starts, first_positions, block_table, table_stride, out,
-                                  q_heads, kv_heads, page_size, window, scale, softcap, shifts, gate, gate_stride, error_flag, stream);
+  CUtensorMap map_q, map_kv;
+  if (!make_map_2d(&map_q, q, tokens, (long long)q_heads * head_dim, q_row_stride, kRowsTC)) return (int)cudaErrorInvalidValue;
+  if (!make_map_2d(&map_kv, pages, (long long)num_pages * 2 * kv_heads * page_size, head_dim, head_dim, kKeysTC)) return (int)cudaErrorInvalidValue;
+  auto launch = head_dim == 64 ? launch_attention_tc<64, 64> : launch_attention_tc<128, 128>;
+  return launch(map_q, map_kv, map_kv, map_kv, tiles, n_tiles, seq_starts, first_positions, block_table, table_stride, out, q_heads, kv_heads, page_size, window, scale, softcap,
+                shifts, gate, gate_stride, error_flag, stream);
 }
+#endif

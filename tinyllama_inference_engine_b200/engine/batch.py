@@ -78,6 +78,7 @@ class StepContext:
     max_q_len: int
     max_seq_len: int
     wants_every_row_in_order: bool = False      # want_rows is 0, 1, ..., num_tokens - 1
+    starts_requests: bool = False               # every entry begins its request: no row sees a token of an earlier step
     plans: dict = field(default_factory=dict)   # name -> int32 [n, columns] work list of a registered step plan
 
     @property
@@ -150,15 +151,16 @@ def pack_step(entries: list[StepEntry], first_positions: list[int], slots: list[
         block_tables=tables, request_ids=[e.request_id for e in entries], host_q_lens=layout["q_lens"],
         host_first_positions=list(first_positions), host_state_slots=list(slots),
         max_q_len=max(layout["q_lens"]), max_seq_len=max(layout["seq_lens"]), wants_every_row_in_order=len(want_rows) == num_tokens and want_rows == list(range(num_tokens)),
-        plans={plan.name: views[8 + i].view(-1, plan.columns) for i, plan in enumerate(plans)},
+        starts_requests=not any(first_positions), plans={plan.name: views[8 + i].view(-1, plan.columns) for i, plan in enumerate(plans)},
     )
 
 
-def step_shape(entries: list[StepEntry]) -> tuple:
-    """What of a step decides its kernels' launch shapes and its buffer's layout: every entry's number of tokens and of wanted
-    places (and whether all rows are wanted in order).  Everything else about it is data the kernels read on the device."""
+def step_shape(entries: list[StepEntry], first_positions: list[int]) -> tuple:
+    """What of a step decides its kernels, their launch shapes and its buffer's layout: every entry's number of tokens and of wanted
+    places, whether all rows are wanted in order, and whether every entry begins its request.  Everything else about it is data the
+    kernels read on the device."""
     in_order = all(entry.want == list(range(len(entry.tokens))) for entry in entries)
-    return tuple((len(entry.tokens), len(entry.want)) for entry in entries) + (in_order,)
+    return tuple((len(entry.tokens), len(entry.want)) for entry in entries) + (in_order, not any(first_positions))
 
 
 def decode_context(buffer: torch.Tensor, count: int, table_width: int, groups: int, max_positions: int, request_ids: list) -> tuple["StepContext", list]:

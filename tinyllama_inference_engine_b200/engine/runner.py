@@ -147,7 +147,7 @@ class ModelRunner:
             slots.append(self.cache.records[entry.request_id].slot)
         ids = [e.request_id for e in entries]
         table_rows = [self.cache.block_table_rows(group, ids) for group in self.cache.page_groups]
-        graphed = self._graphed_step(entries) if timings is None and trace is None else None
+        graphed = self._graphed_step(entries, firsts) if timings is None and trace is None else None
         if graphed is not None:
             logits = graphed.run(self, entries, firsts, slots, table_rows)
         else:
@@ -162,7 +162,7 @@ class ModelRunner:
         clock.finish(timings, ("transfer", "compute"))
         return logits
 
-    def _graphed_step(self, entries: list[StepEntry]):
+    def _graphed_step(self, entries: list[StepEntry], firsts: list[int]):
         """The captured form of steps of this shape, once the shape has come up often enough to be worth capturing (else None).
 
         A prompt portion of a few hundred tokens is some 160 kernels of a few microseconds each: launched one by one the host
@@ -171,7 +171,7 @@ class ModelRunner:
         fixed address that every replay refreshes with one copy."""
         if not (self.engine_config.use_cuda_graphs and self.device.type == "cuda" and self.model.capturable):
             return None   # some part reads the step on the host: kernel by kernel
-        shape = step_shape(entries)
+        shape = step_shape(entries, firsts)
         slot = self._step_graphs.get(shape)
         if slot is None:
             if len(self._step_graphs) >= MAX_STEP_GRAPHS:

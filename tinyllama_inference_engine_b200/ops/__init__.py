@@ -315,12 +315,19 @@ def head_linear(x, weight, out, gate=None) -> None:
     if x.dtype == torch.bfloat16 and rows >= HEAD_LINEAR_LIBRARY_ROWS:
         torch.bmm(x.transpose(0, 1), weight.transpose(1, 2), out=out.transpose(0, 1))
         if gate is not None:
-            _check(core().tlie_sigmoid_gate(_code(out), c_void_p(out.data_ptr()), c_longlong(out.stride(0)), gate_ptr, c_longlong(gate_stride), c_int(rows),
-                                            c_int(heads * n_out), _stream()), "sigmoid_gate")
+            sigmoid_gate(out.as_strided((rows, heads * n_out), (out.stride(0), 1)), gate)
         return
     _check(core().tlie_head_linear(_code(x), c_void_p(x.data_ptr()), c_longlong(x.stride(0)), c_longlong(x.stride(1)), _ptr(weight), c_void_p(out.data_ptr()),
                                    c_longlong(out.stride(0)), c_longlong(out.stride(1)), c_int(rows), c_int(heads), c_int(n_out), c_int(k_in), gate_ptr,
                                    c_longlong(gate_stride), _stream()), "head_linear")
+
+
+def sigmoid_gate(x, gate) -> None:
+    """x[t, i] *= sigmoid(gate[t, i]) in place, 32-bit inside; both may be runs of columns of wider rows."""
+    if gate.shape != x.shape or gate.dtype != x.dtype or gate.stride(1) != 1 or x.stride(1) != 1 or not x.is_cuda:
+        raise KernelError("sigmoid_gate: x and the gate share a shape and a dtype, on a CUDA device", code="invalid_shape")
+    _check(core().tlie_sigmoid_gate(_code(x), c_void_p(x.data_ptr()), c_longlong(x.stride(0)), c_void_p(gate.data_ptr()), c_longlong(gate.stride(0)), c_int(x.shape[0]),
+                                    c_int(x.shape[1]), _stream()), "sigmoid_gate")
 
 
 def linear(x, weight, out) -> None:
@@ -820,17 +827,29 @@ def _latent_plane(cache, width: int):
 
 
 def latent_store(rows, latent_offset: int, weight, eps: float, inv_freq, rot_dims: int, positions, token_seq, cache, queries, heads: int, plain: int, rot: int, rank: int,
-                 interleaved: bool = True, amplitude: float = 1.0, query_rows=None, q_latent=None) -> None:
+                 interleaved: bool = True, amplitude: float = 1.0, query_rows=None, q_latent=None, own_rows=None, in_place: bool = False) -> None:
     """Latent attention's norms, rotation and cache write: ``rows[:, latent_offset:]`` = [rank | rot] becomes [rms-normed latent (32-bit ``weight``) |
     rotated shared key part] in the token's cache row (``rows`` None: this part is left out); the ``rot`` columns behind the ``plain`` ones of
     every query head of ``query_rows`` [T, heads * (plain + rot)] (None: of the first columns of ``rows``) are rotated into ``queries``
     [T, heads * (rank + rot)], behind each head's first ``rank`` columns, which are left alone (``queries`` None: this part is left out).
     The first ``rot_dims`` columns turn by position * inv_freq[i], cosines and sines times ``amplitude``: columns (2i, 2i + 1) together if
     ``interleaved``, else column i with column i + rot_dims / 2.  ``q_latent`` = (offset, 32-bit weight, out): the queries' own latent, the columns of
-    ``rows`` from ``offset`` on, rms-normed into ``out`` [T, its width]."""
+    ``rows`` from ``offset`` on, rms-normed into ``out`` [T, its width].  ``own_rows`` = ([T, rank], [T, rot]): what goes into the cache rows is written
+    there as well.  ``in_place``: the queries' rot parts turn where they are, in ``query_rows`` (``queries`` None)."""
     pages = _latent_plane(cache, rank + rot)
     some = rows if rows is not None else query_rows
     tokens = some.shape[0]
+    own_latent, own_shared = own_rows if own_rows is not None else (None, None)
+    if own_rows is not None and (rows is None or own_latent.shape != (tokens, rank) or own_shared.shape != (tokens, rot) or own_latent.dtype != some.dtype or own_shared.dtype != some.dtype):
+        raise KernelError("latent_store: the step's own rows are [T, rank] and [T, rot] of the rows' dtype", code="invalid_shape")
+    if in_place:
+        if queries is not None or query_rows is None or query_rows.shape != (tokens, heads * (plain + rot)) or rows is not None:
+            raise KernelError("latent_store: rotation in place takes query_rows [T, heads * (plain + rot)] alone", code="invalid_shape")
+        _check(mixed_attention().tlie_latent_store(_code(some), _ptr(None), c_int(0), c_int(0), _ptr(None), c_float(eps), _ptr(inv_freq), c_int(rot_dims), c_int(1 if interleaved else 0),
+                                                   c_float(amplitude), _i32(positions, "positions"), _i32(token_seq, "token_seq"), _ptr(None), c_int(0), _ptr(None), c_longlong(0),
+                                                   c_int(tokens), c_int(heads), c_int(plain), c_int(rot), c_int(plain), c_int(cache.page_size), c_int(0), _ptr(query_rows),
+                                                   c_int(query_rows.shape[1]), _ptr(query_rows), _ptr(None), c_int(0), c_int(0), _ptr(None), _ptr(None), _ptr(None), _stream()), "latent_store")
+        return
     if queries is not None and (queries.shape != (tokens, heads * (rank + rot)) or queries.dtype != some.dtype):
         raise KernelError("latent_store: queries must be [rows, heads * (rank + rot)] of the rows' dtype", code="invalid_shape")
     if pages.dtype != some.dtype or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dims // 2 or weight.dtype != torch.float32 or weight.numel() != rank:
@@ -849,7 +868,7 @@ def latent_store(rows, latent_offset: int, weight, eps: float, inv_freq, rot_dim
                                                c_longlong(cache.page_size * (rank + rot)), c_int(tokens), c_int(heads), c_int(plain), c_int(rot), c_int(rank),
                                                c_int(cache.page_size), c_int(1 if cache.writes else 0), _ptr(source if queries is not None else None),
                                                c_int(0 if queries is None else source.shape[1]), _ptr(queries), _ptr(q_weight), c_int(q_offset),
-                                               c_int(0 if q_out is None else q_out.shape[1]), _ptr(q_out), _stream()), "latent_store")
+                                               c_int(0 if q_out is None else q_out.shape[1]), _ptr(q_out), _ptr(own_latent), _ptr(own_shared), _stream()), "latent_store")
 
 
 def store_kv_planes(rows, k_offset: int, v_offset: int, positions, token_seq, cache, kv_heads: int, key_dim: int, value_dim: int) -> None:

@@ -46,6 +46,7 @@ def build_all() -> list:
         built.append(build_library(f"tlie_attn_mixed_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "PARTS": parts}))
         built.append(build_library(f"tlie_attn_mixed_decode_k{key_dim}_v{value_dim}_g{parts}", ["attention_mixed_decode.cu"],
                                    {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "KV_HEADS": parts}))
+    built.append(build_library("tlie_attn_latent_rows_k192_r64_v128", ["attention_prefill_tc.cu"], {"LATENT_ROWS": 1, "KEY_DIM": 192, "ROT_DIM": 64, "VALUE_DIM": 128}))
     built.append(build_library("tlie_attn_latent_k576_v512", ["attention_latent_prefill.cu"], {"KEY_DIM": 576, "VALUE_DIM": 512}))   # other widths on first use
     for key_dim, value_dim, kv_heads in DEFAULT_SIGMOID_SETS:
         built.append(build_library(f"tlie_attn_sigmoid_k{key_dim}_v{value_dim}_p1", ["attention_mixed_prefill.cu"], {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "PARTS": 1, "SIGMOID_WEIGHTS": 1}))
@@ -835,6 +836,43 @@ def latent_prefill(queries, batch, block_table, pages_ptr, page_stride: int, sin
     if splits > 1:
         ops._check(ops.mixed_attention().tlie_merge_parts(ops._ptr(partial), ops._ptr(out), c_int(tokens), c_int(heads), c_int(value_dim), c_int(splits), ops._ptr(sinks),
                                                           ops._stream()), "merge_parts")
+
+
+# --- latent attention with its keys and values expanded, for steps that begin their requests -------------------------------------------
+use_latent_rows = True
+
+
+def latent_rows_library(key_dim: int, rot: int, value_dim: int):
+    """The kernel set of one (key width, shared rotated width, value width): compiled when a model of these sizes first runs a whole prompt."""
+    return load_library(f"tlie_attn_latent_rows_k{key_dim}_r{rot}_v{value_dim}", ["attention_prefill_tc.cu"],
+                        {"LATENT_ROWS": 1, "KEY_DIM": key_dim, "ROT_DIM": rot, "VALUE_DIM": value_dim})
+
+
+def latent_rows_fit(plain: int, rot: int, value_dim: int, dtype: torch.dtype) -> bool:
+    """Whether the sizes are ones the tensor-memory kernel takes: boxes of 64 columns, keys of up to 192, values of up to 128."""
+    return use_latent_rows and dtype == torch.bfloat16 and plain % 64 == 0 and rot % 64 == 0 and 0 < rot and plain + rot <= 192 and value_dim in (64, 128)
+
+
+def latent_rows_tiles(batch):
+    """The row tiles of a step whose every entry begins its request (no row sees a cached key, so that the step's own rows are all the
+    keys there are), or None for other steps."""
+    if not getattr(batch, "starts_requests", False) or leading_single_rows(batch.host_q_lens):
+        return None
+    tiles = batch.plan("attention_tiles_tc")
+    return tiles if tiles is not None and batch.num_tokens >= TC_ATTENTION_MIN_ROWS_PER_TILE * tiles.shape[0] else None
+
+
+def latent_rows(queries, expanded, shared, tiles, batch, out, heads: int, plain: int, rot: int, value_dim: int, scale: float) -> None:
+    """Causal attention of every request's rows among themselves (csrc/attention_prefill_tc.cu, LATENT_ROWS): ``queries`` [T, heads (plain + rot)], ``expanded``
+    [T, heads plain keys | heads value_dim values], ``shared`` [T, rot] (the key columns all heads share), ``out`` [T, heads value_dim]; bfloat16."""
+    ops = _ops()
+    tokens = queries.shape[0]
+    if (queries.shape[1] != heads * (plain + rot) or expanded.shape != (tokens, heads * (plain + value_dim)) or shared.shape != (tokens, rot) or out.shape != (tokens, heads * value_dim)
+            or not latent_rows_fit(plain, rot, value_dim, queries.dtype)):
+        raise KernelError("latent_rows: queries [T, heads (plain + rot)], expanded [T, heads (plain + value_dim)], shared [T, rot], out [T, heads value_dim], bfloat16", code="invalid_shape")
+    ops._check(latent_rows_library(plain + rot, rot, value_dim).tlie_prefill_attention_rows(
+        ops._ptr(queries), ops._ptr(expanded), ops._ptr(shared), c_int(tokens), ops._i32(tiles, "tiles"), c_int(tiles.shape[0]), ops._i32(batch.seq_starts, "seq_starts"),
+        ops._i32(batch.first_positions, "first_positions"), ops._ptr(out), c_int(heads), c_float(scale), ops._ptr(tcgen05_error_flag(queries.device)), ops._stream()), "latent_rows")
 
 
 # --- attention with mixed heads, steps of few rows on the tensor cores ------------------------------------------------------------------

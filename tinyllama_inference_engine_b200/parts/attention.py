@@ -378,7 +378,9 @@ class LatentAttention(Mixer):
     Only [c | rotated part] is cached (one plane, one head, rank + rot wide).  The products with W_uk and W_uv are moved across the
     attention: q~_h = W_uk,h^T q_plain,h, so that the score is [q~_h | q_rot,h] . [c_j | rot_j] and head h's weighted sum of latents,
     sum_j p_j c_j, is multiplied by W_uv,h afterwards.  All heads then read the same cached rows: attention with one key/value
-    head whose values are the first ``rank`` columns of its keys.
+    head whose values are the first ``rank`` columns of its keys.  A step whose every request begins in it sees no cached key: there, with
+    a query latent and at widths the tensor-memory kernel takes (``ops.fast.latent_rows_fit``), the step's own keys and values are expanded by one
+    product and attended to as they are, a third of the multiplications.
 
     params: ``hidden_size``, ``num_heads``, ``plain_dim``, ``rot_dim``, ``value_dim``, ``rank``, ``scale``, ``eps``, ``rot_dims``, ``rot_base``,
     ``sink``, optional ``query_rank`` (0), ``output_gate`` (False), ``rot_layout`` ("interleaved": columns (2i, 2i + 1) turn together; "halves": column i with
@@ -448,6 +450,9 @@ class LatentAttention(Mixer):
         self.w_uk_t = weights.get(f"{prefix}.uk", dtype).view(self.heads, self.plain, self.rank).transpose(1, 2).contiguous()
         self.w_uv = weights.get(f"{prefix}.uv", dtype).view(self.heads, self.vdim, self.rank).contiguous()
         self.sinks = weights.get(f"{prefix}.sink", torch.float32).contiguous() if spec.get("sink") else None
+        self.w_expand = None   # [heads * plain keys | heads * vdim values] of a latent, for steps that begin their requests
+        if self.query_rank and self.sinks is None and self.w_in.is_cuda and ops.fast.latent_rows_fit(self.plain, self.rot, self.vdim, dtype):
+            self.w_expand = torch.cat([weights.get(f"{prefix}.uk", dtype), weights.get(f"{prefix}.uv", dtype)], dim=0).contiguous()
         self.w_o = weights.get(f"{prefix}.o", dtype).contiguous()
         frequencies, self.amplitude = rotation_frequencies(self.rot_dims, spec["rot_base"], spec.get("rot_scaling"))
         self.inv_freq = torch.from_numpy(frequencies).to(runtime.device)
@@ -463,6 +468,39 @@ class LatentAttention(Mixer):
         else:
             ops.linear(x, self.w_in, rows)
         width = self.rank + self.rot
+        mixed = ws.get("attention", tokens, self.heads * self.vdim, dtype)
+        gate = rows[:, self.gate_offset : self.gate_offset + self.heads * self.vdim] if self.gate_offset >= 0 else None
+        tiles = ops.fast.latent_rows_tiles(ctx) if self.w_expand is not None else None
+        if tiles is not None:
+            self._attend_to_own_rows(rows, tiles, ctx, cache, mixed, gate)
+        else:
+            self._attend_to_cache(rows, width, ctx, cache, mixed, gate)
+        if accumulate_into is not None:
+            ops.linear_accumulate(mixed, self.w_o, accumulate_into, prepare)
+            return None
+        out = ws.get("mixer_out", tokens, self.hidden, dtype)
+        ops.linear(mixed, self.w_o, out)
+        return out
+
+    def _attend_to_own_rows(self, rows, tiles, ctx, cache: LayerCache, mixed, gate) -> None:
+        """The step's keys and values expanded; nothing is read from the cache (its rows are written)."""
+        ws, dtype, tokens = self.runtime.workspace, self.runtime.dtype, rows.shape[0]
+        rotation = (self.inv_freq, self.rot_dims, ctx.positions, ctx.token_seq, cache)
+        sizes = (self.heads, self.plain, self.rot, self.rank, self.interleaved, self.amplitude)
+        latent, shared = ws.get("latent_own", tokens, self.rank, dtype), ws.get("latent_shared_key", tokens, self.rot, dtype)
+        query_latent, query_rows = ws.get("query_latent", tokens, self.query_rank, dtype), ws.get("latent_query_rows", tokens, self.query_width, dtype)
+        ops.latent_store(rows, self.latent_offset, self.latent_weight, self.eps, *rotation, None, *sizes, q_latent=(0, self.query_weight, query_latent), own_rows=(latent, shared))
+        ops.linear(query_latent, self.w_uq, query_rows)
+        ops.latent_store(None, 0, self.latent_weight, self.eps, *rotation, None, *sizes, query_rows=query_rows, in_place=True)
+        expanded = ws.get("latent_expanded", tokens, self.w_expand.shape[0], dtype)
+        ops.linear(latent, self.w_expand, expanded)
+        ops.fast.latent_rows(query_rows, expanded, shared, tiles, ctx, mixed, self.heads, self.plain, self.rot, self.vdim, self.scale)
+        if gate is not None:
+            ops.sigmoid_gate(mixed, gate)
+
+    def _attend_to_cache(self, rows, width: int, ctx, cache: LayerCache, mixed, gate) -> None:
+        """The products with the expansions moved across the attention over the cached rows."""
+        ws, dtype, tokens = self.runtime.workspace, self.runtime.dtype, rows.shape[0]
         flat_queries = ws.get("latent_queries", tokens, self.heads * width, dtype)
         rotation = (self.inv_freq, self.rot_dims, ctx.positions, ctx.token_seq, cache)
         sizes = (self.heads, self.plain, self.rot, self.rank, self.interleaved, self.amplitude)
@@ -481,15 +519,7 @@ class LatentAttention(Mixer):
         summed = ws.get("latent_sums", tokens, self.heads * self.rank, dtype)
         ops.mixed_heads_attention(flat_queries, -1, ctx.positions, ctx.token_seq, cache, None, None, summed, self.heads, 1, width,
                                   self.rank, 0, self.scale, batch=ctx, sinks=self.sinks, values_in_keys=True)
-        mixed = ws.get("attention", tokens, self.heads * self.vdim, dtype)
-        gate = rows[:, self.gate_offset : self.gate_offset + self.heads * self.vdim] if self.gate_offset >= 0 else None
         ops.head_linear(summed.view(tokens, self.heads, self.rank), self.w_uv, mixed.view(tokens, self.heads, self.vdim), gate)
-        if accumulate_into is not None:
-            ops.linear_accumulate(mixed, self.w_o, accumulate_into, prepare)
-            return None
-        out = ws.get("mixer_out", tokens, self.hidden, dtype)
-        ops.linear(mixed, self.w_o, out)
-        return out
 
 
 class DifferentialAttention(Mixer):
