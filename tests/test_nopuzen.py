@@ -478,9 +478,10 @@ def test_sigmoid_attention_in_tensor_memory(dim, heads, kv, page_size, softcap, 
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype,atol", [(torch.float32, 2e-5), (torch.bfloat16, 3e-2)])
-@pytest.mark.parametrize("heads,dim,rot,vdim,rank,q_rank,interleaved", [(4, 16, 16, 32, 32, 24, False), (1, 20, 6, 10, 96, 40, False), (3, 10, 2, 7, 20, 13, True), (16, 32, 64, 32, 128, 48, False)])
-@pytest.mark.parametrize("long_tail", [False, True])
-def test_latent_attention_kernels(dtype, atol, heads, dim, rot, vdim, rank, q_rank, interleaved, long_tail):
+@pytest.mark.parametrize("heads,dim,rot,vdim,rank,q_rank,interleaved", [(4, 16, 16, 32, 32, 24, False), (1, 20, 6, 10, 96, 40, False), (3, 10, 2, 7, 20, 13, True), (16, 32, 64, 32, 128, 48, False),
+                                                                            (20, 16, 16, 16, 64, 32, True), (2, 64, 64, 32, 512, 40, False)])
+@pytest.mark.parametrize("long_tail,singles", [(False, False), (True, False), (True, True)])
+def test_latent_attention_kernels(dtype, atol, heads, dim, rot, vdim, rank, q_rank, interleaved, long_tail, singles):
     """The norms of both latents, the rotations with an amplitude, the cache write, the products moved across the attention and the gate against
     expanded keys and values, in three steps through a scrambled block table."""
     from tinyllama_inference_engine_b200 import ops
@@ -514,7 +515,10 @@ def test_latent_attention_kernels(dtype, atol, heads, dim, rot, vdim, rank, q_ra
     inv_freq = torch.tensor(freq, dtype=torch.float32).cuda()
     uk_t = w_uk.view(heads, dim, rank).transpose(1, 2).contiguous().cuda()
     sizes = (heads, dim, rot, rank, interleaved, amplitude)
-    for pieces in _pieces(lens, firsts):
+    steps = list(_pieces(lens, firsts))
+    if singles:     # the last rows one by one: steps of single tokens, of fewer and fewer requests
+        steps = steps[:2] + [[(r, a + i, 1) for r, a, n in steps[2] if i < n] for i in range(max(n for _, _, n in steps[2]))]
+    for pieces in steps:
         step_rows, positions, token_seq, sub, batch, index = _step_of(rows, cache, pieces)
         tokens = len(index)
         q_latent, queries = torch.zeros(tokens, q_rank, dtype=dtype, device="cuda"), torch.zeros(tokens, heads * (rank + rot), dtype=dtype, device="cuda")

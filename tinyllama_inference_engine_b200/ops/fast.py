@@ -817,10 +817,24 @@ def latent_prefill_takes(batch, queries, key_dim: int, value_dim: int) -> bool:
 def latent_prefill(queries, batch, block_table, pages_ptr, page_stride: int, sinks, out, heads: int, key_dim: int, value_dim: int, page_size: int, scale: float) -> None:
     """Causal attention of ``heads`` query heads per token over one cached row per token whose first ``value_dim`` columns are the
     values (csrc/attention_latent_prefill.cu).  ``queries`` [T, heads * key_dim], ``out`` [T, heads * value_dim].  A step whose CTAs
-    would leave most SMs empty (decoded tokens: one row tile per request) deals every row tile's keys to several CTAs, down to four
-    tiles of 32 keys each, and merges the parts with the general kernel's merge."""
+    would leave most SMs empty (few rows per request) deals every row tile's keys to several CTAs, down to four
+    tiles of 32 keys each, and merges the parts with the general kernel's merge.  Steps of single tokens run on a kernel whose rows are
+    a token's heads, the keys dealt to as many CTAs as there are SMs, down to a tile of 64 keys each."""
     ops = _ops()
     tokens = queries.shape[0]
+    if batch.max_q_len == 1 and latent_prefill_library(key_dim, value_dim).tlie_latent_decode_fits() == 1:
+        splits = max(1, min(sm_count() // (tokens * -(-heads // 16)), -(-batch.max_seq_len // 64), 64))
+        partial = mixed_scratch(queries.device, tokens * splits * (heads * value_dim + 2 * heads), torch.float32) if splits > 1 else None
+        ops._check(
+            latent_prefill_library(key_dim, value_dim).tlie_latent_decode(
+                ops._ptr(queries), pages_ptr, c_longlong(page_stride), ops._i32(batch.first_positions, "first_positions"), ops._i32(block_table, "block_table"),
+                c_int(block_table.shape[1]), ops._ptr(sinks), ops._ptr(out), c_int(tokens), c_int(heads), c_int(page_size), c_float(scale), c_int(splits), ops._ptr(partial),
+                ops._stream()),
+            "latent_decode")
+        if splits > 1:
+            ops._check(ops.mixed_attention().tlie_merge_parts(ops._ptr(partial), ops._ptr(out), c_int(tokens), c_int(heads), c_int(value_dim), c_int(splits), ops._ptr(sinks),
+                                                              ops._stream()), "merge_parts")
+        return
     row_tiles = -(-batch.max_q_len * heads // 64) * batch.num_seqs
     splits, partial = 1, None
     if 2 * row_tiles <= sm_count():
