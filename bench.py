@@ -976,6 +976,13 @@ def run_designs(args) -> dict:
             ms = timed(lambda: ops.mixed_heads_attention(queries, -1, ctx.positions, ctx.token_seq, latent_cache, None, None, summed, LH, 1, rank + rot, rank, 0, (plain + rot) ** -0.5,
                                                          batch=ctx, values_in_keys=True))
             out[f"latent_attention_{name}"] = against_flops(ms, causal * LH * 2.0 * (2 * rank + rot)) if prompt else against_bytes(ms, causal * (rank + rot) * 2.0)
+            if prompt:   # the form of steps that begin their requests: the step's own keys and values expanded
+                tiles, own, w_expand = fast.latent_rows_tiles(ctx), torch.randn(tokens, rank, device=device).to(bf16), (torch.randn(LH * (plain + vdim), rank, device=device) * rank ** -0.5).to(bf16)
+                expanded, shared_key = torch.empty(tokens, LH * (plain + vdim), dtype=bf16, device=device), torch.randn(tokens, rot, device=device).to(bf16)
+                own_queries, heads_out = torch.randn(tokens, LH * (plain + rot), device=device).to(bf16), torch.empty(tokens, LH * vdim, dtype=bf16, device=device)
+                expand_ms = timed(lambda: ops.linear(own, w_expand, expanded))
+                rows_ms = timed(lambda: fast.latent_rows(own_queries, expanded, shared_key, tiles, ctx, heads_out, LH, plain, rot, vdim, (plain + rot) ** -0.5))
+                out["latent_attention_own_rows_prefill"] = against_flops(rows_ms, causal * LH * 2.0 * (plain + rot + vdim), ms, causal * LH * 2.0 * (2 * rank + rot), expansion_ms=expand_ms)
             down_rows, q_latent = torch.randn(tokens, q_rank + rank + rot + LH * vdim, device=device).to(bf16), torch.empty(tokens, q_rank, dtype=bf16, device=device)
             q_rows = torch.randn(tokens, LH * (plain + rot), device=device).to(bf16)
             sizes = (LH, plain, rot, rank, False, 1.1)

@@ -13,7 +13,9 @@
 // ``softcap`` and sigmoid weights (``sigmoid``, ``shifts``) as in the general kernel; a part's maximum is then 0 and the parts' totals add up to 1,
 // so that the merge is the same.
 //
-// Compile-time: KEY_DIM, VALUE_DIM (multiples of 16), KV_HEADS.  Heads per key/value head: at most 16.
+// Heads that are not mixed need not sit in one CTA: gridDim.z CTAs then share the key/value heads, KV_HEADS each.
+//
+// Compile-time: KEY_DIM, VALUE_DIM (multiples of 16), KV_HEADS (of one CTA).  Heads per key/value head: at most 16.
 #include "common.cuh"
 #include "mma_utils.cuh"
 
@@ -56,9 +58,10 @@ __global__ void __launch_bounds__(kThreads)
     mixed_decode_kernel(const __nv_bfloat16* __restrict__ rows, int row_stride, int gate_offset, const __nv_bfloat16* __restrict__ k_pages,
                         long long k_page_stride, const __nv_bfloat16* __restrict__ v_pages, long long v_page_stride, const int* __restrict__ positions,
                         const int* __restrict__ token_seq, const int* __restrict__ block_table, int table_stride, const float* __restrict__ slopes,
-                        const float* __restrict__ mix, __nv_bfloat16* __restrict__ out, int heads, int page_size, int window, float scale,
+                        const float* __restrict__ mix, __nv_bfloat16* __restrict__ out, int all_heads, int page_size, int window, float scale,
                         float* __restrict__ partial, int keep_first, int gate_per_head, float softcap, int sigmoid, const float* __restrict__ shifts) {
   extern __shared__ __align__(16) unsigned char smem[];
+  const int heads = all_heads / (int)gridDim.z, head0 = blockIdx.z * heads, kv0 = blockIdx.z * kG;   // this CTA's heads: head0 .. head0 + heads - 1
   const DecodeSmem at(heads, mix != nullptr);
   long long* k_at = reinterpret_cast<long long*>(smem + at.rows);
   long long* v_at = k_at + kKeys;
@@ -86,7 +89,7 @@ __global__ void __launch_bounds__(kThreads)
     const int chunk = i % kQChunks, r = i / kQChunks;
     const int c = r >> 4, in_group = r & 15;
     uint4 value = make_uint4(0u, 0u, 0u, 0u);
-    if (in_group < group) value = *reinterpret_cast<const uint4*>(row + (size_t)(c * group + in_group) * kD + chunk * 8);
+    if (in_group < group) value = *reinterpret_cast<const uint4*>(row + (size_t)(head0 + c * group + in_group) * kD + chunk * 8);
     *reinterpret_cast<uint4*>(q_s + (size_t)r * kQRow + chunk * 8) = value;
   }
   for (int i = tid; i < kG * 16 * kPRow / 2; i += kThreads) reinterpret_cast<unsigned*>(p_s)[i] = 0u;   // rows of no head stay zero
@@ -131,12 +134,12 @@ __global__ void __launch_bounds__(kThreads)
     for (int i = tid; i < kG * kKeys * kKChunks; i += kThreads) {
       const int chunk = i % kKChunks, j = (i / kKChunks) % kKeys, c = i / (kKChunks * kKeys);
       const bool valid = j < count;
-      cp_async_16(k_t + ((size_t)c * kKeys + j) * kKRow + chunk * 8, valid ? k_pages + k_at[j] + (size_t)c * page_size * kD + chunk * 8 : k_pages, valid);
+      cp_async_16(k_t + ((size_t)c * kKeys + j) * kKRow + chunk * 8, valid ? k_pages + k_at[j] + (size_t)(kv0 + c) * page_size * kD + chunk * 8 : k_pages, valid);
     }
     for (int i = tid; i < kG * kKeys * kVChunks; i += kThreads) {
       const int chunk = i % kVChunks, j = (i / kVChunks) % kKeys, c = i / (kVChunks * kKeys);
       const bool valid = j < count;
-      cp_async_16(v_t + ((size_t)c * kKeys + j) * kVRow + chunk * 8, valid ? v_pages + v_at[j] + (size_t)c * page_size * kVD + chunk * 8 : v_pages, valid);
+      cp_async_16(v_t + ((size_t)c * kKeys + j) * kVRow + chunk * 8, valid ? v_pages + v_at[j] + (size_t)(kv0 + c) * page_size * kVD + chunk * 8 : v_pages, valid);
     }
     cp_async_commit();
     cp_async_wait<0>();
@@ -170,7 +173,7 @@ __global__ void __launch_bounds__(kThreads)
             if (in_group < group) {
               const int h = c * group + in_group;
               float raw = s[j][e] * scale;
-              if (slopes) raw -= slopes[h] * (float)(pos - (base + key < kept ? base + key : lo + (base + key - kept)));
+              if (slopes) raw -= slopes[head0 + h] * (float)(pos - (base + key < kept ? base + key : lo + (base + key - kept)));
               raw_s[h * kKeys + key] = raw;
             }
           }
@@ -197,7 +200,7 @@ __global__ void __launch_bounds__(kThreads)
       }
       if (softcap > 0.0f) score = softcap * tanhf(score / softcap);
       if (sigmoid) {
-        const float p = lane < count ? 1.0f / (1.0f + expf(-(score + (shifts != nullptr ? shifts[h] : 0.0f)))) : 0.0f;
+        const float p = lane < count ? 1.0f / (1.0f + expf(-(score + (shifts != nullptr ? shifts[head0 + h] : 0.0f)))) : 0.0f;
         p_s[(size_t)((h / group) * 16 + h % group) * kPRow + lane] = __float2bfloat16_rn(p);
         if (lane == 0) shrink_s[h] = 1.0f;
         continue;
@@ -247,12 +250,12 @@ __global__ void __launch_bounds__(kThreads)
     }
   }
   __syncthreads();
-  const int outputs = heads * kVD;
-  float* mine = splits > 1 ? partial + ((size_t)t * splits + blockIdx.y) * (outputs + 2 * heads) : nullptr;
+  const int outputs = all_heads * kVD;
+  float* mine = splits > 1 ? partial + ((size_t)t * splits + blockIdx.y) * (outputs + 2 * all_heads) : nullptr;
   if (mine != nullptr)
     for (int i = tid; i < heads; i += kThreads) {
-      mine[outputs + i] = max_s[i];
-      mine[outputs + heads + i] = sum_s[i];
+      mine[outputs + head0 + i] = max_s[i];
+      mine[outputs + all_heads + head0 + i] = sum_s[i];
     }
 #pragma unroll
   for (int u = 0; u < kGroupsPerWarp; ++u) {
@@ -262,8 +265,8 @@ __global__ void __launch_bounds__(kThreads)
     for (int half = 0; half < 2; ++half) {
       const int in_group = g + half * 8;
       if (in_group >= group) continue;
-      const int h = c * group + in_group;
-      const float inv = mine != nullptr ? 1.0f : 1.0f / sum_s[h];
+      const float inv = mine != nullptr ? 1.0f : 1.0f / sum_s[c * group + in_group];
+      const int h = head0 + c * group + in_group;
 #pragma unroll
       for (int i = 0; i < kVD / 8; ++i) {
         const int d = i * 8 + 2 * tq;
@@ -343,20 +346,22 @@ TLIE_EXPORT long long tlie_mixed_decode_smem_bytes(int heads, int mixed) { retur
 // ``splits`` > 1: ``partial`` holds tokens * splits * (heads * VALUE_DIM + 2 * heads) floats.
 TLIE_EXPORT int tlie_mixed_decode(const void* rows, int row_stride, int gate_offset, const void* k_pages, long long k_page_stride, const void* v_pages,
                                   long long v_page_stride, const int* positions, const int* token_seq, const int* block_table, int table_stride,
-                                  const float* slopes, const float* mix, void* out, int tokens, int heads, int page_size, int window, float scale, int splits,
+                                  const float* slopes, const float* mix, void* out, int tokens, int heads, int kv_heads, int page_size, int window, float scale, int splits,
                                   float* partial, int keep_first, int gate_per_head, float softcap, int sigmoid, const float* shifts, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (keep_first < 0) return (int)cudaErrorInvalidValue;
-  if (heads <= 0 || heads % kG != 0 || heads / kG > 16 || row_stride % 8 != 0 || (gate_offset >= 0 && !gate_per_head && gate_offset % 2 != 0) || splits < 1 || splits > 64 ||
+  if (kv_heads <= 0 || kv_heads % kG != 0 || kv_heads / kG > 65535 || (mix != nullptr && kv_heads != kG)) return (int)cudaErrorInvalidValue;
+  if (heads <= 0 || heads % kv_heads != 0 || heads / kv_heads > 16 || row_stride % 8 != 0 || (gate_offset >= 0 && !gate_per_head && gate_offset % 2 != 0) || splits < 1 || splits > 64 ||
       (splits > 1 && partial == nullptr))
     return (int)cudaErrorInvalidValue;
-  const size_t smem = DecodeSmem(heads, mix != nullptr).total;
+  const int shares = kv_heads / kG;
+  const size_t smem = DecodeSmem(heads / shares, mix != nullptr).total;
   if (smem > 227 * 1024) return (int)cudaErrorInvalidValue;
   if (smem > 48 * 1024) {
     const cudaError_t set = cudaFuncSetAttribute(mixed_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (set != cudaSuccess) return (int)set;
   }
-  mixed_decode_kernel<<<dim3(tokens, splits), kThreads, smem, stream>>>((const __nv_bfloat16*)rows, row_stride, gate_offset, (const __nv_bfloat16*)k_pages,
+  mixed_decode_kernel<<<dim3(tokens, splits, shares), kThreads, smem, stream>>>((const __nv_bfloat16*)rows, row_stride, gate_offset, (const __nv_bfloat16*)k_pages,
                                                                        k_page_stride, (const __nv_bfloat16*)v_pages, v_page_stride, positions, token_seq,
                                                                        block_table, table_stride, slopes, mix, (__nv_bfloat16*)out, heads, page_size, window,
                                                                        scale, partial, window > 0 ? keep_first : 0, gate_per_head, softcap, sigmoid, shifts);

@@ -894,13 +894,18 @@ use_mixed_decode = True
 
 
 def mixed_decode_library(key_dim: int, value_dim: int, kv_heads: int):
-    """The kernel set of one (key width, value width, key/value heads): compiled when a model of these sizes first decodes."""
+    """The kernel set of one (key width, value width, key/value heads of a CTA): compiled when a model of these sizes first decodes."""
     lib = load_library(f"tlie_attn_mixed_decode_k{key_dim}_v{value_dim}_g{kv_heads}", ["attention_mixed_decode.cu"],
                        {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "KV_HEADS": kv_heads})
     if not getattr(lib, "_tlie_typed", False):
         lib.tlie_mixed_decode_smem_bytes.restype = c_longlong
         lib._tlie_typed = True
     return lib
+
+
+def mixed_decode_share(kv_heads: int, mixed: bool) -> int:
+    """How many key/value heads one CTA of the decode kernel takes: all of them if the heads are mixed, else the largest divisor up to four (a warp each)."""
+    return kv_heads if mixed else max(n for n in (1, 2, 3, 4) if kv_heads % n == 0)
 
 
 def mixed_decode_takes(rows, heads: int, kv_heads: int, key_dim: int, value_dim: int, gate_offset: int, mixed: bool, gate_per_head: bool = False) -> bool:
@@ -910,7 +915,9 @@ def mixed_decode_takes(rows, heads: int, kv_heads: int, key_dim: int, value_dim:
         return False
     if gate_offset >= 0 and not gate_per_head and gate_offset % 2:
         return False
-    fixed = 512 + kv_heads * (16 * (key_dim + 8) + 32 * (key_dim + 8) + 32 * (value_dim + 8) + 16 * 40) * 2
+    share = mixed_decode_share(kv_heads, mixed)
+    heads = heads // (kv_heads // share)
+    fixed = 512 + share * (16 * (key_dim + 8) + 32 * (key_dim + 8) + 32 * (value_dim + 8) + 16 * 40) * 2
     return fixed + heads * 32 * 4 + (heads * heads * 4 if mixed else 0) + 3 * heads * 4 + 16 <= 200 * 1024
 
 
@@ -924,10 +931,10 @@ def mixed_decode(rows, gate_offset: int, positions, token_seq, block_table, plan
     partial = mixed_scratch(rows.device, tokens * splits * (heads * value_dim + 2 * heads), torch.float32) if splits > 1 else None
     k_ptr, k_stride, v_ptr, v_stride = planes
     ops._check(
-        mixed_decode_library(key_dim, value_dim, kv_heads).tlie_mixed_decode(
+        mixed_decode_library(key_dim, value_dim, mixed_decode_share(kv_heads, mix is not None)).tlie_mixed_decode(
             ops._ptr(rows), c_int(rows.shape[1]), c_int(gate_offset), k_ptr, c_longlong(k_stride), v_ptr, c_longlong(v_stride), ops._i32(positions, "positions"),
             ops._i32(token_seq, "token_seq"), ops._i32(block_table, "block_table"), c_int(block_table.shape[1]), ops._ptr(slopes), ops._ptr(mix), ops._ptr(out),
-            c_int(tokens), c_int(heads), c_int(page_size), c_int(window), c_float(scale), c_int(splits), ops._ptr(partial), c_int(keep_first),
+            c_int(tokens), c_int(heads), c_int(kv_heads), c_int(page_size), c_int(window), c_float(scale), c_int(splits), ops._ptr(partial), c_int(keep_first),
             c_int(1 if gate_per_head else 0), c_float(softcap), c_int(1 if sigmoid else 0), ops._ptr(shifts), ops._stream()),
         "mixed_decode")
 
