@@ -513,25 +513,32 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
         const bool need_mask = key0 + kKeysTC - 1 > t.pos0 || (window > 0 && key0 < t.pos0 + t.rows_here - window);
         if constexpr (kSigmoidTC) {
           // with u = 1 / (1 + e^(2 s / c)): c tanh(s / c) = c - 2 c u, and the weight is 1 / (1 + e^-(c - 2 c u + shift))
+          // (loops without a branch inside, so that the chains of different scores run side by side)
           const Float2Bits to_exp2 = pair_of(sig_to_exp, sig_to_exp), twice_cap2 = pair_of(sig_twice_cap, sig_twice_cap), base2 = pair_of(sig_base, sig_base);
+          if (softcap > 0.0f) {
+#pragma unroll
+            for (int i = 0; i < kKeysTC / 2; ++i) {
+              float x0, x1;
+              unpair(mul2(pair_of(sc[2 * i], sc[2 * i + 1]), to_exp2), x0, x1);
+              inverse_one_plus_exp2(x0, x1, sc[2 * i], sc[2 * i + 1]);
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < kKeysTC / 2; ++i) unpair(mul2(pair_of(sc[2 * i], sc[2 * i + 1]), to_exp2), sc[2 * i], sc[2 * i + 1]);
+          }
 #pragma unroll
           for (int i = 0; i < kKeysTC / 2; ++i) {
             float x0, x1, w0, w1;
-            Float2Bits score = mul2(pair_of(sc[2 * i], sc[2 * i + 1]), to_exp2);
-            if (softcap > 0.0f) {
-              float u0, u1;
-              unpair(score, x0, x1);
-              inverse_one_plus_exp2(x0, x1, u0, u1);
-              score = pair_of(u0, u1);
-            }
-            unpair(fma2(score, twice_cap2, base2), x0, x1);
+            unpair(fma2(pair_of(sc[2 * i], sc[2 * i + 1]), twice_cap2, base2), x0, x1);
             inverse_one_plus_exp2(x0, x1, w0, w1);
-            if (need_mask) {
-              const int key = key0 + 2 * i;
-              w0 = (key >= my_lo && key <= my_pos) ? w0 : 0.0f;
-              w1 = (key + 1 >= my_lo && key + 1 <= my_pos) ? w1 : 0.0f;
-            }
             packed[i] = pack_bf16(w0, w1);
+          }
+          if (need_mask) {
+#pragma unroll
+            for (int i = 0; i < kKeysTC / 2; ++i) {
+              const int key = key0 + 2 * i;
+              packed[i] &= ((key >= my_lo && key <= my_pos) ? 0xffffu : 0u) | ((key + 1 >= my_lo && key + 1 <= my_pos) ? 0xffff0000u : 0u);
+            }
           }
         } else {
         float tile_max = -INFINITY;

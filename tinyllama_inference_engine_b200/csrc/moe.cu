@@ -384,7 +384,7 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_tiled_kernel(const T* __
     float sum[2][TOK];
 #pragma unroll
     for (int i = 0; i < TOK; ++i) sum[0][i] = sum[1][i] = 0.0f;
-    if (e1 >= router_rows) {   // a warp with one row left: eight of its pieces ahead (a token's sum runs over the columns in the same order)
+    if (TOK == 1 && e1 >= router_rows) {   // a warp with one row left: eight of its pieces ahead (a token's sum runs over the columns in the same order)
 #pragma unroll 8
       for (int d = lane * 4; d < width; d += 128) {
         const float4 a0 = *reinterpret_cast<const float4*>(w0 + d);
