@@ -541,67 +541,67 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
             }
           }
         } else {
-        float tile_max = -INFINITY;
-        if (need_mask) {
+          float tile_max = -INFINITY;
+          if (need_mask) {
 #pragma unroll
-          for (int i = 0; i < kKeysTC; ++i) {
-            const int key = key0 + i;
-            sc[i] = (key >= my_lo && key <= my_pos) ? sc[i] : -INFINITY;
-            tile_max = fmaxf(tile_max, sc[i]);
-          }
-        } else {
-          float m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;   // four chains of eight three-way maxima instead of one of 64 dependent ones
-#pragma unroll
-          for (int i = 0; i < kKeysTC; i += 8) {
-            tile_max = max3(tile_max, sc[i], sc[i + 1]);
-            m1 = max3(m1, sc[i + 2], sc[i + 3]);
-            m2 = max3(m2, sc[i + 4], sc[i + 5]);
-            m3 = max3(m3, sc[i + 6], sc[i + 7]);
-          }
-          tile_max = fmaxf(fmaxf(tile_max, m1), fmaxf(m2, m3));
-        }
-        const float scaled_max = tile_max * sl2;
-        if (j == 0) {
-          reference = scaled_max;   // nothing accumulated yet: the first product overwrites O
-        } else {
-          // O (in tensor memory) and the sum are taken against `reference`.  They are brought to a new one only when this
-          // tile's maximum is far above it; the loads and stores are warp-wide, rows that need nothing multiply by one.
-          const bool grown = scaled_max > reference + kLazyRescale;
-          if (__any_sync(0xffffffffu, grown)) {
-            // The product that last added to O must be done (the one of this tile waits for this P, so its barrier cannot be further on).
-            ok = mbar_wait(&sm.v_done[v_before.stage], v_before.phase, abort_flag);
-            if (!ok) break;
-            asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-            const float alpha = grown ? exp2f(reference - scaled_max) : 1.0f;
-#pragma unroll
-            for (int c = 0; c < kSubTiles; ++c) {   // 64 columns of the output at a time
-              float o[64];
-              tmem_ld64(tmem_o + c * 64, o);
-#pragma unroll
-              for (int i = 0; i < 64; ++i) o[i] *= alpha;
-              tmem_st64(tmem_o + c * 64, o);
+            for (int i = 0; i < kKeysTC; ++i) {
+              const int key = key0 + i;
+              sc[i] = (key >= my_lo && key <= my_pos) ? sc[i] : -INFINITY;
+              tile_max = fmaxf(tile_max, sc[i]);
             }
-            row_sum *= alpha;
-            if (grown) reference = scaled_max;
-          }
-        }
-        const float base = (reference == -INFINITY) ? 0.0f : reference;   // a row that has seen no key yet: every p is 0
-        TL(3)
-        const Float2Bits scale2 = pair_of(sl2, sl2), minus_base2 = pair_of(-base, -base);
-        Float2Bits sums = pair_of(0.0f, 0.0f);   // the even keys' sum and the odd keys'
-        // (Taking a share of the exponentials on the FMA pipe, by a polynomial, was measured: a quarter of them gains 2 %, half
-        // of them loses 17 %.)
+          } else {
+            float m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;   // four chains of eight three-way maxima instead of one of 64 dependent ones
 #pragma unroll
-        for (int i = 0; i < kKeysTC / 2; ++i) {
-          float x0, x1;
-          unpair(fma2(pair_of(sc[2 * i], sc[2 * i + 1]), scale2, minus_base2), x0, x1);
-          const float p0 = exp2_approx(x0), p1 = exp2_approx(x1);
-          sums = add2(sums, pair_of(p0, p1));
-          packed[i] = pack_bf16(p0, p1);
-        }
-        float sum0, sum1;
-        unpair(sums, sum0, sum1);
-        row_sum += sum0 + sum1;
+            for (int i = 0; i < kKeysTC; i += 8) {
+              tile_max = max3(tile_max, sc[i], sc[i + 1]);
+              m1 = max3(m1, sc[i + 2], sc[i + 3]);
+              m2 = max3(m2, sc[i + 4], sc[i + 5]);
+              m3 = max3(m3, sc[i + 6], sc[i + 7]);
+            }
+            tile_max = fmaxf(fmaxf(tile_max, m1), fmaxf(m2, m3));
+          }
+          const float scaled_max = tile_max * sl2;
+          if (j == 0) {
+            reference = scaled_max;   // nothing accumulated yet: the first product overwrites O
+          } else {
+            // O (in tensor memory) and the sum are taken against `reference`.  They are brought to a new one only when this
+            // tile's maximum is far above it; the loads and stores are warp-wide, rows that need nothing multiply by one.
+            const bool grown = scaled_max > reference + kLazyRescale;
+            if (__any_sync(0xffffffffu, grown)) {
+              // The product that last added to O must be done (the one of this tile waits for this P, so its barrier cannot be further on).
+              ok = mbar_wait(&sm.v_done[v_before.stage], v_before.phase, abort_flag);
+              if (!ok) break;
+              asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+              const float alpha = grown ? exp2f(reference - scaled_max) : 1.0f;
+#pragma unroll
+              for (int c = 0; c < kSubTiles; ++c) {   // 64 columns of the output at a time
+                float o[64];
+                tmem_ld64(tmem_o + c * 64, o);
+#pragma unroll
+                for (int i = 0; i < 64; ++i) o[i] *= alpha;
+                tmem_st64(tmem_o + c * 64, o);
+              }
+              row_sum *= alpha;
+              if (grown) reference = scaled_max;
+            }
+          }
+          const float base = (reference == -INFINITY) ? 0.0f : reference;   // a row that has seen no key yet: every p is 0
+          TL(3)
+          const Float2Bits scale2 = pair_of(sl2, sl2), minus_base2 = pair_of(-base, -base);
+          Float2Bits sums = pair_of(0.0f, 0.0f);   // the even keys' sum and the odd keys'
+          // (Taking a share of the exponentials on the FMA pipe, by a polynomial, was measured: a quarter of them gains 2 %, half
+          // of them loses 17 %.)
+#pragma unroll
+          for (int i = 0; i < kKeysTC / 2; ++i) {
+            float x0, x1;
+            unpair(fma2(pair_of(sc[2 * i], sc[2 * i + 1]), scale2, minus_base2), x0, x1);
+            const float p0 = exp2_approx(x0), p1 = exp2_approx(x1);
+            sums = add2(sums, pair_of(p0, p1));
+            packed[i] = pack_bf16(p0, p1);
+          }
+          float sum0, sum1;
+          unpair(sums, sum0, sum1);
+          row_sum += sum0 + sum1;
         }
         TL(4)
         // P over the first 32 columns of this tile's scores: key 2 i in the lower half of column i, key 2 i + 1 in the upper.  The
