@@ -147,7 +147,9 @@ __global__ void __launch_bounds__(128) normed_store_kernel(T* __restrict__ rows,
 // ... k at k_offset | ... v at v_offset].  Every vector gets its bias (null: none); q and k are divided by their root mean square and
 // multiplied by a weight (null: neither); their first ``rot_dims`` columns turn by position * inv_freq[i], cosines and sines times
 // ``amplitude``, columns (2i, 2i + 1) together if ``interleaved``, else column i with column i + rot_dims / 2; query head h is multiplied by
-// q_factors[h] (null: not).  q stays in place, k and v go into the token's page.  A warp per vector, which waits in shared memory as
+// q_factors[h] (null: not).  q stays in place, k and v go into the token's page.  ``first_values`` [tokens, kv_heads x value_dim] (null: none): with
+// ``keep_values`` the values are left there as well, otherwise v <- (1 - value_share) v + value_share first_values is what is
+// stored (values drawn towards those of an earlier layer, which left them).  A warp per vector, which waits in shared memory as
 // 32-bit numbers between the passes; gridDim.y CTAs share a token's vectors (steps of few rows).
 template <typename T>
 __global__ void __launch_bounds__(256) norm_rotary_store_kernel(T* __restrict__ rows, int row_stride, int k_offset, int v_offset, const float* __restrict__ q_bias,
@@ -157,7 +159,7 @@ __global__ void __launch_bounds__(256) norm_rotary_store_kernel(T* __restrict__ 
                                                                 const int* __restrict__ positions, const int* __restrict__ token_seq,
                                                                 const int* __restrict__ block_table, int table_stride, T* __restrict__ k_pages, long long k_page_stride,
                                                                 T* __restrict__ v_pages, long long v_page_stride, int heads, int kv_heads, int key_dim, int value_dim,
-                                                                int page_size, int write_cache) {
+                                                                int page_size, int write_cache, T* __restrict__ first_values, int keep_values, float value_share) {
   extern __shared__ float turn_s[];   // the token's cosines [rot_dims / 2], its sines, then a vector per warp [key_dim]
   const int t = blockIdx.x;
   const int pos = positions[t];
@@ -173,11 +175,18 @@ __global__ void __launch_bounds__(256) norm_rotary_store_kernel(T* __restrict__ 
     turn_s[i] = cosine * amplitude;
     turn_s[half + i] = sine * amplitude;
   }
-  if (page >= 0)
-    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < kv_heads * value_dim; i += gridDim.y * blockDim.x) {
-      const int head = i / value_dim, d = i - head * value_dim;
-      v_pages[(size_t)page * v_page_stride + ((size_t)head * page_size + slot) * value_dim + d] = from_float<T>(to_float(row[v_offset + i]) + (v_bias != nullptr ? v_bias[i] : 0.0f));
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < kv_heads * value_dim; i += gridDim.y * blockDim.x) {
+    const int head = i / value_dim, d = i - head * value_dim;
+    float v = to_float(row[v_offset + i]) + (v_bias != nullptr ? v_bias[i] : 0.0f);
+    if (first_values != nullptr) {
+      T* first = first_values + (size_t)t * kv_heads * value_dim + i;
+      if (keep_values)
+        *first = from_float<T>(v);
+      else
+        v = (1.0f - value_share) * v + value_share * to_float(*first);
     }
+    if (page >= 0) v_pages[(size_t)page * v_page_stride + ((size_t)head * page_size + slot) * value_dim + d] = from_float<T>(v);
+  }
   __syncthreads();
   for (int h = blockIdx.y * warps + warp; h < heads + kv_heads; h += gridDim.y * warps) {
     const bool is_key = h >= heads;
@@ -817,7 +826,7 @@ TLIE_EXPORT int tlie_norm_rotary_store(int dtype, void* rows, int row_stride, in
                                        const float* q_weight, const float* k_weight, float eps, const float* q_factors, const float* inv_freq, int rot_dims,
                                        int interleaved, float amplitude, const int* positions, const int* token_seq, const int* block_table, int table_stride,
                                        void* k_pages, long long k_page_stride, void* v_pages, long long v_page_stride, int tokens, int heads, int kv_heads, int key_dim,
-                                       int value_dim, int page_size, int write_cache, cudaStream_t stream) {
+                                       int value_dim, int page_size, int write_cache, void* first_values, int keep_values, float value_share, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   constexpr int kThreads = 256;
   const size_t smem = ((size_t)rot_dims + (size_t)(kThreads / 32) * key_dim) * sizeof(float);
@@ -827,7 +836,7 @@ TLIE_EXPORT int tlie_norm_rotary_store(int dtype, void* rows, int row_stride, in
   norm_rotary_store_kernel<T><<<dim3(tokens, shares), kThreads, smem, stream>>>((T*)rows, row_stride, k_offset, v_offset, q_bias, k_bias, v_bias, q_weight, k_weight, eps, q_factors, \
                                                                   inv_freq, rot_dims, interleaved, amplitude, positions, token_seq, block_table, table_stride,     \
                                                                   (T*)k_pages, k_page_stride, (T*)v_pages, v_page_stride, heads, kv_heads, key_dim, value_dim,       \
-                                                                  page_size, write_cache)
+                                                                  page_size, write_cache, (T*)first_values, keep_values, value_share)
   if (dtype == TLIE_F32)
     TLIE_STORE(float);
   else

@@ -13,6 +13,8 @@
 // ``softcap`` and sigmoid weights (``sigmoid``, ``shifts``) as in the general kernel; a part's maximum is then 0 and the parts' totals add up to 1,
 // so that the merge is the same.
 //
+// ``sinks`` (optional, one per head): the softmax's denominator also holds exp(sink_h), a weight that belongs to no key.
+//
 // Heads that are not mixed need not sit in one CTA: gridDim.z CTAs then share the key/value heads, KV_HEADS each.
 //
 // Compile-time: KEY_DIM, VALUE_DIM (multiples of 16), KV_HEADS (of one CTA).  Heads per key/value head: at most 16.
@@ -59,7 +61,8 @@ __global__ void __launch_bounds__(kThreads)
                         long long k_page_stride, const __nv_bfloat16* __restrict__ v_pages, long long v_page_stride, const int* __restrict__ positions,
                         const int* __restrict__ token_seq, const int* __restrict__ block_table, int table_stride, const float* __restrict__ slopes,
                         const float* __restrict__ mix, __nv_bfloat16* __restrict__ out, int all_heads, int page_size, int window, float scale,
-                        float* __restrict__ partial, int keep_first, int gate_per_head, float softcap, int sigmoid, const float* __restrict__ shifts) {
+                        float* __restrict__ partial, int keep_first, int gate_per_head, float softcap, int sigmoid, const float* __restrict__ shifts,
+                        const float* __restrict__ sinks) {
   extern __shared__ __align__(16) unsigned char smem[];
   const int heads = all_heads / (int)gridDim.z, head0 = blockIdx.z * heads, kv0 = blockIdx.z * kG;   // this CTA's heads: head0 .. head0 + heads - 1
   const DecodeSmem at(heads, mix != nullptr);
@@ -265,8 +268,9 @@ __global__ void __launch_bounds__(kThreads)
     for (int half = 0; half < 2; ++half) {
       const int in_group = g + half * 8;
       if (in_group >= group) continue;
-      const float inv = mine != nullptr ? 1.0f : 1.0f / sum_s[c * group + in_group];
       const int h = head0 + c * group + in_group;
+      float inv = 1.0f;
+      if (mine == nullptr) inv = 1.0f / (sum_s[c * group + in_group] + (sinks != nullptr ? expf(sinks[h] - max_s[c * group + in_group]) : 0.0f));
 #pragma unroll
       for (int i = 0; i < kVD / 8; ++i) {
         const int d = i * 8 + 2 * tq;
@@ -293,7 +297,7 @@ __global__ void __launch_bounds__(kThreads)
 
 // The parts of a row put together (see merge_mixed_kernel of the general kernel): a CTA per (row, head), a thread per output.
 __global__ void merge_mixed_decode_kernel(const float* __restrict__ partial, const __nv_bfloat16* __restrict__ rows, int row_stride, int gate_offset,
-                                          __nv_bfloat16* __restrict__ out, int heads, int splits, int gate_per_head) {
+                                          __nv_bfloat16* __restrict__ out, int heads, int splits, int gate_per_head, const float* __restrict__ sinks) {
   __shared__ float weight_s[64];   // at most 64 parts: each part's e^(max - highest)
   __shared__ float scratch[2];
   const int t = blockIdx.x, h = blockIdx.y;
@@ -309,7 +313,7 @@ __global__ void merge_mixed_decode_kernel(const float* __restrict__ partial, con
       top[i] = s < splits ? mine[s * part_size + outputs + h] : -INFINITY;
       sum[i] = s < splits ? mine[s * part_size + outputs + heads + h] : 0.0f;
     }
-    const float highest = warp_max(fmaxf(top[0], top[1]));
+    const float highest = fmaxf(warp_max(fmaxf(top[0], top[1])), sinks != nullptr ? sinks[h] : -INFINITY);
     float total = 0.0f;
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -318,6 +322,7 @@ __global__ void merge_mixed_decode_kernel(const float* __restrict__ partial, con
       total += sum[i] * weight;
     }
     total = warp_sum(total);
+    if (sinks != nullptr) total += expf(sinks[h] - highest);
     if (lane == 0) scratch[0] = 1.0f / total;
   }
   __syncthreads();
@@ -347,9 +352,10 @@ TLIE_EXPORT long long tlie_mixed_decode_smem_bytes(int heads, int mixed) { retur
 TLIE_EXPORT int tlie_mixed_decode(const void* rows, int row_stride, int gate_offset, const void* k_pages, long long k_page_stride, const void* v_pages,
                                   long long v_page_stride, const int* positions, const int* token_seq, const int* block_table, int table_stride,
                                   const float* slopes, const float* mix, void* out, int tokens, int heads, int kv_heads, int page_size, int window, float scale, int splits,
-                                  float* partial, int keep_first, int gate_per_head, float softcap, int sigmoid, const float* shifts, cudaStream_t stream) {
+                                  float* partial, int keep_first, int gate_per_head, float softcap, int sigmoid, const float* shifts,
+                                  const float* sinks, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (keep_first < 0) return (int)cudaErrorInvalidValue;
+  if (keep_first < 0 || (sigmoid && sinks != nullptr)) return (int)cudaErrorInvalidValue;
   if (kv_heads <= 0 || kv_heads % kG != 0 || kv_heads / kG > 65535 || (mix != nullptr && kv_heads != kG)) return (int)cudaErrorInvalidValue;
   if (heads <= 0 || heads % kv_heads != 0 || heads / kv_heads > 16 || row_stride % 8 != 0 || (gate_offset >= 0 && !gate_per_head && gate_offset % 2 != 0) || splits < 1 || splits > 64 ||
       (splits > 1 && partial == nullptr))
@@ -364,9 +370,9 @@ TLIE_EXPORT int tlie_mixed_decode(const void* rows, int row_stride, int gate_off
   mixed_decode_kernel<<<dim3(tokens, splits, shares), kThreads, smem, stream>>>((const __nv_bfloat16*)rows, row_stride, gate_offset, (const __nv_bfloat16*)k_pages,
                                                                        k_page_stride, (const __nv_bfloat16*)v_pages, v_page_stride, positions, token_seq,
                                                                        block_table, table_stride, slopes, mix, (__nv_bfloat16*)out, heads, page_size, window,
-                                                                       scale, partial, window > 0 ? keep_first : 0, gate_per_head, softcap, sigmoid, shifts);
+                                                                       scale, partial, window > 0 ? keep_first : 0, gate_per_head, softcap, sigmoid, shifts, sinks);
   if (splits > 1)
     merge_mixed_decode_kernel<<<dim3(tokens, heads), kVD >= 128 ? 128 : (kVD > 32 ? 64 : 32), 0, stream>>>(partial, (const __nv_bfloat16*)rows, row_stride,
-                                                                                                        gate_offset, (__nv_bfloat16*)out, heads, splits, gate_per_head);
+                                                                                                        gate_offset, (__nv_bfloat16*)out, heads, splits, gate_per_head, sinks);
   return (int)cudaGetLastError();
 }

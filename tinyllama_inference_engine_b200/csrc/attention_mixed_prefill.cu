@@ -16,7 +16,10 @@
 // SIGMOID_WEIGHTS 1: no softmax; the score is bounded, softcap * tanh(score / softcap), and a key's weight is sigmoid(score + shift_h), not brought
 // to a sum of one.  Nothing is rescaled then.  tanh and sigmoid are written with e^x and a reciprocal, in 32-bit.
 //
-// Compile-time: KEY_DIM, VALUE_DIM (multiples of 16), PARTS (key heads per folded query), SIGMOID_WEIGHTS.
+// SCORE_CAP 1: a softmax over bounded scores, softcap * tanh(score / softcap), the tanh as above.  ``sinks`` (softmax builds; optional, one per head):
+// the denominator also holds exp(sink_h), a weight that belongs to no key.
+//
+// Compile-time: KEY_DIM, VALUE_DIM (multiples of 16), PARTS (key heads per folded query), SIGMOID_WEIGHTS, SCORE_CAP.
 #include "common.cuh"
 #include "mma_utils.cuh"
 
@@ -31,6 +34,9 @@
 #endif
 #ifndef SIGMOID_WEIGHTS
 #define SIGMOID_WEIGHTS 0
+#endif
+#ifndef SCORE_CAP
+#define SCORE_CAP 0
 #endif
 
 namespace tlie {
@@ -143,7 +149,7 @@ __global__ void __launch_bounds__(kThreads, kMinBlocks)
                          long long v_page_stride, const int* __restrict__ seq_starts, const int* __restrict__ first_positions,
                          const int* __restrict__ block_table, int table_stride, const float* __restrict__ slopes, __nv_bfloat16* __restrict__ out,
                          int heads, int kv_heads, int page_size, int window, int mixed, int keep_first, int gate_per_head, float softcap,
-                         const float* __restrict__ shifts) {
+                         const float* __restrict__ shifts, const float* __restrict__ sinks) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __nv_bfloat16* q_smem = reinterpret_cast<__nv_bfloat16*>(smem_raw);            // [kRows][kQRow]
   __nv_bfloat16* k_ring = q_smem + (size_t)kRows * kQRow;                        // [kRing][kPartsPerChunk][64][kKRow]
@@ -222,6 +228,9 @@ __global__ void __launch_bounds__(kThreads, kMinBlocks)
     return __fdividef(1.0f, 1.0f + exp2_approx(minus));
   };
 #else
+#if SCORE_CAP
+  const float cap_to_exp = 2.0f * kLog2e / softcap, cap_log2 = softcap * kLog2e;
+#endif
   float row_max[2] = {-INFINITY, -INFINITY};
   float row_sum[2] = {0.0f, 0.0f};
 #endif
@@ -290,7 +299,12 @@ __global__ void __launch_bounds__(kThreads, kMinBlocks)
         for (int e = 0; e < 4; ++e) {
           const int key = key0 + j * 8 + 2 * t + (e & 1);
           const int r = e >> 1;
-          const float v = ((key >= my_lo[r] || key < keep) && key <= my_pos[r]) ? fmaf(s_frag[j][e], kLog2e, -slope * (float)(my_pos[r] - key)) : -INFINITY;
+#if SCORE_CAP   // no distance bias beside a bound
+          const float score = fmaf(-2.0f * cap_log2, __fdividef(1.0f, 1.0f + exp2_approx(s_frag[j][e] * cap_to_exp)), cap_log2);
+#else
+          const float score = fmaf(s_frag[j][e], kLog2e, -slope * (float)(my_pos[r] - key));
+#endif
+          const float v = ((key >= my_lo[r] || key < keep) && key <= my_pos[r]) ? score : -INFINITY;
           s_frag[j][e] = v;
           tile_max[r] = fmaxf(tile_max[r], v);
         }
@@ -355,7 +369,8 @@ __global__ void __launch_bounds__(kThreads, kMinBlocks)
 #if SIGMOID_WEIGHTS
     const float inv = 1.0f;
 #else
-    const float inv = 1.0f / row_sum[r];
+    // a row sees itself at least: its maximum is finite.  A sink far above it makes the sum infinite and the output zero, as it should be.
+    const float inv = 1.0f / (sinks != nullptr ? row_sum[r] + exp2f(sinks[head] * kLog2e - row_max[r]) : row_sum[r]);
 #endif
     const size_t row = (size_t)(row0 + my_row[r]);
     __nv_bfloat16* dst = out + (row * heads + head) * kVD + 2 * t;
@@ -383,19 +398,21 @@ TLIE_EXPORT int tlie_mixed_prefill_folded_width() { return kParts * kD; }
 
 // ``folded``: scratch for the folded queries, bfloat16 [tokens, heads, PARTS * KEY_DIM].  ``slopes``: the folded slopes (or null).
 // ``folded`` null: the queries are taken from ``rows`` as they are (no mix, the scale already in them).
-// ``softcap`` and ``shifts`` (or null): SIGMOID_WEIGHTS only.
+// ``softcap``: SIGMOID_WEIGHTS (0: unbounded) or SCORE_CAP (positive) only.  ``shifts`` (or null): SIGMOID_WEIGHTS only.  ``sinks`` (or null): 32-bit [heads],
+// softmax builds only.
 // ``mix`` null: PARTS must be 1.  ``longest``: the most rows any entry of the step has.
 TLIE_EXPORT int tlie_mixed_prefill(const void* rows, int row_stride, int gate_offset, const float* mix, float scale, void* folded, const void* k_pages,
                                    long long k_page_stride, const void* v_pages, long long v_page_stride, const int* seq_starts,
                                    const int* first_positions, const int* block_table, int table_stride, const float* slopes, void* out, int tokens,
                                    int entries, int longest, int heads, int kv_heads, int page_size, int window, int keep_first, int gate_per_head,
-                                   float softcap, const float* shifts, cudaStream_t stream) {
+                                   float softcap, const float* shifts, const float* sinks, cudaStream_t stream) {
   if (tokens <= 0 || entries <= 0) return 0;
   if (keep_first < 0) return (int)cudaErrorInvalidValue;
   if (kRows == 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || page_size % 16 != 0 || heads > 65535 || entries > 65535 ||
       (mix != nullptr ? kParts != kv_heads : kParts != 1) || row_stride % 8 != 0 || (gate_offset >= 0 && !gate_per_head && gate_offset % 2 != 0))
     return (int)cudaErrorInvalidValue;
-  if (!SIGMOID_WEIGHTS && (softcap > 0.0f || shifts != nullptr)) return (int)cudaErrorInvalidValue;
+  if ((!SIGMOID_WEIGHTS && (shifts != nullptr || (softcap > 0.0f) != (SCORE_CAP != 0))) || (SIGMOID_WEIGHTS && sinks != nullptr) || (SCORE_CAP && slopes != nullptr))
+    return (int)cudaErrorInvalidValue;
   if (folded == nullptr && mix != nullptr) return (int)cudaErrorInvalidValue;
   const size_t fold_smem = ((size_t)heads * kD + (mix != nullptr ? (size_t)heads * heads : 0)) * sizeof(float);
   if (fold_smem > 200 * 1024) return (int)cudaErrorInvalidValue;
@@ -422,6 +439,6 @@ TLIE_EXPORT int tlie_mixed_prefill(const void* rows, int row_stride, int gate_of
   mixed_prefill_kernel<<<grid, kThreads, smem, stream>>>((const __nv_bfloat16*)(folded != nullptr ? folded : rows), folded_stride, (const __nv_bfloat16*)rows, row_stride, gate_offset,
                                                          (const __nv_bfloat16*)k_pages, k_page_stride, (const __nv_bfloat16*)v_pages, v_page_stride,
                                                          seq_starts, first_positions, block_table, table_stride, slopes, (__nv_bfloat16*)out, heads,
-                                                         kv_heads, page_size, window, mix != nullptr ? 1 : 0, keep_first, gate_per_head, softcap, shifts);
+                                                         kv_heads, page_size, window, mix != nullptr ? 1 : 0, keep_first, gate_per_head, softcap, shifts, sinks);
   return (int)cudaGetLastError();
 }

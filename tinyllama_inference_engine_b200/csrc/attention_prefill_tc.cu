@@ -32,6 +32,8 @@
 // as it is.  tanh and sigmoid are e^x and a reciprocal each, in 32-bit; one reciprocal serves two scores (1 / a = b / (a b)), so that a
 // score costs three operations of the exponential unit.  In both kinds the output may be multiplied by sigmoid(gate), one number per
 // (row, head), as it is read out.
+// SCORE_CAP 1 (a build of its own): a softmax over bounded scores, softcap * tanh(score / softcap), tanh as above.  In both softmax builds ``sinks`` (optional, one
+// per head) puts exp(sink_h) into the denominator, a weight that belongs to no key.
 // LATENT_ROWS 1 (a build of its own, KEY_DIM / ROT_DIM / VALUE_DIM): the keys and values are rows of the step itself and not of pages, which is all a
 // step sees whose requests all start in it.  A key is a head's own columns beside ROT_DIM columns that every head shares (latent
 // attention with its keys and values expanded): the two come from matrices of their own, a box each.
@@ -60,11 +62,14 @@
 #ifndef LATENT_ROWS
 #define LATENT_ROWS 0
 #endif
+#ifndef SCORE_CAP
+#define SCORE_CAP 0
+#endif
 #include <type_traits>
 
 namespace tlie {
 
-constexpr bool kSigmoidTC = SIGMOID_WEIGHTS != 0;
+constexpr bool kSigmoidTC = SIGMOID_WEIGHTS != 0, kCappedTC = SCORE_CAP != 0;
 constexpr int kRowsTC = 128;      // query rows per CTA
 constexpr int kKeysTC = 64;       // keys per tile (one box)
 constexpr int kBoxDims = 64;      // dims of one box: 128 bytes, the swizzle span
@@ -231,7 +236,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
                                 const int* __restrict__ tiles, const int* __restrict__ seq_starts, const int* __restrict__ first_positions,
                                 const int* __restrict__ block_table, int table_stride, __nv_bfloat16* __restrict__ out, int q_heads,
                                 int kv_heads, int page_size, int window, float scale, float softcap, const float* __restrict__ shifts,
-                                const __nv_bfloat16* __restrict__ gate, int gate_stride, int* __restrict__ error_flag) {
+                                const __nv_bfloat16* __restrict__ gate, int gate_stride, const float* __restrict__ sinks, int* __restrict__ error_flag) {
   extern __shared__ uint8_t smem_raw[];
   using Smem = SmemTC<kD, kVD>;
   constexpr int kKStages = Smem::kKStages, kVStages = Smem::kVStages;
@@ -478,7 +483,9 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
     const int sub = warp & 3;
     const int row = sub * 32 + lane;
     const uint32_t lane_base = (uint32_t)(sub * 32) << 16;
-    const float sl2 = scale * kLog2eTC;
+    // bounded scores arrive in the loop as softcap * tanh in units of log2: nothing is left to scale then
+    const float sl2 = kCappedTC ? 1.0f : scale * kLog2eTC;
+    const float cap_to_exp = 2.0f * scale * kLog2eTC / softcap, cap_log2 = softcap * kLog2eTC;
     // sigmoid weights, in units of log2: without a bound the exponent is -(score + shift); with one see the loop
     const float sig_to_exp = softcap > 0.0f ? 2.0f * sl2 / softcap : sl2;
     const float sig_twice_cap = softcap > 0.0f ? 2.0f * softcap * kLog2eTC : -1.0f;
@@ -541,6 +548,16 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
             }
           }
         } else {
+          if constexpr (kCappedTC) {   // c tanh(s / c) = c - 2 c u with u = 1 / (1 + e^(2 s / c)), before the mask
+            const Float2Bits to_exp2 = pair_of(cap_to_exp, cap_to_exp), minus_twice2 = pair_of(-2.0f * cap_log2, -2.0f * cap_log2), cap2 = pair_of(cap_log2, cap_log2);
+#pragma unroll
+            for (int i = 0; i < kKeysTC / 2; ++i) {
+              float x0, x1, u0, u1;
+              unpair(mul2(pair_of(sc[2 * i], sc[2 * i + 1]), to_exp2), x0, x1);
+              inverse_one_plus_exp2(x0, x1, u0, u1);
+              unpair(fma2(pair_of(u0, u1), minus_twice2, cap2), sc[2 * i], sc[2 * i + 1]);
+            }
+          }
           float tile_max = -INFINITY;
           if (need_mask) {
 #pragma unroll
@@ -631,7 +648,8 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
       if (ok) ok = mbar_wait(&sm.o_full[u], 0, abort_flag);
       if (ok) {
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        float inv = kSigmoidTC ? 1.0f : 1.0f / row_sum;
+        // (the reference is near a maximum the row has seen; a sink far above it makes the sum infinite and the output zero, as it should be)
+        float inv = kSigmoidTC ? 1.0f : 1.0f / (sinks != nullptr ? row_sum + exp2f(sinks[head] * kLog2eTC - reference) : row_sum);
         if (gate != nullptr && row < t.rows_here) inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(t.row0 + row) * gate_stride + head])));
 #pragma unroll
         for (int half = 0; half < kSubTiles; ++half) {   // 64 columns of the output at a time (the load is warp-wide: every row takes part)
@@ -692,7 +710,7 @@ template <int kD, int kVD>
 static int launch_attention_tc(const CUtensorMap& map_q, const CUtensorMap& map_kv, const CUtensorMap& map_v, const CUtensorMap& map_rot, const int* tiles, int n_tiles,
                                const int* seq_starts, const int* first_positions, const int* block_table, int table_stride, void* out, int q_heads,
                                int kv_heads, int page_size, int window, float scale, float softcap, const float* shifts, const void* gate, int gate_stride,
-                               int* error_flag, cudaStream_t stream) {
+                               const float* sinks, int* error_flag, cudaStream_t stream) {
   // keys of 128 and more: exactly the structure, no room to align it by hand (the kernel checks that it need not): 1 KB more and two CTAs no longer share an SM
 #ifdef TLIE_ATTN_ONE_PER_SM   // for measurements: so much shared memory that a CTA has its SM to itself
   const int smem = 200 * 1024;
@@ -708,7 +726,7 @@ static int launch_attention_tc(const CUtensorMap& map_q, const CUtensorMap& map_
   dim3 grid(q_heads, n_tiles);
   return (int)launch_pdl(prefill_attention_tc_kernel<kD, kVD>, grid, dim3(kThreadsTC), (size_t)smem, stream, map_q, map_kv, map_v, map_rot, tiles, seq_starts, first_positions,
                          block_table, table_stride, (__nv_bfloat16*)out, q_heads, kv_heads, page_size, window, scale, softcap, shifts, (const __nv_bfloat16*)gate, gate_stride,
-                         error_flag);
+                         sinks, error_flag);
 }
 
 #if LATENT_ROWS
@@ -729,19 +747,20 @@ TLIE_EXPORT int tlie_prefill_attention_rows(const void* q, const void* expanded,
       !make_map_2d(&map_rot, shared, tokens, ROT_DIM, ROT_DIM, kKeysTC))
     return (int)cudaErrorInvalidValue;
   return launch_attention_tc<KEY_DIM, VALUE_DIM>(map_q, map_k, map_v, map_rot, tiles, n_tiles, seq_starts, first_positions, nullptr, 0, out, heads, heads, kKeysTC, 0, scale, 0.0f,
-                                                 nullptr, nullptr, 0, error_flag, stream);
+                                                 nullptr, nullptr, 0, nullptr, error_flag, stream);
 }
 #else
 // q: the step's rows [tokens, q_row_stride] starting with the rotated q heads (head size 64 or 128); pages: one layer's pool
 // [num_pages, 2, kv_heads, page_size, head size]; tiles: int32 [n_tiles, 4] work items of one or two 128-row tiles (request, first
-// row, request or -1, first row); error_flag: device int, zero.  softcap (0: none) and shifts (32-bit [q_heads] or null): SIGMOID_WEIGHTS only.
+// row, request or -1, first row); error_flag: device int, zero.  softcap: SIGMOID_WEIGHTS (0: none) or SCORE_CAP (positive).  shifts (32-bit [q_heads] or
+// null): SIGMOID_WEIGHTS only.  sinks (32-bit [q_heads] or null): not with SIGMOID_WEIGHTS.
 // gate (or null): bfloat16, one number per (token, head), rows gate_stride elements apart; the output is multiplied by its sigmoid.
 TLIE_EXPORT int tlie_prefill_attention_tc(const void* q, int q_row_stride, int tokens, const void* pages, int num_pages, const int* tiles,
                                           int n_tiles, const int* seq_starts, const int* first_positions, const int* block_table,
                                           int table_stride, void* out, int q_heads, int kv_heads, int head_dim, int page_size, int window, float scale,
-                                          float softcap, const float* shifts, const void* gate, int gate_stride, int* error_flag, cudaStream_t stream) {
+                                          float softcap, const float* shifts, const void* gate, int gate_stride, const float* sinks, int* error_flag, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
-  if (!kSigmoidTC && (softcap > 0.0f || shifts != nullptr)) return (int)cudaErrorInvalidValue;
+  if ((!kSigmoidTC && (shifts != nullptr || (softcap > 0.0f) != kCappedTC)) || (kSigmoidTC && sinks != nullptr)) return (int)cudaErrorInvalidValue;
   if (kv_heads <= 0 || q_heads % kv_heads != 0 || n_tiles > 65535 || page_size % kKeysTC != 0 || q_row_stride % 8 != 0 || error_flag == nullptr ||
       (head_dim != 64 && head_dim != 128))
     return (int)cudaErrorInvalidValue;
@@ -750,6 +769,6 @@ TLIE_EXPORT int tlie_prefill_attention_tc(const void* q, int q_row_stride, int t
   if (!make_map_2d(&map_kv, pages, (long long)num_pages * 2 * kv_heads * page_size, head_dim, head_dim, kKeysTC)) return (int)cudaErrorInvalidValue;
   auto launch = head_dim == 64 ? launch_attention_tc<64, 64> : launch_attention_tc<128, 128>;
   return launch(map_q, map_kv, map_kv, map_kv, tiles, n_tiles, seq_starts, first_positions, block_table, table_stride, out, q_heads, kv_heads, page_size, window, scale, softcap,
-                shifts, gate, gate_stride, error_flag, stream);
+                shifts, gate, gate_stride, sinks, error_flag, stream);
 }
 #endif

@@ -322,6 +322,40 @@ __global__ void __launch_bounds__(256) hgrn2_prepare_kernel(const T* __restrict_
   }
 }
 
+// prep rows of the same layout for linear attention with a learned decay per key channel: rows = [q: H dim | k: H dim | v: H vdim] (products),
+// q times ``q_scale``; the decay of channel i is sigmoid(z_i)^(1 / tau) = e^(-softplus(-z_i) / tau) with z = decay_in + bias; beta = 1.  ``a2`` given (then
+// ``decay_in`` [T, rank] is the first half of a low-rank pair): z_i = a2[i] . decay_in + bias_i with a2 [H dim, rank], summed in 32-bit here (a step of
+// few rows then needs no product of its own for it).  A thread per number.
+template <typename T>
+__global__ void __launch_bounds__(256) gla_prepare_kernel(const T* __restrict__ rows, int row_stride, const T* __restrict__ decay_in, long long decay_stride,
+                                                          const T* __restrict__ a2, int rank, const float* __restrict__ bias, float tau, float q_scale,
+                                                          float* __restrict__ prep, int heads, int dim, int vdim) {
+  const int t = blockIdx.x;
+  const T* row = rows + (size_t)t * row_stride;
+  const T* decay_row = decay_in + (size_t)t * decay_stride;
+  const int qk = heads * dim, values = heads * vdim;
+  float* out = prep + (size_t)t * (3 * qk + values + heads);
+  const int w = blockIdx.y * blockDim.x + threadIdx.x;   // one piece of work a thread: a key channel, a value or a head's beta
+  if (w < qk) {
+    out[w] = to_float(row[w]) * q_scale;
+    out[qk + w] = to_float(row[qk + w]);
+    float z = bias[w];
+    if (a2 != nullptr) {
+      const T* weights = a2 + (size_t)w * rank;
+      float sum = 0.0f;
+      for (int r = 0; r < rank; ++r) sum = fmaf(to_float(weights[r]), to_float(decay_row[r]), sum);
+      z += sum;
+    } else {
+      z += to_float(decay_row[w]);
+    }
+    out[2 * qk + values + heads + w] = expf(-softplus_f(-z) / tau);
+  } else if (w < qk + values) {
+    out[2 * qk + (w - qk)] = to_float(row[2 * qk + (w - qk)]);
+  } else if (w < qk + values + heads) {
+    out[2 * qk + values + (w - qk - values)] = 1.0f;
+  }
+}
+
 // prep rows of the same layout for a state-space layer: rows = [z: inner | x: inner | B: G N | C: G N | dt: H] (products, inner = H vdim).
 // x, B and C pass a causal convolution over time per channel (taps [channels, n] with a bias, the last column the current token's;
 // inputs before an entry's first row come from the request's state at ``conv_offset``) and silu; dt = softplus(dt + dt_bias); the
@@ -484,6 +518,21 @@ TLIE_EXPORT int tlie_hgrn2_prepare(int dtype, const void* rows, int row_stride, 
     hgrn2_prepare_kernel<float><<<grid, 256, 0, stream>>>((const float*)rows, row_stride, f_bias, lower, prep, heads, dim, vdim);
   else
     hgrn2_prepare_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)rows, row_stride, f_bias, lower, prep, heads, dim, vdim);
+  return (int)cudaGetLastError();
+}
+
+// ``a2`` null: ``decay_in`` [tokens, heads dim] are the decays' pre-activations; else the first half of a low-rank pair, [tokens, rank].
+TLIE_EXPORT int tlie_gla_prepare(int dtype, const void* rows, int row_stride, const void* decay_in, long long decay_stride, const void* a2, int rank, const float* bias,
+                                 float tau, float q_scale, float* prep, int tokens, int heads, int dim, int vdim, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (decay_in == nullptr || bias == nullptr || (a2 != nullptr && rank <= 0) || !(tau > 0.0f)) return (int)cudaErrorInvalidValue;
+  const dim3 grid(tokens, (heads * dim + heads * vdim + heads + 255) / 256);
+  if (dtype == TLIE_F32)
+    gla_prepare_kernel<float><<<grid, 256, 0, stream>>>((const float*)rows, row_stride, (const float*)decay_in, decay_stride, (const float*)a2, rank, bias, tau, q_scale,
+                                                        prep, heads, dim, vdim);
+  else
+    gla_prepare_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)rows, row_stride, (const __nv_bfloat16*)decay_in, decay_stride,
+                                                                (const __nv_bfloat16*)a2, rank, bias, tau, q_scale, prep, heads, dim, vdim);
   return (int)cudaGetLastError();
 }
 

@@ -291,6 +291,61 @@ __global__ void activation_vec_kernel(const T* __restrict__ in, T* __restrict__ 
   }
 }
 
+// See tlie_dynamic_tanh.  A thread per VEC neighbouring elements.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) dynamic_tanh_kernel(float* __restrict__ residual, const T* __restrict__ a, const T* __restrict__ b, const int* __restrict__ rows,
+                                                           const float* __restrict__ weight, const float* __restrict__ bias, float alpha, T* __restrict__ out, int hidden,
+                                                           size_t pieces) {
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int per_row = hidden / VEC;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < pieces; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / per_row;
+    const int c = (int)(i - t * per_row) * VEC;
+    const size_t from = (size_t)(rows != nullptr ? rows[t] : (int)t) * hidden + c;
+    float v[VEC];
+    if constexpr (VEC == 4) {
+      const float4 r = *reinterpret_cast<const float4*>(residual + from);
+      v[0] = r.x, v[1] = r.y, v[2] = r.z, v[3] = r.w;
+    } else {
+      v[0] = residual[from];
+    }
+    if (a != nullptr || b != nullptr) {
+      float joined[VEC];
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) joined[j] = 0.0f;
+      for (int side = 0; side < 2; ++side) {
+        const T* d = side == 0 ? a : b;
+        if (d == nullptr) continue;
+        __align__(16) T piece[VEC];
+        if constexpr (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(piece) = *reinterpret_cast<const uint2*>(d + from);
+        else if constexpr (VEC == 4) *reinterpret_cast<float4*>(piece) = *reinterpret_cast<const float4*>(d + from);
+        else piece[0] = d[from];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) joined[j] += to_float(piece[j]);
+      }
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] += joined[j];
+      if constexpr (VEC == 4)
+        *reinterpret_cast<float4*>(residual + from) = make_float4(v[0], v[1], v[2], v[3]);
+      else
+        residual[from] = v[0];
+    }
+    if (out != nullptr) {
+      __align__(16) T y[VEC];
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) y[j] = from_float<T>(tanhf(alpha * v[j]) * __ldg(weight + c + j) + __ldg(bias + c + j));
+      T* dst = out + t * hidden + c;
+      if constexpr (VEC == 4 && sizeof(T) == 2) {
+        *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(y);
+      } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) dst[j] = y[j];
+      }
+    }
+  }
+}
+
 }  // namespace tlie
 
 using namespace tlie;
@@ -341,6 +396,29 @@ TLIE_EXPORT int tlie_add_rmsnorm(int dtype, float* residual, const void* delta, 
     add_rmsnorm_kernel<__nv_bfloat16><<<out_rows, block, 0, stream>>>(residual, (const __nv_bfloat16*)delta, rows,
                                                                       weight, eps, (__nv_bfloat16*)out, hidden);
   return (int)cudaGetLastError();
+}
+
+// y (or null: the stream is only completed) = tanh(alpha r) * weight + bias element by element, for the stream r after a and b (each may be null) have joined
+// it: what stands in the place of a norm in a layer that has no statistics.  ``rows`` (then a and b null): only these rows of the stream.
+TLIE_EXPORT int tlie_dynamic_tanh(int dtype, float* residual, const void* a, const void* b, const int* rows, const float* weight, const float* bias, float alpha,
+                                  void* out, int out_rows, int hidden, cudaStream_t stream) {
+  if (out_rows <= 0 || hidden <= 0) return 0;
+  if (rows != nullptr && (a != nullptr || b != nullptr)) return (int)cudaErrorInvalidValue;
+  const size_t total = (size_t)out_rows * hidden;
+  const size_t most = (size_t)device_sm_count() * 16;
+#define TLIE_TANH(T, VEC)                                                                                                                                       \
+  do {                                                                                                                                                         \
+    const size_t pieces = total / VEC, blocks = (pieces + 255) / 256;                                                                                          \
+    return (int)launch_pdl(dynamic_tanh_kernel<T, VEC>, dim3((unsigned)(blocks < most ? blocks : most)), dim3(256), 0, stream, residual, (const T*)a, (const T*)b, rows, \
+                           weight, bias, alpha, (T*)out, hidden, pieces);                                                                                      \
+  } while (0)
+  if (hidden % 4 == 0) {
+    if (dtype == TLIE_F32) TLIE_TANH(float, 4);
+    TLIE_TANH(__nv_bfloat16, 4);
+  }
+  if (dtype == TLIE_F32) TLIE_TANH(float, 1);
+  TLIE_TANH(__nv_bfloat16, 1);
+#undef TLIE_TANH
 }
 
 TLIE_EXPORT int tlie_add(int dtype, float* residual, const void* delta, long long count, cudaStream_t stream) {

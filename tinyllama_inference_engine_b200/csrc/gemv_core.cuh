@@ -28,6 +28,11 @@ struct GemvArgs {
   const float* prepare_weight;   // [N], or nullptr
   __nv_bfloat16* prepare_x;      // [M, N]
   float* prepare_squares;        // [M, tiles of 16 columns]
+  // prepare_curve 1: what is stored is bfloat16(tanh(prepare_alpha r) * prepare_weight + prepare_bias), the next layer's input as it is (a curve per
+  // element needs no sums of squares)
+  int prepare_curve;
+  float prepare_alpha;
+  const float* prepare_bias;     // [N]
   // X_PREPARED: x is such a bfloat16 [M, K]; squares [M, square_tiles] are summed into the row's scale with eps
   const float* squares;
   int square_tiles;
@@ -132,7 +137,7 @@ template <int MT, int XMODE, int EPI, int WARPS = kGemvWarps>
 // prior, prior_weight (ACCUM): the residual element this thread will add to and the next norm's weight for its column, asked for
 // before the k loop (gemv_epilogue_prefetch) so that the end of the tile does not wait for two trips to L2.
 __device__ __forceinline__ void gemv_reduce_store(const GemvArgs& a, const float (&acc)[MT][4], float* red, const float* row_scale, int n0, float prior = 0.0f,
-                                                  float prior_weight = 0.0f) {
+                                                  float prior_weight = 0.0f, float prior_bias = 0.0f) {
   constexpr int kRedRow = MT * 8 + 1;
   constexpr int kTileRows = (EPI == EPI_GATED) ? 8 : 16;      // outputs of a tile
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -177,7 +182,9 @@ __device__ __forceinline__ void gemv_reduce_store(const GemvArgs& a, const float
         value = prior + sum;
         reinterpret_cast<float*>(a.out)[o] = value;
       }
-      if (a.prepare_weight != nullptr) {   // the same for the whole block
+      if (a.prepare_curve) {   // the same for the whole block
+        if (live) a.prepare_x[o] = __float2bfloat16_rn(tanhf(a.prepare_alpha * value) * prior_weight + prior_bias);
+      } else if (a.prepare_weight != nullptr) {
         if (live) a.prepare_x[o] = __float2bfloat16_rn(value * prior_weight);
         float squares = value * value;     // zero where nothing lives; the 16 columns of a row are 16 neighbouring lanes
 #pragma unroll
@@ -256,13 +263,14 @@ struct GemvPhase {
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) acc[mt][0] = acc[mt][1] = acc[mt][2] = acc[mt][3] = 0.0f;
       // what the end of the tile will add to (the epilogue gives a thread at most one output: the block is at least as wide as the tile)
-      float prior = 0.0f, prior_weight = 0.0f;
+      float prior = 0.0f, prior_weight = 0.0f, prior_bias = 0.0f;
       if (EPI == EPI_ACCUM && threadIdx.x < kTileRows * MT * 8) {
         static_assert(kTileRows * MT * 8 <= WARPS * 32, "one output per thread at most");
         const int m = threadIdx.x / kTileRows, r = threadIdx.x - m * kTileRows;
         if (m < a.M && n0 + r < n_rows) {
           prior = __ldcg(reinterpret_cast<const float*>(a.out) + (size_t)m * n_rows + n0 + r);
           if (a.prepare_weight != nullptr) prior_weight = __ldg(a.prepare_weight + n0 + r);
+          if (a.prepare_curve) prior_bias = __ldg(a.prepare_bias + n0 + r);
         }
       }
 
@@ -307,7 +315,7 @@ struct GemvPhase {
       // old one, and the widest products took half as long again.)
       issued = tile_index + tile_step < tiles;
       if (issued) issue(a, (tile_index + tile_step) * kTileRows, warp);
-      gemv_reduce_store<MT, XMODE, EPI, WARPS>(a, acc, red, row_scale, n0, prior, prior_weight);
+      gemv_reduce_store<MT, XMODE, EPI, WARPS>(a, acc, red, row_scale, n0, prior, prior_weight, prior_bias);
     }
   }
 };

@@ -110,7 +110,7 @@ TLIE_EXPORT void tlie_gemv_set_wide_ctas(int on) { gemv_wide_ctas = on; }
 // norm_weight [K] and eps give the RMSNorm.  x_mode 3: x is bf16(residual * norm weight) [M, K] and `squares`
 // [M, square_tiles] the rows' sums of squares, as an earlier call with epilogue 2 and prepare_* left them.
 // prepare_weight (epilogue 2 only, else null): also store bf16(out * prepare_weight) in prepare_x [M, N] and the rows' sums of
-// squares per 16 columns in prepare_squares [M, ceil(N / 16)].  epilogue 0: bf16 out [M, N]; 1: 32-bit out; 2: out (32-bit [M, N]) += result;
+// squares per 16 columns in prepare_squares [M, ceil(N / 16)]; prepare_curve 1 stores bf16(tanh(prepare_alpha out) * prepare_weight + prepare_bias) instead, and no squares.  epilogue 0: bf16 out [M, N]; 1: 32-bit out; 2: out (32-bit [M, N]) += result;
 // 3: w holds [gate rows | up rows] (N even), out = silu(gate) * up as bf16 [M, N / 2] (gate_kind 2: gelu in its tanh form in the place of silu; gate_kind 1: the halves clamped at gate_limit,
 // min(gate) * sigmoid(gate_alpha * min(gate)) * (clamp(up) + gate_shift)).  activation (epilogue 0 only): 1 the square of
 // relu, 2 gelu in its tanh form, 3 silu, 4 act_a z^2 + z / 2 above zero and act_b (e^z - 1 - z) + z / 2 below, applied to the rounded product before
@@ -119,13 +119,15 @@ TLIE_EXPORT void tlie_gemv_set_wide_ctas(int on) { gemv_wide_ctas = on; }
 TLIE_EXPORT int tlie_gemv_fused(int x_mode, const void* x, int ldx, const int* rows, const float* norm_weight, float eps,
                                 const void* w, void* out, int M, int N, int K, int epilogue, const float* squares, int square_tiles,
                                 const float* prepare_weight, void* prepare_x, float* prepare_squares, int activation, int gate_kind, float gate_limit,
-                                float gate_alpha, float gate_shift, float act_a, float act_b, const float* bias, cudaStream_t stream) {
+                                float gate_alpha, float gate_shift, float act_a, float act_b, const float* bias, int prepare_curve, float prepare_alpha,
+                                const float* prepare_bias, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (gate_kind < 0 || gate_kind > 2 || (gate_kind != 0 && epilogue != EPI_GATED)) return (int)cudaErrorInvalidValue;
   if (activation < 0 || activation > 4 || ((activation != 0 || bias != nullptr) && epilogue != EPI_STORE_BF16)) return (int)cudaErrorInvalidValue;
   if (K <= 0 || K % 8 != 0 || M > 16 || ((x_mode == X_PLAIN || x_mode == X_PREPARED) && ldx % 8 != 0) || (epilogue == EPI_GATED && (N & 1)) ||
       (x_mode == X_PREPARED && (squares == nullptr || square_tiles <= 0)) ||
-      (prepare_weight != nullptr && (epilogue != EPI_ACCUM || prepare_x == nullptr || prepare_squares == nullptr)))
+      (prepare_weight != nullptr && (epilogue != EPI_ACCUM || prepare_x == nullptr || (prepare_curve ? prepare_bias == nullptr : prepare_squares == nullptr))) ||
+      (prepare_curve && prepare_weight == nullptr))
     return (int)cudaErrorInvalidValue;
   GemvArgs a;
   a.x = x;
@@ -144,6 +146,9 @@ TLIE_EXPORT int tlie_gemv_fused(int x_mode, const void* x, int ldx, const int* r
   a.prepare_weight = prepare_weight;
   a.prepare_x = (__nv_bfloat16*)prepare_x;
   a.prepare_squares = prepare_squares;
+  a.prepare_curve = prepare_curve;
+  a.prepare_alpha = prepare_alpha;
+  a.prepare_bias = prepare_bias;
   a.activation = activation;
   a.act_a = act_a;
   a.act_b = act_b;

@@ -4,6 +4,8 @@
 //                 Experts form ``groups`` equal groups of neighbours; a group's score is the sum of its two largest choice scores, or
 //                 (``group_best``) its largest; only experts of the ``keep`` best groups can be chosen.  The ``top`` largest choice scores among them are chosen (ties: the lower index); their
 //                 weights are s / (sum of the chosen s + 1e-20) * route_scale (``normalize`` 0: s * route_scale, the scores as they are).
+//                 ``softmax`` 2: s = z, and the weights are the softmax over the chosen z alone, times route_scale.  ``bias`` (optional): one number per
+//                 expert, added to z.
 //                 ``shared_gate``: the router has one row more, and sigmoid of its product with the token is what the shared branch is
 //                 multiplied by.
 //   moe_gate_up   per (token, chosen expert): act(W_gate x) * (W_up x), straight from the expert's rows (steps of few rows, and the
@@ -15,19 +17,12 @@
 //
 // Expert weights are stacked: gate_up [experts][2 ff][width] (gate rows, then up rows), down [experts][width][ff].
 // Activation codes: 0 silu, 1 gelu in its tanh form, both times the up half; 2 the square of relu, for experts without a gate
-// (gate_up is then [experts][ff][width], the up rows alone).
+// (gate_up is then [experts][ff][width], the up rows alone); 3 the clamped gate: with g = min(gate, limit) and u = clamp(up, -limit, limit),
+// g * sigmoid(alpha * g) * (u + shift).
 #include "common.cuh"
+#include "moe_act.cuh"
 
 namespace tlie {
-
-__device__ __forceinline__ float moe_act(float z, int kind) {
-  if (kind == 2) {
-    const float r = fmaxf(z, 0.0f);
-    return r * r;
-  }
-  if (kind == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-  return z / (1.0f + expf(-z));
-}
 
 // the lane's share of w . x: w a row of T in global memory, x 32-bit numbers in shared memory; 16 bytes at a time where rows allow it
 __device__ __forceinline__ float lane_dot(const float* w, const float* x, int width, int lane, bool vector) {
@@ -252,7 +247,7 @@ __device__ __forceinline__ void route_softmax(float* s, float* choice, const flo
 
 // One warp chooses a token's experts from s [experts] and choice [experts] (shared memory, written before); group_score [groups] is scratch.
 __device__ __forceinline__ void route_select(float* s, float* choice, float* group_score, int* __restrict__ ids, float* __restrict__ weights, int t, int lane,
-                                             int experts, int groups, int keep, int top, float route_scale, int normalize, int group_best) {
+                                             int experts, int groups, int keep, int top, float route_scale, int normalize, int group_best, bool logits) {
   const int per = experts / groups;
   if (groups > 1 && keep < groups) {
     for (int g = lane; g < groups; g += 32) {
@@ -309,6 +304,15 @@ __device__ __forceinline__ void route_select(float* s, float* choice, float* gro
     total += s[e];
     __syncwarp();
   }
+  if (logits) {   // s holds logits: the weights are the softmax over the chosen ones
+    float highest = -INFINITY, sum = 0.0f;
+    for (int k = lane; k < top; k += 32) highest = fmaxf(highest, weights[(size_t)t * top + k]);
+    highest = warp_max(highest);
+    for (int k = lane; k < top; k += 32) sum += expf(weights[(size_t)t * top + k] - highest);
+    sum = warp_sum(sum);
+    for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] = expf(weights[(size_t)t * top + k] - highest) / sum * route_scale;
+    return;
+  }
   const float factor = normalize ? route_scale / (total + 1e-20f) : route_scale;   // not normalised: the scores as they are
   for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] *= factor;
 }
@@ -318,7 +322,7 @@ template <typename T>
 __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router, const float* __restrict__ correction,
                                                                      int* __restrict__ ids, float* __restrict__ weights, int tokens, int width, int experts,
                                                                      int groups, int keep, int top, float route_scale, int normalize, int softmax, int group_best,
-                                                                     float* __restrict__ shared_gate) {
+                                                                     float* __restrict__ shared_gate, const float* __restrict__ bias) {
   extern __shared__ float route_smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kRouteWarps + warp;
@@ -334,18 +338,19 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(const T* __
     for (int d = lane; d < width; d += 32) sum = fmaf(w[d], to_float(row[d]), sum);
     sum = warp_sum(sum);
     if (lane == 0) {
+      if (bias != nullptr && e < experts) sum += bias[e];
       const float score = 1.0f / (1.0f + expf(-sum));
       if (e == experts) {
         shared_gate[t] = score;
       } else {
         s[e] = softmax ? sum : score;
-        choice[e] = score + (correction != nullptr ? correction[e] : 0.0f);
+        choice[e] = (softmax == 2 ? sum : score) + (correction != nullptr ? correction[e] : 0.0f);
       }
     }
   }
   __syncwarp();
-  if (softmax) route_softmax(s, choice, correction, lane, experts);
-  route_select(s, choice, group_score, ids, weights, t, lane, experts, groups, keep, top, route_scale, normalize, group_best);
+  if (softmax == 1) route_softmax(s, choice, correction, lane, experts);
+  route_select(s, choice, group_score, ids, weights, t, lane, experts, groups, keep, top, route_scale, normalize, group_best, softmax == 2);
 }
 
 constexpr int kRouteTiledWarps = 8;    // steps of many tokens (four share a CTA); a CTA of one token has 32 warps
@@ -360,7 +365,7 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_tiled_kernel(const T* __
                                                                                 const float* __restrict__ correction, int* __restrict__ ids,
                                                                                 float* __restrict__ weights, int tokens, int width, int experts, int groups, int keep,
                                                                                 int top, float route_scale, int normalize, int softmax, int group_best,
-                                                                                float* __restrict__ shared_gate) {
+                                                                                float* __restrict__ shared_gate, const float* __restrict__ bias) {
   extern __shared__ __align__(16) float route_smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t0 = blockIdx.x * TOK;
@@ -420,16 +425,17 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_tiled_kernel(const T* __
       const int e = j == 0 ? e0 : e1;
       if (e >= router_rows) break;
       const float shift = (correction != nullptr && e < experts) ? correction[e] : 0.0f;
+      const float offset = (bias != nullptr && e < experts) ? bias[e] : 0.0f;
 #pragma unroll
       for (int i = 0; i < TOK; ++i) {
-        const float z = warp_sum(sum[j][i]);
+        const float z = warp_sum(sum[j][i]) + offset;
         if (lane == 0) {
           const float score = 1.0f / (1.0f + expf(-z));
           if (e == experts) {
             if (t0 + i < tokens) shared_gate[t0 + i] = score;
           } else {
             tables[(size_t)i * per_token + e] = softmax ? z : score;
-            tables[(size_t)i * per_token + experts + e] = score + shift;
+            tables[(size_t)i * per_token + experts + e] = (softmax == 2 ? z : score) + shift;
           }
         }
       }
@@ -439,8 +445,8 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_tiled_kernel(const T* __
   for (int i = warp; i < TOK; i += WARPS) {
     if (t0 + i >= tokens) break;
     float* s = tables + (size_t)i * per_token;
-    if (softmax) route_softmax(s, s + experts, correction, lane, experts);
-    route_select(s, s + experts, s + 2 * experts, ids, weights, t0 + i, lane, experts, groups, keep, top, route_scale, normalize, group_best);
+    if (softmax == 1) route_softmax(s, s + experts, correction, lane, experts);
+    route_select(s, s + experts, s + 2 * experts, ids, weights, t0 + i, lane, experts, groups, keep, top, route_scale, normalize, group_best, softmax == 2);
   }
 }
 
@@ -451,7 +457,7 @@ constexpr int kDownOutputs = 32;
 // grid (tokens * top, ceil(ff / (GATED ? 32 : 64))); act [tokens * top][ff].  GATED false: experts of one up matrix, act(W_up x).
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(kMoeWarps * 32) moe_gate_up_kernel(const T* __restrict__ x, const T* __restrict__ gate_up, const int* __restrict__ ids,
-                                                                     const float* __restrict__ input_weights, T* __restrict__ act, int width, int ff, int top, int kind) {
+                                                                     const float* __restrict__ input_weights, T* __restrict__ act, int width, int ff, int top, ExpertGate gate) {
   extern __shared__ __align__(16) float moe_x[];
   const int slot = blockIdx.x, t = slot / top;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -484,7 +490,7 @@ __global__ void __launch_bounds__(kMoeWarps * 32) moe_gate_up_kernel(const T* __
   for (int j = 0; j < kPerWarp; ++j) {
     const float g = warp_sum(sums[GATED ? 2 * j : j]);
     const float u = GATED ? warp_sum(sums[2 * j + 1]) : 1.0f;
-    if (lane == 0 && f[j] < ff) act[(size_t)slot * ff + f[j]] = from_float<T>(moe_act(g, kind) * u);
+    if (lane == 0 && f[j] < ff) act[(size_t)slot * ff + f[j]] = from_float<T>(GATED ? gate(g, u) : gate.ungated(g));
   }
 }
 
@@ -546,8 +552,9 @@ using namespace tlie;
 
 TLIE_EXPORT int tlie_moe_route(int dtype, const void* x, const float* router, const float* correction, int* ids, float* weights, int tokens, int width, int experts,
                                int groups, int keep, int top, float route_scale, int normalize, int softmax, int group_best, float* shared_gate,
-                               cudaStream_t stream) {
+                               const float* bias, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (softmax < 0 || softmax > 2 || (softmax == 2 && !normalize)) return (int)cudaErrorInvalidValue;
   if (experts <= 0 || groups <= 0 || experts % groups != 0 || keep <= 0 || keep > groups || top <= 0 || top > keep * (experts / groups))
     return (int)cudaErrorInvalidValue;
   const size_t tables = (size_t)(2 * experts + groups) * sizeof(float);
@@ -563,7 +570,7 @@ TLIE_EXPORT int tlie_moe_route(int dtype, const void* x, const float* router, co
     if (tiled > 48 * 1024) e = cudaFuncSetAttribute(moe_route_tiled_kernel<T, TOK, (TOK == 1 ? 32 : kRouteTiledWarps)>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tiled);             \
     if (e == cudaSuccess)                                                                                                                                 \
       moe_route_tiled_kernel<T, TOK, (TOK == 1 ? 32 : kRouteTiledWarps)><<<blocks, (TOK == 1 ? 32 : kRouteTiledWarps) * 32, tiled, stream>>>((const T*)x, router, correction, ids, weights, tokens, width, experts, groups, keep, \
-                                                                                     top, route_scale, normalize, softmax, group_best, shared_gate);                \
+                                                                                     top, route_scale, normalize, softmax, group_best, shared_gate, bias);                \
   } while (0)
       if (dtype == TLIE_F32) {
         if (tok == 4) TLIE_ROUTE_TILED(float, 4); else TLIE_ROUTE_TILED(float, 1);
@@ -578,16 +585,16 @@ TLIE_EXPORT int tlie_moe_route(int dtype, const void* x, const float* router, co
   if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
   const int blocks = (tokens + kRouteWarps - 1) / kRouteWarps;
   if (dtype == TLIE_F32)
-    moe_route_kernel<float><<<blocks, kRouteWarps * 32, smem, stream>>>((const float*)x, router, correction, ids, weights, tokens, width, experts, groups, keep, top, route_scale, normalize, softmax, group_best, shared_gate);
+    moe_route_kernel<float><<<blocks, kRouteWarps * 32, smem, stream>>>((const float*)x, router, correction, ids, weights, tokens, width, experts, groups, keep, top, route_scale, normalize, softmax, group_best, shared_gate, bias);
   else
     moe_route_kernel<__nv_bfloat16><<<blocks, kRouteWarps * 32, smem, stream>>>((const __nv_bfloat16*)x, router, correction, ids, weights, tokens, width, experts, groups,
-                                                                              keep, top, route_scale, normalize, softmax, group_best, shared_gate);
+                                                                              keep, top, route_scale, normalize, softmax, group_best, shared_gate, bias);
   return (int)cudaGetLastError();
 }
 
 template <typename T, bool GATED>
-static int launch_moe_first(const void* x, const void* gate_up, const int* ids, const float* input_weights, void* act, int tokens, int width, int ff, int top, int kind,
-                            cudaStream_t stream) {
+static int launch_moe_first(const void* x, const void* gate_up, const int* ids, const float* input_weights, void* act, int tokens, int width, int ff, int top,
+                            const ExpertGate& gate, cudaStream_t stream) {
   const size_t x_smem = (size_t)width * sizeof(float);
   if (x_smem > 200 * 1024) return (int)cudaErrorInvalidValue;
   if (x_smem > 48 * 1024) {
@@ -596,13 +603,13 @@ static int launch_moe_first(const void* x, const void* gate_up, const int* ids, 
   }
   constexpr int kOutputs = GATED ? kGateUpOutputs : 2 * kGateUpOutputs;
   moe_gate_up_kernel<T, GATED><<<dim3(tokens * top, (ff + kOutputs - 1) / kOutputs), kMoeWarps * 32, x_smem, stream>>>((const T*)x, (const T*)gate_up, ids, input_weights,
-                                                                                                                    (T*)act, width, ff, top, kind);
+                                                                                                                    (T*)act, width, ff, top, gate);
   return (int)cudaGetLastError();
 }
 
 template <typename T>
 static int launch_moe_experts(const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, const float* shared_gate, void* act,
-                              void* out, int tokens, int width, int ff, int top, int kind, int weight_input, cudaStream_t stream) {
+                              void* out, int tokens, int width, int ff, int top, const ExpertGate& gate, int weight_input, cudaStream_t stream) {
   const size_t act_smem = (size_t)top * ff * sizeof(float);
   if (act_smem > 200 * 1024) return (int)cudaErrorInvalidValue;
   if (act_smem > 48 * 1024) {
@@ -610,8 +617,8 @@ static int launch_moe_experts(const void* x, const void* gate_up, const void* do
     if (e != cudaSuccess) return (int)e;
   }
   const float* input_weights = weight_input ? weights : nullptr;
-  const int rc = kind == 2 ? launch_moe_first<T, false>(x, gate_up, ids, input_weights, act, tokens, width, ff, top, kind, stream)
-                           : launch_moe_first<T, true>(x, gate_up, ids, input_weights, act, tokens, width, ff, top, kind, stream);
+  const int rc = gate.kind == 2 ? launch_moe_first<T, false>(x, gate_up, ids, input_weights, act, tokens, width, ff, top, gate, stream)
+                                : launch_moe_first<T, true>(x, gate_up, ids, input_weights, act, tokens, width, ff, top, gate, stream);
   if (rc != 0) return rc;
   moe_down_kernel<T><<<dim3(tokens, (width + kDownOutputs - 1) / kDownOutputs), kMoeWarps * 32, act_smem, stream>>>(
       (const T*)act, (const T*)down, ids, weight_input ? nullptr : weights, (const T*)shared, shared_gate, (T*)out, width, ff, top);
@@ -620,12 +627,14 @@ static int launch_moe_experts(const void* x, const void* gate_up, const void* do
 
 // ``act``: scratch [tokens * top, ff] of ``dtype``; ``shared`` [tokens, width] or null, times ``shared_gate`` [tokens] (32-bit) unless that is null; ``out`` [tokens, width].
 // ``weight_input`` 1: a chosen expert reads the token times its weight and its output is added as it is (out[t] = sum_k expert_k(weight_k x[t])); 0: the weight
-// multiplies the expert's output.  ``kind`` 2: experts without a gate.
+// multiplies the expert's output.  ``kind`` 2: experts without a gate.  ``limit``, ``alpha``, ``shift``: kind 3 only.
 TLIE_EXPORT int tlie_moe_experts(int dtype, const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared,
-                                 const float* shared_gate, void* act, void* out, int tokens, int width, int ff, int top, int kind, int weight_input, cudaStream_t stream) {
+                                 const float* shared_gate, void* act, void* out, int tokens, int width, int ff, int top, int kind, int weight_input, float limit, float alpha,
+                                 float shift, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if ((long long)tokens * top > 2147483647LL / 2 || kind < 0 || kind > 2) return (int)cudaErrorInvalidValue;
+  const ExpertGate gate{kind, limit, alpha, shift};
+  if ((long long)tokens * top > 2147483647LL / 2 || kind < 0 || kind > 3) return (int)cudaErrorInvalidValue;
   if (dtype == TLIE_F32)
-    return launch_moe_experts<float>(x, gate_up, down, ids, weights, shared, shared_gate, act, out, tokens, width, ff, top, kind, weight_input, stream);
-  return launch_moe_experts<__nv_bfloat16>(x, gate_up, down, ids, weights, shared, shared_gate, act, out, tokens, width, ff, top, kind, weight_input, stream);
+    return launch_moe_experts<float>(x, gate_up, down, ids, weights, shared, shared_gate, act, out, tokens, width, ff, top, gate, weight_input, stream);
+  return launch_moe_experts<__nv_bfloat16>(x, gate_up, down, ids, weights, shared, shared_gate, act, out, tokens, width, ff, top, gate, weight_input, stream);
 }

@@ -16,21 +16,13 @@
 //                sum does not depend on what else is in the step.
 #include "common.cuh"
 #include "mma_utils.cuh"
+#include "moe_act.cuh"
 
 namespace tlie {
 
 constexpr int kGM = 64, kGN = 64, kGK = 32;
 constexpr int kGRow = kGK + 8;   // padded shared-memory rows (elements)
 constexpr int kGThreads = 128;
-
-__device__ __forceinline__ float grouped_act(float z, int kind) {
-  if (kind == 2) {
-    const float r = fmaxf(z, 0.0f);
-    return r * r;
-  }
-  if (kind == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-  return z / (1.0f + expf(-z));
-}
 
 // meta: [0] number of tiles, then (expert, first sorted row, rows) per tile
 __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ ids, int slots, int experts, int* __restrict__ sorted_slots, int* __restrict__ meta) {
@@ -66,7 +58,7 @@ enum { GROUPED_DOWN = 0, GROUPED_GATED = 1, GROUPED_PLAIN = 2 };
 template <int MODE>
 __global__ void __launch_bounds__(kGThreads) moe_grouped_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __restrict__ w, const int* __restrict__ sorted_slots,
                                                                 const int* __restrict__ meta, const float* __restrict__ weights, void* __restrict__ out, int N, int K,
-                                                                int top, int kind, int weight_input) {
+                                                                int top, ExpertGate gate, int weight_input) {
   constexpr bool FIRST = MODE != GROUPED_DOWN;   // the rows are the tokens' own, gathered
   constexpr int kB = MODE == GROUPED_GATED ? 2 : 1;
   __shared__ __align__(16) __nv_bfloat16 a_s[2][kGM][kGRow];
@@ -141,7 +133,7 @@ __global__ void __launch_bounds__(kGThreads) moe_grouped_kernel(const __nv_bfloa
         for (int c = 0; c < 2; ++c) {
           const int n = n0 + j * 8 + 2 * t + c;
           const float up = MODE == GROUPED_GATED ? scale * acc[kB - 1][j][r * 2 + c] : 1.0f;
-          if (n < N) dst[n] = __float2bfloat16_rn(grouped_act(scale * acc[0][j][r * 2 + c], kind) * up);
+          if (n < N) dst[n] = __float2bfloat16_rn(gate(scale * acc[0][j][r * 2 + c], up));
         }
     } else {
       const int slot = row_slot[row];
@@ -178,21 +170,22 @@ using namespace tlie;
 // y 32-bit [tokens * top, width].  ``shared`` bfloat16 [tokens, width] or null, times ``shared_gate`` [tokens] unless that is null.
 TLIE_EXPORT int tlie_moe_grouped(const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, const float* shared_gate, int* sorted_slots,
                                  int* meta, void* act, float* y, void* out, int tokens, int width, int ff, int experts, int top, int kind, int weight_input,
-                                 cudaStream_t stream) {
+                                 float limit, float alpha, float shift, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   const long long slots = (long long)tokens * top;
-  if (width % 8 != 0 || ff % 8 != 0 || experts <= 0 || experts > 4096 || slots > (1LL << 30) || kind < 0 || kind > 2) return (int)cudaErrorInvalidValue;
+  if (width % 8 != 0 || ff % 8 != 0 || experts <= 0 || experts > 4096 || slots > (1LL << 30) || kind < 0 || kind > 3) return (int)cudaErrorInvalidValue;
+  const ExpertGate gate{kind, limit, alpha, shift};
   const int max_tiles = (int)(slots / kGM) + experts;
   moe_sort_kernel<<<1, 1024, 2 * experts * sizeof(int), stream>>>(ids, (int)slots, experts, sorted_slots, meta);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   auto first = kind == 2 ? moe_grouped_kernel<GROUPED_PLAIN> : moe_grouped_kernel<GROUPED_GATED>;
   first<<<dim3(max_tiles, (ff + kGN - 1) / kGN), kGThreads, 0, stream>>>((const __nv_bfloat16*)x, (const __nv_bfloat16*)gate_up, sorted_slots, meta, weights, act, ff, width,
-                                                                         top, kind, weight_input);
+                                                                         top, gate, weight_input);
   e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   moe_grouped_kernel<GROUPED_DOWN><<<dim3(max_tiles, (width + kGN - 1) / kGN), kGThreads, 0, stream>>>((const __nv_bfloat16*)act, (const __nv_bfloat16*)down, sorted_slots, meta,
-                                                                                                weights, y, width, ff, top, kind, weight_input);
+                                                                                                weights, y, width, ff, top, gate, weight_input);
   e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   const size_t total = (size_t)tokens * width;

@@ -18,6 +18,7 @@
 // tensor memory and the bounded waits are those of gemm_tcgen05.cu.  Tiles are walked with the row tile fastest: the CTAs that
 // run together then work on few column blocks of every expert, whose weights come from memory once and from L2 for the
 // expert's other row tiles, while the gathered rows stay in L2 from one column block to the next.
+#include "moe_act.cuh"
 #include "tcgen05_utils.cuh"
 
 namespace tlie {
@@ -31,16 +32,6 @@ constexpr int kTcStoreBytes = kStoreWarps * kTcStoreBuffers * kTcBoxBytes;
 constexpr int kTcSmemBytes = kTcStages * kTcStageBytes + kTcStoreBytes + 1024 + 256;
 constexpr int kTcTmemCols = 512;            // two accumulators of 256 columns
 static_assert(kTcSmemBytes <= 227 * 1024, "shared memory of one CTA");
-
-template <int ACT>
-__device__ __forceinline__ float tc_act(float z) {
-  if (ACT == 2) {
-    const float r = fmaxf(z, 0.0f);
-    return r * r;
-  }
-  if (ACT == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-  return z / (1.0f + expf(-z));
-}
 
 // meta: [0] number of 128-row tiles, [1 + i] the expert of tile i.  row_of_slot [slots]; token_of_row [max_rows] holds the row's slot (token * top + k).
 __global__ void __launch_bounds__(1024) moe_layout_kernel(const int* __restrict__ ids, int slots, int experts, int top, int max_rows, int* __restrict__ row_of_slot,
@@ -99,7 +90,8 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const __nv_bfloat16* __
 // One warp's 32 rows of a gated tile: act(gate) * up of 32 columns at a time (GATED false: act of a plain tile's columns) as bfloat16 into
 // a staging box, written by a bulk tensor store (columns past N are clipped by the tensor map).
 template <int ACT, bool GATED>
-__device__ __forceinline__ void tc_store_activated(uint32_t tmem_acc, int row0, int n0, int N, const CUtensorMap* map_out, uint8_t* staging, int lane, int& boxes) {
+__device__ __forceinline__ void tc_store_activated(uint32_t tmem_acc, int row0, int n0, int N, const CUtensorMap* map_out, uint8_t* staging, int lane, int& boxes,
+                                                   const ExpertGate& params) {
   const int swizzle = (lane >> 1) & 3;   // 64-byte swizzle: 16-byte chunk j of row r lies at chunk j ^ ((r / 2) % 4)
 #pragma unroll 1
   for (int c = 0; c < (GATED ? kTcBN / 2 : kTcBN) / kStoreCols && n0 + c * kStoreCols < N; ++c) {
@@ -108,9 +100,13 @@ __device__ __forceinline__ void tc_store_activated(uint32_t tmem_acc, int row0, 
     if (GATED) tmem_load_32(tmem_acc + kTcBN / 2 + c * kStoreCols, up);
     asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
 #pragma unroll
-    for (int i = 0; i < kStoreCols / 2; ++i)
-      packed[i] = GATED ? pack_bf16(tc_act<ACT>(__uint_as_float(gate[2 * i])) * __uint_as_float(up[2 * i]), tc_act<ACT>(__uint_as_float(gate[2 * i + 1])) * __uint_as_float(up[2 * i + 1]))
-                        : pack_bf16(tc_act<ACT>(__uint_as_float(gate[2 * i])), tc_act<ACT>(__uint_as_float(gate[2 * i + 1])));
+    for (int i = 0; i < kStoreCols / 2; ++i) {
+      float v[2];
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+        v[j] = expert_gate<ACT>(__uint_as_float(gate[2 * i + j]), GATED ? __uint_as_float(up[2 * i + j]) : 1.0f, params.limit, params.alpha, params.shift);
+      packed[i] = pack_bf16(v[0], v[1]);
+    }
     uint8_t* box = staging + (boxes % kTcStoreBuffers) * kTcBoxBytes;
     ++boxes;
     if (lane == 0) bulk_wait_read<kTcStoreBuffers - 1>();   // the store that last read this box is done with it
@@ -161,7 +157,7 @@ enum { TC_DOWN = 0, TC_GATED = 1, TC_PLAIN = 2 };
 template <int MODE, int ACT>
 __global__ void __launch_bounds__(kGemmThreads)
     moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const __grid_constant__ CUtensorMap map_out,
-                  const int* __restrict__ meta, int N, int K, int* __restrict__ error_flag) {
+                  const int* __restrict__ meta, int N, int K, const ExpertGate params, int* __restrict__ error_flag) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* tiles = reinterpret_cast<uint8_t*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);   // swizzled tiles need 1024-byte alignment
   uint8_t* staging = tiles + kTcStages * kTcStageBytes;
@@ -266,7 +262,7 @@ __global__ void __launch_bounds__(kGemmThreads)
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
       const uint32_t tmem_acc = tmem_base + acc * kTcBN + ((uint32_t)(sub * 32) << 16);
       if (MODE != TC_DOWN)
-        tc_store_activated<ACT, GATED>(tmem_acc, m0 + sub * 32, n0, N, &map_out, my_staging, lane, boxes);
+        tc_store_activated<ACT, GATED>(tmem_acc, m0 + sub * 32, n0, N, &map_out, my_staging, lane, boxes, params);
       else
         tc_store_f32(tmem_acc, m0 + sub * 32, n0, N, &map_out, my_staging, lane, boxes);
       asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -319,7 +315,8 @@ __global__ void __launch_bounds__(256) moe_tc_combine_kernel(const float* __rest
 }
 
 template <int MODE, int ACT>
-static int launch_moe_tc(const void* a, const void* b, void* out, const int* meta, int max_rows, int b_rows, int N, int K, int* error_flag, cudaStream_t stream) {
+static int launch_moe_tc(const void* a, const void* b, void* out, const int* meta, int max_rows, int b_rows, int N, int K, const ExpertGate& params, int* error_flag,
+                         cudaStream_t stream) {
   constexpr bool GATED = MODE == TC_GATED;
   CUtensorMap map_a, map_b, map_out;
   if (!make_map(&map_a, a, max_rows, K, kBM) || !make_map(&map_b, b, b_rows, K, GATED ? kTcBN / 2 : kTcBN)) return (int)cudaErrorInvalidValue;
@@ -334,7 +331,7 @@ static int launch_moe_tc(const void* a, const void* b, void* out, const int* met
   const long long most = (long long)(max_rows / kBM) * ((N + kTileN - 1) / kTileN);
   const int sm_count = device_sm_count();
   return (int)launch_pdl(moe_tc_kernel<MODE, ACT>, dim3((unsigned)(most < sm_count ? most : sm_count)), dim3(kGemmThreads), kTcSmemBytes, stream, map_a, map_b, map_out,
-                         meta, N, K, error_flag);
+                         meta, N, K, params, error_flag);
 }
 
 }  // namespace tlie
@@ -346,11 +343,12 @@ using namespace tlie;
 // ``shared`` bfloat16 [tokens, width] or null, times ``shared_gate`` [tokens] unless that is null.  All of 16-byte aligned bases; width and ff multiples of 8.
 TLIE_EXPORT int tlie_moe_grouped_tc(const void* x, const void* gate_up, const void* down, const int* ids, const float* weights, const void* shared, const float* shared_gate, int* row_of_slot,
                                     int* token_of_row, int* meta, void* xs, void* act, float* y, void* out, int tokens, int width, int ff, int experts, int top,
-                                    int kind, int weight_input, int* error_flag, cudaStream_t stream) {
+                                    int kind, int weight_input, float limit, float alpha, float shift, int* error_flag, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   const long long slots = (long long)tokens * top;
-  if (width % 8 != 0 || ff % 8 != 0 || experts <= 0 || experts > 4096 || slots > (1LL << 30) || kind < 0 || kind > 2 || error_flag == nullptr) return (int)cudaErrorInvalidValue;
+  if (width % 8 != 0 || ff % 8 != 0 || experts <= 0 || experts > 4096 || slots > (1LL << 30) || kind < 0 || kind > 3 || error_flag == nullptr) return (int)cudaErrorInvalidValue;
   if ((long long)experts * 2 * ff > 2147483647LL || (long long)experts * width > 2147483647LL) return (int)cudaErrorInvalidValue;
+  const ExpertGate params{kind, limit, alpha, shift};
   const int max_rows = ((int)(slots / kBM) + experts) * kBM;
   moe_layout_kernel<<<1, 1024, 2 * experts * sizeof(int), stream>>>(ids, (int)slots, experts, top, max_rows, row_of_slot, token_of_row, meta);
   cudaError_t e = cudaGetLastError();
@@ -358,11 +356,12 @@ TLIE_EXPORT int tlie_moe_grouped_tc(const void* x, const void* gate_up, const vo
   moe_gather_kernel<<<max_rows / 8, 256, 0, stream>>>((const __nv_bfloat16*)x, token_of_row, meta, weight_input ? weights : nullptr, (__nv_bfloat16*)xs, width, top);
   e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
-  int rc = kind == 2   ? launch_moe_tc<TC_PLAIN, 2>(xs, gate_up, act, meta, max_rows, experts * ff, ff, width, error_flag, stream)
-           : kind == 1 ? launch_moe_tc<TC_GATED, 1>(xs, gate_up, act, meta, max_rows, experts * 2 * ff, ff, width, error_flag, stream)
-                       : launch_moe_tc<TC_GATED, 0>(xs, gate_up, act, meta, max_rows, experts * 2 * ff, ff, width, error_flag, stream);
+  int rc = kind == 2   ? launch_moe_tc<TC_PLAIN, 2>(xs, gate_up, act, meta, max_rows, experts * ff, ff, width, params, error_flag, stream)
+           : kind == 3 ? launch_moe_tc<TC_GATED, 3>(xs, gate_up, act, meta, max_rows, experts * 2 * ff, ff, width, params, error_flag, stream)
+           : kind == 1 ? launch_moe_tc<TC_GATED, 1>(xs, gate_up, act, meta, max_rows, experts * 2 * ff, ff, width, params, error_flag, stream)
+                       : launch_moe_tc<TC_GATED, 0>(xs, gate_up, act, meta, max_rows, experts * 2 * ff, ff, width, params, error_flag, stream);
   if (rc != 0) return rc;
-  rc = launch_moe_tc<TC_DOWN, 0>(act, down, y, meta, max_rows, experts * width, width, ff, error_flag, stream);
+  rc = launch_moe_tc<TC_DOWN, 0>(act, down, y, meta, max_rows, experts * width, width, ff, params, error_flag, stream);
   if (rc != 0) return rc;
   const size_t quads = (size_t)tokens * (width / 4);
   const size_t blocks = (quads + 255) / 256;

@@ -95,6 +95,10 @@ class DecoderModel:
             return None
         from .. import ops
 
+        if isinstance(prepared, ops.FinishedNorm):
+            if prepared.norm is self.final_norm and prepared.finished is not None and want_rows.shape[0] == prepared.shape[0]:
+                return self.head.forward(prepared.finished)
+            prepared = None
         if self.final_norm.supports_lazy and want_rows.shape[0] <= ops.fused_rows_limit(self.runtime.dtype, residual.device):
             if prepared is not None and prepared.weight is self.final_norm.weight and prepared.shape[0] == want_rows.shape[0]:
                 return self.head.forward(prepared)

@@ -196,6 +196,25 @@ def silu_mul(gate_up, out) -> None:
     _check(core().tlie_silu_mul(_code(out), _ptr(gate_up), _ptr(out), c_int(rows), c_int(inter), _stream()), "silu_mul")
 
 
+def dynamic_tanh(residual, a, b, rows, weight, bias, alpha: float, out) -> None:
+    """``residual += a + b`` in 32-bit (each may be None), then ``out = tanh(alpha * residual[rows]) * weight + bias`` element by element, 32-bit inside
+    (``out`` None: the stream is only completed; ``rows`` None: every row in order, and only then may ``a`` or ``b`` be given)."""
+    width = residual.shape[1]
+    count = residual.shape[0] if rows is None else rows.shape[0]
+    if residual.dtype != torch.float32 or weight.dtype != torch.float32 or bias.dtype != torch.float32 or weight.numel() != width or bias.numel() != width:
+        raise KernelError("dynamic_tanh: the stream, the weight and the bias are 32-bit and one width", code="invalid_shape")
+    given = [t for t in (a, b) if t is not None]
+    if any(t.shape != residual.shape for t in given) or (given and rows is not None) or (out is not None and out.shape != (count, width)):
+        raise KernelError("dynamic_tanh: what joins the stream has its shape (and no rows are gathered then), out is [rows, width]", code="invalid_shape")
+    dtypes = {t.dtype for t in given + ([out] if out is not None else [])}
+    if not dtypes:
+        return
+    if len(dtypes) != 1:
+        raise KernelError("dynamic_tanh: what joins the stream and the output share a dtype", code="invalid_dtype")
+    _check(core().tlie_dynamic_tanh(_code(out if out is not None else given[0]), _ptr(residual), _ptr(a), _ptr(b), _i32(rows, "rows"), _ptr(weight), _ptr(bias),
+                                    c_float(alpha), _ptr(out), c_int(count), c_int(width), _stream()), "dynamic_tanh")
+
+
 GATE_KINDS = {"silu": 0, "gelu_tanh": 1}
 
 
@@ -389,6 +408,17 @@ class StreamCopy(LazyNorm):
         self.copy = copy
 
 
+class FinishedNorm(LazyNorm):
+    """A norm of the whole residual stream that needs no statistics and is therefore finished by whoever completes the stream: ``norm`` names the part
+    whose output it is, ``finished`` is that output once somebody has left it there (None until then), ``curve`` = (alpha, weight, bias) of
+    tanh(alpha x) * weight + bias and ``buffer`` are what a completing product needs to do so."""
+
+    def __init__(self, norm, residual, curve, buffer):
+        super().__init__(residual, None, 0.0, None, lambda: self.finished)   # nobody's RMS weight is this one's
+        self.norm, self.curve, self.buffer = norm, curve, buffer
+        self.finished = None
+
+
 def norm_linear(x: "LazyNorm", weight, out, gated: bool = False, clamp=None) -> None:
     """out = rmsnorm(residual) * norm_weight . weight^T in one kernel (``gated``: silu(gate) * up of the two halves; with ``clamp`` =
     (limit, alpha, shift) the clamped gate of ``clamped_gate_mul`` instead)."""
@@ -455,6 +485,13 @@ def linear_accumulate(x, weight, residual, prepare: "LazyNorm | None" = None) ->
     ``prepare``: the lazy norm of this residual (all rows) that the next product will consume; the kernel then leaves that
     norm's input beside the residual (``prepare.prepared``), written by the threads that hold the finished sums."""
     rows = x.shape[0]
+    if isinstance(prepare, FinishedNorm):
+        # the next layer's input in full, where one kernel completes the stream; otherwise it stays unfinished and the block norms the stream itself
+        if prepare.residual is residual and prepare.buffer is not None and fast.gemv_fits(rows, weight.shape[1], norm=False, N=weight.shape[0]):
+            fast.gemv_fused(x, weight, residual, epilogue="accumulate", prepare_curve=(*prepare.curve, prepare.buffer))
+            prepare.finished = prepare.buffer
+            return
+        prepare = None
     preparing = (prepare is not None and prepare.rows is None and prepare.residual is residual and use_prepared_norms
                  and residual.shape[0] >= PREPARED_NORM_MIN_ROWS)
     if fast.gemv_fits(rows, weight.shape[1], norm=False, N=weight.shape[0]):
@@ -705,6 +742,23 @@ def hgrn2_prepare(rows, f_bias, lower, prep, heads: int, dim: int, vdim: int) ->
                                                    c_int(heads), c_int(dim), c_int(vdim), _stream()), "hgrn2_prepare")
 
 
+def gla_prepare(rows, decay_in, a2, bias, tau: float, q_scale: float, prep, heads: int, dim: int, vdim: int) -> None:
+    """What the plain recurrence reads for linear attention with a learned decay per key channel: ``rows`` = [q: H dim | k: H dim | v: H vdim | ...]
+    (products); ``prep[t]`` = [q * q_scale | k | v | 1 | sigmoid(z)^(1 / tau)], all 32-bit, with z = decay_in + bias (``bias`` 32-bit [H dim], ``decay_in``
+    [T, H dim]), or with ``a2`` [H dim, rank] given z = a2 decay_in + bias for ``decay_in`` [T, rank].  ``decay_in`` may be a run of columns of wider rows."""
+    tokens = rows.shape[0]
+    if rows.shape[1] < 2 * heads * dim + heads * vdim or rows.stride(1) != 1 or prep.dtype != torch.float32 or prep.shape != (tokens, 3 * heads * dim + heads * vdim + heads):
+        raise KernelError("gla_prepare: rows [T, >= 2 H dim + H vdim], prep 32-bit [T, 3 H dim + H vdim + H]", code="invalid_shape")
+    rank = heads * dim if a2 is None else a2.shape[1]
+    if decay_in.shape != (tokens, rank) or decay_in.dtype != rows.dtype or decay_in.stride(1) != 1 or not decay_in.is_cuda or bias.dtype != torch.float32 or bias.numel() != heads * dim:
+        raise KernelError("gla_prepare: decay_in [T, H dim] (with a2: [T, rank]) of the rows' dtype, bias 32-bit [H dim]", code="invalid_shape")
+    if a2 is not None and (a2.shape[0] != heads * dim or a2.dtype != rows.dtype):
+        raise KernelError("gla_prepare: a2 [H dim, rank] of the rows' dtype", code="invalid_shape")
+    _check(delta_rule_library().tlie_gla_prepare(_code(rows), c_void_p(rows.data_ptr()), c_int(rows.stride(0)), c_void_p(decay_in.data_ptr()), c_longlong(decay_in.stride(0)),
+                                                 _ptr(a2), c_int(rank), _ptr(bias), c_float(tau), c_float(q_scale), _ptr(prep), c_int(tokens), c_int(heads), c_int(dim),
+                                                 c_int(vdim), _stream()), "gla_prepare")
+
+
 def ssd_prepare(rows, taps, conv_bias, a_log, dt_bias, state, conv_offset: int, ctx, prep, heads: int, groups: int, n: int, vdim: int) -> None:
     """What the plain recurrence reads for a state-space layer: ``rows`` = [z: inner | x: inner | B: G n | C: G n | dt: H] (products, inner = H vdim).
     x, B, C pass a causal convolution per channel (``taps`` 32-bit [inner + 2 G n, taps], ``conv_bias`` or None; the inputs before an entry's first row
@@ -905,13 +959,16 @@ def rotary_store_planes(rows, k_offset: int, v_offset: int, biases, inv_freq, ro
 
 
 def norm_rotary_store(rows, k_offset: int, v_offset: int, biases, q_weight, k_weight, eps: float, q_factors, inv_freq, rot_dims: int, interleaved: bool, amplitude: float,
-                      positions, token_seq, cache, heads: int, kv_heads: int, key_dim: int, value_dim: int) -> None:
+                      positions, token_seq, cache, heads: int, kv_heads: int, key_dim: int, value_dim: int, first_values=None, value_share: float | None = None) -> None:
     """Biases, a norm, a partial rotation and the cache write in one kernel.  Every q, k and v vector of ``rows`` gets its bias (``biases`` =
     (q, k, v), 32-bit or None each, or None); q and k are divided by their root mean square (``eps`` inside the root) and multiplied by
     ``q_weight`` / ``k_weight`` (32-bit [key_dim]; None: no norm); their first ``rot_dims`` columns turn by position * inv_freq[i], cosines and
     sines times ``amplitude``, columns (2i, 2i + 1) together if ``interleaved``, else column i with column i + rot_dims / 2; query head h is
     multiplied by ``q_factors[h]`` (32-bit [heads] or None).  q is left in place, k goes into the key plane and v into the value plane of the
-    token's page."""
+    token's page.  ``first_values`` [T, kv_heads * value_dim] (or None): with ``value_share`` None the values are left there as well; otherwise the stored
+    values are (1 - value_share) v + value_share * first_values (32-bit inside)."""
+    if first_values is not None and (first_values.shape != (rows.shape[0], kv_heads * value_dim) or first_values.dtype != rows.dtype):
+        raise KernelError("norm_rotary_store: the earlier layer's values are [T, kv_heads * value_dim] of the rows' dtype", code="invalid_shape")
     pages, k_ptr, k_stride, v_ptr, v_stride = _plane_pointers(cache, kv_heads, key_dim, value_dim)
     if pages.dtype != rows.dtype or rot_dims % 2 or rot_dims > key_dim or (rot_dims > 0 and (inv_freq is None or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dims // 2)):
         raise KernelError("norm_rotary_store: pages of the rows' dtype; inv_freq 32-bit [rot_dims / 2], rot_dims even and at most key_dim", code="invalid_shape")
@@ -925,7 +982,8 @@ def norm_rotary_store(rows, k_offset: int, v_offset: int, biases, q_weight, k_we
                                                     c_int(1 if interleaved else 0), c_float(amplitude), _i32(positions, "positions"), _i32(token_seq, "token_seq"),
                                                     _i32(table, "block_table"), c_int(table.shape[1]), k_ptr, c_longlong(k_stride), v_ptr, c_longlong(v_stride),
                                                     c_int(rows.shape[0]), c_int(heads), c_int(kv_heads), c_int(key_dim), c_int(value_dim), c_int(cache.page_size),
-                                                    c_int(1 if cache.writes else 0), _stream()), "norm_rotary_store")
+                                                    c_int(1 if cache.writes else 0), _ptr(first_values), c_int(1 if value_share is None else 0),
+                                                    c_float(0.0 if value_share is None else value_share), _stream()), "norm_rotary_store")
 
 
 def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, slopes, mix, out, heads: int, kv_heads: int, key_dim: int, value_dim: int,
@@ -970,25 +1028,25 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
             and fast.latent_prefill_takes(batch, rows, key_dim, value_dim)):
         fast.latent_prefill(rows, batch, table, k_ptr, k_stride, sinks, out, heads, key_dim, value_dim, cache.page_size, scale)
         return
-    plain_options = sinks is None and not values_in_keys   # what the tensor-core kernels with two planes know
-    if (plain_options and sigmoid and slopes is None and mix is None and window == 0 and rows.dtype == torch.bfloat16 and cache.pages is not None and key_dim == value_dim
+    two_planes = not values_in_keys   # what the tensor-core kernels below read
+    if (two_planes and slopes is None and mix is None and window == 0 and rows.dtype == torch.bfloat16 and cache.pages is not None and key_dim == value_dim
             and rows.shape[1] % 8 == 0 and (gate_offset < 0 or gate_per_head) and _tensor_memory_attention(rows, gate_offset, positions, token_seq, cache, out, heads, kv_heads, key_dim,
-                                                                                                           scale, batch, softcap, shifts)):
+                                                                                                           scale, batch, softcap, sigmoid, shifts, sinks)):
         return
-    if plain_options and (sigmoid or softcap == 0.0) and rows.dtype == torch.bfloat16 and fast.mixed_prefill_takes(batch, rows, cache.page_size, kv_heads if mix is not None else 1, key_dim, value_dim, gate_offset,
-                                                                                   gate_per_head, sigmoid):
+    if two_planes and (sigmoid or softcap == 0.0 or slopes is None) and rows.dtype == torch.bfloat16 and fast.mixed_prefill_takes(
+            batch, rows, cache.page_size, kv_heads if mix is not None else 1, key_dim, value_dim, gate_offset, gate_per_head, sigmoid, softcap > 0.0):
         folded = folded_slopes if folded_slopes is not None else fast.folded_slopes(slopes, mix)
         fast.mixed_prefill(rows, gate_offset, batch, table, (k_ptr, k_stride, v_ptr, v_stride), folded, mix, out, heads, kv_heads, key_dim, value_dim,
-                           cache.page_size, window, scale, keep_first if window > 0 else 0, gate_per_head, softcap, sigmoid, shifts)
+                           cache.page_size, window, scale, keep_first if window > 0 else 0, gate_per_head, softcap, sigmoid, shifts, sinks)
         return
     # few rows over long contexts (decode steps): every row's keys are dealt to several CTAs
     splits, partial = 1, None
     if batch is not None and tokens * 2 <= fast.sm_count():
         reach = min(window + keep_first, batch.max_seq_len) if window > 0 else batch.max_seq_len
         splits = max(1, min(2 * fast.sm_count() // tokens, -(-reach // 32), 64))   # down to one tile of 32 keys per CTA
-        if plain_options and fast.mixed_decode_takes(rows, heads, kv_heads, key_dim, value_dim, gate_offset, mix is not None, gate_per_head):
+        if two_planes and fast.mixed_decode_takes(rows, heads, kv_heads, key_dim, value_dim, gate_offset, mix is not None, gate_per_head):
             fast.mixed_decode(rows, gate_offset, positions, token_seq, table, (k_ptr, k_stride, v_ptr, v_stride), slopes, mix, out, heads, kv_heads, key_dim,
-                              value_dim, cache.page_size, window, scale, splits, keep_first if window > 0 else 0, gate_per_head, softcap, sigmoid, shifts)
+                              value_dim, cache.page_size, window, scale, splits, keep_first if window > 0 else 0, gate_per_head, softcap, sigmoid, shifts, sinks)
             return
         if splits > 1:
             partial = fast.mixed_scratch(rows.device, tokens * splits * (heads * value_dim + 2 * heads), torch.float32)
@@ -1001,9 +1059,10 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
            "mixed_heads_attention")
 
 
-def _tensor_memory_attention(rows, gate_offset: int, positions, token_seq, cache, out, heads: int, kv_heads: int, dim: int, scale: float, batch, softcap: float, shifts) -> bool:
-    """Attention with sigmoid weights for a step that carries prompt portions, on the tensor-memory kernel; decoding requests at the step's head
-    run on the kernel of few rows.  False: the step or the sizes are not for it."""
+def _tensor_memory_attention(rows, gate_offset: int, positions, token_seq, cache, out, heads: int, kv_heads: int, dim: int, scale: float, batch, softcap: float,
+                             sigmoid: bool, shifts, sinks) -> bool:
+    """Attention of a step that carries prompt portions on the tensor-memory kernel (sigmoid weights, bounded scores and sinks each in a build that has them);
+    decoding requests at the step's head run on the kernel of few rows.  False: the step or the sizes are not for it."""
     host_q_lens = getattr(batch, "host_q_lens", None)
     if host_q_lens is None:
         return False
@@ -1015,9 +1074,9 @@ def _tensor_memory_attention(rows, gate_offset: int, positions, token_seq, cache
         planes = _plane_pointers(cache, kv_heads, dim, dim)[1:]
         splits = max(1, min(2 * fast.sm_count() // lead, -(-batch.max_seq_len // 32), 64))
         fast.mixed_decode(rows[:lead], gate_offset, positions[:lead], token_seq[:lead], cache.block_table, planes, None, None, out[:lead], heads, kv_heads, dim, dim, cache.page_size, 0,
-                          scale, splits, 0, True, softcap, True, shifts)
-    fast.prefill_attention_tc(rows, cache.pages, tiles, batch.seq_starts, batch.first_positions, cache.block_table, out, heads, kv_heads, dim, cache.page_size, 0, scale, softcap, True,
-                              shifts, gate_offset)
+                          scale, splits, 0, True, softcap, sigmoid, shifts, sinks)
+    fast.prefill_attention_tc(rows, cache.pages, tiles, batch.seq_starts, batch.first_positions, cache.block_table, out, heads, kv_heads, dim, cache.page_size, 0, scale, softcap, sigmoid,
+                              shifts, gate_offset, sinks)
     return True
 
 
@@ -1092,23 +1151,26 @@ def moe_library():
     return load_library("tlie_moe", MOE_SOURCES)
 
 
-ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}
+ROUTER_SCORES = {"sigmoid": 0, "softmax": 1, "logits": 2}
 GROUP_SCORES = {"two_best": 0, "best": 1}
 
 
 def moe_route(x, router, correction, ids, weights, groups: int, keep: int, route_scale: float, normalize: bool = True, scores: str = "sigmoid",
-              group_score: str = "two_best", shared_gate=None) -> None:
+              group_score: str = "two_best", shared_gate=None, bias=None) -> None:
     """Per token of ``x`` [T, width]: s = sigmoid(router x), or with ``scores`` "softmax" softmax(router x) over all experts (``router`` 32-bit
     [experts, width], sums in 32-bit), choice = s + ``correction`` (32-bit [experts] or None).  Experts form ``groups`` equal groups of
     neighbours; a group's score is the sum of its two largest choice scores (``group_score`` "best": its largest) and only experts of the
     ``keep`` best groups can be chosen.  ``ids`` int32 [T, top] receives the experts of the ``top`` largest
     choice scores (the lower index on ties), ``weights`` 32-bit [T, top] their s / (sum of the chosen s + 1e-20) * ``route_scale``
     (``normalize`` False: s * ``route_scale``, the scores as they are).  ``shared_gate`` (32-bit [T]): the router then has one row more, and
-    ``shared_gate`` receives the sigmoid of that row's product with the token."""
+    ``shared_gate`` receives the sigmoid of that row's product with the token.  ``scores`` "logits": s = router x itself, and the weights are the softmax
+    over the chosen ones alone, times ``route_scale``.  ``bias`` (32-bit [experts] or None) is added to the router's products."""
     tokens, width = x.shape
     experts, top = router.shape[0] - (0 if shared_gate is None else 1), ids.shape[1]
     if scores not in ROUTER_SCORES or group_score not in GROUP_SCORES:
         raise KernelError(f"moe_route: no scores {scores!r} or no group score {group_score!r}", code="invalid_argument")
+    if (scores == "logits" and not normalize) or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != experts)):
+        raise KernelError("moe_route: weights over logits are always brought to a sum of one; a bias is 32-bit [experts]", code="invalid_shape")
     if shared_gate is not None and (shared_gate.dtype != torch.float32 or shared_gate.numel() != tokens):
         raise KernelError("moe_route: the shared branch's gate is 32-bit, one number per token", code="invalid_shape")
     if router.dtype != torch.float32 or router.shape[1] != width or ids.dtype != torch.int32 or ids.shape != (tokens, top) or weights.dtype != torch.float32 or weights.shape != (tokens, top):
@@ -1117,20 +1179,22 @@ def moe_route(x, router, correction, ids, weights, groups: int, keep: int, route
         raise KernelError("moe_route: the correction is 32-bit [experts]", code="invalid_shape")
     _check(moe_library().tlie_moe_route(_code(x), _ptr(x), _ptr(router), _ptr(correction), _ptr(ids), _ptr(weights), c_int(tokens), c_int(width), c_int(experts),
                                         c_int(groups), c_int(keep), c_int(top), c_float(route_scale), c_int(1 if normalize else 0), c_int(ROUTER_SCORES[scores]),
-                                        c_int(GROUP_SCORES[group_score]), _ptr(shared_gate), _stream()), "moe_route")
+                                        c_int(GROUP_SCORES[group_score]), _ptr(shared_gate), _ptr(bias), _stream()), "moe_route")
 
 
-EXPERT_KINDS = {**GATE_KINDS, "relu_squared": 2}   # the last: experts without a gate
+EXPERT_KINDS = {**GATE_KINDS, "relu_squared": 2, "clamped_sigmoid": 3}   # "relu_squared": experts without a gate
 
 
-def moe_experts(x, gate_up, down, ids, weights, shared, out, activation: str = "silu", batch=None, weight_input: bool = False, shared_gate=None) -> None:
+def moe_experts(x, gate_up, down, ids, weights, shared, out, activation: str = "silu", batch=None, weight_input: bool = False, shared_gate=None, clamp=None) -> None:
     """out[t] = sum_k weights[t, k] * W_down[e] (act(W_gate[e] x[t]) * (W_up[e] x[t])) for e = ids[t, k], plus ``shared[t]`` if given.
     ``gate_up`` [experts, 2 ff, width] (an expert's gate rows, then its up rows), ``down`` [experts, width, ff].  Steps of few rows and the
     32-bit path read each chosen expert's rows directly; bfloat16 prompt portions sort the (token, expert) pairs by expert and run
     the experts' products on the tensor cores.  ``weight_input``: the weight multiplies what the expert reads instead of what it returns,
     out[t] = sum_k expert_e(weights[t, k] x[t]) (the two differ: the experts are not linear).  ``activation`` "relu_squared": experts without a
     gate, W_down[e] act(W_up[e] x[t]), ``gate_up`` [experts, ff, width] holding the up rows alone.  ``shared_gate`` (32-bit [T]): ``shared[t]`` is
-    multiplied by it."""
+    multiplied by it.  ``activation`` "clamped_sigmoid" with ``clamp`` = (limit, alpha, shift): the halves meet as in ``clamped_gate_mul``."""
+    if (activation == "clamped_sigmoid") != (clamp is not None):
+        raise KernelError("moe_experts: a clamped gate, and only that, has a clamp = (limit, alpha, shift)", code="invalid_argument")
     if activation not in EXPERT_KINDS:
         raise KernelError(f"moe_experts: no activation {activation!r}", code="invalid_argument")
     kind = EXPERT_KINDS[activation]
@@ -1144,11 +1208,12 @@ def moe_experts(x, gate_up, down, ids, weights, shared, out, activation: str = "
     if shared_gate is not None and (shared is None or shared_gate.dtype != torch.float32 or shared_gate.numel() != tokens):
         raise KernelError("moe_experts: the shared branch's gate is 32-bit, one number per token, beside a shared branch", code="invalid_shape")
     if x.dtype == torch.bfloat16 and fast.moe_grouped_takes(tokens, top, width, ff, experts):
-        fast.moe_grouped(x, gate_up, down, ids, weights, shared, out, kind, weight_input, shared_gate)
+        fast.moe_grouped(x, gate_up, down, ids, weights, shared, out, kind, weight_input, shared_gate, clamp)
         return
     act = fast.mixed_scratch(x.device, tokens * top * ff, x.dtype)
     _check(moe_library().tlie_moe_experts(_code(x), _ptr(x), _ptr(gate_up), _ptr(down), _ptr(ids), _ptr(weights), _ptr(shared), _ptr(shared_gate), _ptr(act), _ptr(out),
-                                          c_int(tokens), c_int(width), c_int(ff), c_int(top), c_int(kind), c_int(1 if weight_input else 0), _stream()), "moe_experts")
+                                          c_int(tokens), c_int(width), c_int(ff), c_int(top), c_int(kind), c_int(1 if weight_input else 0),
+                                          *(c_float(float(v)) for v in clamp or (0.0, 0.0, 0.0)), _stream()), "moe_experts")
 
 
 # --- sampling ------------------------------------------------------------------------------

@@ -41,6 +41,7 @@ def build_all() -> list:
     built.append(build_library("tlie_gemm_tcgen05", TCGEN05_SOURCES))
     built.append(build_library("tlie_attn_prefill_tc", ["attention_prefill_tc.cu"]))
     built.append(build_library("tlie_attn_prefill_tc_sigmoid", ["attention_prefill_tc.cu"], {"SIGMOID_WEIGHTS": 1}))
+    built.append(build_library("tlie_attn_prefill_tc_capped", ["attention_prefill_tc.cu"], {"SCORE_CAP": 1}))
     built.append(build_library("tlie_probes", ["probes.cu"]))
     for key_dim, value_dim, parts in DEFAULT_MIXED_PREFILL_SETS:
         built.append(build_library(f"tlie_attn_mixed_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "PARTS": parts}))
@@ -112,7 +113,7 @@ GEMV_GATES = {"silu": 0, "gelu_tanh": 2}   # the gated epilogue's activation (1 
 
 
 def gemv_fused(x, weight, out, *, norm=None, epilogue: str = "store", prepared=None, prepare=None, activation: str | None = None, constants=(0.0, 0.0),
-               clamp=None, gate: str = "silu", bias=None) -> None:
+               clamp=None, gate: str = "silu", bias=None, prepare_curve=None) -> None:
     """out (+)= f(x) . weight^T for up to 16 rows, one kernel.
 
     norm      None: ``x`` is bfloat16 [M, K].  (norm_weight, eps, rows): ``x`` is the 32-bit residual stream and
@@ -128,6 +129,8 @@ def gemv_fused(x, weight, out, *, norm=None, epilogue: str = "store", prepared=N
     bias      ("store" into bfloat16 only) 32-bit [N], added to the sums before they are rounded.
     prepare   ("accumulate" only) (norm_weight [N], x_out bfloat16 [M, N], squares_out [M, ceil(N / 16)]): also store
               bfloat16(out * norm_weight) and the rows' sums of squares per 16 columns, for a later call with ``prepared``.
+    prepare_curve ("accumulate" only, in the place of ``prepare``) (alpha, weight [N], bias [N], x_out bfloat16 [M, N]): also store
+              bfloat16(tanh(alpha * out) * weight + bias), the finished operand of the product after this one.
     """
     ops = _ops()
     N, K = weight.shape
@@ -170,9 +173,17 @@ def gemv_fused(x, weight, out, *, norm=None, epilogue: str = "store", prepared=N
                 or squares_out.dtype != torch.float32 or squares_out.shape != (M, -(-N // 16)) or not x_out.is_contiguous() or not squares_out.is_contiguous()):
             raise KernelError("gemv_fused: prepare takes a 32-bit norm weight [N], bfloat16 [M, N] and 32-bit [M, ceil(N / 16)], with accumulate", code="invalid_shape")
         emit = (ops._ptr(norm_weight), ops._ptr(x_out), ops._ptr(squares_out))
+    curve = (c_int(0), c_float(0.0), c_void_p(0))
+    if prepare_curve is not None:
+        alpha, curve_weight, curve_bias, x_out = prepare_curve
+        if (epilogue != "accumulate" or prepare is not None or curve_weight.dtype != torch.float32 or curve_weight.numel() != N or curve_bias.dtype != torch.float32
+                or curve_bias.numel() != N or x_out.dtype != torch.bfloat16 or x_out.shape != (M, N) or not x_out.is_contiguous()):
+            raise KernelError("gemv_fused: prepare_curve takes a number, 32-bit weight and bias [N] and bfloat16 [M, N], with accumulate", code="invalid_shape")
+        emit = (ops._ptr(curve_weight), ops._ptr(x_out), c_void_p(0))
+        curve = (c_int(1), c_float(alpha), ops._ptr(curve_bias))
     ops._check(gemv_library().tlie_gemv_fused(*args, ops._ptr(weight), ops._ptr(out), c_int(M), c_int(N), c_int(K), c_int(code), *consume, *emit, c_int(GEMV_ACTIVATIONS[activation]),
                                              c_int(GEMV_GATES[gate] if clamp is None else 1), *(c_float(float(v)) for v in (clamp or (0.0, 0.0, 0.0))), *(c_float(float(v)) for v in constants), ops._ptr(bias),
-                                             ops._stream()), "gemv_fused")
+                                             *curve, ops._stream()), "gemv_fused")
 
 
 # --- tensor-core product for 17 to 127 rows (tcgen05 with the operands swapped, K cut over a cluster) -----------------
@@ -654,7 +665,9 @@ TC_ATTENTION_HEAD_DIMS = (64, 128)
 TC_ATTENTION_MIN_ROWS_PER_TILE = 32
 
 
-def tc_attention_library(sigmoid: bool = False):
+def tc_attention_library(sigmoid: bool = False, capped: bool = False):
+    if capped and not sigmoid:
+        return load_library("tlie_attn_prefill_tc_capped", ["attention_prefill_tc.cu"], {"SCORE_CAP": 1})
     if sigmoid:
         return load_library("tlie_attn_prefill_tc_sigmoid", ["attention_prefill_tc.cu"], {"SIGMOID_WEIGHTS": 1})
     return load_library("tlie_attn_prefill_tc", ["attention_prefill_tc.cu"])
@@ -670,21 +683,23 @@ def tc_attention_tiles(batch, head_dim: int, page_size: int, lead: int):
 
 
 def prefill_attention_tc(qkv, pages, tiles, seq_starts, first_positions, block_table, out, q_heads: int, kv_heads: int, head_dim: int, page_size: int,
-                         window: int, scale: float, softcap: float = 0.0, sigmoid: bool = False, shifts=None, gate_offset: int = -1) -> None:
+                         window: int, scale: float, softcap: float = 0.0, sigmoid: bool = False, shifts=None, gate_offset: int = -1,
+                         sinks=None) -> None:
     """Flash attention of the work items in ``tiles`` (int32 [n, 4], see ``paired_attention_tiles``) on the 5th-generation tensor cores; head size 64 or 128, bfloat16.
     ``sigmoid``, ``softcap``, ``shifts``: weights without a softmax (see ``ops.mixed_heads_attention``), a build of its own.  ``gate_offset`` >= 0: the column
-    of ``qkv`` where one gate per head starts, whose sigmoid multiplies the head's output."""
+    of ``qkv`` where one gate per head starts, whose sigmoid multiplies the head's output.  ``softcap`` without ``sigmoid``: a softmax over bounded scores, a build of
+    its own; ``sinks`` (32-bit [heads]): exp(sink) joins the softmax's denominator."""
     ops = _ops()
     if head_dim not in TC_ATTENTION_HEAD_DIMS or page_size % 64 != 0:
         raise KernelError("the tensor-memory attention takes head sizes 64 and 128 and pages of a multiple of 64 keys", code="invalid_shape")
-    lib = tc_attention_library(sigmoid)
+    lib = tc_attention_library(sigmoid, softcap > 0.0)
     gate = c_void_p(0) if gate_offset < 0 else c_void_p(qkv.data_ptr() + gate_offset * qkv.element_size())
     ops._check(
         lib.tlie_prefill_attention_tc(
             ops._ptr(qkv), c_int(qkv.shape[1]), c_int(qkv.shape[0]), ops._ptr(pages), c_int(pages.shape[0]), ops._i32(tiles, "tiles"), c_int(tiles.shape[0]),
             ops._i32(seq_starts, "seq_starts"), ops._i32(first_positions, "first_positions"), ops._i32(block_table, "block_table"),
             c_int(block_table.shape[1]), ops._ptr(out), c_int(q_heads), c_int(kv_heads), c_int(head_dim), c_int(page_size), c_int(window), c_float(scale),
-            c_float(softcap), ops._ptr(shifts), gate, c_int(qkv.shape[1]), ops._ptr(tcgen05_error_flag(qkv.device)), ops._stream(),
+            c_float(softcap), ops._ptr(shifts), gate, c_int(qkv.shape[1]), ops._ptr(sinks), ops._ptr(tcgen05_error_flag(qkv.device)), ops._stream(),
         ),
         "prefill_attention_tc",
     )
@@ -725,16 +740,18 @@ use_mixed_prefill = True
 MIXED_PREFILL_MIN_ROWS = 8    # a step whose longest entry has fewer rows stays on the general kernel (a tile is at least 16 rows)
 
 
-def mixed_prefill_library(key_dim: int, value_dim: int, parts: int, sigmoid: bool = False):
+def mixed_prefill_library(key_dim: int, value_dim: int, parts: int, sigmoid: bool = False, capped: bool = False):
     """The kernel set of one (key width, value width, key heads per folded query, kind of weights): compiled when a model of these sizes first runs a prompt."""
     defines = {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "PARTS": parts}
     if sigmoid:
         return load_library(f"tlie_attn_sigmoid_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], {**defines, "SIGMOID_WEIGHTS": 1})
+    if capped:
+        return load_library(f"tlie_attn_capped_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], {**defines, "SCORE_CAP": 1})
     return load_library(f"tlie_attn_mixed_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], defines)
 
 
 def mixed_prefill_takes(batch, rows, page_size: int, parts: int, key_dim: int, value_dim: int, gate_offset: int, gate_per_head: bool = False,
-                        sigmoid: bool = False) -> bool:
+                        sigmoid: bool = False, capped: bool = False) -> bool:
     """Whether a step's attention with mixed heads runs on the tensor-core kernel: bfloat16, a prompt portion among the entries,
     widths that are multiples of 16, and tiles that fit shared memory (the kernel set says how many rows its tile has: 0 = none)."""
     if not use_mixed_prefill or batch is None or batch.max_q_len < MIXED_PREFILL_MIN_ROWS or rows.dtype != torch.bfloat16:
@@ -743,7 +760,7 @@ def mixed_prefill_takes(batch, rows, page_size: int, parts: int, key_dim: int, v
         return False
     if ((parts * key_dim + 8) * 16 + 3 * 64 * (key_dim + 8) + (3 if parts == 1 else 2) * 64 * (value_dim + 8)) * 2 > 227 * 1024:
         return False   # not even 16 rows of folded queries fit beside the rings of keys and values
-    return mixed_prefill_library(key_dim, value_dim, parts, sigmoid).tlie_mixed_prefill_tile_rows() > 0
+    return mixed_prefill_library(key_dim, value_dim, parts, sigmoid, capped).tlie_mixed_prefill_tile_rows() > 0
 
 
 def folded_slopes(slopes, mix):
@@ -769,13 +786,13 @@ def mixed_scratch(device: torch.device, elements: int, dtype: torch.dtype) -> to
 
 def mixed_prefill(rows, gate_offset: int, batch, block_table, planes, folded, mix, out, heads: int, kv_heads: int, key_dim: int, value_dim: int,
                   page_size: int, window: int, scale: float, keep_first: int = 0, gate_per_head: bool = False, softcap: float = 0.0, sigmoid: bool = False,
-                  shifts=None) -> None:
+                  shifts=None, sinks=None) -> None:
     """Attention with mixed heads for a step that carries prompt portions (csrc/attention_mixed_prefill.cu): the mix is folded into
     the queries by a first kernel, the second is flash attention over the concatenated key heads.  ``planes``: (key plane pointer,
     its page stride in elements, value plane pointer, its page stride); ``folded``: the folded slopes (``folded_slopes``) or None.
     ``keep_first``: with a window, the keys below this position stay visible; ``gate_per_head``: the gate is one column per head.
     With nothing to fold (no mix, ``scale`` 1) the first kernel is left out and the queries are read where they are.  ``sigmoid``, ``softcap``,
-    ``shifts``: see ``ops.mixed_heads_attention``."""
+    ``shifts``, ``sinks``: see ``ops.mixed_heads_attention``."""
     ops = _ops()
     parts = kv_heads if mix is not None else 1
     tokens = rows.shape[0]
@@ -783,12 +800,12 @@ def mixed_prefill(rows, gate_offset: int, batch, block_table, planes, folded, mi
     held = None if mix is None and scale == 1.0 else mixed_scratch(rows.device, need, torch.bfloat16)
     k_ptr, k_stride, v_ptr, v_stride = planes
     ops._check(
-        mixed_prefill_library(key_dim, value_dim, parts, sigmoid).tlie_mixed_prefill(
+        mixed_prefill_library(key_dim, value_dim, parts, sigmoid, softcap > 0.0).tlie_mixed_prefill(
             ops._ptr(rows), c_int(rows.shape[1]), c_int(gate_offset), ops._ptr(mix), c_float(scale), ops._ptr(held), k_ptr, c_longlong(k_stride), v_ptr,
             c_longlong(v_stride), ops._i32(batch.seq_starts, "seq_starts"), ops._i32(batch.first_positions, "first_positions"), ops._i32(block_table, "block_table"),
             c_int(block_table.shape[1]), ops._ptr(folded), ops._ptr(out), c_int(tokens), c_int(batch.num_seqs), c_int(batch.max_q_len),
             c_int(heads), c_int(kv_heads), c_int(page_size), c_int(window), c_int(keep_first), c_int(1 if gate_per_head else 0), c_float(softcap),
-            ops._ptr(shifts), ops._stream()),
+            ops._ptr(shifts), ops._ptr(sinks), ops._stream()),
         "mixed_prefill")
     ops.launch_count += 0 if held is None else 1   # two kernels: the fold and the attention
 
@@ -923,7 +940,7 @@ def mixed_decode_takes(rows, heads: int, kv_heads: int, key_dim: int, value_dim:
 
 def mixed_decode(rows, gate_offset: int, positions, token_seq, block_table, planes, slopes, mix, out, heads: int, kv_heads: int, key_dim: int, value_dim: int,
                  page_size: int, window: int, scale: float, splits: int, keep_first: int = 0, gate_per_head: bool = False, softcap: float = 0.0,
-                 sigmoid: bool = False, shifts=None) -> None:
+                 sigmoid: bool = False, shifts=None, sinks=None) -> None:
     """Attention with mixed heads for a step of few rows (csrc/attention_mixed_decode.cu).  ``planes`` as in ``mixed_prefill``;
     ``splits``: CTAs that share a row's key tiles (their parts are merged by a second kernel)."""
     ops = _ops()
@@ -935,7 +952,7 @@ def mixed_decode(rows, gate_offset: int, positions, token_seq, block_table, plan
             ops._ptr(rows), c_int(rows.shape[1]), c_int(gate_offset), k_ptr, c_longlong(k_stride), v_ptr, c_longlong(v_stride), ops._i32(positions, "positions"),
             ops._i32(token_seq, "token_seq"), ops._i32(block_table, "block_table"), c_int(block_table.shape[1]), ops._ptr(slopes), ops._ptr(mix), ops._ptr(out),
             c_int(tokens), c_int(heads), c_int(kv_heads), c_int(page_size), c_int(window), c_float(scale), c_int(splits), ops._ptr(partial), c_int(keep_first),
-            c_int(1 if gate_per_head else 0), c_float(softcap), c_int(1 if sigmoid else 0), ops._ptr(shifts), ops._stream()),
+            c_int(1 if gate_per_head else 0), c_float(softcap), c_int(1 if sigmoid else 0), ops._ptr(shifts), ops._ptr(sinks), ops._stream()),
         "mixed_decode")
 
 
@@ -1048,8 +1065,9 @@ def moe_grouped_takes(tokens: int, top: int, width: int, ff: int, experts: int) 
     return use_moe_grouped and tokens >= MOE_GROUPED_MIN_ROWS and tokens * top >= MOE_GROUPED_MIN_SLOTS and width % 8 == 0 and ff % 8 == 0 and experts <= 4096
 
 
-def moe_grouped(x, gate_up, down, ids, weights, shared, out, kind: int, weight_input: bool = False, shared_gate=None) -> None:
+def moe_grouped(x, gate_up, down, ids, weights, shared, out, kind: int, weight_input: bool = False, shared_gate=None, clamp=None) -> None:
     ops = _ops()
+    clamp = tuple(c_float(float(v)) for v in clamp or (0.0, 0.0, 0.0))
     tokens, width = x.shape
     experts, _, ff = down.shape
     top = ids.shape[1]
@@ -1067,7 +1085,7 @@ def moe_grouped(x, gate_up, down, ids, weights, shared, out, kind: int, weight_i
         ops._check(ops.moe_library().tlie_moe_grouped_tc(ops._ptr(x), ops._ptr(gate_up), ops._ptr(down), ops._ptr(ids), ops._ptr(weights), ops._ptr(shared), ops._ptr(shared_gate),
                                                          ops._ptr(row_of_slot),
                                                          ops._ptr(token_of_row), ops._ptr(meta), ops._ptr(xs), ops._ptr(act), ops._ptr(y), ops._ptr(out), c_int(tokens), c_int(width),
-                                                         c_int(ff), c_int(experts), c_int(top), c_int(kind), c_int(1 if weight_input else 0), ops._ptr(tcgen05_error_flag(device)), ops._stream()), "moe_grouped_tc")
+                                                         c_int(ff), c_int(experts), c_int(top), c_int(kind), c_int(1 if weight_input else 0), *clamp, ops._ptr(tcgen05_error_flag(device)), ops._stream()), "moe_grouped_tc")
         ops.launch_count += 4   # five kernels: the layout, the gathered rows, two products over all experts, the sum
         return
     sorted_slots = named_scratch(device, "moe_sorted", slots, torch.int32)
@@ -1076,5 +1094,5 @@ def moe_grouped(x, gate_up, down, ids, weights, shared, out, kind: int, weight_i
     y = named_scratch(device, "moe_by_slot", slots * width, torch.float32)
     ops._check(ops.moe_library().tlie_moe_grouped(ops._ptr(x), ops._ptr(gate_up), ops._ptr(down), ops._ptr(ids), ops._ptr(weights), ops._ptr(shared), ops._ptr(shared_gate), ops._ptr(sorted_slots),
                                                   ops._ptr(meta), ops._ptr(act), ops._ptr(y), ops._ptr(out), c_int(tokens), c_int(width), c_int(ff), c_int(experts), c_int(top),
-                                                  c_int(kind), c_int(1 if weight_input else 0), ops._stream()), "moe_grouped")
+                                                  c_int(kind), c_int(1 if weight_input else 0), *clamp, ops._stream()), "moe_grouped")
     ops.launch_count += 3   # four kernels: the sort, two products per expert, the sum

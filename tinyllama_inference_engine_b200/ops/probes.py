@@ -88,7 +88,7 @@ def attention_phase_cycles(tokens: int, q_heads: int, kv_heads: int, head_dim: i
             ops._check(lib.tlie_prefill_attention_tc(ops._ptr(qkv), c_int(qkv.shape[1]), c_int(tokens), ops._ptr(pool), c_int(pages), ops._i32(tiles, "tiles"), c_int(tiles.shape[0]),
                                                      ops._i32(starts, "seq_starts"), ops._i32(first, "first_positions"), ops._i32(table, "block_table"), c_int(pages), ops._ptr(out),
                                                      c_int(q_heads), c_int(kv_heads), c_int(head_dim), c_int(page), c_int(0), c_float(head_dim ** -0.5), c_float(0.0), ops._ptr(None),
-                                                     ops._ptr(None), c_int(0), ops._ptr(ops.error_flag(device)), ops._stream()), "prefill_attention_tc")
+                                                     ops._ptr(None), c_int(0), ops._ptr(None), ops._ptr(ops.error_flag(device)), ops._stream()), "prefill_attention_tc")
         torch.cuda.synchronize(device)
         ops.check_device_errors(device)
         stamps = (ctypes.c_longlong * 24)()

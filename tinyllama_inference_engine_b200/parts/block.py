@@ -294,7 +294,88 @@ class StreamInputMixBlock(Block):
         return mixed, None
 
 
+class ParallelBlock(Block):
+    """x -> x + (mixer(h) + feed_forward(h)) with h = norm(x): one norm, both sublayers read its output.
+
+    params: ``norm``, ``mixer``, ``feed_forward`` (or None), each a PartSpec with its tensor-name suffix (``*_name``).  The norm is one that can be finished
+    by whoever completes the stream (``DynamicTanh``).  h stays as it is while the sublayers run, so a sublayer whose last product can add into the
+    32-bit stream does so; what does not join the stream that way joins it in the kernel of the norm that reads the stream next, which
+    the block hands on finished (``ops.FinishedNorm``)."""
+
+    _SLOTS = (("norm", "norm"), ("mixer", "mixer"), ("feed_forward", "feed_forward"))
+
+    capturable = True
+    accepts_next_norm = True
+
+    @classmethod
+    def _slots(cls, spec: PartSpec):
+        return [pair for pair in cls._SLOTS if spec.get("feed_forward") is not None or pair[0] != "feed_forward"]
+
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
+        specs: list[TensorSpec] = []
+        for slot, category in cls._slots(spec):
+            child = spec[slot]
+            specs += part_class(category, child).tensor_specs(child, f"{prefix}.{spec[slot + '_name']}")
+        return specs
+
+    @classmethod
+    def cache_need(cls, spec: PartSpec) -> CacheNeed:
+        return part_class("mixer", spec["mixer"]).cache_need(spec["mixer"])
+
+    def __init__(self, spec, prefix, weights, runtime):
+        super().__init__(spec, prefix, weights, runtime)
+        self.feed_forward = None
+        for slot, category in self._slots(spec):
+            setattr(self, slot, build_part(category, spec[slot], f"{prefix}.{spec[slot + '_name']}", weights, runtime))
+
+    @property
+    def first_norm(self):
+        return self.norm
+
+    def _normed(self, residual, pending):
+        from .. import ops
+
+        if isinstance(pending, ops.FinishedNorm) and pending.norm is self.norm and pending.finished is not None:
+            return pending.finished
+        return self.norm.forward(residual, None if isinstance(pending, ops.LazyNorm) else pending)
+
+    @staticmethod
+    def _adds(part, rows: int, fused: bool) -> bool:
+        """Whether the sublayer's last product adds into the stream itself."""
+        return part.fuses_residual_add and (fused or part.adds_to_residual(rows))
+
+    def forward(self, residual, pending, ctx, cache: LayerCache, next_norm=None):
+        from .. import ops
+
+        rows = residual.shape[0]
+        fused = rows <= ops.fused_rows_limit(self.runtime.dtype, residual.device)
+        following = next_norm if hasattr(next_norm, "pending") and hasattr(next_norm, "join") else None   # a norm that can be handed on finished
+        h = self._normed(residual, pending)
+        sublayers = [(self.mixer, (ctx, cache))] + ([] if self.feed_forward is None else [(self.feed_forward, (ctx,))])
+        # where both add, the last product completes the stream and finishes the norm that reads it next
+        adding = [self._adds(part, rows, fused) for part, _ in sublayers]
+        branches, handle = [], None
+        for index, (part, args) in enumerate(sublayers):
+            if not adding[index]:
+                branches.append(part.forward(h, *args))
+                continue
+            if fused and following is not None and part.prepares_next_norm and index == len(sublayers) - 1 and not branches:
+                handle = following.pending(residual)
+                part.forward(h, *args, accumulate_into=residual, prepare=handle)
+            else:
+                part.forward(h, *args, accumulate_into=residual)
+        if handle is not None and handle.finished is not None:
+            return residual, handle
+        if following is not None:
+            return residual, following.join(residual, *branches) if branches else following.join(residual, None)
+        for branch in branches[1:]:
+            ops.add_(residual, branch)
+        return residual, branches[0] if branches else None
+
+
 register_part("block", "output_norm", OutputNormBlock)
+register_part("block", "parallel", ParallelBlock)
 register_part("block", "pre_norm_residual", PreNormResidualBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)
 register_part("block", "stream_input_mix", StreamInputMixBlock)

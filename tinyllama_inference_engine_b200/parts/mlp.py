@@ -169,10 +169,12 @@ class RoutedExperts(FeedForward):
     ``scores`` "softmax": s = softmax(z) over all experts.  ``group_score`` "best": a group's score is its largest choice score.
     ``activation`` "relu_squared": experts (and the shared one) without a gate, W_down act(W_up x).  ``shared_gate`` True: the shared expert's output is
     multiplied by sigmoid(w x), one number per token, w the tensor ``<prefix>.shared.sg`` [1, hidden]: a row more in the router's product.
+    ``scores`` "logits": s = z, and the weights are the softmax over the chosen z alone (times ``route_scale``).  ``router_bias`` True: z = W_router x + b, b the
+    tensor ``<prefix>.router.b`` [experts].  ``activation`` "clamped_sigmoid": experts' halves meet as in ``GatedMLP`` (params ``limit``, ``alpha``, ``shift``).
 
     params: ``hidden_size``, ``experts``, ``top``, ``expert_size`` (an expert's inner width), ``groups``, ``keep_groups``, ``route_scale``,
-    ``activation`` ("silu" or "gelu_tanh"), ``shared_size`` (0 or None: no shared expert), ``correction`` (whether the tensor exists),
-    ``normalize`` (True), ``weight_input`` (False), ``scores`` ("sigmoid"), ``group_score`` ("two_best"), ``shared_gate`` (False).
+    ``activation`` ("silu", "gelu_tanh", "relu_squared" or "clamped_sigmoid"), ``shared_size`` (0 or None: no shared expert), ``correction`` (whether the tensor exists),
+    ``normalize`` (True), ``weight_input`` (False), ``scores`` ("sigmoid"), ``group_score`` ("two_best"), ``shared_gate`` (False), ``router_bias`` (False).
     tensors: ``<prefix>.router`` [experts, hidden], ``<prefix>.correction`` [experts], ``<prefix>.e<i>.{gate,up,down}``,
     ``<prefix>.shared.{gate,up,down}`` (without a gate: up and down).  The experts' gate and up rows are stacked per expert at load time, [experts, 2 ff, hidden].
     """
@@ -185,11 +187,12 @@ class RoutedExperts(FeedForward):
         if size <= 0:
             return None
         sizes = {"hidden_size": spec["hidden_size"], "intermediate_size": size, "activation": spec.get("activation", "silu")}
+        sizes.update({key: spec[key] for key in ("limit", "alpha", "shift") if spec.get(key) is not None})
         return PartSpec("gated_mlp", {**sizes, "names": ("gate", "up", "down")}) if cls._gated(spec) else PartSpec("dense_mlp", sizes)
 
     @classmethod
     def _gated(cls, spec: PartSpec) -> bool:
-        return spec.get("activation", "silu") in ops.GATE_KINDS
+        return spec.get("activation", "silu") != "relu_squared"
 
     @classmethod
     def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
@@ -200,6 +203,8 @@ class RoutedExperts(FeedForward):
                 specs.append(TensorSpec(f"{prefix}.e{e}.gate", (ff, hidden), std=hidden ** -0.5))
             specs += [TensorSpec(f"{prefix}.e{e}.up", (ff, hidden), std=hidden ** -0.5), TensorSpec(f"{prefix}.e{e}.down", (hidden, ff), std=ff ** -0.5)]
         specs.append(TensorSpec(f"{prefix}.router", (int(spec["experts"]), hidden), std=hidden ** -0.5))
+        if spec.get("router_bias"):
+            specs.append(TensorSpec(f"{prefix}.router.b", (int(spec["experts"]),), std=0.2))
         if spec.get("correction", True):
             specs.append(TensorSpec(f"{prefix}.correction", (int(spec["experts"]),), std=0.1))
         shared = cls._shared_spec(spec)
@@ -225,6 +230,8 @@ class RoutedExperts(FeedForward):
         self.w_gate_up = torch.stack([torch.cat([weights.get(f"{prefix}.e{e}.{name}", dtype) for name in first], dim=0) for e in range(self.experts)]).contiguous()
         self.w_down = torch.stack([weights.get(f"{prefix}.e{e}.down", dtype) for e in range(self.experts)]).contiguous()
         self.router = weights.get(f"{prefix}.router", torch.float32).contiguous()
+        self.router_bias = weights.get(f"{prefix}.router.b", torch.float32).contiguous() if spec.get("router_bias") else None
+        self.clamp = tuple(float(spec[key]) for key in ("limit", "alpha", "shift")) if self.activation == "clamped_sigmoid" else None
         self.correction = weights.get(f"{prefix}.correction", torch.float32).contiguous() if spec.get("correction", True) else None
         self.scores, self.group_score = spec.get("scores", "sigmoid"), spec.get("group_score", "two_best")
         if self.scores not in ops.ROUTER_SCORES or self.group_score not in ops.GROUP_SCORES:
@@ -241,11 +248,11 @@ class RoutedExperts(FeedForward):
         weights = ws.get("expert_weights", tokens, self.top, torch.float32)
         shared_gate = ws.get("shared_gate", tokens, 1, torch.float32) if self.gates_shared else None
         ops.moe_route(x, self.router, self.correction, ids, weights, self.groups, self.keep, self.route_scale, normalize=self.normalize, scores=self.scores,
-                      group_score=self.group_score, shared_gate=shared_gate)
+                      group_score=self.group_score, shared_gate=shared_gate, bias=self.router_bias)
         shared = None if self.shared is None else self.shared.forward(x, ctx)
         out = ws.get("routed_out", tokens, self.hidden, dtype)
         ops.moe_experts(x, self.w_gate_up, self.w_down, ids, weights, shared, out, self.activation, batch=ctx, weight_input=self.weight_input,
-                        shared_gate=shared_gate)
+                        shared_gate=shared_gate, clamp=self.clamp)
         return out
 
 

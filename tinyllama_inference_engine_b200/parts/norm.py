@@ -1,4 +1,4 @@
-"""RMSNorm, with the residual add fused in front of it; and the layer norm, with and without a bias."""
+"""RMSNorm, with the residual add fused in front of it; the layer norm, with and without a bias; and the curve that may stand in a norm's place."""
 from __future__ import annotations
 
 import torch
@@ -131,6 +131,56 @@ class GroupedRMSNorm(LayerNorm):
             self.weight = (self.weight * scale).contiguous()
 
 
+class DynamicTanh(Norm):
+    """y = tanh(alpha x) * weight + bias element by element: what stands in the place of a norm where no statistics are taken.
+
+    params: ``size``, optional ``suffix`` (what follows the prefix in the tensor's name, ".weight" unless given).
+    tensors: ``<prefix><suffix>`` [size], ``<prefix><suffix>.b`` [size], ``<prefix><suffix>.alpha`` [].  The residual sum, the curve, weight and bias are 32-bit.
+    ``forward`` takes one output that is still to join the stream, as the other norms do; ``join`` takes up to two and hands the result over as an
+    ``ops.FinishedNorm``.  Since an element's value needs nothing of its row, a product that completes the stream can leave this norm's output
+    beside it (``pending``, ``ops.linear_accumulate``)."""
+
+    capturable = True
+    supports_lazy = False
+
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
+        name = f"{prefix}{spec.get('suffix', '.weight')}"
+        return [TensorSpec(name, (spec["size"],), init="norm", std=0.1), TensorSpec(f"{name}.b", (spec["size"],), std=0.2), TensorSpec(f"{name}.alpha", (), init="uniform", std=1.0)]
+
+    def __init__(self, spec, prefix, weights, runtime):
+        super().__init__(spec, prefix, weights, runtime)
+        self.size = int(spec["size"])
+        name = f"{prefix}{spec.get('suffix', '.weight')}"
+        self.weight = weights.get(name, torch.float32).contiguous()
+        self.bias = weights.get(f"{name}.b", torch.float32).contiguous()
+        self.alpha = float(weights.get(f"{name}.alpha", torch.float32))
+
+    def _out(self, rows: int, name: str = "normed"):
+        return self.runtime.workspace.get(name, rows, self.size, self.runtime.dtype)
+
+    def forward(self, residual, delta=None, rows=None, lazy: bool = False):
+        out = self._out(residual.shape[0]) if rows is None else self._out(rows.shape[0], "normed_rows")
+        if rows is not None and delta is not None:
+            ops.add_(residual, delta)
+            delta = None
+        ops.dynamic_tanh(residual, delta, None, rows, self.weight, self.bias, self.alpha, out)
+        return out
+
+    def pending(self, residual) -> "ops.FinishedNorm":
+        """This norm of ``residual`` as it will be: for the product that completes it to finish."""
+        buffer = self._out(residual.shape[0]) if self.runtime.dtype == torch.bfloat16 else None
+        return ops.FinishedNorm(self, residual, (self.alpha, self.weight, self.bias), buffer)
+
+    def join(self, residual, first, second=None) -> "ops.FinishedNorm":
+        """``residual += first + second`` (either may be None) and this norm of the result, one kernel."""
+        handle = ops.FinishedNorm(self, residual, (self.alpha, self.weight, self.bias), None)
+        handle.finished = self._out(residual.shape[0])
+        ops.dynamic_tanh(residual, first, second, None, self.weight, self.bias, self.alpha, handle.finished)
+        return handle
+
+
+register_part("norm", "dynamic_tanh", DynamicTanh)
 register_part("norm", "grouped_rmsnorm", GroupedRMSNorm)
 register_part("norm", "rmsnorm", RMSNorm)
 register_part("norm", "layernorm", LayerNorm)

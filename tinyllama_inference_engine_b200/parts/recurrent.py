@@ -1,6 +1,6 @@
-"""Recurrent mixers: a state of fixed size per request instead of a cache that grows: a gated recurrence per channel, and four mixers
+"""Recurrent mixers: a state of fixed size per request instead of a cache that grows: a gated recurrence per channel, and five mixers
 over a matrix of fast weights per head (the gated delta rule with a decay per key channel and with one per head, linear attention whose
-forget gate also writes, a state-space layer with a scalar decay per head), which share one recurrence kernel."""
+forget gate also writes and linear attention with a decay beside its keys, a state-space layer with a scalar decay per head), which share one recurrence kernel."""
 from __future__ import annotations
 
 import torch
@@ -342,6 +342,85 @@ class Hgrn2(_MatrixRecurrence):
         return self._project(normed, accumulate_into, prepare)
 
 
+class GatedLinearAttention(_MatrixRecurrence):
+    """Linear attention whose key channels each fade at a rate of their own, learned from the token.
+
+    q = W_q x * dim^(-1/2) and k = W_k x (``heads`` of ``dim``), v = W_v x (``heads`` of ``vdim``); decay = sigmoid(W_a2 W_a1 x + b)^(1 / ``tau``) per head and key
+    channel (a low-rank pair).  Per head S <- diag(decay) S + k v^T, o = S^T q.  Each head's o is divided by its root mean square over vdim (``eps``), times
+    ``<prefix>.norm`` [vdim], times silu(W_g x); heads concatenated; W_o.  State (32-bit, zero for a new request): the heads' matrices.  Decays and
+    everything after the projections are 32-bit.  q, k, v, the gate and the pair's first half are one stacked product; the second half is a product
+    of its own for many rows and part of the preparation for few.
+    params: ``hidden_size``, ``num_heads``, ``key_dim``, ``value_dim``, ``tau``, ``decay_rank``, ``eps``.
+    tensors: ``<prefix>.q``, ``<prefix>.k`` [heads dim, hidden], ``<prefix>.v``, ``<prefix>.g`` [heads vdim, hidden], ``<prefix>.o`` [hidden, heads vdim],
+    ``<prefix>.norm`` [vdim], ``<prefix>.a1`` [decay_rank, hidden], ``<prefix>.a2`` [heads dim, decay_rank], ``<prefix>.a2.b`` [heads dim].
+    """
+
+    fuses_residual_add = True
+    prepares_next_norm = True
+
+    @classmethod
+    def _sizes(cls, spec: PartSpec):
+        return tuple(int(spec[k]) for k in ("hidden_size", "num_heads", "key_dim", "value_dim", "decay_rank"))
+
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
+        hidden, heads, dim, vdim, rank = cls._sizes(spec)
+        std = hidden ** -0.5
+        return [TensorSpec(f"{prefix}.q", (heads * dim, hidden), std=std), TensorSpec(f"{prefix}.k", (heads * dim, hidden), std=std),
+                TensorSpec(f"{prefix}.v", (heads * vdim, hidden), std=std), TensorSpec(f"{prefix}.g", (heads * vdim, hidden), std=std),
+                TensorSpec(f"{prefix}.o", (hidden, heads * vdim), std=(heads * vdim) ** -0.5), TensorSpec(f"{prefix}.norm", (vdim,), init="norm", std=0.1),
+                TensorSpec(f"{prefix}.a1", (rank, hidden), std=std), TensorSpec(f"{prefix}.a2", (heads * dim, rank), std=rank ** -0.5),
+                TensorSpec(f"{prefix}.a2.b", (heads * dim,), std=1.0)]
+
+    @classmethod
+    def cache_need(cls, spec: PartSpec) -> CacheNeed:
+        _, heads, dim, vdim, _ = cls._sizes(spec)
+        return CacheNeed("state", state_shape=(ops.delta_state_words(heads, dim, vdim, 0, 1)[0],))
+
+    def __init__(self, spec, prefix, weights, runtime):
+        super().__init__(spec, prefix, weights, runtime)
+        self.hidden, self.heads, self.dim, self.vdim, self.rank = self._sizes(spec)
+        self.eps, self.tau = float(spec["eps"]), float(spec["tau"])
+        dtype = runtime.dtype
+        stacked, offsets, width = [], [], 0
+        for name in ("q", "k", "v", "g", "a1"):
+            piece = weights.get(f"{prefix}.{name}", dtype)
+            if name in ("g", "a1") and width % 8:   # pieces that are read as a product's operand or a gate start on a 16-byte boundary of their row
+                stacked.append(torch.zeros((8 - width % 8, self.hidden), dtype=dtype, device=piece.device))
+                width += stacked[-1].shape[0]
+            offsets.append(width)
+            stacked.append(piece)
+            width += piece.shape[0]
+        if width % 8:
+            stacked.append(torch.zeros((8 - width % 8, self.hidden), dtype=dtype, device=stacked[0].device))
+        self.gate_offset, self.a1_offset = offsets[3], offsets[4]
+        self.w_in = torch.cat(stacked, dim=0).contiguous()
+        self.w_a2 = weights.get(f"{prefix}.a2", dtype).contiguous()
+        self.decay_bias = weights.get(f"{prefix}.a2.b", torch.float32).contiguous()
+        self.out_weight = weights.get(f"{prefix}.norm", torch.float32).contiguous()
+        self.w_o = weights.get(f"{prefix}.o", dtype).contiguous()
+
+    def adds_to_residual(self, rows: int) -> bool:
+        return ops.can_accumulate(rows, self.w_o)
+
+    def forward(self, x, ctx, cache: LayerCache, accumulate_into=None, prepare=None):
+        ws, dtype, tokens = self.runtime.workspace, self.runtime.dtype, x.shape[0]
+        rows = ws.get("gla_in", tokens, self.w_in.shape[0], dtype)
+        ops.linear(x, self.w_in, rows)
+        decay_in, a2 = rows[:, self.a1_offset : self.a1_offset + self.rank], self.w_a2
+        if tokens > ops.fused_rows_limit(dtype, rows.device):
+            pre = ws.get("gla_decay_in", tokens, self.heads * self.dim, dtype)
+            ops.linear(decay_in, self.w_a2, pre)
+            decay_in, a2 = pre, None
+        prep = ws.get("gla_prep", tokens, 3 * self.heads * self.dim + self.heads * self.vdim + self.heads, torch.float32)
+        ops.gla_prepare(rows, decay_in, a2, self.decay_bias, self.tau, self.dim ** -0.5, prep, self.heads, self.dim, self.vdim)
+        read = self._recur(prep, ctx, cache, self.heads, self.heads, self.dim, self.vdim, plain=True)
+        gated = ws.get("recurrent_out", tokens, self.heads * self.vdim, dtype)
+        ops.delta_gate_norm(read, rows[:, self.gate_offset : self.gate_offset + self.heads * self.vdim], self.out_weight, gated, self.eps, self.heads, self.vdim,
+                            gate_kind="silu")
+        return self._project(gated, accumulate_into, prepare)
+
+
 class StateSpaceDuality(_MatrixRecurrence):
     """A state-space layer with a scalar decay per head (the form that is also linear attention).
 
@@ -414,6 +493,7 @@ class StateSpaceDuality(_MatrixRecurrence):
 
 
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)
+register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "hgrn2", Hgrn2)
 register_part("mixer", "state_space_duality", StateSpaceDuality)
 register_part("mixer", "mingru", MinGRU)
