@@ -61,8 +61,8 @@ def rotate(x, positions, rot, interleaved):
 
 
 def mixed_values(v, first, lam):
-    """The layer's values drawn towards those of the first layer that mixes (None: this is that layer)."""
-    return v if first is None else (1.0 - lam) * v + lam * first
+    """The layer's values drawn towards those of the first layer that mixes (None: this is that layer), number by number whatever the heads' widths are."""
+    return v if first is None else (1.0 - lam) * v + lam * first.reshape(v.shape)
 
 
 def one_more_softmax_heads(q, k, v, scale, positions):

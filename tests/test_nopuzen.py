@@ -5,7 +5,6 @@ from __future__ import annotations
 
 import json
 import math
-from types import SimpleNamespace
 
 import numpy as np
 import pytest
@@ -13,6 +12,7 @@ import torch
 
 import plain_nopuzen
 import trace_tools
+from kernel_steps import pieces_of, scrambled_table, step_of
 from tinyllama_inference_engine_b200 import EngineConfig
 from tinyllama_inference_engine_b200.cache import CacheManager
 from tinyllama_inference_engine_b200.config import architecture_for, load_model_config
@@ -337,37 +337,6 @@ def test_product_per_head_behind_a_gate(dtype, atol, tokens, heads, n, k):
     assert float((out.cpu().double() - want).abs().max()) <= atol * max(1.0, float(want.abs().max()))
 
 
-def _scrambled_table(totals, page_size, g):
-    width = max(-(-t // page_size) for t in totals)
-    count = sum(-(-t // page_size) for t in totals) + 3
-    order = torch.randperm(count, generator=g).tolist()
-    table = torch.full((len(totals), width), -1, dtype=torch.int32)
-    for r, t in enumerate(totals):
-        for p in range(-(-t // page_size)):
-            table[r, p] = order.pop()
-    return table, count
-
-
-def _step_of(rows, cache, pieces):
-    """The context of a step that brings request r's rows [a, a + n) for (r, a, n) in ``pieces``."""
-    index = [(r, a + i) for r, a, n in pieces for i in range(n)]
-    step_rows = torch.stack([rows[r][p] for r, p in index]).cuda().contiguous()
-    positions = torch.tensor([p for _, p in index], dtype=torch.int32).cuda()
-    token_seq = torch.tensor([j for j, (_, _, n) in enumerate(pieces) for _ in range(n)], dtype=torch.int32).cuda()
-    starts = torch.tensor(np.concatenate([[0], np.cumsum([n for _, _, n in pieces])]), dtype=torch.int32).cuda()
-    sub = type(cache)(cache.need, True, cache.pages, cache.block_table[[r for r, _, _ in pieces]].contiguous(), cache.page_size, None, cache.plane_pages)
-    batch = SimpleNamespace(max_q_len=max(n for _, _, n in pieces), num_seqs=len(pieces), max_seq_len=max(a + n for _, a, n in pieces), seq_starts=starts,
-                            first_positions=torch.tensor([a for _, a, _ in pieces], dtype=torch.int32).cuda(), num_tokens=len(index), plan=lambda name: None)
-    return step_rows, positions, token_seq, sub, batch, index
-
-
-def _pieces(lens, firsts):
-    """Every request in three steps: rows before ``firsts``, a portion behind them, and its last rows as a step of few rows of their own."""
-    tails = [min(n, 3 + r) for r, n in enumerate(lens)]
-    return ([(r, 0, f) for r, f in enumerate(firsts) if f > 0], [(r, f, n - t) for r, (n, f, t) in enumerate(zip(lens, firsts, tails)) if n > t],
-            [(r, f + n - t, t) for r, (n, f, t) in enumerate(zip(lens, firsts, tails))])
-
-
 SIGMOID_SHAPES = [(4, 2, 16, 32, 8, True, 1.0), (2, 1, 32, 16, 32, True, 1.2), (3, 3, 16, 16, 0, True, 1.0), (6, 1, 64, 64, 20, False, 1.0), (1, 1, 40, 24, 10, False, 1.3), (5, 5, 10, 6, 4, True, 1.0),
                   (8, 2, 128, 128, 64, True, 1.0), (20, 1, 16, 16, 16, True, 1.0), (4, 2, 80, 48, 80, True, 1.0), (4, 4, 64, 64, 64, True, 1.0)]
 
@@ -386,7 +355,7 @@ def test_sigmoid_attention_kernels(dtype, atol, heads, kv, dim, vdim, rot, inter
 
     lens, firsts = ([37, 1, 18], [30, 52, 0]) if not long_tail else ([5, 200, 9], [330, 0, 61])
     g = torch.Generator().manual_seed(heads * 100 + dim)
-    table, count = _scrambled_table([f + n for n, f in zip(lens, firsts)], page_size, g)
+    table, count = scrambled_table([f + n for n, f in zip(lens, firsts)], page_size, g)
     columns = heads * dim + kv * dim + kv * vdim + heads
     columns += -columns % 8
     rows = [torch.randn(f + n, columns, generator=g).to(dtype) for n, f in zip(lens, firsts)]
@@ -412,8 +381,8 @@ def test_sigmoid_attention_kernels(dtype, atol, heads, kv, dim, vdim, rot, inter
         want.append((o * torch.sigmoid(x[:, gate_offset : gate_offset + heads])[:, :, None]).reshape(total, heads * vdim))
     got = [torch.zeros_like(w) for w in want]
     device = [t.cuda() for t in (*biases, q_weight, k_weight, temps * sizes["scale"], shifts)]
-    for pieces in _pieces(lens, firsts):
-        step_rows, positions, token_seq, sub, batch, index = _step_of(rows, cache, pieces)
+    for pieces in pieces_of(lens, firsts):
+        step_rows, positions, token_seq, sub, batch, index = step_of(rows, cache, pieces)
         ops.norm_rotary_store(step_rows, k_offset, v_offset, device[:3], device[3], device[4], eps, device[5], inv_freq, rot, interleaved, amplitude, positions, token_seq, sub,
                               heads, kv, dim, vdim)
         out = torch.zeros(len(index), heads * vdim, dtype=dtype, device="cuda")
@@ -439,7 +408,7 @@ def test_sigmoid_attention_in_tensor_memory(dim, heads, kv, page_size, softcap, 
     g = torch.Generator().manual_seed(dim + heads)
     lens, firsts = [1, 1, 300, 129, 200], [70, 200, 0, 130, 1]
     totals = [f + n for n, f in zip(lens, firsts)]
-    table, count = _scrambled_table(totals, page_size, g)
+    table, count = scrambled_table(totals, page_size, g)
     columns = (heads + 2 * kv) * dim + heads
     columns += -columns % 8
     rows = [torch.randn(t, columns, generator=g).bfloat16() for t in totals]
@@ -489,7 +458,7 @@ def test_latent_attention_kernels(dtype, atol, heads, dim, rot, vdim, rank, q_ra
 
     lens, firsts, page_size = ([37, 1, 18], [30, 52, 0], 16) if not long_tail else ([5, 150, 9], [330, 0, 61], 16)
     g = torch.Generator().manual_seed(rank)
-    table, count = _scrambled_table([f + n for n, f in zip(lens, firsts)], page_size, g)
+    table, count = scrambled_table([f + n for n, f in zip(lens, firsts)], page_size, g)
     latent_offset, gate_offset = q_rank + (-q_rank % 8), q_rank + (-q_rank % 8) + rank + rot
     rows = [torch.randn(f + n, gate_offset + heads * vdim, generator=g).to(dtype) for n, f in zip(lens, firsts)]
     pages = torch.full((count, 1, 1, page_size, rank + rot), float("nan")).to(dtype).cuda()
@@ -515,11 +484,11 @@ def test_latent_attention_kernels(dtype, atol, heads, dim, rot, vdim, rank, q_ra
     inv_freq = torch.tensor(freq, dtype=torch.float32).cuda()
     uk_t = w_uk.view(heads, dim, rank).transpose(1, 2).contiguous().cuda()
     sizes = (heads, dim, rot, rank, interleaved, amplitude)
-    steps = list(_pieces(lens, firsts))
+    steps = list(pieces_of(lens, firsts))
     if singles:     # the last rows one by one: steps of single tokens, of fewer and fewer requests
         steps = steps[:2] + [[(r, a + i, 1) for r, a, n in steps[2] if i < n] for i in range(max(n for _, _, n in steps[2]))]
     for pieces in steps:
-        step_rows, positions, token_seq, sub, batch, index = _step_of(rows, cache, pieces)
+        step_rows, positions, token_seq, sub, batch, index = step_of(rows, cache, pieces)
         tokens = len(index)
         q_latent, queries = torch.zeros(tokens, q_rank, dtype=dtype, device="cuda"), torch.zeros(tokens, heads * (rank + rot), dtype=dtype, device="cuda")
         ops.latent_store(step_rows, latent_offset, weight.cuda(), eps, inv_freq, rot, positions, token_seq, sub, None, *sizes, q_latent=(0, q_weight.cuda(), q_latent))

@@ -61,7 +61,7 @@ def build_vogusun_spec(config: VogusunConfig) -> ModelSpec:
         })))
     spec = ModelSpec(
         architecture="Vogusun", hidden_size=width, vocab_size=config.vocab, max_positions=MAX_POSITIONS,
-        embedding=PartSpec("token_embedding", {"vocab_size": config.vocab, "hidden_size": width, "tensor": "embed"}),
+        embedding=PartSpec("token_embedding", {"vocab_size": config.vocab, "hidden_size": width, "tensor": "embed", "init_std": 1.0}),
         layers=tuple(layers), order=tuple(OrderEntry(layer=i, cache=i) for i in range(len(layers))),
         final_norm=PartSpec("dynamic_tanh", {**curve, "name": "final.norm"}),
         head=PartSpec("linear_head", {"vocab_size": config.vocab, "hidden_size": width, "tensor": "head", "tied_to": None}),

@@ -16,7 +16,8 @@ def _tensor_name(spec: PartSpec) -> str:
 class TokenEmbedding(Part):
     """hidden = table[token], a row copy without scaling (src/model.cpp:94-97).
 
-    params: ``vocab_size``, ``hidden_size``, ``name`` (the tensor is ``<name>.weight``, or ``tensor`` in full).  The row is widened into the
+    params: ``vocab_size``, ``hidden_size``, ``name`` (the tensor is ``<name>.weight``, or ``tensor`` in full), optional ``init_std`` (of the random-weights mode,
+    0.02 unless given: without a norm that divides by a row's own size the stream wants numbers of its own).  The row is widened into the
     32-bit residual stream by a gather kernel (the reference copies one row per token
     with a device memcpy, src/cuda/model.cu:572-576).
     """
@@ -26,7 +27,7 @@ class TokenEmbedding(Part):
 
     @classmethod
     def tensor_specs(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
-        return [TensorSpec(_tensor_name(spec), (spec["vocab_size"], spec["hidden_size"]))]
+        return [TensorSpec(_tensor_name(spec), (spec["vocab_size"], spec["hidden_size"]), std=float(spec.get("init_std", 0.02)))]
 
     def __init__(self, spec, prefix, weights, runtime):
         super().__init__(spec, prefix, weights, runtime)

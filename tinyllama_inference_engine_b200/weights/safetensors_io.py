@@ -124,7 +124,7 @@ def write_safetensors(path: str | Path, tensors: dict[str, torch.Tensor], metada
         tensor = tensor.detach().cpu().contiguous()
         if tensor.dtype not in _NAMES:
             raise EngineError(f"cannot store dtype {tensor.dtype} for {name!r}", code="invalid_dtype")
-        raw = tensor.view(torch.uint8).numpy().tobytes() if tensor.numel() else b""
+        raw = tensor.reshape(-1).view(torch.uint8).numpy().tobytes() if tensor.numel() else b""
         header[name] = {
             "dtype": _NAMES[tensor.dtype],
             "shape": list(tensor.shape),
