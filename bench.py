@@ -489,6 +489,38 @@ def nopuzen_config(size: dict, extra: dict) -> dict:
     return {"architecture": "Nopuzen", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-5}, "layers": layers}
 
 
+# `--designs vogusun`: Vogusun (one curve per element in a norm's place and both sublayers side by side behind it; softmax attention with normed and
+# rotated queries and keys, one more in the denominator and a gate per head; softmax attention with biased projections, a stretched rotation and
+# bounded scores, values drawn towards the first layer's; gated linear attention; gated feed-forwards with gelu, every second layer a
+# mixture of experts with clamped gates) beside Redasun, the closest of the engine's designs (attention with normed and rotated queries and keys
+# over pages, gated feed-forwards with gelu, every second layer a mixture of gated experts), at equal width, layer count, vocabulary,
+# feed-forward and expert widths.
+VOGUSUN_SIZES = {
+    "w2048": dict(attention=dict(heads=16, kv_heads=4, dim=128, vdim=128), attention_2=dict(heads=32, kv_heads=8, dim=64, vdim=64, softcap=30.0),
+                  gla=dict(heads=16, dim=128, vdim=128, tau=16.0, decay_rank=16), experts=32, top=4, expert_ff=1408, limit=7.0, pattern=("attention", "gla", "attention_2", "gla")),
+    "w4096": dict(attention=dict(heads=32, kv_heads=8, dim=128, vdim=128), attention_2=dict(heads=32, kv_heads=8, dim=192, vdim=128, softcap=30.0),
+                  gla=dict(heads=32, dim=128, vdim=128, tau=16.0, decay_rank=16), experts=32, top=4, expert_ff=3584, limit=7.0, pattern=("attention", "gla", "attention_2", "attention")),
+}
+
+
+def vogusun_config(size: dict, extra: dict) -> dict:
+    layers = []
+    for index in range(size["layers"]):
+        kind = extra["pattern"][index % len(extra["pattern"])]
+        mixer = dict(extra[kind])
+        if kind != "gla":
+            rot = {"base": 500000.0, "dims": mixer["dim"]}
+            if kind == "attention_2":
+                rot["scaling"] = {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+            mixer |= {"scale": mixer["dim"] ** -0.5, "rot": rot, "v_mix": True}
+        if index % 2 == 0:
+            mlp = {"kind": "dense", "ff": size["ff"]}
+        else:
+            mlp = {"kind": "moe", "expert": {"ff": extra["expert_ff"], "limit": extra["limit"]}, "router": {"experts": extra["experts"], "top": extra["top"]}}
+        layers.append({"type": kind, "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Vogusun", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-5}, "layers": layers}
+
+
 def run_designs(args) -> dict:
     import numpy as np
     import torch
@@ -1033,13 +1065,129 @@ def run_designs(args) -> dict:
             out[f"norms_{name}"] = against_bytes(ms, tokens * W * 12.0, like_ms)
         return out
 
+    def vogusun_kernel_numbers(size: dict, extra: dict) -> dict:
+        """Vogusun's own kernels alone against their rooflines, beside like kernels of the other designs at the same sizes: either softmax attention beside
+        the Llama path's, their store beside the one without the drawn values; the recurrence's preparation beside the one whose forget gate
+        also writes (the recurrence and the gated norm behind it are those designs' kernels); the router over chosen logits beside the
+        sigmoid one; clamped experts beside silu ones; the curve beside the RMS norm with its add; the dense feed-forward beside silu's."""
+        W, page, bf16, r = size["width"], 64, torch.bfloat16, extra["gla"]
+        E, top, F = extra["experts"], extra["top"], extra["expert_ff"]
+        RH, RD, RV, rank = r["heads"], r["dim"], r["vdim"], r["decay_rank"]
+        out = {}
+        pages_needed = -(-(context + 1) // page) * batch + -(-prompt_tokens // page)
+        ones = torch.ones(max(W, RH * RD, 4096), device=device)
+        gate_up, down = (torch.randn(E, 2 * F, W, device=device) * W ** -0.5).to(bf16), (torch.randn(E, W, F, device=device) * F ** -0.5).to(bf16)
+        router = torch.randn(E, W, device=device) * W ** -0.5
+        w_gate_up, w_down = (torch.randn(2 * size["ff"], W, device=device) * W ** -0.5).to(bf16), (torch.randn(W, size["ff"], device=device) * size["ff"] ** -0.5).to(bf16)
+        w_a2 = torch.randn(RH * RD, rank, device=device).to(bf16)
+
+        def context_for(lens, firsts):
+            table_width = size["positions"] // page
+            rows, at = [], 0
+            for n, f in zip(lens, firsts):
+                count = -(-(f + n) // page)
+                rows.append(list(range(at, at + count)) + [-1] * (table_width - count))
+                at += count
+            entries = [StepEntry(i, [0] * n, []) for i, n in enumerate(lens)]
+            return pack_step(entries, list(firsts), list(range(len(lens))), [rows], device)
+
+        def against_bytes(ms, moved, like_ms=None, like_moved=None, **more):
+            line = {"ms": ms, "gbs": moved / ms / 1e6, "frac": moved / (ms / 1e3) / 1e9 / peak["hbm_gbs"], **more}
+            return line if like_ms is None else {**line, "like_ms": like_ms, "like_frac": (like_moved or moved) / (like_ms / 1e3) / 1e9 / peak["hbm_gbs"]}
+
+        def against_flops(ms, flops, like_ms=None, like_flops=None, **more):
+            line = {"ms": ms, "tflops": flops / ms / 1e9, "frac": flops / (ms / 1e3) / (peak["bf16_tflops"] * 1e12), **more}
+            return line if like_ms is None else {**line, "like_ms": like_ms, "like_frac": (like_flops or flops) / (like_ms / 1e3) / (peak["bf16_tflops"] * 1e12)}
+
+        for name, lens, firsts in (("prefill", [prompt_tokens], [0]), ("decode", [1] * batch, [context] * batch)):
+            ctx, tokens, prompt = context_for(lens, firsts), sum(lens), name == "prefill"
+            causal = sum(f + i + 1 for n, f in zip(lens, firsts) for i in range(n))
+            for kind in ("attention", "attention_2"):
+                a = extra[kind]
+                H, G, D, V = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+                if D == V:
+                    cache = LayerCache(CacheNeed("pages"), True, torch.randn(pages_needed, 2, G, page, D, device=device).to(bf16), ctx.block_tables[0], page)
+                else:
+                    planes = tuple(torch.randn(pages_needed, G, page, w, device=device).to(bf16) for w in (D, V))
+                    cache = LayerCache(CacheNeed("pages"), True, None, ctx.block_tables[0], page, None, planes)
+                inv_freq = torch.tensor([10000.0 ** (-2.0 * i / D) for i in range(D // 2)], dtype=torch.float32, device=device)
+                gate_at, columns = (H + G) * D + G * V, (H + G) * D + G * V + -(-H // 8) * 8
+                rows, kept = torch.randn(tokens, columns, device=device).to(bf16), torch.randn(tokens, G * V, device=device).to(bf16)
+                factors, plain = torch.full((H,), D ** -0.5, device=device), kind == "attention"
+                biases = None if plain else (ones[: H * D], ones[: G * D], ones[: G * V]) if max(H * D, G * V) <= ones.numel() else tuple(torch.ones(n, device=device) for n in (H * D, G * D, G * V))
+                norm = (ones[:D], ones[:D]) if plain else (None, None)
+                store = lambda **k: ops.norm_rotary_store(rows, H * D, (H + G) * D, biases, *norm, 1e-5, factors, inv_freq, D, plain, 1.0, ctx.positions, ctx.token_seq, cache, H, G, D, V, **k)
+                ms, like_ms = timed(lambda: store(first_values=kept, value_share=0.3)), timed(store)
+                moved = tokens * 2.0 * (2 * H * D + 2 * G * (D + V))
+                out[f"{kind}_store_{name}"] = against_bytes(ms, moved + tokens * 2.0 * G * V, like_ms, moved)
+                mixed = torch.empty(tokens, H * V, dtype=bf16, device=device)
+                options = dict(gate_per_head=True, sinks=torch.zeros(H, device=device)) if plain else dict(gate_per_head=True, softcap=a["softcap"])
+                ms = timed(lambda: ops.mixed_heads_attention(rows, gate_at if plain else -1, ctx.positions, ctx.token_seq, cache, None, None, mixed, H, G, D, V, 0, 1.0, batch=ctx, **options))
+                L = min(D, V)   # the Llama path knows one width for keys and values
+                pages = torch.randn(pages_needed, 2, G, page, L, device=device).to(bf16)
+                qkv, like_out = torch.randn(tokens, (H + 2 * G) * L, device=device).to(bf16), torch.empty(tokens, H * L, dtype=bf16, device=device)
+                like_ms = timed(lambda: ops.paged_attention(qkv, pages, ctx.positions, ctx.token_seq, ctx.block_tables[0], like_out, H, G, L, page, 0, L ** -0.5, batch=ctx))
+                out[f"{kind}_{name}"] = (against_flops(ms, causal * H * 2.0 * (D + V), like_ms, causal * H * 4.0 * L) if prompt
+                                         else against_bytes(ms, causal * G * 2.0 * (D + V), like_ms, causal * G * 4.0 * L))
+            # gated linear attention
+            qk, values = RH * RD, RH * RV
+            rows = torch.randn(tokens, 2 * qk + 2 * values + rank, device=device).to(bf16)
+            prep, state = torch.zeros(tokens, 3 * qk + values + RH, device=device), torch.zeros(batch + 1, ops.delta_state_words(RH, RD, RV, 0, 1)[0], device=device)
+            pre, first = torch.empty(tokens, qk, dtype=bf16, device=device), rows[:, 2 * qk + 2 * values :]
+
+            def prepare():
+                if prompt:
+                    ops.linear(first, w_a2, pre)
+                    ops.gla_prepare(rows, pre, None, ones[:qk], r["tau"], RD ** -0.5, prep, RH, RD, RV)
+                else:
+                    ops.gla_prepare(rows, first, w_a2, ones[:qk], r["tau"], RD ** -0.5, prep, RH, RD, RV)
+
+            ms, like_ms = timed(prepare), timed(lambda: ops.hgrn2_prepare(rows, ones[:qk], ones[:qk], prep, RH, RD, RV))
+            moved = tokens * (2.0 * (2 * qk + values) + 4.0 * (3 * qk + values))
+            out[f"gla_prepare_{name}"] = against_bytes(ms, moved + (tokens * 4.0 * qk if prompt else 2.0 * qk * rank), like_ms, moved)
+            read, gated = torch.empty(tokens, values, device=device), torch.empty(tokens, values, dtype=bf16, device=device)
+            ms = timed(lambda: ops.delta_rule(prep, state, ctx, read, RH, RH, RD, RV, plain=True))
+            like_ms = timed(lambda: ops.delta_rule(prep, state, ctx, read, RH, RH, RD, RV))
+            out[f"gla_recurrence_{name}"] = against_bytes(ms, tokens * 4.0 * (3 * qk + 2 * values) + len(lens) * 8.0 * RH * RD * RV, like_ms)
+            ms = timed(lambda: ops.delta_gate_norm(read, rows[:, 2 * qk + values : 2 * qk + 2 * values], ones[:RV], gated, 1e-5, RH, RV, gate_kind="silu"))
+            out[f"gla_gate_norm_{name}"] = against_bytes(ms, tokens * 8.0 * values)
+            # router and experts
+            x = torch.randn(tokens, W, device=device).to(bf16)
+            ids, weights = torch.empty(tokens, top, dtype=torch.int32, device=device), torch.empty(tokens, top, device=device)
+            like_ms = timed(lambda: ops.moe_route(x, router, None, ids, weights, 1, 1, 2.0))
+            ms = timed(lambda: ops.moe_route(x, router, None, ids, weights, 1, 1, 1.0, scores="logits", bias=ones[:E]))
+            out[f"router_{name}"] = against_bytes(ms, tokens * W * 2.0 + E * W * 4.0, like_ms)
+            routed = torch.empty(tokens, W, dtype=bf16, device=device)
+            ms = timed(lambda: ops.moe_experts(x, gate_up, down, ids, weights, None, routed, "clamped_sigmoid", batch=ctx, clamp=(extra["limit"], 1.702, 1.0)))
+            like_ms = timed(lambda: ops.moe_experts(x, gate_up, down, ids, weights, None, routed, "silu", batch=ctx))
+            chosen = len(torch.unique(ids))
+            out[f"experts_{name}"] = (against_flops(ms, tokens * top * 6.0 * F * W, like_ms) if prompt else against_bytes(ms, chosen * 6.0 * F * W, like_ms, experts_read=chosen))
+            # the dense feed-forward, adding into the stream as the block lets it
+            act, stream = torch.empty(tokens, size["ff"], dtype=bf16, device=device), torch.zeros(tokens, W, device=device)
+
+            def dense(kind):
+                ops.linear_gated(x, w_gate_up, act, activation=kind)
+                ops.linear_accumulate(act, w_down, stream)
+
+            ms, like_ms = timed(lambda: dense("gelu_tanh")), timed(lambda: dense("silu"))
+            out[f"dense_{name}"] = against_flops(ms, tokens * 6.0 * size["ff"] * W, like_ms) if prompt else against_bytes(ms, 6.0 * size["ff"] * W, like_ms)
+            # the curve in the norm's place
+            normed = torch.empty(tokens, W, dtype=bf16, device=device)
+            for joins, delta in (("alone", None), ("joining", x)):
+                ms = timed(lambda: ops.dynamic_tanh(stream, delta, None, None, ones[:W], ones[:W], 0.5, normed))
+                like_ms = timed(lambda: ops.add_rmsnorm(stream, delta, ones[:W], 1e-5, normed))
+                out[f"curve_{joins}_{name}"] = against_bytes(ms, tokens * W * (6.0 if delta is None else 12.0), like_ms)
+        return out
+
     results = {}
     which = args.designs
     with ClockSampler() as clocks:
         for key, size in DESIGN_SIZES.items():
             marutar, llama = design_configs(size)
             base = Path(tempfile.gettempdir()) / f"tlie_b200_designs_{os.getuid()}_{key}"
-            if which == "nopuzen":
+            if which == "vogusun":
+                pair = (("vogusun", vogusun_config(size, VOGUSUN_SIZES[key])), ("redasun", redasun_config(size, REDASUN_SIZES[key])))
+            elif which == "nopuzen":
                 pair = (("nopuzen", nopuzen_config(size, NOPUZEN_SIZES[key])), ("redasun", redasun_config(size, REDASUN_SIZES[key])))
             elif which == "kilurax":
                 pair = (("kilurax", kilurax_config(size, KILURAX_SIZES[key])), ("redasun", redasun_config(size, REDASUN_SIZES[key])))
@@ -1053,7 +1201,9 @@ def run_designs(args) -> dict:
                 if not (folders[name] / "model.safetensors").exists():
                     write_random_model(folders[name], config, seed=0)
             results[key] = {name: model_numbers(folders[name]) for name, _ in pair}
-            if which == "nopuzen":
+            if which == "vogusun":
+                results[key]["kernels"] = vogusun_kernel_numbers(size, VOGUSUN_SIZES[key])
+            elif which == "nopuzen":
                 results[key]["kernels"] = nopuzen_kernel_numbers(size, NOPUZEN_SIZES[key])
             elif which == "kilurax":
                 results[key]["kernels"] = kilurax_kernel_numbers(size, KILURAX_SIZES[key], ZIRUTAR_SIZES[key])
@@ -1064,6 +1214,8 @@ def run_designs(args) -> dict:
             results[key]["sizes"] = {k: v for k, v in size.items() if k != "pattern"} | {"pattern": "/".join(size["pattern"])}
             if which == "redasun":
                 results[key]["sizes"] = {k: v for k, v in size.items() if k in ("width", "ff", "vocab", "layers")} | {k: (list(v) if isinstance(v, tuple) else v) for k, v in REDASUN_SIZES[key].items()}
+            if which == "vogusun":
+                results[key]["sizes"] = {k: v for k, v in size.items() if k in ("width", "ff", "vocab", "layers")} | {k: (list(v) if isinstance(v, tuple) else v) for k, v in VOGUSUN_SIZES[key].items()}
             if which == "nopuzen":
                 results[key]["sizes"] = {k: v for k, v in size.items() if k in ("width", "ff", "vocab", "layers")} | {k: (list(v) if isinstance(v, tuple) else v) for k, v in NOPUZEN_SIZES[key].items()}
             if which == "kilurax":
@@ -1071,7 +1223,7 @@ def run_designs(args) -> dict:
             if which == "zirutar":
                 results[key]["sizes"] |= {k: v for k, v in ZIRUTAR_SIZES[key].items() if k != "pattern"} | {"zirutar_pattern": "/".join(ZIRUTAR_SIZES[key]["pattern"])}
     names = {"marutar": "Marutar beside the Llama decoder", "zirutar": "Zirutar beside Marutar", "redasun": "Redasun beside the Llama decoder",
-             "kilurax": "Kilurax beside Redasun", "nopuzen": "Nopuzen beside Redasun"}[which]
+             "kilurax": "Kilurax beside Redasun", "nopuzen": "Nopuzen beside Redasun", "vogusun": "Vogusun beside Redasun"}[which]
     return {"metric": f"prompt and decode throughput of {names} at equal sizes", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16",
             "data": "synthetic (random weights, uniform random token ids)", "impl": "engine", "higher_is_better": True,
             "config": {"prompt_tokens": prompt_tokens, "decode_context": context, "decode_batch": batch, "decode_steps": steps, "page_size": 64, "peaks": peak_kind,
@@ -1132,9 +1284,9 @@ def main() -> int:
     parser.add_argument("--impl", default="engine", choices=["engine", "reference"])
     parser.add_argument("--reference-points", action="store_true", help="with --impl reference: also time batch 1 and 64 (minutes)")
     parser.add_argument("--sections", default="decode,e2e,prefill,points,mixed", help="which measurements to take (fewer for profiling runs; `mixed` adds requests of mixed length through the scheduler)")
-    parser.add_argument("--designs", nargs="?", const="marutar", default=None, choices=["marutar", "zirutar", "redasun", "kilurax", "nopuzen"],
+    parser.add_argument("--designs", nargs="?", const="marutar", default=None, choices=["marutar", "zirutar", "redasun", "kilurax", "nopuzen", "vogusun"],
                         help="instead of the headline workload: another design beside the closest existing one at equal sizes (prompt and decode throughput through "
-                             "the engine, and the design's own kernels against their rooflines): Marutar beside the Llama decoder (the default), Zirutar beside Marutar, Redasun beside the Llama decoder, Kilurax beside Redasun, or Nopuzen beside Redasun")
+                             "the engine, and the design's own kernels against their rooflines): Marutar beside the Llama decoder (the default), Zirutar beside Marutar, Redasun beside the Llama decoder, Kilurax beside Redasun, Nopuzen beside Redasun, or Vogusun beside Redasun")
     args = parser.parse_args()
     if args.gpus != 1:
         print(f"bench.py measures one GPU only: this engine is single-GPU by design (asked for {args.gpus})")
