@@ -32,8 +32,13 @@
 // as it is.  tanh and sigmoid are e^x and a reciprocal each, in 32-bit; one reciprocal serves two scores (1 / a = b / (a b)), so that a
 // score costs three operations of the exponential unit.  In both kinds the output may be multiplied by sigmoid(gate), one number per
 // (row, head), as it is read out.
-// SCORE_CAP 1 (a build of its own): a softmax over bounded scores, softcap * tanh(score / softcap), tanh as above.  In both softmax builds ``sinks`` (optional, one
-// per head) puts exp(sink_h) into the denominator, a weight that belongs to no key.
+// SCORE_CAP 1 (a build of its own): a softmax over bounded scores, softcap * tanh(score / softcap).  A warp whose scores of a tile all lie within 0.6 of the
+// bound takes tanh from an odd polynomial (t P(t^2), P of degree four fitted on [0, 0.36]: relative error 7e-8), which leaves the exponential unit to the
+// softmax; other tiles take it as above.  Bounded scores need no running maximum while e^softcap is far from overflow: weights are then taken
+// against zero.  In both softmax builds ``sinks`` (optional, one per head) puts exp(sink_h) into the denominator, a weight that belongs to no key.
+// PLANES 1 (a build of its own, KEY_DIM / VALUE_DIM): keys and values are planes with a pointer and a page stride each and of any widths that are multiples
+// of 8: KEY_DIM and VALUE_DIM are the widths rounded up to whole boxes of 64, and a box past a row's end arrives with zeros there (of the
+// queries it holds the next head's numbers, which meet the keys' zeros).
 // LATENT_ROWS 1 (a build of its own, KEY_DIM / ROT_DIM / VALUE_DIM): the keys and values are rows of the step itself and not of pages, which is all a
 // step sees whose requests all start in it.  A key is a head's own columns beside ROT_DIM columns that every head shares (latent
 // attention with its keys and values expanded): the two come from matrices of their own, a box each.
@@ -64,6 +69,9 @@
 #endif
 #ifndef SCORE_CAP
 #define SCORE_CAP 0
+#endif
+#ifndef PLANES
+#define PLANES 0
 #endif
 #include <type_traits>
 
@@ -176,6 +184,15 @@ __device__ __forceinline__ Float2Bits mul2(Float2Bits a, Float2Bits b) {
   asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(r.bits) : "l"(a.bits), "l"(b.bits));
   return r;
 }
+// tanh(t) = t P(t^2) for |t| <= kTanhReach: least maximum of the relative error over the interval (7e-8), found by reweighted least squares.
+constexpr float kTanhReach = 0.6f;
+__host__ __device__ constexpr float tanh_poly(int n) {
+  constexpr float p[5] = {0.9999999268688395f, -0.33332309973338137f, 0.13310173643287185f, -0.05210147946595585f, 0.015475426588089806f};
+  return p[n];
+}
+// e^(+-40) is 2^58: a row's weights and their sum stay far inside 32-bit numbers without a maximum taken off.
+constexpr float kCapWithoutMaximum = 40.0f;
+
 __device__ __forceinline__ float reciprocal_approx(float x) {
   float r;
   asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(x));
@@ -236,7 +253,8 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
                                 const int* __restrict__ tiles, const int* __restrict__ seq_starts, const int* __restrict__ first_positions,
                                 const int* __restrict__ block_table, int table_stride, __nv_bfloat16* __restrict__ out, int q_heads,
                                 int kv_heads, int page_size, int window, float scale, float softcap, const float* __restrict__ shifts,
-                                const __nv_bfloat16* __restrict__ gate, int gate_stride, const float* __restrict__ sinks, int* __restrict__ error_flag) {
+                                const __nv_bfloat16* __restrict__ gate, int gate_stride, const float* __restrict__ sinks, int key_dim, int value_dim, int k_page_rows,
+                                int v_page_rows, int* __restrict__ error_flag) {
   extern __shared__ uint8_t smem_raw[];
   using Smem = SmemTC<kD, kVD>;
   constexpr int kKStages = Smem::kKStages, kVStages = Smem::kVStages;
@@ -355,7 +373,11 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
         }
         const int page = t.table[page_index];
         TL(0)
+#if PLANES
+        row = page * (kIsV ? v_page_rows : k_page_rows) + kvh * page_size + in_page;   // row of the plane's [rows, width] view
+#else
         row = ((page * 2 + (kIsV ? 1 : 0)) * kv_heads + kvh) * page_size + in_page;   // row of the [rows, head size] view of the pool
+#endif
 #endif
         if (!mbar_wait(empty + 8 * ring.stage, ring.phase ^ 1, abort_flag)) return false;
         TL(1)
@@ -373,7 +395,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
           else
             tma_load_2d(dst, &map_rot, c * kBoxDims - kPlain, row, bar);
 #else
-          tma_load_2d(dst, &map_kv, c * kBoxDims, row, bar);
+          tma_load_2d(dst, kIsV && PLANES ? &map_v : &map_kv, c * kBoxDims, row, bar);
 #endif
         }
         ring.advance();
@@ -384,7 +406,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
       auto load_q = [&](const RowTile& t) {
         mbar_expect_tx(&sm.q_full, kRowsTC * kD * 2);
 #pragma unroll
-        for (int c = 0; c < kKSubTiles; ++c) tma_load_2d(sm.q + c * kRowsTC * kBoxDims, &map_q, head * kD + c * kBoxDims, t.row0, &sm.q_full);
+        for (int c = 0; c < kKSubTiles; ++c) tma_load_2d(sm.q + c * kRowsTC * kBoxDims, &map_q, head * (PLANES ? key_dim : kD) + c * kBoxDims, t.row0, &sm.q_full);
       };
       bool ok = G > 0;
       if (ok) {
@@ -485,7 +507,8 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
     const uint32_t lane_base = (uint32_t)(sub * 32) << 16;
     // bounded scores arrive in the loop as softcap * tanh in units of log2: nothing is left to scale then
     const float sl2 = kCappedTC ? 1.0f : scale * kLog2eTC;
-    const float cap_to_exp = 2.0f * scale * kLog2eTC / softcap, cap_log2 = softcap * kLog2eTC;
+    const float cap_log2 = softcap * kLog2eTC, cap_inverse = scale / softcap;
+    const bool without_maximum = kCappedTC && softcap <= kCapWithoutMaximum;
     // sigmoid weights, in units of log2: without a bound the exponent is -(score + shift); with one see the loop
     const float sig_to_exp = softcap > 0.0f ? 2.0f * sl2 / softcap : sl2;
     const float sig_twice_cap = softcap > 0.0f ? 2.0f * softcap * kLog2eTC : -1.0f;
@@ -503,7 +526,7 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
       const int my_lo = (window > 0 && my_pos - window + 1 > 0) ? my_pos - window + 1 : 0;
       const uint32_t tmem_o = tmem + lane_base + kOutCol0 + u * kOutStride;
       // The row's reference maximum (times scale * log2 e) that the exponents are taken against, and the sum against it.
-      float reference = -INFINITY, row_sum = 0.0f;
+      float reference = without_maximum ? 0.0f : -INFINITY, row_sum = 0.0f;
       for (int j = 0; j < t.num_kt && ok; ++j, ++g, v_before = v_at, v_at.advance(), at.advance()) {
         const int b = g & 1;
         const int key0 = (t.first_kt + j) * kKeysTC;
@@ -548,14 +571,39 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
             }
           }
         } else {
-          if constexpr (kCappedTC) {   // c tanh(s / c) = c - 2 c u with u = 1 / (1 + e^(2 s / c)), before the mask
-            const Float2Bits to_exp2 = pair_of(cap_to_exp, cap_to_exp), minus_twice2 = pair_of(-2.0f * cap_log2, -2.0f * cap_log2), cap2 = pair_of(cap_log2, cap_log2);
+          if constexpr (kCappedTC) {   // the bound, before the mask
+            float largest = 0.0f, l1 = 0.0f, l2 = 0.0f, l3 = 0.0f;
 #pragma unroll
-            for (int i = 0; i < kKeysTC / 2; ++i) {
-              float x0, x1, u0, u1;
-              unpair(mul2(pair_of(sc[2 * i], sc[2 * i + 1]), to_exp2), x0, x1);
-              inverse_one_plus_exp2(x0, x1, u0, u1);
-              unpair(fma2(pair_of(u0, u1), minus_twice2, cap2), sc[2 * i], sc[2 * i + 1]);
+            for (int i = 0; i < kKeysTC; i += 8) {
+              largest = max3(largest, fabsf(sc[i]), fabsf(sc[i + 1]));
+              l1 = max3(l1, fabsf(sc[i + 2]), fabsf(sc[i + 3]));
+              l2 = max3(l2, fabsf(sc[i + 4]), fabsf(sc[i + 5]));
+              l3 = max3(l3, fabsf(sc[i + 6]), fabsf(sc[i + 7]));
+            }
+            largest = fmaxf(fmaxf(largest, l1), fmaxf(l2, l3));
+            if (__all_sync(0xffffffffu, largest * cap_inverse <= kTanhReach)) {
+              const Float2Bits inverse2 = pair_of(cap_inverse, cap_inverse);
+              Float2Bits poly2[5];
+#pragma unroll
+              for (int n = 0; n < 5; ++n) poly2[n] = pair_of(tanh_poly(n) * cap_log2, tanh_poly(n) * cap_log2);
+#pragma unroll
+              for (int i = 0; i < kKeysTC / 2; ++i) {
+                const Float2Bits t2 = mul2(pair_of(sc[2 * i], sc[2 * i + 1]), inverse2), u2 = mul2(t2, t2);
+                Float2Bits r2 = poly2[4];
+#pragma unroll
+                for (int n = 3; n >= 0; --n) r2 = fma2(r2, u2, poly2[n]);
+                unpair(mul2(t2, r2), sc[2 * i], sc[2 * i + 1]);
+              }
+            } else {   // c tanh(s / c) = c - 2 c u with u = 1 / (1 + e^(2 s / c))
+              const float to_exp = 2.0f * cap_inverse * kLog2eTC;
+              const Float2Bits to_exp2 = pair_of(to_exp, to_exp), minus_twice2 = pair_of(-2.0f * cap_log2, -2.0f * cap_log2), cap2 = pair_of(cap_log2, cap_log2);
+#pragma unroll
+              for (int i = 0; i < kKeysTC / 2; ++i) {
+                float x0, x1, u0, u1;
+                unpair(mul2(pair_of(sc[2 * i], sc[2 * i + 1]), to_exp2), x0, x1);
+                inverse_one_plus_exp2(x0, x1, u0, u1);
+                unpair(fma2(pair_of(u0, u1), minus_twice2, cap2), sc[2 * i], sc[2 * i + 1]);
+              }
             }
           }
           float tile_max = -INFINITY;
@@ -564,9 +612,10 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
             for (int i = 0; i < kKeysTC; ++i) {
               const int key = key0 + i;
               sc[i] = (key >= my_lo && key <= my_pos) ? sc[i] : -INFINITY;
-              tile_max = fmaxf(tile_max, sc[i]);
+              if (!kCappedTC) tile_max = fmaxf(tile_max, sc[i]);
             }
-          } else {
+          }
+          if (kCappedTC ? !without_maximum : !need_mask) {
             float m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;   // four chains of eight three-way maxima instead of one of 64 dependent ones
 #pragma unroll
             for (int i = 0; i < kKeysTC; i += 8) {
@@ -578,7 +627,9 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
             tile_max = fmaxf(fmaxf(tile_max, m1), fmaxf(m2, m3));
           }
           const float scaled_max = tile_max * sl2;
-          if (j == 0) {
+          if (without_maximum) {
+            // every weight is taken against zero
+          } else if (j == 0) {
             reference = scaled_max;   // nothing accumulated yet: the first product overwrites O
           } else {
             // O (in tensor memory) and the sum are taken against `reference`.  They are brought to a new one only when this
@@ -656,9 +707,11 @@ __global__ void __launch_bounds__(kThreadsTC, 2)
           float o[64];
           tmem_ld64(tmem_o + half * 64, o);
           if (row < t.rows_here) {
-            __nv_bfloat16* dst = out + ((size_t)(t.row0 + row) * q_heads + head) * kVD + half * 64;
+            const int width = PLANES ? value_dim : kVD;
+            __nv_bfloat16* dst = out + ((size_t)(t.row0 + row) * q_heads + head) * width + half * 64;
 #pragma unroll
             for (int c = 0; c < 8; ++c)
+              if (!PLANES || half * 64 + c * 8 < value_dim)
               *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(pack_bf16(o[c * 8] * inv, o[c * 8 + 1] * inv), pack_bf16(o[c * 8 + 2] * inv, o[c * 8 + 3] * inv),
                                                                  pack_bf16(o[c * 8 + 4] * inv, o[c * 8 + 5] * inv), pack_bf16(o[c * 8 + 6] * inv, o[c * 8 + 7] * inv));
           }
@@ -710,7 +763,7 @@ template <int kD, int kVD>
 static int launch_attention_tc(const CUtensorMap& map_q, const CUtensorMap& map_kv, const CUtensorMap& map_v, const CUtensorMap& map_rot, const int* tiles, int n_tiles,
                                const int* seq_starts, const int* first_positions, const int* block_table, int table_stride, void* out, int q_heads,
                                int kv_heads, int page_size, int window, float scale, float softcap, const float* shifts, const void* gate, int gate_stride,
-                               const float* sinks, int* error_flag, cudaStream_t stream) {
+                               const float* sinks, int key_dim, int value_dim, int k_page_rows, int v_page_rows, int* error_flag, cudaStream_t stream) {
   // keys of 128 and more: exactly the structure, no room to align it by hand (the kernel checks that it need not): 1 KB more and two CTAs no longer share an SM
 #ifdef TLIE_ATTN_ONE_PER_SM   // for measurements: so much shared memory that a CTA has its SM to itself
   const int smem = 200 * 1024;
@@ -726,7 +779,7 @@ static int launch_attention_tc(const CUtensorMap& map_q, const CUtensorMap& map_
   dim3 grid(q_heads, n_tiles);
   return (int)launch_pdl(prefill_attention_tc_kernel<kD, kVD>, grid, dim3(kThreadsTC), (size_t)smem, stream, map_q, map_kv, map_v, map_rot, tiles, seq_starts, first_positions,
                          block_table, table_stride, (__nv_bfloat16*)out, q_heads, kv_heads, page_size, window, scale, softcap, shifts, (const __nv_bfloat16*)gate, gate_stride,
-                         sinks, error_flag);
+                         sinks, key_dim, value_dim, k_page_rows, v_page_rows, error_flag);
 }
 
 #if LATENT_ROWS
@@ -747,7 +800,29 @@ TLIE_EXPORT int tlie_prefill_attention_rows(const void* q, const void* expanded,
       !make_map_2d(&map_rot, shared, tokens, ROT_DIM, ROT_DIM, kKeysTC))
     return (int)cudaErrorInvalidValue;
   return launch_attention_tc<KEY_DIM, VALUE_DIM>(map_q, map_k, map_v, map_rot, tiles, n_tiles, seq_starts, first_positions, nullptr, 0, out, heads, heads, kKeysTC, 0, scale, 0.0f,
-                                                 nullptr, nullptr, 0, nullptr, error_flag, stream);
+                                                 nullptr, nullptr, 0, nullptr, KEY_DIM, VALUE_DIM, 0, 0, error_flag, stream);
+}
+#elif PLANES
+// q: the step's rows [tokens, q_row_stride] starting with the rotated q heads of key_dim; k_pages / v_pages: the planes, a page's rows (kv_heads x page_size of
+// key_dim / value_dim) k_page_rows / v_page_rows rows apart; num_pages: pages in the pool.  The rest as in tlie_prefill_attention_tc.
+TLIE_EXPORT int tlie_prefill_attention_tc_planes(const void* q, int q_row_stride, int tokens, const void* k_pages, int k_page_rows, const void* v_pages, int v_page_rows, int num_pages,
+                                                 const int* tiles, int n_tiles, const int* seq_starts, const int* first_positions, const int* block_table, int table_stride,
+                                                 void* out, int q_heads, int kv_heads, int key_dim, int value_dim, int page_size, int window, float scale, float softcap,
+                                                 const void* gate, int gate_stride, const float* sinks, int* error_flag, cudaStream_t stream) {
+  if (n_tiles <= 0) return 0;
+  static_assert(KEY_DIM % kBoxDims == 0 && VALUE_DIM % kBoxDims == 0 && KEY_DIM <= 192 && VALUE_DIM <= 128 && !SIGMOID_WEIGHTS, "widths are multiples of a box");
+  if ((softcap > 0.0f) != kCappedTC || kv_heads <= 0 || q_heads % kv_heads != 0 || n_tiles > 65535 || page_size % kKeysTC != 0 || q_row_stride % 8 != 0 || error_flag == nullptr ||
+      key_dim <= 0 || key_dim > KEY_DIM || key_dim % 8 != 0 || value_dim <= 0 || value_dim > VALUE_DIM || value_dim % 8 != 0 || num_pages <= 0)
+    return (int)cudaErrorInvalidValue;
+  const long long plane_rows = (long long)kv_heads * page_size;
+  const long long k_rows = (long long)(num_pages - 1) * k_page_rows + plane_rows, v_rows = (long long)(num_pages - 1) * v_page_rows + plane_rows;
+  if (k_page_rows < plane_rows || v_page_rows < plane_rows) return (int)cudaErrorInvalidValue;
+  CUtensorMap map_q, map_k, map_v;
+  if (!make_map_2d(&map_q, q, tokens, (long long)q_heads * key_dim, q_row_stride, kRowsTC) || !make_map_2d(&map_k, k_pages, k_rows, key_dim, key_dim, kKeysTC) ||
+      !make_map_2d(&map_v, v_pages, v_rows, value_dim, value_dim, kKeysTC))
+    return (int)cudaErrorInvalidValue;
+  return launch_attention_tc<KEY_DIM, VALUE_DIM>(map_q, map_k, map_v, map_k, tiles, n_tiles, seq_starts, first_positions, block_table, table_stride, out, q_heads, kv_heads, page_size,
+                                                 window, scale, softcap, nullptr, gate, gate_stride, sinks, key_dim, value_dim, k_page_rows, v_page_rows, error_flag, stream);
 }
 #else
 // q: the step's rows [tokens, q_row_stride] starting with the rotated q heads (head size 64 or 128); pages: one layer's pool
@@ -769,6 +844,6 @@ TLIE_EXPORT int tlie_prefill_attention_tc(const void* q, int q_row_stride, int t
   if (!make_map_2d(&map_kv, pages, (long long)num_pages * 2 * kv_heads * page_size, head_dim, head_dim, kKeysTC)) return (int)cudaErrorInvalidValue;
   auto launch = head_dim == 64 ? launch_attention_tc<64, 64> : launch_attention_tc<128, 128>;
   return launch(map_q, map_kv, map_kv, map_kv, tiles, n_tiles, seq_starts, first_positions, block_table, table_stride, out, q_heads, kv_heads, page_size, window, scale, softcap,
-                shifts, gate, gate_stride, sinks, error_flag, stream);
+                shifts, gate, gate_stride, sinks, head_dim, head_dim, 0, 0, error_flag, stream);
 }
 #endif

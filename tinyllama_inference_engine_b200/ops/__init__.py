@@ -1029,15 +1029,20 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
         fast.latent_prefill(rows, batch, table, k_ptr, k_stride, sinks, out, heads, key_dim, value_dim, cache.page_size, scale)
         return
     two_planes = not values_in_keys   # what the tensor-core kernels below read
-    if (two_planes and slopes is None and mix is None and window == 0 and rows.dtype == torch.bfloat16 and cache.pages is not None and key_dim == value_dim
-            and rows.shape[1] % 8 == 0 and (gate_offset < 0 or gate_per_head) and _tensor_memory_attention(rows, gate_offset, positions, token_seq, cache, out, heads, kv_heads, key_dim,
-                                                                                                           scale, batch, softcap, sigmoid, shifts, sinks)):
+    unmixed = two_planes and slopes is None and mix is None and window == 0 and rows.dtype == torch.bfloat16
+    planes = (k_ptr, k_stride, v_ptr, v_stride)
+    if (unmixed and rows.shape[1] % 8 == 0 and (gate_offset < 0 or gate_per_head)
+            and _tensor_memory_attention(rows, gate_offset, positions, token_seq, cache, planes, out, heads, kv_heads, key_dim, value_dim, scale, batch, softcap, sigmoid, shifts, sinks)):
         return
     if two_planes and (sigmoid or softcap == 0.0 or slopes is None) and rows.dtype == torch.bfloat16 and fast.mixed_prefill_takes(
             batch, rows, cache.page_size, kv_heads if mix is not None else 1, key_dim, value_dim, gate_offset, gate_per_head, sigmoid, softcap > 0.0):
         folded = folded_slopes if folded_slopes is not None else fast.folded_slopes(slopes, mix)
         fast.mixed_prefill(rows, gate_offset, batch, table, (k_ptr, k_stride, v_ptr, v_stride), folded, mix, out, heads, kv_heads, key_dim, value_dim,
                            cache.page_size, window, scale, keep_first if window > 0 else 0, gate_per_head, softcap, sigmoid, shifts, sinks)
+        return
+    if unmixed and batch is not None and not sigmoid and fast.heads_decode_takes(rows, cache.page_size, heads, kv_heads, key_dim, value_dim):
+        fast.heads_decode(rows, gate_offset, gate_per_head, positions, token_seq, table, planes, out, heads, kv_heads, key_dim, value_dim, cache.page_size, scale, softcap, sinks,
+                          batch.max_seq_len)
         return
     # few rows over long contexts (decode steps): every row's keys are dealt to several CTAs
     splits, partial = 1, None
@@ -1059,24 +1064,36 @@ def mixed_heads_attention(rows, gate_offset: int, positions, token_seq, cache, s
            "mixed_heads_attention")
 
 
-def _tensor_memory_attention(rows, gate_offset: int, positions, token_seq, cache, out, heads: int, kv_heads: int, dim: int, scale: float, batch, softcap: float,
-                             sigmoid: bool, shifts, sinks) -> bool:
-    """Attention of a step that carries prompt portions on the tensor-memory kernel (sigmoid weights, bounded scores and sinks each in a build that has them);
-    decoding requests at the step's head run on the kernel of few rows.  False: the step or the sizes are not for it."""
+def _tensor_memory_attention(rows, gate_offset: int, positions, token_seq, cache, planes, out, heads: int, kv_heads: int, key_dim: int, value_dim: int, scale: float, batch,
+                             softcap: float, sigmoid: bool, shifts, sinks) -> bool:
+    """Attention of a step that carries prompt portions on the tensor-memory kernel (sigmoid weights, bounded scores, and planes of two widths each in a build
+    that has them); decoding requests at the step's head run on the kernels of few rows.  False: the step or the sizes are not for it."""
     host_q_lens = getattr(batch, "host_q_lens", None)
     if host_q_lens is None:
         return False
     lead = fast.leading_single_rows(host_q_lens)
-    tiles = fast.tc_attention_tiles(batch, dim, cache.page_size, lead)
-    if tiles is None or (lead and not fast.mixed_decode_takes(rows, heads, kv_heads, dim, dim, gate_offset, False, True)):
+    one_tensor = cache.pages is not None and key_dim == value_dim and key_dim in fast.TC_ATTENTION_HEAD_DIMS
+    if not one_tensor and (sigmoid or not fast.tc_planes_fit(key_dim, value_dim)):
         return False
-    if lead:
-        planes = _plane_pointers(cache, kv_heads, dim, dim)[1:]
+    tiles = fast.tc_attention_tiles(batch, key_dim if one_tensor else None, cache.page_size, lead)
+    if tiles is None:
+        return False
+    by_heads = not sigmoid and fast.heads_decode_takes(rows, cache.page_size, heads, kv_heads, key_dim, value_dim)
+    if lead and not by_heads and not fast.mixed_decode_takes(rows, heads, kv_heads, key_dim, value_dim, gate_offset, False, True):
+        return False
+    if lead and by_heads:
+        fast.heads_decode(rows[:lead], gate_offset, True, positions[:lead], token_seq[:lead], cache.block_table, planes, out[:lead], heads, kv_heads, key_dim, value_dim, cache.page_size,
+                          scale, softcap, sinks, batch.max_seq_len)
+    elif lead:
         splits = max(1, min(2 * fast.sm_count() // lead, -(-batch.max_seq_len // 32), 64))
-        fast.mixed_decode(rows[:lead], gate_offset, positions[:lead], token_seq[:lead], cache.block_table, planes, None, None, out[:lead], heads, kv_heads, dim, dim, cache.page_size, 0,
-                          scale, splits, 0, True, softcap, sigmoid, shifts, sinks)
-    fast.prefill_attention_tc(rows, cache.pages, tiles, batch.seq_starts, batch.first_positions, cache.block_table, out, heads, kv_heads, dim, cache.page_size, 0, scale, softcap, sigmoid,
-                              shifts, gate_offset, sinks)
+        fast.mixed_decode(rows[:lead], gate_offset, positions[:lead], token_seq[:lead], cache.block_table, planes, None, None, out[:lead], heads, kv_heads, key_dim, value_dim,
+                          cache.page_size, 0, scale, splits, 0, True, softcap, sigmoid, shifts, sinks)
+    if one_tensor:
+        fast.prefill_attention_tc(rows, cache.pages, tiles, batch.seq_starts, batch.first_positions, cache.block_table, out, heads, kv_heads, key_dim, cache.page_size, 0, scale, softcap,
+                                  sigmoid, shifts, gate_offset, sinks)
+    else:
+        fast.prefill_attention_tc_planes(rows, cache.pages if cache.pages is not None else cache.plane_pages[0], planes, tiles, batch.seq_starts, batch.first_positions, cache.block_table, out,
+                                         heads, kv_heads, key_dim, value_dim, cache.page_size, scale, softcap, gate_offset, sinks)
     return True
 
 

@@ -28,6 +28,7 @@ def sm_count() -> int:
 DEFAULT_HEAD_DIMS = (64, 128)
 DEFAULT_MIXED_PREFILL_SETS = ((64, 64, 4), (128, 128, 8))   # (key width, value width, key heads per folded query) built ahead; others on first use
 DEFAULT_SIGMOID_SETS = ((64, 64, 4), (128, 128, 4))   # (key width, value width, key/value heads) of attention with sigmoid weights built ahead; others on first use
+DEFAULT_HEADS_DECODE_SETS = ((64, 64), (128, 128), (192, 128))   # (key width, value width) of softmax attention of single rows built ahead; others on first use
 DEFAULT_DIFF_SETS = ((64, 128), (128, 128))   # (key width per map, value width) of differential attention built ahead; others on first use
 _scratch: dict[torch.device, list[torch.Tensor]] = {}
 
@@ -42,6 +43,8 @@ def build_all() -> list:
     built.append(build_library("tlie_attn_prefill_tc", ["attention_prefill_tc.cu"]))
     built.append(build_library("tlie_attn_prefill_tc_sigmoid", ["attention_prefill_tc.cu"], {"SIGMOID_WEIGHTS": 1}))
     built.append(build_library("tlie_attn_prefill_tc_capped", ["attention_prefill_tc.cu"], {"SCORE_CAP": 1}))
+    built.append(build_library("tlie_attn_prefill_tc_planes_k192_v128_capped", ["attention_prefill_tc.cu"], {"PLANES": 1, "KEY_DIM": 192, "VALUE_DIM": 128, "SCORE_CAP": 1}))
+    built += [build_library(f"tlie_attn_heads_decode_k{k}_v{v}", ["attention_heads_decode.cu"], {"KEY_DIM": k, "VALUE_DIM": v}) for k, v in DEFAULT_HEADS_DECODE_SETS]
     built.append(build_library("tlie_probes", ["probes.cu"]))
     for key_dim, value_dim, parts in DEFAULT_MIXED_PREFILL_SETS:
         built.append(build_library(f"tlie_attn_mixed_k{key_dim}_v{value_dim}_p{parts}", ["attention_mixed_prefill.cu"], {"KEY_DIM": key_dim, "VALUE_DIM": value_dim, "PARTS": parts}))
@@ -673,11 +676,11 @@ def tc_attention_library(sigmoid: bool = False, capped: bool = False):
     return load_library("tlie_attn_prefill_tc", ["attention_prefill_tc.cu"])
 
 
-def tc_attention_tiles(batch, head_dim: int, page_size: int, lead: int):
+def tc_attention_tiles(batch, head_dim: int | None, page_size: int, lead: int):
     """The step's row tiles for the tensor-memory kernel, or None if the step or the sizes are not for it (``lead``: the single rows at the
-    step's head, which the tiles leave out)."""
+    step's head, which the tiles leave out; ``head_dim`` None: the widths have been looked at)."""
     tiles = batch.plan("attention_tiles_tc")
-    if not use_tc_attention or tiles is None or head_dim not in TC_ATTENTION_HEAD_DIMS or page_size % 64 != 0:
+    if not use_tc_attention or tiles is None or (head_dim is not None and head_dim not in TC_ATTENTION_HEAD_DIMS) or page_size % 64 != 0:
         return None
     return tiles if batch.num_tokens - lead >= TC_ATTENTION_MIN_ROWS_PER_TILE * tiles.shape[0] else None
 
@@ -703,6 +706,38 @@ def prefill_attention_tc(qkv, pages, tiles, seq_starts, first_positions, block_t
         ),
         "prefill_attention_tc",
     )
+
+
+def tc_planes_fit(key_dim: int, value_dim: int) -> bool:
+    """Whether the tensor-memory kernel has a build for keys and values of these widths in planes of their own."""
+    return key_dim % 8 == 0 and value_dim % 8 == 0 and 0 < key_dim <= 192 and 0 < value_dim <= 128
+
+
+def tc_planes_library(key_dim: int, value_dim: int, capped: bool):
+    """One build per (widths rounded up to whole 64-wide boxes, bounded scores or not): compiled when a model of these sizes first runs a prompt."""
+    k, v = -(-key_dim // 64) * 64, -(-value_dim // 64) * 64
+    defines = {"PLANES": 1, "KEY_DIM": k, "VALUE_DIM": v}
+    return load_library(f"tlie_attn_prefill_tc_planes_k{k}_v{v}" + ("_capped" if capped else ""), ["attention_prefill_tc.cu"], {**defines, "SCORE_CAP": 1} if capped else defines)
+
+
+def prefill_attention_tc_planes(rows, pool, planes, tiles, seq_starts, first_positions, block_table, out, heads: int, kv_heads: int, key_dim: int, value_dim: int, page_size: int,
+                                scale: float, softcap: float = 0.0, gate_offset: int = -1, sinks=None) -> None:
+    """``prefill_attention_tc`` for keys and values in planes of any two widths (``tc_planes_fit``): ``planes`` = (key plane, its page stride in elements, value plane, its
+    page stride), ``pool`` the tensor whose first axis counts the pages.  A softmax; ``softcap``, ``sinks`` and one gate per head as there."""
+    ops = _ops()
+    if not tc_planes_fit(key_dim, value_dim) or page_size % 64 != 0:
+        raise KernelError("the tensor-memory attention takes widths that are multiples of 8 up to 192 and 128 and pages of a multiple of 64 keys", code="invalid_shape")
+    k_ptr, k_stride, v_ptr, v_stride = planes
+    if k_stride % key_dim or v_stride % value_dim:
+        raise KernelError("a plane's page stride is whole rows", code="invalid_shape")
+    gate = c_void_p(0) if gate_offset < 0 else c_void_p(rows.data_ptr() + gate_offset * rows.element_size())
+    ops._check(
+        tc_planes_library(key_dim, value_dim, softcap > 0.0).tlie_prefill_attention_tc_planes(
+            ops._ptr(rows), c_int(rows.shape[1]), c_int(rows.shape[0]), k_ptr, c_int(k_stride // key_dim), v_ptr, c_int(v_stride // value_dim), c_int(pool.shape[0]), ops._i32(tiles, "tiles"),
+            c_int(tiles.shape[0]), ops._i32(seq_starts, "seq_starts"), ops._i32(first_positions, "first_positions"), ops._i32(block_table, "block_table"), c_int(block_table.shape[1]),
+            ops._ptr(out), c_int(heads), c_int(kv_heads), c_int(key_dim), c_int(value_dim), c_int(page_size), c_int(0), c_float(scale), c_float(softcap), gate, c_int(rows.shape[1]),
+            ops._ptr(sinks), ops._ptr(tcgen05_error_flag(rows.device)), ops._stream()),
+        "prefill_attention_tc_planes")
 
 
 def paged_attention_bf16(qkv, pages, positions, token_seq, block_table, out, q_heads, kv_heads, head_dim, page_size, window, scale, batch) -> bool:
@@ -954,6 +989,43 @@ def mixed_decode(rows, gate_offset: int, positions, token_seq, block_table, plan
             c_int(tokens), c_int(heads), c_int(kv_heads), c_int(page_size), c_int(window), c_float(scale), c_int(splits), ops._ptr(partial), c_int(keep_first),
             c_int(1 if gate_per_head else 0), c_float(softcap), c_int(1 if sigmoid else 0), ops._ptr(shifts), ops._ptr(sinks), ops._stream()),
         "mixed_decode")
+
+
+# --- softmax attention of single rows, heads unmixed, planes of any two widths --------------------------------------------------------
+use_heads_decode = True
+
+
+def heads_decode_library(key_dim: int, value_dim: int):
+    """The kernel set of one pair of widths: compiled when a model of these sizes first decodes."""
+    lib = load_library(f"tlie_attn_heads_decode_k{key_dim}_v{value_dim}", ["attention_heads_decode.cu"], {"KEY_DIM": key_dim, "VALUE_DIM": value_dim})
+    if not getattr(lib, "_tlie_typed", False):
+        lib.tlie_heads_decode_scratch_floats.restype = c_longlong
+        lib._tlie_typed = True
+    return lib
+
+
+def heads_decode_takes(rows, page_size: int, heads: int, kv_heads: int, key_dim: int, value_dim: int) -> bool:
+    """Whether a step of few rows per request runs its (unmixed, unwindowed) softmax attention on csrc/attention_heads_decode.cu."""
+    return (use_heads_decode and rows.dtype == torch.bfloat16 and key_dim % 16 == 0 and value_dim % 16 == 0 and key_dim <= 256 and value_dim <= 128 and heads // kv_heads <= 16
+            and rows.stride(0) % 2 == 0 and page_size % 16 == 0 and rows.shape[0] * kv_heads <= 16384)
+
+
+def heads_decode(rows, gate_offset: int, gate_per_head: bool, positions, token_seq, block_table, planes, out, heads: int, kv_heads: int, key_dim: int, value_dim: int, page_size: int,
+                 scale: float, softcap: float, sinks, max_seq_len: int) -> None:
+    """Every row of ``rows`` over its request's keys up to its own position; ``planes`` as in ``mixed_prefill``.  A row's keys are dealt to several CTAs where there are
+    fewer (row, key/value head) pairs than SMs."""
+    ops = _ops()
+    tokens = rows.shape[0]
+    lib = heads_decode_library(key_dim, value_dim)
+    splits = decode_splits(tokens, kv_heads, max_seq_len)
+    buffer = scratch(rows.device, lib.tlie_heads_decode_scratch_floats(c_int(tokens), c_int(heads), c_int(splits)))
+    k_ptr, k_stride, v_ptr, v_stride = planes
+    ops._check(
+        lib.tlie_heads_decode(
+            ops._ptr(rows), c_int(rows.stride(0)), c_int(gate_offset), c_int(1 if gate_per_head else 0), k_ptr, c_longlong(k_stride), v_ptr, c_longlong(v_stride),
+            ops._i32(positions, "positions"), ops._i32(token_seq, "token_seq"), ops._i32(block_table, "block_table"), c_int(block_table.shape[1]), ops._ptr(out), ops._ptr(buffer),
+            c_int(tokens), c_int(heads), c_int(kv_heads), c_int(page_size), c_float(scale), c_float(softcap), ops._ptr(sinks), c_int(splits), ops._stream()),
+        "heads_decode")
 
 
 if os.environ.get("TLIE_SKINNY", "0") == "1":
