@@ -553,6 +553,49 @@ def test_gated_linear_attention_kernels(dtype, atol, heads, dim, vdim, rank, tau
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("heads,dim,vdim", [(2, 16, 32), (1, 200, 40), (3, 33, 7), (2, 128, 64)])
+@pytest.mark.parametrize("lens", [[600, 1, 128, 129, 256, 257], [30, 513], [1024]])
+def test_long_entries_of_the_recurrence_in_chunks(heads, dim, vdim, lens):
+    """Entries of all lengths around whole chunks beside short ones, from states that are not zero, strong and weak decays: what the chunks give is what the
+    rows in order give, and so is the state they leave."""
+    from types import SimpleNamespace
+
+    from tinyllama_inference_engine_b200 import ops
+
+    assert max(lens) >= ops.RECURRENCE_CHUNKS_MIN_ROWS
+    g = torch.Generator().manual_seed(sum(lens) + dim)
+    qk, values, total = heads * dim, heads * vdim, sum(lens)
+    starts = np.concatenate([[0], np.cumsum(lens)])
+    parts = [torch.randn(total, n, generator=g) for n in (qk, qk, values)]
+    decay = torch.sigmoid(torch.randn(total, qk, generator=g) + torch.linspace(-1.0, 8.0, qk)) ** 0.25
+    prep = torch.cat([*parts, torch.ones(total, heads), decay], dim=1).cuda().contiguous()
+    slots = list(range(len(lens)))[::-1]
+    words = ops.delta_state_words(heads, dim, vdim, 0, 1)[0]
+    step = lambda a, b, order: SimpleNamespace(seq_starts=torch.tensor(np.concatenate([[0], np.cumsum([y - x for x, y in zip(a, b)])]), dtype=torch.int32).cuda(),
+                                               state_slots=torch.tensor([slots[i] for i in order], dtype=torch.int32).cuda(), num_seqs=len(order), max_q_len=max(y - x for x, y in zip(a, b)))
+    before, state = torch.zeros(len(lens), words, device="cuda"), None
+    ops.delta_rule(prep[: len(lens)].contiguous(), before, step([0] * len(lens), [1] * len(lens), range(len(lens))), torch.zeros(len(lens), values, device="cuda"), heads, heads, dim, vdim, plain=True)
+    results = {}
+    for chunks in (True, False):
+        kept, ops.use_recurrence_chunks = ops.use_recurrence_chunks, chunks
+        try:
+            state, out = before.clone(), torch.full((total, values), float("nan"), device="cuda")
+            launches = ops.launch_count
+            ops.delta_rule(prep, state, step(starts[:-1], starts[1:], range(len(lens))), out, heads, heads, dim, vdim, plain=True)
+            assert ops.launch_count - launches == (3 if chunks else 1)
+            results[chunks] = (out.cpu(), state.cpu())
+        finally:
+            ops.use_recurrence_chunks = kept
+    for got, want in zip(*results.values()):
+        assert torch.isfinite(got).all() and float((got - want).abs().max()) <= 2e-6 * float(want.abs().max())
+    q, k, v, fade = (t.double() for t in (*parts, decay))
+    for e, (a, b) in enumerate(zip(starts[:-1], starts[1:])):      # the row that wrote the state a request starts from comes first
+        rows = [torch.cat([t[e:e + 1], t[a:b]]).view(b - a + 1, heads, -1) for t in (q, k, v, fade)]
+        want = plain_vogusun.gated_linear_recurrence(*rows)[1:].reshape(b - a, values)
+        assert float((results[True][0][a:b].double() - want).abs().max()) <= 2e-5 * max(1.0, float(want.abs().max())), e
+
+
+@pytest.mark.gpu
 @pytest.mark.parametrize("tokens", [50, 1300])    # a CTA per token; four tokens per CTA (a step of many rows), the last CTA short of rows
 @pytest.mark.parametrize("experts,top,width", [(8, 3, 64), (6, 2, 44), (4, 1, 32), (64, 8, 128), (5, 5, 24), (40, 36, 48), (10, 3, 42), (7, 7, 17)])
 def test_router_over_chosen_logits(tokens, experts, top, width):

@@ -125,31 +125,76 @@ __device__ __forceinline__ void delta_commit() { asm volatile("cp.async.commit_g
 template <int N>
 __device__ __forceinline__ void delta_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
 
+// A long entry of the plain recurrence is cut into chunks of kChunkRows rows that run side by side, since without the correction a row only scales the state
+// and adds to it: the state behind a chunk is (the product of its decays) times the state in front of it plus what the chunk alone would leave.
+//   CHUNKED_LOCAL  a CTA per (entry, head, columns, chunk but the last): the chunk from a zero state, nothing read out; leaves its end and its decays' product
+//   delta_chunk_starts_kernel   every state element by itself: from the request's state through the chunks' ends to the state in front of every chunk
+//   CHUNKED_READ   every chunk from the state in front of it, with the read-outs; the last one leaves the request's state
+// The chunks are enough CTAs for a thread to own COLS columns of the state, which its reads of a row's q, k and decays then serve: with one column a
+// thread the reads of shared memory set the pace (16 heads of 128 x 128, 2,048 rows: 0.43 ms in chunks, 0.57 in one run).
+// All of it in 32-bit.  Chunk c of entry e has the place seq_starts[e] / kChunkRows + e + c in the scratch: no two chunks share one, and there are at most
+// tokens / kChunkRows + entries.
+constexpr int kChunkRows = 128;
+enum { WHOLE = 0, CHUNKED_LOCAL = 1, CHUNKED_READ = 2 };
+
 // R: key channels a lane has registers for (a multiple of 4, dim <= 8 R); the state holds 4 ceil(dim / 32) of them per lane.
 // A row's operands ([q | k | g] of the head, the CTA's 16 values, beta) are copied asynchronously into a ring of kDeltaStages
 // buffers, several rows ahead, so that a row's turn never waits for memory; padding words are zeroed once and never copied.
 // PLAIN: u = beta v needs nothing of the state, so the chain from one row to the next is S <- g S + k u alone and the read-out's sums and
 // shuffles (o = S^T q of the new state) hang off it; with the correction u waits for k . S_j, reduced over the column's lanes, in every row.
-template <int R, bool PLAIN>
+// The sums over a column's lanes of COLS columns at once: the first steps halve what a lane holds (it keeps one half of the columns and hands over the other), so
+// that COLS columns cost COLS - 1 shuffles and a few more instead of log2(lanes) each.  Returns the finished sum and which column it belongs to; the
+// kDeltaLanes / COLS lanes that share a column hold the same.
+template <int COLS>
+__device__ __forceinline__ float sum_columns(float (&reads)[COLS], int lane, int& which) {
+  which = 0;
+  int offset = kDeltaLanes / 2;
+#pragma unroll
+  for (int held = COLS; held > 1; held >>= 1, offset >>= 1) {
+    const bool upper = (lane & offset) != 0;
+#pragma unroll
+    for (int i = 0; i < held / 2; ++i) {
+      const float keep = upper ? reads[i + held / 2] : reads[i], send = upper ? reads[i] : reads[i + held / 2];
+      reads[i] = keep + __shfl_xor_sync(0xffffffffu, send, offset);
+    }
+    if (upper) which += held / 2;
+  }
+#pragma unroll
+  for (; offset > 0; offset >>= 1) reads[0] += __shfl_xor_sync(0xffffffffu, reads[0], offset);
+  return reads[0];
+}
+
+template <int R, bool PLAIN, int MODE = WHOLE, int COLS = 1>
 __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(const float* __restrict__ prep, float* __restrict__ state, long long state_stride,
                                                                   const int* __restrict__ seq_starts, const int* __restrict__ state_slots, float* __restrict__ out,
-                                                                  int heads, int kv_heads, int dim, int vdim) {
-  extern __shared__ __align__(16) float stage_s[];   // kDeltaStages buffers of [q: 8 R | k: 8 R | g: 8 R | v: 16 | beta | 3 unused]
+                                                                  int heads, int kv_heads, int dim, int vdim, float* __restrict__ chunk_states,
+                                                                  float* __restrict__ chunk_decays) {
+  static_assert((PLAIN || MODE == WHOLE) && (MODE != WHOLE || COLS == 1) && COLS <= kDeltaLanes, "only the plain recurrence is cut into chunks, and only chunks have several columns a thread");
+  extern __shared__ __align__(16) float stage_s[];   // kDeltaStages buffers of [q: 8 R | k: 8 R | g: 8 R | v: 16 COLS | beta | 3 unused]
   constexpr int kPadded = kDeltaLanes * R;
-  constexpr int kRow = 3 * kPadded + kDeltaColumns + 4;
+  constexpr int kBlockColumns = kDeltaColumns * COLS;
+  constexpr int kRow = 3 * kPadded + kBlockColumns + 4;
   constexpr int kLoads = (kRow + kDeltaThreads - 1) / kDeltaThreads;
-  const int column_blocks = (vdim + kDeltaColumns - 1) / kDeltaColumns;
+  const int column_blocks = (vdim + kBlockColumns - 1) / kBlockColumns;
   const int head = blockIdx.x / column_blocks, block = blockIdx.x - head * column_blocks;
   const int entry = blockIdx.y;
-  const int tid = threadIdx.x, lane = tid & (kDeltaLanes - 1), column = block * kDeltaColumns + tid / kDeltaLanes;
+  const int tid = threadIdx.x, lane = tid & (kDeltaLanes - 1), column = block * kBlockColumns + tid / kDeltaLanes;   // a thread's columns: this one and every kDeltaColumns-th behind it
   const bool live = column < vdim;
-  const int first = seq_starts[entry], count = seq_starts[entry + 1] - first;
+  const int entry_first = seq_starts[entry], entry_count = seq_starts[entry + 1] - entry_first;
+  const int chunk = MODE == WHOLE ? 0 : blockIdx.z;
+  const bool last_chunk = MODE == WHOLE || (chunk + 1) * kChunkRows >= entry_count;
+  if (MODE != WHOLE && (chunk * kChunkRows >= entry_count || (MODE == CHUNKED_LOCAL && last_chunk))) return;
+  const int first = entry_first + chunk * kChunkRows, count = MODE == WHOLE ? entry_count : min(kChunkRows, entry_count - chunk * kChunkRows);
   const int kv = head / (heads / kv_heads);
   const int qk = kv_heads * dim;
   const int width = 2 * qk + heads * vdim + heads + heads * dim;
   const int held = 4 * ((dim + 4 * kDeltaLanes - 1) / (4 * kDeltaLanes));   // key channels per lane that are stored
   const size_t matrix = (size_t)held * vdim * kDeltaLanes;
   float* mine = state + (size_t)state_slots[entry] * state_stride + (size_t)head * matrix;
+  // where this run starts from and what it leaves: the request's state, or a chunk's place in the scratch
+  const size_t place = MODE == WHOLE ? 0 : (size_t)(entry_first / kChunkRows + entry + chunk) * heads + head;
+  const float* from_state = (MODE == CHUNKED_READ && entry_count > kChunkRows) ? chunk_states + place * matrix : mine;
+  float* to_state = MODE == CHUNKED_LOCAL ? chunk_states + place * matrix : mine;
 
   // where each word of a staged row comes from in a prep row (-1: padding, stays zero)
   int source[kLoads];
@@ -157,18 +202,24 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(const float* 
   for (int i = 0; i < kLoads; ++i) {
     const int w = tid + i * kDeltaThreads;
     int at = -1;
-    if (w < kPadded) at = w < dim ? kv * dim + w : -1;
+    if (w < kPadded) at = w < dim && MODE != CHUNKED_LOCAL ? kv * dim + w : -1;
     else if (w < 2 * kPadded) at = w - kPadded < dim ? qk + kv * dim + (w - kPadded) : -1;
     else if (w < 3 * kPadded) at = w - 2 * kPadded < dim ? 2 * qk + heads * vdim + heads + head * dim + (w - 2 * kPadded) : -1;
-    else if (w < 3 * kPadded + kDeltaColumns) at = block * kDeltaColumns + (w - 3 * kPadded) < vdim ? 2 * qk + head * vdim + block * kDeltaColumns + (w - 3 * kPadded) : -1;
-    else if (w == 3 * kPadded + kDeltaColumns) at = 2 * qk + heads * vdim + head;
+    else if (w < 3 * kPadded + kBlockColumns) at = block * kBlockColumns + (w - 3 * kPadded) < vdim ? 2 * qk + head * vdim + block * kBlockColumns + (w - 3 * kPadded) : -1;
+    else if (w == 3 * kPadded + kBlockColumns) at = 2 * qk + heads * vdim + head;
     source[i] = at;
   }
   for (int i = tid; i < kDeltaStages * kRow; i += kDeltaThreads) stage_s[i] = 0.0f;
   __syncthreads();
-  float S[R];
+  float S[COLS][R];
 #pragma unroll
-  for (int i = 0; i < R; ++i) S[i] = (live && i < held) ? mine[((size_t)i * vdim + column) * kDeltaLanes + lane] : 0.0f;
+  for (int n = 0; n < COLS; ++n)
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+      S[n][i] = (MODE != CHUNKED_LOCAL && column + n * kDeltaColumns < vdim && i < held) ? from_state[((size_t)i * vdim + column + n * kDeltaColumns) * kDeltaLanes + lane] : 0.0f;
+  float faded[MODE == CHUNKED_LOCAL ? R : 1];   // the product of the chunk's decays: every column of a head fades alike, so the first columns' CTA has it
+#pragma unroll
+  for (int i = 0; i < (MODE == CHUNKED_LOCAL ? R : 1); ++i) faded[i] = 1.0f;
 
   auto issue = [&](int block_of_rows) {   // one group per block of rows, empty past the end, so that the count of groups in flight is the same at every step
 #pragma unroll
@@ -195,39 +246,60 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(const float* 
     if constexpr (PLAIN) {
       // the block's four rows: the state's chain first, every row leaving its share of the read-out; then the four sums across the column's
       // lanes side by side, so that a round of shuffles is waited for once per block and not once per row
-      float reads[kDeltaBlock];
+      float reads[kDeltaBlock][COLS];
 #pragma unroll
       for (int n = 0; n < kDeltaBlock; ++n) {
         const int row = block_of_rows * kDeltaBlock + n;
-        reads[n] = 0.0f;
+#pragma unroll
+        for (int m = 0; m < COLS; ++m) reads[n][m] = 0.0f;
         if (row < count) {
           const float* cur = stage_s + (row % kDeltaStages) * kRow;
-          const float u = cur[3 * kPadded + kDeltaColumns] * cur[3 * kPadded + (tid / kDeltaLanes)];   // beta v
-          float read2[2] = {0.0f, 0.0f};
+          float u[COLS], read2[COLS][2];
+#pragma unroll
+          for (int m = 0; m < COLS; ++m) {
+            u[m] = cur[3 * kPadded + kBlockColumns] * cur[3 * kPadded + tid / kDeltaLanes + m * kDeltaColumns];   // beta v
+            read2[m][0] = read2[m][1] = 0.0f;
+          }
 #pragma unroll
           for (int j = 0; j < R / 4; ++j) {
-            const float4 q4 = *reinterpret_cast<const float4*>(cur + j * 4 * kDeltaLanes + lane * 4);
             const float4 k4 = *reinterpret_cast<const float4*>(cur + kPadded + j * 4 * kDeltaLanes + lane * 4);
             const float4 g4 = *reinterpret_cast<const float4*>(cur + 2 * kPadded + j * 4 * kDeltaLanes + lane * 4);
-            const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, g[4] = {g4.x, g4.y, g4.z, g4.w};
+            const float k[4] = {k4.x, k4.y, k4.z, k4.w}, g[4] = {g4.x, g4.y, g4.z, g4.w};
+            float q[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+            if constexpr (MODE != CHUNKED_LOCAL) {
+              const float4 q4 = *reinterpret_cast<const float4*>(cur + j * 4 * kDeltaLanes + lane * 4);
+              q[0] = q4.x, q[1] = q4.y, q[2] = q4.z, q[3] = q4.w;
+            }
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
               const int i = 4 * j + c;
-              S[i] = S[i] * g[c] + k[c] * u;
-              read2[c & 1] += q[c] * S[i];
+#pragma unroll
+              for (int m = 0; m < COLS; ++m) {
+                S[m][i] = S[m][i] * g[c] + k[c] * u[m];
+                if constexpr (MODE != CHUNKED_LOCAL) read2[m][c & 1] += q[c] * S[m][i];
+              }
+              if constexpr (MODE == CHUNKED_LOCAL) {
+                if (block == 0) faded[i] *= g[c];
+              }
             }
           }
-          reads[n] = read2[0] + read2[1];
+#pragma unroll
+          for (int m = 0; m < COLS; ++m) reads[n][m] = read2[m][0] + read2[m][1];
         }
       }
+      if constexpr (MODE != CHUNKED_LOCAL) {
+        float total[kDeltaBlock];
+        int which = 0;
 #pragma unroll
-      for (int offset = kDeltaLanes / 2; offset > 0; offset >>= 1)
+        for (int n = 0; n < kDeltaBlock; ++n) total[n] = sum_columns(reads[n], lane, which);
+        const int mine_at = column + which * kDeltaColumns;
+        if (mine_at < vdim && (lane & (kDeltaLanes / COLS - 1)) == 0) {
 #pragma unroll
-        for (int n = 0; n < kDeltaBlock; ++n) reads[n] += __shfl_xor_sync(0xffffffffu, reads[n], offset);
-#pragma unroll
-      for (int n = 0; n < kDeltaBlock; ++n) {
-        const int row = block_of_rows * kDeltaBlock + n;
-        if (row < count && live && lane == 0) out[(size_t)(first + row) * heads * vdim + head * vdim + column] = reads[n];
+          for (int n = 0; n < kDeltaBlock; ++n) {
+            const int row = block_of_rows * kDeltaBlock + n;
+            if (row < count) out[(size_t)(first + row) * heads * vdim + head * vdim + mine_at] = total[n];
+          }
+        }
       }
     } else {
 #pragma unroll
@@ -247,9 +319,9 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(const float* 
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           const int i = 4 * j + c;
-          S[i] *= g[c];
-          reach2[c & 1] += k[c] * S[i];
-          read2[c & 1] += q[c] * S[i];
+          S[0][i] *= g[c];
+          reach2[c & 1] += k[c] * S[0][i];
+          read2[c & 1] += q[c] * S[0][i];
           both2[c & 1] += q[c] * k[c];
           kk[i] = k[c];
         }
@@ -264,16 +336,61 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(const float* 
       const float v = cur[3 * kPadded + (tid / kDeltaLanes)], beta = cur[3 * kPadded + kDeltaColumns];
       const float u = beta * (v - reach);
 #pragma unroll
-      for (int i = 0; i < R; ++i) S[i] += kk[i] * u;
+      for (int i = 0; i < R; ++i) S[0][i] += kk[i] * u;
       if (live && lane == 0) out[(size_t)(first + row) * heads * vdim + head * vdim + column] = read + both * u;
     }
     }
   }
   delta_wait<0>();
-  if (live && count > 0) {
+  if (count > 0 && (MODE == CHUNKED_LOCAL || last_chunk)) {
 #pragma unroll
-    for (int i = 0; i < R; ++i)
-      if (i < held) mine[((size_t)i * vdim + column) * kDeltaLanes + lane] = S[i];
+    for (int n = 0; n < COLS; ++n)
+#pragma unroll
+      for (int i = 0; i < R; ++i)
+        if (column + n * kDeltaColumns < vdim && i < held) to_state[((size_t)i * vdim + column + n * kDeltaColumns) * kDeltaLanes + lane] = S[n][i];
+  }
+  if constexpr (MODE == CHUNKED_LOCAL) {
+    if (column == 0) {
+#pragma unroll
+      for (int i = 0; i < R; ++i)
+        if (i < held) chunk_decays[(place * held + i) * kDeltaLanes + lane] = faded[i];
+    }
+  }
+}
+
+// chunk_states [place][head][held][vdim][lanes] holds what every chunk but an entry's last leaves by itself and receives the state in front of every chunk.
+// A thread per element of the heads' matrices, blockIdx.y an entry; entries of one chunk are read and left in the request's state directly.
+__global__ void __launch_bounds__(256) delta_chunk_starts_kernel(const float* __restrict__ state, long long state_stride, const int* __restrict__ seq_starts,
+                                                                 const int* __restrict__ state_slots, float* __restrict__ chunk_states, const float* __restrict__ chunk_decays,
+                                                                 int heads, int held, int vdim) {
+  const int entry = blockIdx.y;
+  const int first = seq_starts[entry], count = seq_starts[entry + 1] - first;
+  const int chunks = (count + kChunkRows - 1) / kChunkRows;
+  const size_t matrix = (size_t)held * vdim * kDeltaLanes, all = heads * matrix;
+  const size_t at = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (chunks < 2 || at >= all) return;
+  const size_t head = at / matrix, in_matrix = at - head * matrix;
+  const size_t i = in_matrix / ((size_t)vdim * kDeltaLanes), lane = in_matrix % kDeltaLanes;
+  const size_t place0 = (size_t)(first / kChunkRows + entry);
+  float* mine = chunk_states + place0 * all + at;
+  const float* decays = chunk_decays + ((place0 * heads + head) * held + i) * kDeltaLanes + lane;
+  const size_t decay_step = (size_t)heads * held * kDeltaLanes;
+  float S = state[(size_t)state_slots[entry] * state_stride + at];
+  constexpr int kAhead = 8;   // chunks whose numbers are asked for before the first is used
+  for (int c0 = 0; c0 < chunks; c0 += kAhead) {
+    float left[kAhead], decay[kAhead];
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j) {
+      const bool inner = c0 + j + 1 < chunks;
+      left[j] = inner ? mine[(size_t)(c0 + j) * all] : 0.0f;
+      decay[j] = inner ? decays[(size_t)(c0 + j) * decay_step] : 0.0f;
+    }
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j) {
+      if (c0 + j >= chunks) break;
+      mine[(size_t)(c0 + j) * all] = S;
+      S = S * decay[j] + left[j];
+    }
   }
 }
 
@@ -431,18 +548,34 @@ __global__ void __launch_bounds__(256) ssd_finish_kernel(const float* __restrict
   }
 }
 
-template <int R, bool PLAIN>
+template <int R, bool PLAIN, int MODE = WHOLE, int COLS = 1>
 static int launch_delta_rule(const float* prep, float* state, long long state_stride, const int* seq_starts, const int* state_slots, float* out, int entries,
-                             int heads, int kv_heads, int dim, int vdim, cudaStream_t stream) {
-  const int column_blocks = (vdim + kDeltaColumns - 1) / kDeltaColumns;
-  const size_t smem = kDeltaStages * (size_t)(3 * kDeltaLanes * R + kDeltaColumns + 4) * sizeof(float);
+                             int heads, int kv_heads, int dim, int vdim, cudaStream_t stream, int chunks = 1, float* chunk_states = nullptr, float* chunk_decays = nullptr) {
+  constexpr int kBlockColumns = kDeltaColumns * COLS;
+  const int column_blocks = (vdim + kBlockColumns - 1) / kBlockColumns;
+  const size_t smem = kDeltaStages * (size_t)(3 * kDeltaLanes * R + kBlockColumns + 4) * sizeof(float);
   if (smem > 48 * 1024) {   // the widest heads' ring of staged rows is beyond what a kernel may ask for without saying so
-    cudaError_t e = cudaFuncSetAttribute(delta_rule_kernel<R, PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(delta_rule_kernel<R, PLAIN, MODE, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  delta_rule_kernel<R, PLAIN><<<dim3(heads * column_blocks, entries), kDeltaThreads, smem, stream>>>(prep, state, state_stride, seq_starts, state_slots, out, heads,
-                                                                                                  kv_heads, dim, vdim);
+  delta_rule_kernel<R, PLAIN, MODE, COLS><<<dim3(heads * column_blocks, entries, chunks), kDeltaThreads, smem, stream>>>(prep, state, state_stride, seq_starts, state_slots, out, heads,
+                                                                                                                kv_heads, dim, vdim, chunk_states, chunk_decays);
   return (int)cudaGetLastError();
+}
+
+template <int R>
+static int launch_plain_chunks(const float* prep, float* state, long long state_stride, const int* seq_starts, const int* state_slots, float* out, int entries, int heads, int kv_heads,
+                               int dim, int vdim, int chunks, float* chunk_states, float* chunk_decays, cudaStream_t stream) {
+  constexpr int kCols = R <= 16 ? 4 : 2;   // as many columns a thread as its registers hold
+  int rc = launch_delta_rule<R, true, CHUNKED_LOCAL, kCols>(prep, state, state_stride, seq_starts, state_slots, out, entries, heads, kv_heads, dim, vdim, stream, chunks - 1, chunk_states,
+                                                     chunk_decays);
+  if (rc != 0) return rc;
+  const int held = 4 * ((dim + 4 * kDeltaLanes - 1) / (4 * kDeltaLanes));
+  const size_t all = (size_t)heads * held * vdim * kDeltaLanes;
+  delta_chunk_starts_kernel<<<dim3((unsigned)((all + 255) / 256), entries), 256, 0, stream>>>(state, state_stride, seq_starts, state_slots, chunk_states, chunk_decays, heads, held, vdim);
+  rc = (int)cudaGetLastError();
+  if (rc != 0) return rc;
+  return launch_delta_rule<R, true, CHUNKED_READ, kCols>(prep, state, state_stride, seq_starts, state_slots, out, entries, heads, kv_heads, dim, vdim, stream, chunks, chunk_states, chunk_decays);
 }
 
 }  // namespace tlie
@@ -494,6 +627,29 @@ TLIE_EXPORT int tlie_delta_rule(const float* prep, float* state, long long state
   TLIE_DELTA(24);
   TLIE_DELTA(32);
 #undef TLIE_DELTA
+  return (int)cudaErrorInvalidValue;
+}
+
+TLIE_EXPORT int tlie_delta_chunk_rows() { return kChunkRows; }
+
+// The plain recurrence with long entries cut into chunks (see CHUNKED_LOCAL).  ``longest``: the most rows any entry has.  Scratch for places = tokens / kChunkRows +
+// entries: chunk_states [places, a request's matrices], chunk_decays [places, heads, 4 lanes ceil(dim / (4 lanes))], 32-bit.
+TLIE_EXPORT int tlie_delta_rule_chunks(const float* prep, float* state, long long state_stride, const int* seq_starts, const int* state_slots, float* out, int entries, int heads,
+                                       int kv_heads, int dim, int vdim, int longest, float* chunk_states, float* chunk_decays, cudaStream_t stream) {
+  if (entries <= 0) return 0;
+  const int chunks = (longest + kChunkRows - 1) / kChunkRows;
+  if (dim < 1 || dim > 256 || kv_heads < 1 || heads % kv_heads != 0 || chunks < 2 || chunks > 65535 || entries > 65535 || chunk_states == nullptr || chunk_decays == nullptr)
+    return (int)cudaErrorInvalidValue;
+  const int r = 4 * ((dim + 4 * kDeltaLanes - 1) / (4 * kDeltaLanes));
+#define TLIE_CHUNKS(R) \
+  if (r <= R) return launch_plain_chunks<R>(prep, state, state_stride, seq_starts, state_slots, out, entries, heads, kv_heads, dim, vdim, chunks, chunk_states, chunk_decays, stream)
+  TLIE_CHUNKS(4);
+  TLIE_CHUNKS(8);
+  TLIE_CHUNKS(12);
+  TLIE_CHUNKS(16);
+  TLIE_CHUNKS(24);
+  TLIE_CHUNKS(32);
+#undef TLIE_CHUNKS
   return (int)cudaErrorInvalidValue;
 }
 

@@ -646,6 +646,10 @@ import os as _os
 DELTA_LANES = int(_os.environ.get("TLIE_DELTA_LANES", "8"))
 
 
+use_recurrence_chunks = True
+RECURRENCE_CHUNKS_MIN_ROWS = 512   # the longest entry's rows from which the plain recurrence runs in chunks
+
+
 def delta_rule_library():
     return load_library(f"tlie_delta_rule_l{DELTA_LANES}", DELTA_RULE_SOURCES, {"TLIE_DELTA_LANES": DELTA_LANES})
 
@@ -707,6 +711,20 @@ def delta_rule(prep, state, ctx, out, heads: int, kv_heads: int, dim: int, vdim:
     if out.shape != (tokens, heads * vdim) or out.dtype != torch.float32 or prep.dtype != torch.float32 or prep.shape[1] != 2 * kv_heads * dim + heads * (vdim + 1 + dim):
         raise KernelError("delta_rule: prep [rows, 2 G dim + H vdim + H + H dim] and out [rows, H vdim] are 32-bit", code="invalid_shape")
     state_ptr, state_stride = _state_rows(state, "delta_rule")
+    longest = getattr(ctx, "max_q_len", 0)
+    if plain and use_recurrence_chunks and longest >= RECURRENCE_CHUNKS_MIN_ROWS:
+        # a long entry's rows in chunks side by side (without the correction a chunk's end is a scaled start plus what the chunk adds)
+        library = delta_rule_library()
+        places = tokens // library.tlie_delta_chunk_rows() + ctx.num_seqs
+        matrices, _ = delta_state_words(heads, dim, vdim, 0, 1)
+        states = fast.named_scratch(prep.device, "recurrence_states", places * matrices, torch.float32)
+        decays = fast.named_scratch(prep.device, "recurrence_decays", places * (matrices // vdim), torch.float32)
+        _check(library.tlie_delta_rule_chunks(_ptr(prep), state_ptr, state_stride, _i32(ctx.seq_starts, "seq_starts"), _i32(ctx.state_slots, "state_slots"), _ptr(out),
+                                              c_int(ctx.num_seqs), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(longest), _ptr(states), _ptr(decays), _stream()),
+               "delta_rule_chunks")
+        global launch_count
+        launch_count += 2   # three kernels: the chunks by themselves, the states in front of them, the chunks with their read-outs
+        return
     _check(delta_rule_library().tlie_delta_rule(_ptr(prep), state_ptr, state_stride, _i32(ctx.seq_starts, "seq_starts"), _i32(ctx.state_slots, "state_slots"),
                                                 _ptr(out), c_int(ctx.num_seqs), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(1 if plain else 0), _stream()),
            "delta_rule")
