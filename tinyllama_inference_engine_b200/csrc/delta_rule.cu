@@ -165,7 +165,7 @@ __device__ __forceinline__ float sum_columns(float (&reads)[COLS], int lane, int
 }
 
 template <int R, bool PLAIN, int MODE = WHOLE, int COLS = 1>
-__global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(const float* __restrict__ prep, float* __restrict__ state, long long state_stride,
+__global__ void __launch_bounds__(kDeltaThreads, MODE != WHOLE && R <= 16 ? 4 : 1) delta_rule_kernel(const float* __restrict__ prep, float* __restrict__ state, long long state_stride,
                                                                   const int* __restrict__ seq_starts, const int* __restrict__ state_slots, float* __restrict__ out,
                                                                   int heads, int kv_heads, int dim, int vdim, float* __restrict__ chunk_states,
                                                                   float* __restrict__ chunk_decays) {

@@ -647,7 +647,7 @@ DELTA_LANES = int(_os.environ.get("TLIE_DELTA_LANES", "8"))
 
 
 use_recurrence_chunks = True
-RECURRENCE_CHUNKS_MIN_ROWS = 512   # the longest entry's rows from which the plain recurrence runs in chunks
+RECURRENCE_CHUNKS_MIN_ROWS = 384   # the longest entry's rows from which the plain recurrence runs in chunks (16 heads of 128 x 128: 0.10 ms against 0.12 in one run)
 
 
 def delta_rule_library():
