@@ -14,11 +14,13 @@
 //   delta_conv_state per entry: the last taps - 1 inputs of the convolution, kept for the next step
 //   delta_rule       the recurrence: one CTA per (entry, head, 16 columns), rows in order, the operands of the next twelve rows
 //                    on their way (asynchronous copies into a ring of 16) while a block of four is worked on between two barriers
+//   delta_chunk, delta_chunk_starts   the same recurrence without the correction for long entries: chunks of one entry side by side
 //   delta_gate_norm  per (token, head): o / sqrt(mean(o^2) + eps) * weight * sigmoid(gate)
 //
 // The same recurrence without the correction (``plain``: u = beta v) serves other linear-attention mixers: with decay f, key 1 - f and
 // beta 1 it is S <- diag(f) S + (1 - f) v^T (hgrn2_prepare); with one decay per head, key B, value x, beta dt and query C it is the
-// state-space model S <- a S + dt B x^T, y = S^T C (ssd_prepare, and ssd_finish for the skip term, the gate and the grouped norm).
+// state-space model S <- a S + dt B x^T, y = S^T C (ssd_prepare, and ssd_finish for the skip term, the gate and the grouped norm); with a
+// decay of its own per key channel beside key and query it is gated linear attention (gla_prepare).
 // ``decay_per_head``: one decay per head (g = exp(-exp(A_log_h) softplus(a_h + dt_bias_h))), written to all the head's key channels.
 //
 // State of a request (32-bit words): for every head the matrix in the order the recurrence reads it,
@@ -125,6 +127,158 @@ __device__ __forceinline__ void delta_commit() { asm volatile("cp.async.commit_g
 template <int N>
 __device__ __forceinline__ void delta_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
 
+// R: key channels a lane has registers for (a multiple of 4, dim <= 8 R); the state holds 4 ceil(dim / 32) of them per lane.
+// A row's operands ([q | k | g] of the head, the CTA's 16 values, beta) are copied asynchronously into a ring of kDeltaStages
+// buffers, several rows ahead, so that a row's turn never waits for memory; padding words are zeroed once and never copied.
+// PLAIN: u = beta v needs nothing of the state, so the chain from one row to the next is S <- g S + k u alone and the read-out's sums and
+// shuffles (o = S^T q of the new state) hang off it; with the correction u waits for k . S_j, reduced over the column's lanes, in every row.
+template <int R, bool PLAIN>
+__global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(const float* __restrict__ prep, float* __restrict__ state, long long state_stride,
+                                                                  const int* __restrict__ seq_starts, const int* __restrict__ state_slots, float* __restrict__ out,
+                                                                  int heads, int kv_heads, int dim, int vdim) {
+  extern __shared__ __align__(16) float stage_s[];   // kDeltaStages buffers of [q: 8 R | k: 8 R | g: 8 R | v: 16 | beta | 3 unused]
+  constexpr int kPadded = kDeltaLanes * R;
+  constexpr int kRow = 3 * kPadded + kDeltaColumns + 4;
+  constexpr int kLoads = (kRow + kDeltaThreads - 1) / kDeltaThreads;
+  const int column_blocks = (vdim + kDeltaColumns - 1) / kDeltaColumns;
+  const int head = blockIdx.x / column_blocks, block = blockIdx.x - head * column_blocks;
+  const int entry = blockIdx.y;
+  const int tid = threadIdx.x, lane = tid & (kDeltaLanes - 1), column = block * kDeltaColumns + tid / kDeltaLanes;
+  const bool live = column < vdim;
+  const int first = seq_starts[entry], count = seq_starts[entry + 1] - first;
+  const int kv = head / (heads / kv_heads);
+  const int qk = kv_heads * dim;
+  const int width = 2 * qk + heads * vdim + heads + heads * dim;
+  const int held = 4 * ((dim + 4 * kDeltaLanes - 1) / (4 * kDeltaLanes));   // key channels per lane that are stored
+  const size_t matrix = (size_t)held * vdim * kDeltaLanes;
+  float* mine = state + (size_t)state_slots[entry] * state_stride + (size_t)head * matrix;
+
+  // where each word of a staged row comes from in a prep row (-1: padding, stays zero)
+  int source[kLoads];
+#pragma unroll
+  for (int i = 0; i < kLoads; ++i) {
+    const int w = tid + i * kDeltaThreads;
+    int at = -1;
+    if (w < kPadded) at = w < dim ? kv * dim + w : -1;
+    else if (w < 2 * kPadded) at = w - kPadded < dim ? qk + kv * dim + (w - kPadded) : -1;
+    else if (w < 3 * kPadded) at = w - 2 * kPadded < dim ? 2 * qk + heads * vdim + heads + head * dim + (w - 2 * kPadded) : -1;
+    else if (w < 3 * kPadded + kDeltaColumns) at = block * kDeltaColumns + (w - 3 * kPadded) < vdim ? 2 * qk + head * vdim + block * kDeltaColumns + (w - 3 * kPadded) : -1;
+    else if (w == 3 * kPadded + kDeltaColumns) at = 2 * qk + heads * vdim + head;
+    source[i] = at;
+  }
+  for (int i = tid; i < kDeltaStages * kRow; i += kDeltaThreads) stage_s[i] = 0.0f;
+  __syncthreads();
+  float S[R];
+#pragma unroll
+  for (int i = 0; i < R; ++i) S[i] = (live && i < held) ? mine[((size_t)i * vdim + column) * kDeltaLanes + lane] : 0.0f;
+
+  auto issue = [&](int block_of_rows) {   // one group per block of rows, empty past the end, so that the count of groups in flight is the same at every step
+#pragma unroll
+    for (int n = 0; n < kDeltaBlock; ++n) {
+      const int row = block_of_rows * kDeltaBlock + n;
+      if (row < count) {
+        const float* from = prep + (size_t)(first + row) * width;
+        float* to = stage_s + (row % kDeltaStages) * kRow;
+#pragma unroll
+        for (int i = 0; i < kLoads; ++i)
+          if (source[i] >= 0) delta_copy_word(to + tid + i * kDeltaThreads, from + source[i]);
+      }
+    }
+    delta_commit();
+  };
+  constexpr int kBlocksAhead = kDeltaStages / kDeltaBlock - 1;
+#pragma unroll
+  for (int ahead = 0; ahead < kBlocksAhead; ++ahead) issue(ahead);
+  const int blocks = (count + kDeltaBlock - 1) / kDeltaBlock;
+  for (int block_of_rows = 0; block_of_rows < blocks; ++block_of_rows) {
+    delta_wait<kBlocksAhead - 1>();   // this thread's copies of this block's rows have landed ...
+    __syncthreads();                  // ... and so have everyone's; and everyone is done with the block before, whose buffers are written next
+    issue(block_of_rows + kBlocksAhead);
+    if constexpr (PLAIN) {
+      // the block's four rows: the state's chain first, every row leaving its share of the read-out; then the four sums across the column's
+      // lanes side by side, so that a round of shuffles is waited for once per block and not once per row
+      float reads[kDeltaBlock];
+#pragma unroll
+      for (int n = 0; n < kDeltaBlock; ++n) {
+        const int row = block_of_rows * kDeltaBlock + n;
+        reads[n] = 0.0f;
+        if (row < count) {
+          const float* cur = stage_s + (row % kDeltaStages) * kRow;
+          const float u = cur[3 * kPadded + kDeltaColumns] * cur[3 * kPadded + (tid / kDeltaLanes)];   // beta v
+          float read2[2] = {0.0f, 0.0f};
+#pragma unroll
+          for (int j = 0; j < R / 4; ++j) {
+            const float4 q4 = *reinterpret_cast<const float4*>(cur + j * 4 * kDeltaLanes + lane * 4);
+            const float4 k4 = *reinterpret_cast<const float4*>(cur + kPadded + j * 4 * kDeltaLanes + lane * 4);
+            const float4 g4 = *reinterpret_cast<const float4*>(cur + 2 * kPadded + j * 4 * kDeltaLanes + lane * 4);
+            const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, g[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+              const int i = 4 * j + c;
+              S[i] = S[i] * g[c] + k[c] * u;
+              read2[c & 1] += q[c] * S[i];
+            }
+          }
+          reads[n] = read2[0] + read2[1];
+        }
+      }
+#pragma unroll
+      for (int offset = kDeltaLanes / 2; offset > 0; offset >>= 1)
+#pragma unroll
+        for (int n = 0; n < kDeltaBlock; ++n) reads[n] += __shfl_xor_sync(0xffffffffu, reads[n], offset);
+#pragma unroll
+      for (int n = 0; n < kDeltaBlock; ++n) {
+        const int row = block_of_rows * kDeltaBlock + n;
+        if (row < count && live && lane == 0) out[(size_t)(first + row) * heads * vdim + head * vdim + column] = reads[n];
+      }
+    } else {
+#pragma unroll
+    for (int n = 0; n < kDeltaBlock; ++n) {
+      const int row = block_of_rows * kDeltaBlock + n;
+      if (row >= count) break;
+      const float* cur = stage_s + (row % kDeltaStages) * kRow;
+      // k . (g S)_j, q . (g S)_j, q . k (this lane's share), each in two chains of sums
+      float reach2[2] = {0.0f, 0.0f}, read2[2] = {0.0f, 0.0f}, both2[2] = {0.0f, 0.0f};
+      float kk[R];
+#pragma unroll
+      for (int j = 0; j < R / 4; ++j) {
+        const float4 q4 = *reinterpret_cast<const float4*>(cur + j * 4 * kDeltaLanes + lane * 4);
+        const float4 k4 = *reinterpret_cast<const float4*>(cur + kPadded + j * 4 * kDeltaLanes + lane * 4);
+        const float4 g4 = *reinterpret_cast<const float4*>(cur + 2 * kPadded + j * 4 * kDeltaLanes + lane * 4);
+        const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, g[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const int i = 4 * j + c;
+          S[i] *= g[c];
+          reach2[c & 1] += k[c] * S[i];
+          read2[c & 1] += q[c] * S[i];
+          both2[c & 1] += q[c] * k[c];
+          kk[i] = k[c];
+        }
+      }
+      float reach = reach2[0] + reach2[1], read = read2[0] + read2[1], both = both2[0] + both2[1];
+#pragma unroll
+      for (int offset = kDeltaLanes / 2; offset > 0; offset >>= 1) {
+        reach += __shfl_xor_sync(0xffffffffu, reach, offset);
+        read += __shfl_xor_sync(0xffffffffu, read, offset);
+        both += __shfl_xor_sync(0xffffffffu, both, offset);
+      }
+      const float v = cur[3 * kPadded + (tid / kDeltaLanes)], beta = cur[3 * kPadded + kDeltaColumns];
+      const float u = beta * (v - reach);
+#pragma unroll
+      for (int i = 0; i < R; ++i) S[i] += kk[i] * u;
+      if (live && lane == 0) out[(size_t)(first + row) * heads * vdim + head * vdim + column] = read + both * u;
+    }
+    }
+  }
+  delta_wait<0>();
+  if (live && count > 0) {
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+      if (i < held) mine[((size_t)i * vdim + column) * kDeltaLanes + lane] = S[i];
+  }
+}
+
 // A long entry of the plain recurrence is cut into chunks of kChunkRows rows that run side by side, since without the correction a row only scales the state
 // and adds to it: the state behind a chunk is (the product of its decays) times the state in front of it plus what the chunk alone would leave.
 //   CHUNKED_LOCAL  a CTA per (entry, head, columns, chunk but the last): the chunk from a zero state, nothing read out; leaves its end and its decays' product
@@ -135,13 +289,8 @@ __device__ __forceinline__ void delta_wait() { asm volatile("cp.async.wait_group
 // All of it in 32-bit.  Chunk c of entry e has the place seq_starts[e] / kChunkRows + e + c in the scratch: no two chunks share one, and there are at most
 // tokens / kChunkRows + entries.
 constexpr int kChunkRows = 128;
-enum { WHOLE = 0, CHUNKED_LOCAL = 1, CHUNKED_READ = 2 };
+enum { CHUNKED_LOCAL = 1, CHUNKED_READ = 2 };
 
-// R: key channels a lane has registers for (a multiple of 4, dim <= 8 R); the state holds 4 ceil(dim / 32) of them per lane.
-// A row's operands ([q | k | g] of the head, the CTA's 16 values, beta) are copied asynchronously into a ring of kDeltaStages
-// buffers, several rows ahead, so that a row's turn never waits for memory; padding words are zeroed once and never copied.
-// PLAIN: u = beta v needs nothing of the state, so the chain from one row to the next is S <- g S + k u alone and the read-out's sums and
-// shuffles (o = S^T q of the new state) hang off it; with the correction u waits for k . S_j, reduced over the column's lanes, in every row.
 // The sums over a column's lanes of COLS columns at once: the first steps halve what a lane holds (it keeps one half of the columns and hands over the other), so
 // that COLS columns cost COLS - 1 shuffles and a few more instead of log2(lanes) each.  Returns the finished sum and which column it belongs to; the
 // kDeltaLanes / COLS lanes that share a column hold the same.
@@ -164,12 +313,12 @@ __device__ __forceinline__ float sum_columns(float (&reads)[COLS], int lane, int
   return reads[0];
 }
 
-template <int R, bool PLAIN, int MODE = WHOLE, int COLS = 1>
-__global__ void __launch_bounds__(kDeltaThreads, MODE != WHOLE && R <= 16 ? 4 : 1) delta_rule_kernel(const float* __restrict__ prep, float* __restrict__ state, long long state_stride,
+template <int R, int MODE, int COLS>
+__global__ void __launch_bounds__(kDeltaThreads, R <= 16 ? 4 : 1) delta_chunk_kernel(const float* __restrict__ prep, float* __restrict__ state, long long state_stride,
                                                                   const int* __restrict__ seq_starts, const int* __restrict__ state_slots, float* __restrict__ out,
                                                                   int heads, int kv_heads, int dim, int vdim, float* __restrict__ chunk_states,
                                                                   float* __restrict__ chunk_decays) {
-  static_assert((PLAIN || MODE == WHOLE) && (MODE != WHOLE || COLS == 1) && COLS <= kDeltaLanes, "only the plain recurrence is cut into chunks, and only chunks have several columns a thread");
+  static_assert(COLS <= kDeltaLanes, "the lanes of a column share its columns out");
   extern __shared__ __align__(16) float stage_s[];   // kDeltaStages buffers of [q: 8 R | k: 8 R | g: 8 R | v: 16 COLS | beta | 3 unused]
   constexpr int kPadded = kDeltaLanes * R;
   constexpr int kBlockColumns = kDeltaColumns * COLS;
@@ -179,12 +328,11 @@ __global__ void __launch_bounds__(kDeltaThreads, MODE != WHOLE && R <= 16 ? 4 : 
   const int head = blockIdx.x / column_blocks, block = blockIdx.x - head * column_blocks;
   const int entry = blockIdx.y;
   const int tid = threadIdx.x, lane = tid & (kDeltaLanes - 1), column = block * kBlockColumns + tid / kDeltaLanes;   // a thread's columns: this one and every kDeltaColumns-th behind it
-  const bool live = column < vdim;
   const int entry_first = seq_starts[entry], entry_count = seq_starts[entry + 1] - entry_first;
-  const int chunk = MODE == WHOLE ? 0 : blockIdx.z;
-  const bool last_chunk = MODE == WHOLE || (chunk + 1) * kChunkRows >= entry_count;
-  if (MODE != WHOLE && (chunk * kChunkRows >= entry_count || (MODE == CHUNKED_LOCAL && last_chunk))) return;
-  const int first = entry_first + chunk * kChunkRows, count = MODE == WHOLE ? entry_count : min(kChunkRows, entry_count - chunk * kChunkRows);
+  const int chunk = blockIdx.z;
+  const bool last_chunk = (chunk + 1) * kChunkRows >= entry_count;
+  if (chunk * kChunkRows >= entry_count || (MODE == CHUNKED_LOCAL && last_chunk)) return;
+  const int first = entry_first + chunk * kChunkRows, count = min(kChunkRows, entry_count - chunk * kChunkRows);
   const int kv = head / (heads / kv_heads);
   const int qk = kv_heads * dim;
   const int width = 2 * qk + heads * vdim + heads + heads * dim;
@@ -192,7 +340,7 @@ __global__ void __launch_bounds__(kDeltaThreads, MODE != WHOLE && R <= 16 ? 4 : 
   const size_t matrix = (size_t)held * vdim * kDeltaLanes;
   float* mine = state + (size_t)state_slots[entry] * state_stride + (size_t)head * matrix;
   // where this run starts from and what it leaves: the request's state, or a chunk's place in the scratch
-  const size_t place = MODE == WHOLE ? 0 : (size_t)(entry_first / kChunkRows + entry + chunk) * heads + head;
+  const size_t place = (size_t)(entry_first / kChunkRows + entry + chunk) * heads + head;
   const float* from_state = (MODE == CHUNKED_READ && entry_count > kChunkRows) ? chunk_states + place * matrix : mine;
   float* to_state = MODE == CHUNKED_LOCAL ? chunk_states + place * matrix : mine;
 
@@ -243,102 +391,62 @@ __global__ void __launch_bounds__(kDeltaThreads, MODE != WHOLE && R <= 16 ? 4 : 
     delta_wait<kBlocksAhead - 1>();   // this thread's copies of this block's rows have landed ...
     __syncthreads();                  // ... and so have everyone's; and everyone is done with the block before, whose buffers are written next
     issue(block_of_rows + kBlocksAhead);
-    if constexpr (PLAIN) {
-      // the block's four rows: the state's chain first, every row leaving its share of the read-out; then the four sums across the column's
-      // lanes side by side, so that a round of shuffles is waited for once per block and not once per row
-      float reads[kDeltaBlock][COLS];
-#pragma unroll
-      for (int n = 0; n < kDeltaBlock; ++n) {
-        const int row = block_of_rows * kDeltaBlock + n;
-#pragma unroll
-        for (int m = 0; m < COLS; ++m) reads[n][m] = 0.0f;
-        if (row < count) {
-          const float* cur = stage_s + (row % kDeltaStages) * kRow;
-          float u[COLS], read2[COLS][2];
-#pragma unroll
-          for (int m = 0; m < COLS; ++m) {
-            u[m] = cur[3 * kPadded + kBlockColumns] * cur[3 * kPadded + tid / kDeltaLanes + m * kDeltaColumns];   // beta v
-            read2[m][0] = read2[m][1] = 0.0f;
-          }
-#pragma unroll
-          for (int j = 0; j < R / 4; ++j) {
-            const float4 k4 = *reinterpret_cast<const float4*>(cur + kPadded + j * 4 * kDeltaLanes + lane * 4);
-            const float4 g4 = *reinterpret_cast<const float4*>(cur + 2 * kPadded + j * 4 * kDeltaLanes + lane * 4);
-            const float k[4] = {k4.x, k4.y, k4.z, k4.w}, g[4] = {g4.x, g4.y, g4.z, g4.w};
-            float q[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            if constexpr (MODE != CHUNKED_LOCAL) {
-              const float4 q4 = *reinterpret_cast<const float4*>(cur + j * 4 * kDeltaLanes + lane * 4);
-              q[0] = q4.x, q[1] = q4.y, q[2] = q4.z, q[3] = q4.w;
-            }
-#pragma unroll
-            for (int c = 0; c < 4; ++c) {
-              const int i = 4 * j + c;
-#pragma unroll
-              for (int m = 0; m < COLS; ++m) {
-                S[m][i] = S[m][i] * g[c] + k[c] * u[m];
-                if constexpr (MODE != CHUNKED_LOCAL) read2[m][c & 1] += q[c] * S[m][i];
-              }
-              if constexpr (MODE == CHUNKED_LOCAL) {
-                if (block == 0) faded[i] *= g[c];
-              }
-            }
-          }
-#pragma unroll
-          for (int m = 0; m < COLS; ++m) reads[n][m] = read2[m][0] + read2[m][1];
-        }
-      }
-      if constexpr (MODE != CHUNKED_LOCAL) {
-        float total[kDeltaBlock];
-        int which = 0;
-#pragma unroll
-        for (int n = 0; n < kDeltaBlock; ++n) total[n] = sum_columns(reads[n], lane, which);
-        const int mine_at = column + which * kDeltaColumns;
-        if (mine_at < vdim && (lane & (kDeltaLanes / COLS - 1)) == 0) {
-#pragma unroll
-          for (int n = 0; n < kDeltaBlock; ++n) {
-            const int row = block_of_rows * kDeltaBlock + n;
-            if (row < count) out[(size_t)(first + row) * heads * vdim + head * vdim + mine_at] = total[n];
-          }
-        }
-      }
-    } else {
+    // the block's four rows: the state's chain first, every row leaving its share of the read-out; then the four sums across the column's
+    // lanes side by side, so that a round of shuffles is waited for once per block and not once per row
+    float reads[kDeltaBlock][COLS];
 #pragma unroll
     for (int n = 0; n < kDeltaBlock; ++n) {
       const int row = block_of_rows * kDeltaBlock + n;
-      if (row >= count) break;
-      const float* cur = stage_s + (row % kDeltaStages) * kRow;
-      // k . (g S)_j, q . (g S)_j, q . k (this lane's share), each in two chains of sums
-      float reach2[2] = {0.0f, 0.0f}, read2[2] = {0.0f, 0.0f}, both2[2] = {0.0f, 0.0f};
-      float kk[R];
 #pragma unroll
-      for (int j = 0; j < R / 4; ++j) {
-        const float4 q4 = *reinterpret_cast<const float4*>(cur + j * 4 * kDeltaLanes + lane * 4);
-        const float4 k4 = *reinterpret_cast<const float4*>(cur + kPadded + j * 4 * kDeltaLanes + lane * 4);
-        const float4 g4 = *reinterpret_cast<const float4*>(cur + 2 * kPadded + j * 4 * kDeltaLanes + lane * 4);
-        const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, g[4] = {g4.x, g4.y, g4.z, g4.w};
+      for (int m = 0; m < COLS; ++m) reads[n][m] = 0.0f;
+      if (row < count) {
+        const float* cur = stage_s + (row % kDeltaStages) * kRow;
+        float u[COLS], read2[COLS][2];
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          const int i = 4 * j + c;
-          S[0][i] *= g[c];
-          reach2[c & 1] += k[c] * S[0][i];
-          read2[c & 1] += q[c] * S[0][i];
-          both2[c & 1] += q[c] * k[c];
-          kk[i] = k[c];
+        for (int m = 0; m < COLS; ++m) {
+          u[m] = cur[3 * kPadded + kBlockColumns] * cur[3 * kPadded + tid / kDeltaLanes + m * kDeltaColumns];   // beta v
+          read2[m][0] = read2[m][1] = 0.0f;
+        }
+#pragma unroll
+        for (int j = 0; j < R / 4; ++j) {
+          const float4 k4 = *reinterpret_cast<const float4*>(cur + kPadded + j * 4 * kDeltaLanes + lane * 4);
+          const float4 g4 = *reinterpret_cast<const float4*>(cur + 2 * kPadded + j * 4 * kDeltaLanes + lane * 4);
+          const float k[4] = {k4.x, k4.y, k4.z, k4.w}, g[4] = {g4.x, g4.y, g4.z, g4.w};
+          float q[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+          if constexpr (MODE != CHUNKED_LOCAL) {
+            const float4 q4 = *reinterpret_cast<const float4*>(cur + j * 4 * kDeltaLanes + lane * 4);
+            q[0] = q4.x, q[1] = q4.y, q[2] = q4.z, q[3] = q4.w;
+          }
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const int i = 4 * j + c;
+#pragma unroll
+            for (int m = 0; m < COLS; ++m) {
+              S[m][i] = S[m][i] * g[c] + k[c] * u[m];
+              if constexpr (MODE != CHUNKED_LOCAL) read2[m][c & 1] += q[c] * S[m][i];
+            }
+            if constexpr (MODE == CHUNKED_LOCAL) {
+              if (block == 0) faded[i] *= g[c];
+            }
+          }
+        }
+#pragma unroll
+        for (int m = 0; m < COLS; ++m) reads[n][m] = read2[m][0] + read2[m][1];
+      }
+    }
+    if constexpr (MODE != CHUNKED_LOCAL) {
+      float total[kDeltaBlock];
+      int which = 0;
+#pragma unroll
+      for (int n = 0; n < kDeltaBlock; ++n) total[n] = sum_columns(reads[n], lane, which);
+      const int mine_at = column + which * kDeltaColumns;
+      if (mine_at < vdim && (lane & (kDeltaLanes / COLS - 1)) == 0) {
+#pragma unroll
+        for (int n = 0; n < kDeltaBlock; ++n) {
+          const int row = block_of_rows * kDeltaBlock + n;
+          if (row < count) out[(size_t)(first + row) * heads * vdim + head * vdim + mine_at] = total[n];
         }
       }
-      float reach = reach2[0] + reach2[1], read = read2[0] + read2[1], both = both2[0] + both2[1];
-#pragma unroll
-      for (int offset = kDeltaLanes / 2; offset > 0; offset >>= 1) {
-        reach += __shfl_xor_sync(0xffffffffu, reach, offset);
-        read += __shfl_xor_sync(0xffffffffu, read, offset);
-        both += __shfl_xor_sync(0xffffffffu, both, offset);
-      }
-      const float v = cur[3 * kPadded + (tid / kDeltaLanes)], beta = cur[3 * kPadded + kDeltaColumns];
-      const float u = beta * (v - reach);
-#pragma unroll
-      for (int i = 0; i < R; ++i) S[0][i] += kk[i] * u;
-      if (live && lane == 0) out[(size_t)(first + row) * heads * vdim + head * vdim + column] = read + both * u;
-    }
     }
   }
   delta_wait<0>();
@@ -548,18 +656,32 @@ __global__ void __launch_bounds__(256) ssd_finish_kernel(const float* __restrict
   }
 }
 
-template <int R, bool PLAIN, int MODE = WHOLE, int COLS = 1>
+template <int R, bool PLAIN>
 static int launch_delta_rule(const float* prep, float* state, long long state_stride, const int* seq_starts, const int* state_slots, float* out, int entries,
-                             int heads, int kv_heads, int dim, int vdim, cudaStream_t stream, int chunks = 1, float* chunk_states = nullptr, float* chunk_decays = nullptr) {
+                             int heads, int kv_heads, int dim, int vdim, cudaStream_t stream) {
+  const int column_blocks = (vdim + kDeltaColumns - 1) / kDeltaColumns;
+  const size_t smem = kDeltaStages * (size_t)(3 * kDeltaLanes * R + kDeltaColumns + 4) * sizeof(float);
+  if (smem > 48 * 1024) {   // the widest heads' ring of staged rows is beyond what a kernel may ask for without saying so
+    cudaError_t e = cudaFuncSetAttribute(delta_rule_kernel<R, PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  delta_rule_kernel<R, PLAIN><<<dim3(heads * column_blocks, entries), kDeltaThreads, smem, stream>>>(prep, state, state_stride, seq_starts, state_slots, out, heads,
+                                                                                                  kv_heads, dim, vdim);
+  return (int)cudaGetLastError();
+}
+
+template <int R, int MODE, int COLS>
+static int launch_chunks(const float* prep, float* state, long long state_stride, const int* seq_starts, const int* state_slots, float* out, int entries, int heads, int kv_heads, int dim,
+                         int vdim, int chunks, float* chunk_states, float* chunk_decays, cudaStream_t stream) {
   constexpr int kBlockColumns = kDeltaColumns * COLS;
   const int column_blocks = (vdim + kBlockColumns - 1) / kBlockColumns;
   const size_t smem = kDeltaStages * (size_t)(3 * kDeltaLanes * R + kBlockColumns + 4) * sizeof(float);
-  if (smem > 48 * 1024) {   // the widest heads' ring of staged rows is beyond what a kernel may ask for without saying so
-    cudaError_t e = cudaFuncSetAttribute(delta_rule_kernel<R, PLAIN, MODE, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<R, MODE, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  delta_rule_kernel<R, PLAIN, MODE, COLS><<<dim3(heads * column_blocks, entries, chunks), kDeltaThreads, smem, stream>>>(prep, state, state_stride, seq_starts, state_slots, out, heads,
-                                                                                                                kv_heads, dim, vdim, chunk_states, chunk_decays);
+  delta_chunk_kernel<R, MODE, COLS><<<dim3(heads * column_blocks, entries, chunks), kDeltaThreads, smem, stream>>>(prep, state, state_stride, seq_starts, state_slots, out, heads, kv_heads,
+                                                                                                                  dim, vdim, chunk_states, chunk_decays);
   return (int)cudaGetLastError();
 }
 
@@ -567,15 +689,15 @@ template <int R>
 static int launch_plain_chunks(const float* prep, float* state, long long state_stride, const int* seq_starts, const int* state_slots, float* out, int entries, int heads, int kv_heads,
                                int dim, int vdim, int chunks, float* chunk_states, float* chunk_decays, cudaStream_t stream) {
   constexpr int kCols = R <= 16 ? 4 : 2;   // as many columns a thread as its registers hold
-  int rc = launch_delta_rule<R, true, CHUNKED_LOCAL, kCols>(prep, state, state_stride, seq_starts, state_slots, out, entries, heads, kv_heads, dim, vdim, stream, chunks - 1, chunk_states,
-                                                     chunk_decays);
+  int rc = launch_chunks<R, CHUNKED_LOCAL, kCols>(prep, state, state_stride, seq_starts, state_slots, out, entries, heads, kv_heads, dim, vdim, chunks - 1, chunk_states, chunk_decays,
+                                                  stream);
   if (rc != 0) return rc;
   const int held = 4 * ((dim + 4 * kDeltaLanes - 1) / (4 * kDeltaLanes));
   const size_t all = (size_t)heads * held * vdim * kDeltaLanes;
   delta_chunk_starts_kernel<<<dim3((unsigned)((all + 255) / 256), entries), 256, 0, stream>>>(state, state_stride, seq_starts, state_slots, chunk_states, chunk_decays, heads, held, vdim);
   rc = (int)cudaGetLastError();
   if (rc != 0) return rc;
-  return launch_delta_rule<R, true, CHUNKED_READ, kCols>(prep, state, state_stride, seq_starts, state_slots, out, entries, heads, kv_heads, dim, vdim, stream, chunks, chunk_states, chunk_decays);
+  return launch_chunks<R, CHUNKED_READ, kCols>(prep, state, state_stride, seq_starts, state_slots, out, entries, heads, kv_heads, dim, vdim, chunks, chunk_states, chunk_decays, stream);
 }
 
 }  // namespace tlie
