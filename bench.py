@@ -1114,12 +1114,14 @@ def run_designs(args) -> dict:
                 gate_at, columns = (H + G) * D + G * V, (H + G) * D + G * V + -(-H // 8) * 8
                 rows, kept = torch.randn(tokens, columns, device=device).to(bf16), torch.randn(tokens, G * V, device=device).to(bf16)
                 factors, plain = torch.full((H,), D ** -0.5, device=device), kind == "attention"
-                biases = None if plain else (ones[: H * D], ones[: G * D], ones[: G * V]) if max(H * D, G * V) <= ones.numel() else tuple(torch.ones(n, device=device) for n in (H * D, G * D, G * V))
+                biases = None if plain else tuple(torch.zeros(n, device=device) for n in (H * D, G * D, G * V))
                 norm = (ones[:D], ones[:D]) if plain else (None, None)
                 store = lambda **k: ops.norm_rotary_store(rows, H * D, (H + G) * D, biases, *norm, 1e-5, factors, inv_freq, D, plain, 1.0, ctx.positions, ctx.token_seq, cache, H, G, D, V, **k)
                 ms, like_ms = timed(lambda: store(first_values=kept, value_share=0.3)), timed(store)
                 moved = tokens * 2.0 * (2 * H * D + 2 * G * (D + V))
                 out[f"{kind}_store_{name}"] = against_bytes(ms, moved + tokens * 2.0 * G * V, like_ms, moved)
+                rows = torch.randn(tokens, columns, device=device).to(bf16)   # the store has turned and scaled the queries in place again and again
+                rows[:, : H * D] *= D ** -0.5
                 mixed = torch.empty(tokens, H * V, dtype=bf16, device=device)
                 options = dict(gate_per_head=True, sinks=torch.zeros(H, device=device)) if plain else dict(gate_per_head=True, softcap=a["softcap"])
                 ms = timed(lambda: ops.mixed_heads_attention(rows, gate_at if plain else -1, ctx.positions, ctx.token_seq, cache, None, None, mixed, H, G, D, V, 0, 1.0, batch=ctx, **options))

@@ -706,6 +706,7 @@ def delta_rule(prep, state, ctx, out, heads: int, kv_heads: int, dim: int, vdim:
     """The gated delta rule over every entry's rows in order, from and into the entries' state slots: per head
     S <- diag(decay) S; u = beta (v - S^T k); S <- S + k u^T; out = S^T q.  ``out`` is 32-bit [T, heads * vdim].
     ``plain``: u = beta v, the recurrence of linear attention with a decay (nothing is taken back before the write).
+    Long entries of the plain recurrence run in chunks side by side (``RECURRENCE_CHUNKS_MIN_ROWS``; other orders of 32-bit sums, nothing else).
     ``prep`` rows are [q: kv_heads dim | k: kv_heads dim | v: heads vdim | beta: heads | decay: heads dim]."""
     tokens = prep.shape[0]
     if out.shape != (tokens, heads * vdim) or out.dtype != torch.float32 or prep.dtype != torch.float32 or prep.shape[1] != 2 * kv_heads * dim + heads * (vdim + 1 + dim):
